@@ -79,7 +79,7 @@ class CacheLayout:
     def runtime_groups(self, runtime, page_size: int, num_pages: int):
         """GroupSpec list for the host CacheManager, one pool per paged group."""
         return [runtime.GroupSpec(self.page_size_of(g, page_size), self.num_pages_of(g, page_size, num_pages), g.spec.window,
-                                  g.spec.keep_first if g.spec.window else 0)
+                                  g.spec.keep_first if g.spec.window else 0, bool(g.spec.chunked and g.spec.window))
                 for g in self.paged]
 
     def bytes_per_token(self, elem_size: int) -> int:

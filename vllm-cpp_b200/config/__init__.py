@@ -5,5 +5,6 @@ from .rimopel import RimopelConfig
 from .nagavik import NagavikConfig
 from .fifudra import FifudraConfig
 from .mefupel import MefupelConfig
+from .nufetar import NufetarConfig
 
-__all__ = ["ConfigError", "ModelConfig", "EngineConfig", "Qwen3Config", "RimopelConfig", "NagavikConfig", "FifudraConfig", "MefupelConfig", "load_config_dict"]
+__all__ = ["ConfigError", "ModelConfig", "EngineConfig", "Qwen3Config", "RimopelConfig", "NagavikConfig", "FifudraConfig", "MefupelConfig", "NufetarConfig", "load_config_dict"]

@@ -20,6 +20,11 @@
 // scaled: w_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j)).  The sink enters as the
 // starting state (maximum sink_h, sum 1) of the item's first key slice, so sliced
 // items merge as they are.
+// The window may stand still (`chunked`): a query at pos then sees the keys of its own chunk of W positions, counted
+// from position 0.  Query rows may be wide (`wide`): a row has one block of lanes per KV head, the score of key j is the
+// sum over the KV heads of block . that head's key (queries mixed across heads, see rope_store.cu), while its values are
+// still those of the row's own KV head.  A gate per (token, head) may multiply the result (`out_gate`).  Key rows may be as
+// wide as shared memory has room for; values wider than a block's threads hold are dealt to further blocks (grid z).
 // Items whose key range is sliced write (max, sum, unnormalised output) partials,
 // merged by attn_merge_kernel in slice order.
 #include "common.cuh"
@@ -62,6 +67,9 @@ struct AttnArgs {
     const float* slope;
     int sink;
     const float* sink_value;    // with a sink: its score per head (null: 0); it is not scaled
+    int chunked;                // the window is the chunk of `window` positions that pos lies in
+    int wide;                   // q rows are [nkv][hd] lanes, one block per KV head
+    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
 };
 
 template <typename T> struct Vec8;
@@ -84,18 +92,26 @@ template <> struct Vec8<__nv_bfloat16> {
     }
 };
 
+// the first key a query at `pos` sees (kept first keys aside)
+__device__ __forceinline__ int first_key(int pos, int W, int chunked) {
+    if (W <= 0) return 0;
+    return max(0, chunked ? pos - pos % W : pos - W + 1);
+}
+
 template <typename T, int RMAX>
 __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
     extern __shared__ float smem[];
     const int hd = a.hd;
-    float* q_s = smem;                      // [RMAX][hd], pre-scaled
-    float* p_s = q_s + RMAX * hd;           // [RMAX][TK]
+    const int qw = a.wide ? a.nkv * hd : hd;
+    float* q_s = smem;                      // [RMAX][qw], pre-scaled
+    float* p_s = q_s + RMAX * qw;           // [RMAX][TK]
     float* m_s = p_s + RMAX * TK;           // [RMAX] running maximum
     float* l_s = m_s + RMAX;                // [RMAX] running sum
     float* al_s = l_s + RMAX;               // [RMAX] rescale factor of the current tile
     float* da_s = al_s + RMAX;              // [RMAX] distance penalty of the row's head: a, b
     float* db_s = da_s + RMAX;
-    long long* voff_s = reinterpret_cast<long long*>(db_s + RMAX);  // [TK] element offset of each key's V row
+    int* lo_s = reinterpret_cast<int*>(db_s + RMAX);   // [RMAX] first key of the row's window
+    long long* voff_s = reinterpret_cast<long long*>(lo_s + RMAX);  // [TK] element offset of each key's V row
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int* item = a.items + (size_t)blockIdx.x * ITEM_INTS;
@@ -134,7 +150,7 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
     const int W = a.window;
 
     // key range of the whole item, then of this slice (in pages)
-    const int lo = W > 0 ? max(0, pos0 - W + 1) : 0;
+    const int lo = first_key(pos0, W, a.chunked);
     const int hi = pos_last + 1;
     const int ps = a.page_size;
     const int pb_lo = lo / ps, pb_hi = (hi + ps - 1) / ps;
@@ -150,10 +166,10 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
 
     // queries -> shared memory, scaled
     const T* qg = reinterpret_cast<const T*>(a.q);
-    for (int idx = tid; idx < R * hd; idx += TK) {
-        const int r = idx / hd, d = idx % hd;
+    for (int idx = tid; idx < R * qw; idx += TK) {
+        const int r = idx / qw, d = idx % qw;
         const int iq = r / gq, ih = r % gq;
-        q_s[r * hd + d] = to_f32(qg[((size_t)(row0 + iq) * a.nh + head0 + ih) * hd + d]) * a.scale;
+        q_s[r * qw + d] = to_f32(qg[((size_t)(row0 + iq) * a.nh + head0 + ih) * qw + d]) * a.scale;
     }
     if (tid < RMAX) {
         const bool with_sink = a.sink && slice == 0;
@@ -162,8 +178,10 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
         l_s[tid] = with_sink ? 1.f : 0.f;
         da_s[tid] = a.dist_a != nullptr && tid < R ? a.dist_a[h] : (a.slope != nullptr && tid < R ? a.slope[h] : 0.f);
         db_s[tid] = a.dist_a != nullptr && tid < R ? a.dist_b[h] : 0.f;
+        lo_s[tid] = first_key(pos0 + tid / gq, W, a.chunked);
     }
     constexpr int DPT = VCB_MAX_HEAD_DIM / TK;  // output dims per thread
+    const int d0 = blockIdx.z * VCB_MAX_HEAD_DIM;   // first output dim of this block
     float acc_o[RMAX][DPT];
 #pragma unroll
     for (int r = 0; r < RMAX; ++r)
@@ -191,31 +209,32 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
                     valid = false;
                     voff_s[tid] = -1;
                 } else {
-                    const long long in_page = (long long)kvh * ps + kidx % ps;
-                    const long long base = (long long)page * a.page_stride + in_page * hd;
-                    voff_s[tid] = (long long)page * a.page_stride + (long long)a.nkv * ps * hd + in_page * hdv;
-                    const T* kp = pages + base;
-                    if (!vec_ok) {
-                        // a head size that is no multiple of 8: element by element
-                        for (int c = 0; c < hd; ++c) {
-                            const float kf = to_f32(kp[c]);
+                    voff_s[tid] = (long long)page * a.page_stride + (long long)a.nkv * ps * hd + ((long long)kvh * ps + kidx % ps) * hdv;
+                    for (int b = 0; b < (a.wide ? a.nkv : 1); ++b) {
+                        const T* kp = pages + (long long)page * a.page_stride + ((long long)(a.wide ? b : kvh) * ps + kidx % ps) * hd;
+                        const float* q_b = q_s + b * hd;
+                        if (!vec_ok) {
+                            // a head size that is no multiple of 8: element by element
+                            for (int c = 0; c < hd; ++c) {
+                                const float kf = to_f32(kp[c]);
 #pragma unroll
-                            for (int r = 0; r < RMAX; ++r)
-                                if (r < R) s[r] = fmaf(kf, q_s[r * hd + c], s[r]);
+                                for (int r = 0; r < RMAX; ++r)
+                                    if (r < R) s[r] = fmaf(kf, q_b[r * qw + c], s[r]);
+                            }
                         }
-                    }
-                    for (int c = 0; vec_ok && c < hd; c += 8) {
-                        float kf[8];
-                        Vec8<T>::load(kp + c, kf);
+                        for (int c = 0; vec_ok && c < hd; c += 8) {
+                            float kf[8];
+                            Vec8<T>::load(kp + c, kf);
 #pragma unroll
-                        for (int r = 0; r < RMAX; ++r) {
-                            if (r < R) {
-                                const float4 qa = *reinterpret_cast<const float4*>(q_s + r * hd + c);
-                                const float4 qb = *reinterpret_cast<const float4*>(q_s + r * hd + c + 4);
-                                s[r] = fmaf(kf[0], qa.x, s[r]); s[r] = fmaf(kf[1], qa.y, s[r]);
-                                s[r] = fmaf(kf[2], qa.z, s[r]); s[r] = fmaf(kf[3], qa.w, s[r]);
-                                s[r] = fmaf(kf[4], qb.x, s[r]); s[r] = fmaf(kf[5], qb.y, s[r]);
-                                s[r] = fmaf(kf[6], qb.z, s[r]); s[r] = fmaf(kf[7], qb.w, s[r]);
+                            for (int r = 0; r < RMAX; ++r) {
+                                if (r < R) {
+                                    const float4 qa = *reinterpret_cast<const float4*>(q_b + r * qw + c);
+                                    const float4 qb = *reinterpret_cast<const float4*>(q_b + r * qw + c + 4);
+                                    s[r] = fmaf(kf[0], qa.x, s[r]); s[r] = fmaf(kf[1], qa.y, s[r]);
+                                    s[r] = fmaf(kf[2], qa.z, s[r]); s[r] = fmaf(kf[3], qa.w, s[r]);
+                                    s[r] = fmaf(kf[4], qb.x, s[r]); s[r] = fmaf(kf[5], qb.y, s[r]);
+                                    s[r] = fmaf(kf[6], qb.z, s[r]); s[r] = fmaf(kf[7], qb.w, s[r]);
+                                }
                             }
                         }
                     }
@@ -225,7 +244,7 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
             for (int r = 0; r < RMAX; ++r) {
                 if (r < R) {
                     const int pos = pos0 + r / gq;
-                    const bool seen = valid && kidx <= pos && (W <= 0 || kidx > pos - W || kidx < KF);
+                    const bool seen = valid && kidx <= pos && (kidx >= lo_s[r] || kidx < KF);
                     float sc = s[r];
                     if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
                     if (a.dist_a != nullptr && seen) sc -= da_s[r] * logf(1.f + db_s[r] * (float)(pos - kidx));
@@ -266,7 +285,7 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
         // ---- phase 3: output dims dealt to threads ----
 #pragma unroll
         for (int i = 0; i < DPT; ++i) {
-            const int d = tid + i * TK;
+            const int d = d0 + tid + i * TK;
             if (d < hdv) {
 #pragma unroll
                 for (int r = 0; r < RMAX; ++r)
@@ -289,14 +308,17 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
         T* og = reinterpret_cast<T*>(a.out);
 #pragma unroll
         for (int i = 0; i < DPT; ++i) {
-            const int d = tid + i * TK;
+            const int d = d0 + tid + i * TK;
             if (d < hdv) {
 #pragma unroll
                 for (int r = 0; r < RMAX; ++r) {
                     if (r < R) {
                         const float l = l_s[r];
                         const int iq = r / gq, ih = r % gq;
-                        og[((size_t)(row0 + iq) * a.nh + head0 + ih) * hdv + d] = from_f32<T>(l > 0.f ? acc_o[r][i] / l : 0.f);
+                        const size_t row = (size_t)(row0 + iq) * a.nh + head0 + ih;
+                        float o = l > 0.f ? acc_o[r][i] / l : 0.f;
+                        if (a.out_gate != nullptr) o *= a.out_gate[row];
+                        og[row * hdv + d] = from_f32<T>(o);
                     }
                 }
             }
@@ -309,10 +331,10 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
                 const size_t prow = ((size_t)dec_index * a.nh + head0 + r) * nslices + slice;
 #pragma unroll
                 for (int i = 0; i < DPT; ++i) {
-                    const int d = tid + i * TK;
+                    const int d = d0 + tid + i * TK;
                     if (d < hdv) a.part_o[prow * hdv + d] = acc_o[r][i];
                 }
-                if (tid == 0) {
+                if (tid == 0 && blockIdx.z == 0) {
                     a.part_ml[prow * 2] = m_s[r];
                     a.part_ml[prow * 2 + 1] = l_s[r];
                 }
@@ -324,7 +346,8 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
 // merge the slices of sliced items: grid (decode tokens, heads)
 template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                  const int* __restrict__ dec_rows, T* __restrict__ out, int nh, int hd, int nslices) {
+                                  const int* __restrict__ dec_rows, T* __restrict__ out, int nh, int hd, int nslices,
+                                  const float* __restrict__ out_gate) {
     pdl_trigger();
     pdl_wait();
     const int n = blockIdx.x, h = blockIdx.y;
@@ -342,7 +365,9 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
             l += part_ml[(prow0 + s) * 2 + 1] * w;
             o += part_o[(prow0 + s) * hd + d] * w;
         }
-        out[((size_t)row * nh + h) * hd + d] = from_f32<T>(l > 0.f ? o / l : 0.f);
+        o = l > 0.f ? o / l : 0.f;
+        if (out_gate != nullptr) o *= out_gate[(size_t)row * nh + h];
+        out[((size_t)row * nh + h) * hd + d] = from_f32<T>(o);
     }
 }
 
@@ -351,7 +376,10 @@ int launch_attn(const AttnArgs& a, int n_items, cudaStream_t stream) {
     const int g = a.nh / a.nkv;
     const int gq_max = g < RMAX ? g : RMAX;
     const int hchunks = (g + gq_max - 1) / gq_max;
-    const size_t smem = ((size_t)RMAX * a.hd + (size_t)RMAX * TK + 5 * RMAX) * sizeof(float) + TK * sizeof(long long);
+    const size_t qw = a.wide ? (size_t)a.nkv * a.hd : (size_t)a.hd;
+    const int zblocks = (a.hd_v + VCB_MAX_HEAD_DIM - 1) / VCB_MAX_HEAD_DIM;
+    const size_t smem = ((size_t)RMAX * qw + (size_t)RMAX * TK + 6 * RMAX) * sizeof(float) + TK * sizeof(long long);
+    VCB_CHECK_ARG(smem <= 227 * 1024, "attn_paged: %d rows of %zu query lanes are more than a block's shared memory holds", RMAX, qw);
     auto kern = attn_paged_kernel<T, RMAX>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -360,7 +388,7 @@ int launch_attn(const AttnArgs& a, int n_items, cudaStream_t stream) {
             return -2;
         }
     }
-    kern<<<dim3(n_items, a.nkv * hchunks), TK, smem, stream>>>(a);
+    kern<<<dim3(n_items, a.nkv * hchunks, zblocks), TK, smem, stream>>>(a);
     VCB_CHECK_LAUNCH("attn_paged");
     return 0;
 }
@@ -369,18 +397,18 @@ int launch_attn(const AttnArgs& a, int n_items, cudaStream_t stream) {
 
 // rows_max: 8 for items of single decoded tokens (key range may be sliced), 32 for prompt portions
 // keep_first, dist_a / dist_b (float [nh] each, or null) and hd_v (0: as hd): the options named at the top of this file.
-// With them the key head size may be any number up to the largest; values likewise.
+// chunked, wide, out_gate: likewise.  With them the key head size may be any number; values likewise.
 VCB_API int vcb_attn_paged_ex(const void* q, void* out, int dtype, const void* pages, long long page_stride,
                               const int* block_table, const int* table_row, int max_blocks, const int* q_start, const int* q_len,
                               const int* ctx_len, const int* items, int n_items, int rows_max, float* part_o,
                               float* part_ml, int nh, int nkv, int hd, int page_size, int num_pages, int window,
                               float scale, int keep_first, const float* dist_a, const float* dist_b, int hd_v,
-                              float softcap, const float* slope, int sink, const float* sink_value, int* status, cudaStream_t stream) {
+                              float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
+                              const float* out_gate, int* status, cudaStream_t stream) {
     if (n_items == 0) return 0;
     if (hd_v <= 0) hd_v = hd;
     VCB_CHECK_ARG(nh > 0 && nkv > 0 && nh % nkv == 0, "attn_paged: %d query heads are not a multiple of %d KV heads", nh, nkv);
-    VCB_CHECK_ARG(hd >= 1 && hd <= VCB_MAX_HEAD_DIM && hd_v >= 1 && hd_v <= VCB_MAX_HEAD_DIM,
-                  "attn_paged: head sizes %d (keys) and %d (values) must lie in [1, %d]", hd, hd_v, VCB_MAX_HEAD_DIM);
+    VCB_CHECK_ARG(hd >= 1 && hd_v >= 1, "attn_paged: head sizes %d (keys) and %d (values)", hd, hd_v);
     VCB_CHECK_ARG(hd % 8 != 0 || (page_stride % 8 == 0 && ((long long)nkv * page_size * hd) % 8 == 0),
                   "attn_paged: pages whose keys do not start on 8 elements (stride %lld)", page_stride);
     VCB_CHECK_ARG(rows_max == 8 || rows_max == 32, "attn_paged: rows_max must be 8 or 32");
@@ -390,7 +418,7 @@ VCB_API int vcb_attn_paged_ex(const void* q, void* out, int dtype, const void* p
     VCB_CHECK_ARG(softcap >= 0.f, "attn_paged: a negative cap");
     AttnArgs a{q, out, pages, page_stride, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items, part_o, part_ml,
                nh, nkv, hd, page_size, num_pages, window, scale, status, 0, 0, keep_first, dist_a, dist_b, hd_v,
-               softcap, slope, sink, sink_value};
+               softcap, slope, sink, sink_value, chunked, wide, out_gate};
     if (dtype == VCB_F32) return rows_max == 8 ? launch_attn<float, 8>(a, n_items, stream) : launch_attn<float, 32>(a, n_items, stream);
     return rows_max == 8 ? launch_attn<__nv_bfloat16, 8>(a, n_items, stream) : launch_attn<__nv_bfloat16, 32>(a, n_items, stream);
 }
@@ -412,13 +440,13 @@ VCB_API int vcb_attn_paged(const void* q, void* out, int dtype, const void* page
 }
 
 VCB_API int vcb_attn_merge(const float* part_o, const float* part_ml, const int* dec_rows, void* out, int dtype,
-                           int n_dec, int nh, int hd, int nslices, cudaStream_t stream) {
+                           int n_dec, int nh, int hd, int nslices, const float* out_gate, cudaStream_t stream) {
     if (n_dec == 0) return 0;
     const int threads = hd <= 64 ? 64 : (hd <= 128 ? 128 : 256);
     if (dtype == VCB_F32)
-        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices);
+        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices, out_gate);
     else
-        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices);
+        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices, out_gate);
     VCB_CHECK_LAUNCH("attn_merge");
     return 0;
 }
@@ -502,9 +530,9 @@ VCB_API int vcb_attn_decode_no_alloc(const void* q, void* out, int dtype, const 
     if (rc) return rc;
     const int threads = hd <= 64 ? 64 : (hd <= 128 ? 128 : 256);
     if (dtype == VCB_F32)
-        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices);
+        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices, (const float*)nullptr);
     else
-        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices);
+        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices, (const float*)nullptr);
     VCB_CHECK_LAUNCH("attn_decode_no_alloc merge");
     return 0;
 }

@@ -18,6 +18,10 @@
 // Rows beyond the item's real rows and keys beyond the slice are zero-filled and
 // masked, never read from memory that is not theirs.
 //
+// Options: see AttnArgs.  With wide query rows (WIDE: a row has one block of HD lanes per KV head, see attention.cu) a
+// tile's keys come in as one stage per KV head, each meeting its block of the query rows, and their products add up in
+// the same accumulators; the values of the block's own KV head come with the last of them.
+//
 // Two loaders feed the same multiply code.  With pages of 8, 16, 32 or 64 tokens a fifth warp issues TMA
 // tile loads (cp.async.bulk.tensor with 128-byte swizzle, one box per page and 64 lanes of head_dim) into a
 // ring of three stages guarded by full/empty mbarriers, so the four multiplying warps spend no instructions
@@ -92,6 +96,8 @@ struct AttnArgs {
     const float* slope;
     int sink;
     const float* sink_value;    // with a sink: the silent key's score per head, not scaled (null: 0)
+    int chunked;                // the window stands still: the chunk of `window` positions that a query's position lies in
+    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, int src_bytes) {
@@ -158,12 +164,18 @@ __device__ __forceinline__ float2 ld_cluster_f2(const void* local, uint32_t rank
     return v;
 }
 
+// the first key a query at `pos` sees (kept first keys aside)
+__device__ __forceinline__ int first_key(int pos, int W, int chunked) {
+    if (W <= 0) return 0;
+    return max(0, chunked ? pos - pos % W : pos - W + 1);
+}
+
 // WR row groups x WK key groups multiplying warps, MR tiles of 16 rows each; TMA adds one warp that only issues
 // tile loads.
 // DEEP: a ring of six stages instead of three, for launches whose blocks have an SM each anyway (one or two requests
 // decoding): a short key slice is then all on its way before the block's wait is over, where a ring of three brought
 // the second half one memory latency after the first.
-template <int HD, int WR, int WK, int MR, bool TMA, bool DEEP = false>
+template <int HD, int WR, int WK, int MR, bool TMA, bool DEEP = false, bool WIDE = false>
 __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel(const __grid_constant__ CUtensorMap kv_map,
                                                                         AttnArgs a) {
     static_assert(HD % 64 == 0 && BN % (16 * WK) == 0, "layout");
@@ -184,8 +196,9 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     uint8_t* smem = smem_raw + (base_u32 - smem_u32(smem_raw));
     uint8_t* k_s = smem;                              // STAGES tiles
     uint8_t* v_s = k_s + STAGES * TILE_BYTES;         // STAGES tiles
-    uint8_t* q_s = v_s + STAGES * TILE_BYTES;         // RMAX rows
-    uint8_t* bar_s = q_s + RMAX * ROWB;               // 2 * STAGES mbarriers, then the abort flag
+    uint8_t* q_s = v_s + STAGES * TILE_BYTES;         // RMAX rows (WIDE: of every block)
+    const int NG = WIDE ? a.nkv : 1;                  // blocks of a query row = stages of a tile
+    uint8_t* bar_s = q_s + NG * RMAX * ROWB;          // 2 * STAGES mbarriers, then the abort flag
     auto full_bar = [&](int st) { return smem_u32(bar_s) + 8u * st; };
     auto empty_bar = [&](int st) { return smem_u32(bar_s) + 8u * (STAGES + st); };
     volatile int* abort_flag = reinterpret_cast<volatile int*>(bar_s + 16 * STAGES);
@@ -222,7 +235,7 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     const int pos_last = pos0 + nq - 1;
     const int W = a.window;
     const int ps = a.page_size;
-    const int lo = W > 0 ? max(0, pos0 - W + 1) : 0;
+    const int lo = first_key(pos0, W, a.chunked);
     const int hi = pos_last + 1;
     const int pb_lo = lo / ps, pb_hi = (hi + ps - 1) / ps;
     const int pps = (pb_hi - pb_lo + nslices - 1) / nslices;
@@ -236,6 +249,7 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     const int n_first = slice == 0 ? min(KF, lo) : 0;
     const int n_ft = (n_first + BN - 1) / BN;
     const int n_tiles = n_ft + n_own;
+    const int n_loads = n_tiles * NG;      // stages that come in: load i is tile i / NG's keys of KV head i % NG (WIDE)
     auto tile_t0 = [&](int it) { return it < n_ft ? it * BN : t_first + (it - n_ft) * BN; };
     auto tile_beg = [&](int it) { return it < n_ft ? 0 : k_begin; };
     auto tile_end = [&](int it) { return it < n_ft ? n_first : k_end; };
@@ -262,7 +276,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     const int first_pb_hi = (n_first + ps - 1) / ps;   // pages that hold the kept first keys read here
     auto tile_pb0 = [&](int it) { return it < n_ft ? it * pages_per_tile : my_pb_lo + (it - n_ft) * pages_per_tile; };
     auto tile_pb_hi = [&](int it) { return it < n_ft ? first_pb_hi : my_pb_hi; };
-    auto page_of = [&](int it) {
+    auto page_of = [&](int load) {
+        const int it = load / NG;
         const int pb = tile_pb0(it) + my_pg;
         return (it < n_tiles && my_pg < pages_per_tile && pb < tile_pb_hi(it)) ? bt[pb] : -1;
     };
@@ -277,28 +292,30 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
 #pragma unroll
     for (int k = 0; k < AHEAD; ++k) ahead_page[k] = -1;
     // asks for tile `it` once its stage is free (the producer warp, all lanes); false: give up
-    auto issue_tile = [&](int it) {
-        const int st = it % STAGES;
+    auto issue_tile = [&](int load) {
+        const int it = load / NG, st = load % STAGES;
+        const int key_head = WIDE ? load % NG : kvh;
+        const bool with_v = !WIDE || load % NG == NG - 1;
         bool ok = true;
-        if (lane == 0) ok = mbar_wait(empty_bar(st), ((it / STAGES) & 1) ^ 1u, abort_flag, a.status);
+        if (lane == 0) ok = mbar_wait(empty_bar(st), ((load / STAGES) & 1) ^ 1u, abort_flag, a.status);
         if (!__shfl_sync(0xffffffffu, ok, 0)) return false;
         const int pb0 = tile_pb0(it);
         const int np = min(pages_per_tile, tile_pb_hi(it) - pb0);
-        if (lane == 0) mbar_expect_tx(full_bar(st), (uint32_t)(np * ps * ROWB * 2));
+        if (lane == 0) mbar_expect_tx(full_bar(st), (uint32_t)(np * ps * ROWB * (with_v ? 2 : 1)));
         __syncwarp();
-        if (my_pg < np) {
+        if (my_pg < np && (with_v || !my_v)) {
             int page = ahead_page[0];
             if (page < 0 || page >= a.num_pages) {
                 atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                 page = 0;   // keep the byte count whole; the status word reports the fault
             }
-            const int group = (page * 2 * a.nkv + kvh) * groups_page + (my_v ? groups_kv : 0);
+            const int group = (page * 2 * a.nkv + (my_v ? kvh : key_head)) * groups_page + (my_v ? groups_kv : 0);
             const uint32_t dst = smem_u32((my_v ? v_s : k_s) + st * TILE_BYTES) + my_pg * ps * ROWB;
             tma_load_groups(dst, &kv_map, full_bar(st), group);
         }
 #pragma unroll
         for (int k = 0; k + 1 < AHEAD; ++k) ahead_page[k] = ahead_page[k + 1];
-        ahead_page[AHEAD - 1] = page_of(it + AHEAD);
+        ahead_page[AHEAD - 1] = page_of(load + AHEAD);
         return true;
     };
     int pre_tiles = 0;
@@ -312,8 +329,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
             const int first_new = ctx - qlen;
 #pragma unroll
             for (int k = 0; k < AHEAD; ++k) ahead_page[k] = page_of(k);
-            while (pre_tiles < n_tiles && pre_tiles < STAGES &&
-                   min(tile_pb_hi(pre_tiles), tile_pb0(pre_tiles) + pages_per_tile) * ps <= first_new) {
+            while (pre_tiles < n_loads && pre_tiles < STAGES &&
+                   min(tile_pb_hi(pre_tiles / NG), tile_pb0(pre_tiles / NG) + pages_per_tile) * ps <= first_new) {
                 if (!issue_tile(pre_tiles)) break;
                 ++pre_tiles;
             }
@@ -453,19 +470,23 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
         }
     } else {
         // ---- Q rows -> shared memory (rows beyond R are zero) ----
-        for (int idx = tid; idx < RMAX * CH; idx += blockDim.x) {
-            const int r = idx / CH, c = idx % CH;
+        const int QCH = NG * CH;
+        for (int idx = tid; idx < RMAX * QCH; idx += blockDim.x) {
+            const int r = idx / QCH, c = idx % QCH;
             uint4 v = make_uint4(0, 0, 0, 0);
             if (r < R) {
                 const int iq = r / gq, ih = r % gq;
-                v = *reinterpret_cast<const uint4*>(a.q + ((size_t)(row0 + iq) * a.nh + head0 + ih) * HD + c * 8);
+                v = *reinterpret_cast<const uint4*>(a.q + ((size_t)(row0 + iq) * a.nh + head0 + ih) * (NG * HD) + c * 8);
             }
-            *reinterpret_cast<uint4*>(q_s + swz<RMAX>(r, c)) = v;
+            *reinterpret_cast<uint4*>(q_s + (c / CH) * (RMAX * ROWB) + swz<RMAX>(r, c % CH)) = v;
         }
     }
 
     // ---- cp.async loader (all threads): 64 keys x HD of K and of V, gathered page by page ----
-    auto load_tile = [&](int stage, int t0, int t_end) {
+    auto load_tile = [&](int load) {
+        const int stage = load % STAGES, t0 = tile_t0(load / NG), t_end = tile_end(load / NG);
+        const int key_head = WIDE ? load % NG : kvh;
+        const bool with_v = !WIDE || load % NG == NG - 1;
         uint8_t* kd = k_s + stage * TILE_BYTES;
         uint8_t* vd = v_s + stage * TILE_BYTES;
 #pragma unroll
@@ -480,18 +501,18 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                 if (page < 0 || page >= a.num_pages) {
                     atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                 } else {
-                    src = a.pages + (size_t)page * a.page_stride + ((size_t)kvh * ps + kidx % ps) * HD + c * 8;
+                    src = a.pages + (size_t)page * a.page_stride + ((size_t)key_head * ps + kidx % ps) * HD + c * 8;
                     bytes = 16;
                 }
             }
             const int off = swz_kv<HD / 64>(j, c);
             cp_async16(smem_u32(kd + off), src, bytes);
-            cp_async16(smem_u32(vd + off), bytes ? src + (size_t)a.nkv * ps * HD : src, bytes);
+            if (with_v) cp_async16(smem_u32(vd + off), bytes ? src + ((size_t)a.nkv + kvh - key_head) * ps * HD : src, bytes);
         }
     };
 
     if (!TMA) {
-        if (n_tiles > 0) load_tile(0, tile_t0(0), tile_end(0));
+        if (n_tiles > 0) load_tile(0);
         cp_async_commit();
     }
     __syncthreads();   // Q and the barriers are in shared memory
@@ -499,9 +520,9 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     if (TMA && warp == NW) {
         // ---- TMA producer: the tiles after the ones asked for before the wait ----
         int armed = pre_tiles;
-        for (int it = pre_tiles; it < n_tiles; ++it) {
-            if (!issue_tile(it)) break;
-            armed = it + 1;
+        for (int load = pre_tiles; load < n_loads; ++load) {
+            if (!issue_tile(load)) break;
+            armed = load + 1;
         }
         if (lane == 0 && *abort_flag) {   // let copies in flight land before the block goes away
             for (int i = max(0, armed - STAGES); i < armed; ++i) {
@@ -513,7 +534,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
 
     float o[MR][ND][4];
     float m_run[MR][2], l_run[MR][2];   // rows lane/4 and lane/4 + 8 of each of this warp's 16-row tiles
-    int r_a[MR], pos_a[MR], pos_b[MR];
+    int r_a[MR], pos_a[MR], pos_b[MR], lo_a[MR], lo_b[MR];
+    const int lo_last = first_key(pos_last, W, a.chunked);
     bool ok_a[MR], ok_b[MR];
 #pragma unroll
     for (int mr = 0; mr < MR; ++mr) {
@@ -523,6 +545,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
         r_a[mr] = (wr * MR + mr) * 16 + (lane >> 2);
         pos_a[mr] = pos0 + r_a[mr] / gq;
         pos_b[mr] = pos0 + (r_a[mr] + 8) / gq;
+        lo_a[mr] = first_key(pos_a[mr], W, a.chunked);
+        lo_b[mr] = first_key(pos_b[mr], W, a.chunked);
         ok_a[mr] = r_a[mr] < R;
         ok_b[mr] = r_a[mr] + 8 < R;
         const bool scored = with_sink && a.sink_value != nullptr;
@@ -554,20 +578,23 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
 
     if (warp < NW) {
         // ---- one 16-row tile per warp: its Q fragments stay in registers; two: they are re-read per key tile ----
-        uint32_t qf[MR == 1 ? HD / 16 : 1][4];
-        if (MR == 1) {
+        uint32_t qf[MR == 1 && !WIDE ? HD / 16 : 1][4];
+        if (MR == 1 && !WIDE) {
 #pragma unroll
             for (int ks = 0; ks < HD / 16; ++ks)
-                ldmatrix_x4(qf[MR == 1 ? ks : 0], smem_u32(q_s + swz<RMAX>(wr * 16 + (lane & 15), ks * 2 + (lane >> 4))));
+                ldmatrix_x4(qf[MR == 1 && !WIDE ? ks : 0], smem_u32(q_s + swz<RMAX>(wr * 16 + (lane & 15), ks * 2 + (lane >> 4))));
         }
 
-        for (int it = 0; it < n_tiles; ++it) {
-            const int st = it % STAGES;
+        float s[MR][NS][4];
+        for (int load = 0; load < n_loads; ++load) {
+            const int it = load / NG, st = load % STAGES;
+            const int blk = load - it * NG;                   // (WIDE: the block of the query rows that meets these keys)
+            const bool scored = blk == NG - 1;                // the tile's scores are complete, its values are there
             const int t0 = tile_t0(it);
             const int kb = tile_beg(it), ke = tile_end(it);   // the keys of this tile that count
             if (TMA) {
-                if (!mbar_wait(full_bar(st), (it / STAGES) & 1, abort_flag, a.status)) break;
-                if (t0 + BN > ke) {
+                if (!mbar_wait(full_bar(st), (load / STAGES) & 1, abort_flag, a.status)) break;
+                if (scored && t0 + BN > ke) {
                     // the last page may hold slots beyond the sequence (and rows of pages not loaded are stale):
                     // their V must be finite, because a zero weight times NaN is NaN.  Each warp clears what it reads.
                     for (int idx = lane; idx < KW * CH; idx += 32) {
@@ -577,8 +604,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                     __syncwarp();
                 }
             } else {
-                if (it + 1 < n_tiles) {
-                    load_tile((it + 1) & 1, tile_t0(it + 1), tile_end(it + 1));
+                if (load + 1 < n_loads) {
+                    load_tile(load + 1);
                     cp_async_commit();
                     cp_async_wait<1>();
                 } else {
@@ -591,21 +618,22 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
             const int key0 = t0 + wk * KW;   // first key this warp multiplies
 
             // S = Q K^T
-            float s[MR][NS][4];
+            if (blk == 0) {
 #pragma unroll
-            for (int mr = 0; mr < MR; ++mr)
+                for (int mr = 0; mr < MR; ++mr)
 #pragma unroll
-                for (int i = 0; i < NS; ++i) s[mr][i][0] = s[mr][i][1] = s[mr][i][2] = s[mr][i][3] = 0.f;
+                    for (int i = 0; i < NS; ++i) s[mr][i][0] = s[mr][i][1] = s[mr][i][2] = s[mr][i][3] = 0.f;
+            }
 #pragma unroll
             for (int ks = 0; ks < HD / 16; ++ks) {
                 uint32_t qk[MR][4];
 #pragma unroll
                 for (int mr = 0; mr < MR; ++mr) {
-                    if (MR == 1) {
-                        qk[mr][0] = qf[MR == 1 ? ks : 0][0]; qk[mr][1] = qf[MR == 1 ? ks : 0][1];
-                        qk[mr][2] = qf[MR == 1 ? ks : 0][2]; qk[mr][3] = qf[MR == 1 ? ks : 0][3];
+                    if constexpr (MR == 1 && !WIDE) {
+                        qk[mr][0] = qf[ks][0]; qk[mr][1] = qf[ks][1];
+                        qk[mr][2] = qf[ks][2]; qk[mr][3] = qf[ks][3];
                     } else {
-                        ldmatrix_x4(qk[mr], smem_u32(q_s + swz<RMAX>((wr * MR + mr) * 16 + (lane & 15), ks * 2 + (lane >> 4))));
+                        ldmatrix_x4(qk[mr], smem_u32(q_s + blk * (RMAX * ROWB) + swz<RMAX>((wr * MR + mr) * 16 + (lane & 15), ks * 2 + (lane >> 4))));
                     }
                 }
 #pragma unroll
@@ -621,10 +649,19 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                     }
                 }
             }
+            if (WIDE && !scored) {       // further blocks of the rows to come before these scores are whole
+                if (TMA) {
+                    __syncwarp();
+                    if (lane == 0) mbar_arrive(empty_bar(st));
+                } else {
+                    __syncthreads();
+                }
+                continue;
+            }
             // mask (only where the tile touches an edge of some row's key range), running maximum
             // rows beyond R hold zero queries and are never written, so they need no mask of their own
             const bool inner = key0 >= kb && key0 + KW <= ke && key0 + KW - 1 <= pos0 &&
-                               (W <= 0 || key0 > pos_last - W || key0 + KW <= KF);
+                               (W <= 0 || key0 >= lo_last || key0 + KW <= KF);
             const bool penal = a.dist_a != nullptr;
             const int kq = key0 + 2 * (lane & 3);   // this thread's first key of the tile
             const bool all_inner = __all_sync(0xffffffffu, inner);
@@ -678,8 +715,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                         for (int c = 0; c < 2; ++c) {
                             const int kidx = key0 + i * 8 + 2 * (lane & 3) + c;
                             const bool in = kidx >= kb && kidx < ke;
-                            const bool sa = ok_a[mr] && in && kidx <= pos_a[mr] && (W <= 0 || kidx > pos_a[mr] - W || kidx < KF);
-                            const bool sb = ok_b[mr] && in && kidx <= pos_b[mr] && (W <= 0 || kidx > pos_b[mr] - W || kidx < KF);
+                            const bool sa = ok_a[mr] && in && kidx <= pos_a[mr] && (kidx >= lo_a[mr] || kidx < KF);
+                            const bool sb = ok_b[mr] && in && kidx <= pos_b[mr] && (kidx >= lo_b[mr] || kidx < KF);
                             float va = s[mr][i][c] * a.scale, vb = s[mr][i][2 + c] * a.scale;
                             if (penal) {
                                 const float k = (float)(i * 8 + c);
@@ -809,7 +846,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
         }
         const int iq = r / gq, ih = r % gq;
         if (nslices == 1) {
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            float inv = l > 0.f ? 1.f / l : 0.f;
+            if (a.out_gate != nullptr) inv *= a.out_gate[(size_t)(row0 + iq) * a.nh + head0 + ih];
             *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)(row0 + iq) * a.nh + head0 + ih) * HD + d) =
                 __floats2bfloat162_rn(o0 * inv, o1 * inv);
         } else if (in_cluster) {
@@ -857,7 +895,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                         o1 += ov[j].y * w;
                     }
                 }
-                const float inv = l > 0.f ? 1.f / l : 0.f;
+                float inv = l > 0.f ? 1.f / l : 0.f;
+                if (a.out_gate != nullptr) inv *= a.out_gate[(size_t)out_row * a.nh + head0 + ih];
                 *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)out_row * a.nh + head0 + ih) * HD + d) =
                     __floats2bfloat162_rn(o0 * inv, o1 * inv);
             }
@@ -935,7 +974,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                             }
                         }
                     }
-                    const float inv = l > 0.f ? 1.f / l : 0.f;
+                    float inv = l > 0.f ? 1.f / l : 0.f;
+                    if (a.out_gate != nullptr) inv *= a.out_gate[(size_t)out_row * a.nh + head0 + ih];
                     *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)out_row * a.nh + head0 + ih) * HD + d) =
                         __floats2bfloat162_rn(o0 * inv, o1 * inv);
                 }
@@ -1020,6 +1060,8 @@ bool kv_tensor_map(const void* pages, long long rows, int hd, int page_size, CUt
     return true;
 }
 
+constexpr size_t MAX_SMEM = 227 * 1024;   // shared memory of a block
+
 int sm_count() {
     static int n = 0;
     if (n == 0) {
@@ -1030,19 +1072,21 @@ int sm_count() {
     return n;
 }
 
-template <int HD, int WR, int WK, int MR, bool TMA, bool DEEP = false>
+template <int HD, int WR, int WK, int MR, bool TMA, bool DEEP = false, bool WIDE = false>
 int launch(const AttnArgs& a, int n_items, cudaStream_t stream) {
     constexpr int RMAX = 16 * WR * MR;
     constexpr int STAGES = (TMA && WK == 4) ? (DEEP ? 6 : 3) : 2;
     if constexpr (TMA && WK == 4 && !DEEP) {
-        // blocks that have an SM to themselves anyway take the deep ring
+        // blocks that have an SM to themselves anyway take the deep ring (if wide query rows leave room for it)
         const int g0 = a.nh / a.nkv, gq0 = g0 < RMAX ? g0 : RMAX;
-        if ((long long)n_items * a.nkv * ((g0 + gq0 - 1) / gq0) <= sm_count()) return launch<HD, WR, WK, MR, TMA, true>(a, n_items, stream);
+        const size_t deep = 2 * (size_t)6 * BN * HD * 2 + (WIDE ? (size_t)a.nkv : 1) * RMAX * HD * 2 + 16 * 6 + 16 + 1024;
+        if ((long long)n_items * a.nkv * ((g0 + gq0 - 1) / gq0) <= sm_count() && deep <= MAX_SMEM)
+            return launch<HD, WR, WK, MR, TMA, true, WIDE>(a, n_items, stream);
     }
     const int g = a.nh / a.nkv;
     const int gq_max = g < RMAX ? g : RMAX;
     const int hchunks = (g + gq_max - 1) / gq_max;
-    const size_t stages = 2 * (size_t)STAGES * BN * HD * 2 + (size_t)RMAX * HD * 2 + 16 * STAGES + 16;
+    const size_t stages = 2 * (size_t)STAGES * BN * HD * 2 + (WIDE ? (size_t)a.nkv : 1) * RMAX * HD * 2 + 16 * STAGES + 16;
     const size_t merge = ((size_t)WK * RMAX * HD + (size_t)WK * RMAX * 2 + (size_t)RMAX * HD + (size_t)RMAX * 2) * sizeof(float);
     const size_t smem = (stages > merge ? stages : merge) + 1024;   // + alignment slack
     CUtensorMap map;
@@ -1055,15 +1099,15 @@ int launch(const AttnArgs& a, int n_items, cudaStream_t stream) {
         }
         if (!kv_tensor_map(a.pages, rows, HD, a.page_size, &map, true)) return -3;
     }
-    auto kern = attn_mma_kernel<HD, WR, WK, MR, TMA, DEEP>;
-    static bool opted = false;
-    if (!opted) {
+    auto kern = attn_mma_kernel<HD, WR, WK, MR, TMA, DEEP, WIDE>;
+    static size_t opted = 0;
+    if (opted < smem) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) {
             vcb_set_error("attn_mma: %zu bytes of shared memory refused: %s", smem, cudaGetErrorString(e));
             return -2;
         }
-        opted = true;
+        opted = smem;
     }
     if (a.cluster > 1) {
         if (a.cluster > 8 || n_items % a.cluster != 0 || a.slice_counters == nullptr || a.dec_rows == nullptr) {
@@ -1076,6 +1120,19 @@ int launch(const AttnArgs& a, int n_items, cudaStream_t stream) {
     }
     VCB_CHECK_LAUNCH("attn_mma");
     return 0;
+}
+
+// rows of a prompt block whose query rows are wide: 128 where their blocks fit beside the stages, else 64; 0: neither
+int wide_rows(int hd, int nkv) {
+    const size_t fixed = (size_t)2 * 2 * BN * hd * 2 + 2048, per_row = (size_t)nkv * hd * 2;
+    return fixed + 128 * per_row <= MAX_SMEM ? 128 : (fixed + 64 * per_row <= MAX_SMEM ? 64 : 0);
+}
+
+template <int HD, bool TMA>
+int launch_wide(const AttnArgs& a, int n_items, int rows_max, cudaStream_t stream) {
+    if (rows_max == 16) return launch<HD, 1, 4, 1, TMA, false, true>(a, n_items, stream);
+    if (rows_max == 64) return launch<HD, 4, 1, 1, TMA, false, true>(a, n_items, stream);
+    return launch<HD, 8, 1, 1, TMA, false, true>(a, n_items, stream);
 }
 
 template <int HD, bool TMA>
@@ -1096,6 +1153,8 @@ bool vcb_kv_tensor_map(const void* pages, long long rows, int hd, int page_size,
 // rows_max: 16 (single decoded tokens; four warps split each tile's keys) or 128 (prompt portions; eight warps of
 // 16 rows each share the K and V tiles, enough independent MMA chains per SM to keep the tensor pipe fed).
 // Only bfloat16 and head_dim 64 or 128; the caller falls back to vcb_attn_paged otherwise.
+// Rows of a prompt block (rows_max) for query rows of one block per KV head; 0: not taken (the decode form then neither).
+VCB_API int vcb_attn_mma_wide_rows(int dtype, int hd, int nkv) { return dtype == VCB_BF16 && (hd == 64 || hd == 128) ? wide_rows(hd, nkv) : 0; }
 VCB_API int vcb_attn_mma_supported(int dtype, int hd) { return dtype == VCB_BF16 && (hd == 64 || hd == 128); }
 
 VCB_API int vcb_attn_mma_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
@@ -1103,7 +1162,8 @@ VCB_API int vcb_attn_mma_ex(const void* q, void* out, const void* pages, long lo
                             const int* ctx_len, const int* items, int n_items, int rows_max, float* part_o,
                             float* part_ml, int* slice_counters, const int* dec_rows, int nh, int nkv, int hd,
                             int page_size, int num_pages, int window, float scale, int keep_first, const float* dist_a,
-                            const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int* status, int allow_tma, int cluster, cudaStream_t stream);
+                            const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
+                            const float* out_gate, int* status, int allow_tma, int cluster, cudaStream_t stream);
 
 VCB_API int vcb_attn_mma(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                          const int* table_row, int max_blocks, const int* q_start, const int* q_len,
@@ -1113,28 +1173,32 @@ VCB_API int vcb_attn_mma(const void* q, void* out, const void* pages, long long 
                          int cluster, cudaStream_t stream) {
     return vcb_attn_mma_ex(q, out, pages, page_stride, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items,
                            n_items, rows_max, part_o, part_ml, slice_counters, dec_rows, nh, nkv, hd, page_size, num_pages,
-                           window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, status, allow_tma, cluster, stream);
+                           window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, 0, 0, nullptr, status, allow_tma, cluster, stream);
 }
 
-// keep_first, dist_a, dist_b, softcap, slope, sink: the options described with AttnArgs.
+// keep_first, dist_a, dist_b, softcap, slope, sink, chunked, wide, out_gate: the options described with AttnArgs.
 VCB_API int vcb_attn_mma_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                             const int* table_row, int max_blocks, const int* q_start, const int* q_len,
                             const int* ctx_len, const int* items, int n_items, int rows_max, float* part_o,
                             float* part_ml, int* slice_counters, const int* dec_rows, int nh, int nkv, int hd,
                             int page_size, int num_pages, int window, float scale, int keep_first, const float* dist_a,
-                            const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int* status, int allow_tma, int cluster, cudaStream_t stream) {
+                            const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
+                            const float* out_gate, int* status, int allow_tma, int cluster, cudaStream_t stream) {
     if (n_items == 0) return 0;
     VCB_CHECK_ARG(keep_first >= 0 && (dist_a == nullptr) == (dist_b == nullptr), "attn_mma: bad keep_first %d or half a distance penalty", keep_first);
     VCB_CHECK_ARG(nh > 0 && nkv > 0 && nh % nkv == 0, "attn_mma: %d query heads are not a multiple of %d KV heads", nh, nkv);
     VCB_CHECK_ARG(hd == 64 || hd == 128, "attn_mma: head_dim %d is not 64 or 128", hd);
-    VCB_CHECK_ARG(rows_max == 16 || rows_max == 128, "attn_mma: rows_max must be 16 or 128");
+    VCB_CHECK_ARG(rows_max == 16 || rows_max == 128 || (wide && rows_max == 64), "attn_mma: rows_max must be 16 or 128 (64: wide rows only)");
+    VCB_CHECK_ARG(!wide || wide_rows(hd, nkv) >= (rows_max == 16 ? 64 : rows_max), "attn_mma: %d rows of %d x %d lanes are more than a block holds", rows_max, nkv, hd);
     VCB_CHECK_ARG(page_size > 0 && window >= 0, "attn_mma: bad page_size %d or window %d", page_size, window);
     AttnArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)pages, page_stride, block_table,
                table_row, max_blocks, q_start, q_len, ctx_len, items, part_o, part_ml, slice_counters, dec_rows, nh, nkv,
-               page_size, num_pages, window, scale, status, FusedQkv{}, cluster, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value};
+               page_size, num_pages, window, scale, status, FusedQkv{}, cluster, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate};
     VCB_CHECK_ARG(softcap >= 0.f && (dist_a == nullptr || slope == nullptr), "attn_mma: a negative cap, or a logarithmic penalty and a slope at once");
     const bool tma = allow_tma && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64) &&
                      ((uintptr_t)pages % 16 == 0) && page_stride == (long long)2 * nkv * page_size * hd;
+    if (wide && hd == 64) return tma ? launch_wide<64, true>(a, n_items, rows_max, stream) : launch_wide<64, false>(a, n_items, rows_max, stream);
+    if (wide) return tma ? launch_wide<128, true>(a, n_items, rows_max, stream) : launch_wide<128, false>(a, n_items, rows_max, stream);
     if (hd == 64) return tma ? launch_rows<64, true>(a, n_items, rows_max, stream) : launch_rows<64, false>(a, n_items, rows_max, stream);
     return tma ? launch_rows<128, true>(a, n_items, rows_max, stream) : launch_rows<128, false>(a, n_items, rows_max, stream);
 }

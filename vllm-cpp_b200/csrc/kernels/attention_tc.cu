@@ -31,6 +31,12 @@
 // step from one group of 8 keys to the next by the same stride (halves x 1 KB) and from one half of head_dim to the
 // other by 1 KB, so the keys keep their order in a tile whatever the page size.  (One copy per page and half, the
 // obvious way, made the copying warp the slowest role of the block: about 100 clocks a copy, 16 copies a tile.)
+// Wide query rows (WIDE; a row has one block of head_dim lanes per KV head, see attention.cu): S is the sum over the KV
+// heads of block . that head's keys, one MMA chain over all of them into the same accumulator.  The rows' blocks stay in
+// shared memory for the whole unit (up to 512 lanes, 128 KB: one block an SM then), the K ring's stages hold one KV
+// head's keys each and are given back by the products themselves, and the rows of the next unit come in by cp.async
+// as soon as the last scores of this one are there, behind its last weights and output.
+//
 // All hand-offs are mbarriers; every wait is bounded by the clock, and a wait that runs out sets a bit in the
 // status word and an abort flag that the other roles see, after which the block frees its TMEM and returns.
 #include "common.cuh"
@@ -81,7 +87,18 @@ struct TcArgs {
     const float* slope;
     int sink;
     const float* sink_value;    // with a sink: the silent key's score per head, not scaled (null: 0)
+    int chunked;                // the window stands still: the chunk of `window` positions that a query's position lies in
+    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
 };
+
+// the first key a query at `pos` sees (kept first keys aside)
+template <bool OPT> __device__ __forceinline__ int first_key(const TcArgs& a, int pos) {
+    if (a.window <= 0) return 0;
+    return max(0, OPT && a.chunked ? pos - pos % a.window : pos - a.window + 1);
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, int src_bytes) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
+}
 
 // a box of whole groups of 8 tokens, all lanes: coordinates (lane 0, token 0, half 0, group)
 __device__ __forceinline__ void tma_load_groups(uint32_t dst, const CUtensorMap* map, uint32_t bar, int group) {
@@ -206,11 +223,12 @@ __device__ __forceinline__ int tile_pb0(const Unit& u, int it, int pages_per_til
 __device__ __forceinline__ int tile_pb_hi(const Unit& u, int it, int ps) { return it < u.n_ft ? (u.n_first + ps - 1) / ps : u.pb_hi; }
 constexpr int UNIT_INTS = sizeof(Unit) / sizeof(int);
 
-template <int HD, int KS, int VS>
+// MAXQ: blocks of HD lanes that a query row has room for (1, or with wide rows the most there may be: the tiles lie behind them)
+template <int HD, int KS, int VS, int MAXQ = 1>
 struct Layout {
     static constexpr int Q_BYTES = ROWS * HD * 2;
     static constexpr int KV_BYTES = BNK * HD * 2;       // one K or V tile
-    static constexpr int K_OFF = Q_BYTES;
+    static constexpr int K_OFF = MAXQ * Q_BYTES;
     static constexpr int V_OFF = K_OFF + KS * KV_BYTES;
     static constexpr int BAR_OFF = V_OFF + VS * KV_BYTES;
     static constexpr int NUM_BARS = 2 * KS + VS + 7;
@@ -218,12 +236,16 @@ struct Layout {
     static constexpr int TOTAL = BAR_OFF + NUM_BARS * 8 + 16 + 4 * UNIT_RING * (UNIT_INTS + 2);   // + TMEM address, abort flag, the units to come
     static constexpr uint32_t TMEM_COLS = 256;                  // S, S (64 each; P over the first half of its S), O (head_dim)
     static_assert(2 * BNK + HD <= 256, "TMEM columns");
-    static_assert(2 * (TOTAL + 1024) <= 228 * 1024, "two blocks per SM");
+    static_assert(MAXQ > 1 || 2 * (TOTAL + 1024) <= 228 * 1024, "two blocks per SM");
+    static_assert(TOTAL <= 227 * 1024, "shared memory of a block");
 };
 
 constexpr float RESCALE_STEP = 8.0f;   // log2 of how far a row's maximum may outgrow its reference
 
+constexpr int wide_blocks(int hd) { return 512 / hd; }   // blocks of a wide query row that stay in shared memory
+
 // false: the unit has nothing to do (an item laid out for a longer portion than is there)
+template <bool OPT>
 __device__ __forceinline__ bool read_unit(const TcArgs& a, int unit, Unit& u) {
     const int g = a.nh / a.nkv;
     const int gq_max = g < ROWS ? g : ROWS;
@@ -244,7 +266,7 @@ __device__ __forceinline__ bool read_unit(const TcArgs& a, int unit, Unit& u) {
     u.pos0 = ctx - qlen + q0;
     u.pos_last = u.pos0 + u.nq - 1;
     const int ps = a.page_size;
-    const int lo = a.window > 0 ? max(0, u.pos0 - a.window + 1) : 0;
+    const int lo = first_key<OPT>(a, u.pos0);
     u.k_end = u.pos_last + 1;
     u.pb_lo = lo / ps;
     u.pb_hi = (u.k_end + ps - 1) / ps;
@@ -270,9 +292,10 @@ __device__ __forceinline__ bool read_unit(const TcArgs& a, int unit, Unit& u) {
 // Barrier phases, ring stages and score buffers go on counting from unit to unit, so `t0` below is the number of
 // tiles of the units before.
 // OPT: built with the options of TcArgs (kept first keys, distance penalty); without, they cost nothing
-template <int HD, int KS, int VS, bool OPT>
-__global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_constant__ CUtensorMap kv_map, TcArgs a) {
-    using L = Layout<HD, KS, VS>;
+template <int HD, int KS, int VS, bool OPT, bool WIDE>
+__global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const __grid_constant__ CUtensorMap kv_map, TcArgs a) {
+    using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1>;
+    const int NG = WIDE ? a.nkv : 1;    // blocks of a query row = stages of a K tile
     constexpr int CH = HD / 8;          // 16-byte chunks per row of head_dim
     constexpr int ROWB = HD * 2;
     constexpr int HALVES = HD / 64;
@@ -378,7 +401,7 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
         tl.begin(VCB_TL_ATTN_TC, 0, lane == 0);
         Unit u;
         int unit = (int)blockIdx.x;
-        bool has = read_unit(a, unit, u);
+        bool has = read_unit<OPT>(a, unit, u);
         // this lane's page id for the first tile of the unit (see page_of below)
         auto first_page = [&](const Unit& w) {
             const int pb = tile_pb0(w, 0, pages_per_tile) + pl;
@@ -407,7 +430,7 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                         after = -1;
                         break;
                     }
-                    if (read_unit(a, after, un)) break;
+                    if (read_unit<OPT>(a, after, un)) break;
                     if (lane == 0) raw = atomicAdd(a.work, 1);
                 }
                 if (after >= 0) after_page = first_page(un);
@@ -435,10 +458,10 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                     const int pb = tile_pb0(u, it, pages_per_tile) + pl;
                     return (lane < 16 && it < u.n_tiles && pl < pages_per_tile && pb < tile_pb_hi(u, it, ps)) ? bt[pb] : -1;
                 };
-                // loads K tile itk and V tile itv of the unit (either may be -1: none) once their stages are free;
-                // false: give up
+                // loads stage itk of the unit's K tiles (tile itk / NG, with wide rows KV head itk % NG) and V tile itv
+                // (either may be -1: none) once their stages are free; false: give up
                 auto load_tiles = [&](int itk, int itv) {
-                    const int gk = t0 + itk, gv = t0 + itv;
+                    const int gk = t0 * NG + itk, gv = t0 + itv;
                     bool free = true;
                     tl.mark(TL_LOAD_ASKS, gv);
                     if (lane == 0) {
@@ -449,9 +472,10 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                     }
                     tl.mark(TL_LOAD_FREE, gv);
                     if (!__shfl_sync(0xffffffffu, free, 0)) return false;
-                    const int it = copies_v ? itv : itk;
+                    const int it = copies_v ? itv : (itk >= 0 ? itk / NG : -1);
+                    const int key_head = WIDE && itk >= 0 ? itk % NG : u.kvh;
                     const bool mine = lane < 16 && it >= 0;
-                    const int st = mine ? (t0 + it) % (copies_v ? VS : KS) : 0;
+                    const int st = mine ? (copies_v ? gv % VS : gk % KS) : 0;
                     const uint32_t fullb = copies_v ? v_full(st) : k_full(st);
                     const int np = mine ? min(pages_per_tile, tile_pb_hi(u, it, ps) - tile_pb0(u, it, pages_per_tile)) : 0;
                     if (mine && pl == 0) mbar_expect_tx(fullb, (uint32_t)(np * ps * ROWB));
@@ -462,22 +486,34 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                             atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                             page = 0;   // keep the byte count whole; the status word reports the fault
                         }
-                        const int group = (page * 2 * a.nkv + u.kvh) * groups_page + (copies_v ? groups_kv : 0);
+                        const int group = (page * 2 * a.nkv + (copies_v ? u.kvh : key_head)) * groups_page + (copies_v ? groups_kv : 0);
                         const uint32_t dst = base + (copies_v ? L::V_OFF : L::K_OFF) + st * L::KV_BYTES;
                         tma_load_groups(dst + pl * ps * ROWB, &kv_map, fullb, group);
                     }
                     tl.mark(TL_LOAD_SENT, gv);
-                    if (mine) next_page = page_of(it + 1);
+                    if (mine && (copies_v || !WIDE || key_head == NG - 1)) next_page = page_of(it + 1);
                     if (itk >= 0) armed[0] = gk + 1;
                     if (itv >= 0) armed[1] = gv + 1;
                     return true;
                 };
-                ok = load_tiles(0, -1);
-                if (ok && u.n_tiles > 1) ok = load_tiles(1, -1);
-                for (int it = 0; it < u.n_tiles && ok; ++it) {
-                    if (it == max(0, u.n_tiles - 4)) ask();
-                    if (it == max(0, u.n_tiles - 2)) make_known();
-                    ok = load_tiles(it + 2 < u.n_tiles ? it + 2 : -1, it);   // keys two tiles ahead of the values
+                if constexpr (WIDE) {
+                    // keys one tile ahead of the values: the products of a tile's stages take several times as long
+                    for (int b = 0; b < NG && ok; ++b) ok = load_tiles(b, -1);
+                    for (int it = 0; it < u.n_tiles && ok; ++it) {
+                        if (it == max(0, u.n_tiles - 4)) ask();
+                        if (it == max(0, u.n_tiles - 2)) make_known();
+                        if (it + 1 < u.n_tiles)
+                            for (int b = 0; b < NG && ok; ++b) ok = load_tiles((it + 1) * NG + b, -1);
+                        if (ok) ok = load_tiles(-1, it);
+                    }
+                } else {
+                    ok = load_tiles(0, -1);
+                    if (ok && u.n_tiles > 1) ok = load_tiles(1, -1);
+                    for (int it = 0; it < u.n_tiles && ok; ++it) {
+                        if (it == max(0, u.n_tiles - 4)) ask();
+                        if (it == max(0, u.n_tiles - 2)) make_known();
+                        ok = load_tiles(it + 2 < u.n_tiles ? it + 2 : -1, it);   // keys two tiles ahead of the values
+                    }
                 }
                 t0 += u.n_tiles;
             }
@@ -508,7 +544,7 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
             tl.begin(VCB_TL_ATTN_TC, 1, true);
             Unit u;
             int unit = (int)blockIdx.x;
-            bool has = read_unit(a, unit, u);
+            bool has = read_unit<OPT>(a, unit, u);
             for (int seq = 0; unit >= 0 && ok; unit = next_unit(seq, u), has = unit >= 0, ++seq) {
                 if (!has) continue;
                 // The rows have read the output of the unit before and written this unit's queries.
@@ -516,18 +552,22 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                 // S[j & 1] = Q . K_j^T once the tile has landed.  The buffer's last user was P . V of tile j - 2, issued
                 // before this by the same thread, and the tensor cores work through their queue in order.
                 auto issue_qk = [&](int j) {
-                    const int gj = t0 + j, st = gj % KS, b = gj & 1;
-                    tl.mark(TL_QK_ASKS, gj);
-                    if (!mbar_wait(k_full(st), (gj / KS) & 1, abort_flag, a.status)) return false;
-                    tl.mark(TL_QK_KEYS, gj);
-                    tc_fence_after();
-                    const uint32_t qa = base, ka = base + L::K_OFF + st * L::KV_BYTES;
+                    const int gj = t0 + j, b = gj & 1;
+                    for (int blk = 0; blk < NG; ++blk) {
+                        const int gk = gj * NG + blk, st = gk % KS;
+                        tl.mark(TL_QK_ASKS, gj);
+                        if (!mbar_wait(k_full(st), (gk / KS) & 1, abort_flag, a.status)) return false;
+                        tl.mark(TL_QK_KEYS, gj);
+                        tc_fence_after();
+                        const uint32_t qa = base + blk * L::Q_BYTES, ka = base + L::K_OFF + st * L::KV_BYTES;
 #pragma unroll
-                    for (int ks = 0; ks < HD / 16; ++ks) {
-                        // 16 lanes of head_dim = 32 bytes along the 128-byte rows; the second 64 lanes are the next block
-                        const uint64_t da = desc_k_major(qa + (ks / 4) * (ROWS * 128) + (ks % 4) * 32, 1024);
-                        const uint64_t db = desc_k_major(ka + (ks / 4) * 1024 + (ks % 4) * 32, HALVES * 1024);
-                        tc_mma(tmem_s + b * BNK, da, db, idesc_qk, ks > 0);
+                        for (int ks = 0; ks < HD / 16; ++ks) {
+                            // 16 lanes of head_dim = 32 bytes along the 128-byte rows; the second 64 lanes are the next block
+                            const uint64_t da = desc_k_major(qa + (ks / 4) * (ROWS * 128) + (ks % 4) * 32, 1024);
+                            const uint64_t db = desc_k_major(ka + (ks / 4) * 1024 + (ks % 4) * 32, HALVES * 1024);
+                            tc_mma(tmem_s + b * BNK, da, db, idesc_qk, (blk > 0 || ks > 0) ? 1u : 0u);
+                        }
+                        if constexpr (WIDE) tc_commit(k_empty(st));
                     }
                     tc_commit(s_full(b));   // the row that sees it first gives the K stage back (a commit less for this thread)
                     tl.mark(TL_QK_ISSUED, gj);
@@ -573,17 +613,33 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
         // This row's query of the unit to come is asked for before the row finishes the unit it is on (the loader
         // names the next unit two or three tiles early), so that the load's latency passes behind the last product
         // and the output of the old unit; it goes to shared memory when that is done.
-        uint4 qv[CH];
+        // Wide rows go straight to shared memory (cp.async, a warp's 32 rows by its lanes together): every product that
+        // reads the old ones is through when the last scores of a unit are there, which is before this is called.
+        uint4 qv[WIDE ? 1 : CH];
         auto ask_query = [&](const Unit& w, bool there) {   // writes all of qv in any case: what it held is dead
+            if constexpr (WIDE) {
+                if (!there) return;
+                const int per_row = NG * CH;
+                for (int rr = 0; rr < 32; ++rr) {
+                    const int row = qtr * 32 + rr;
+                    const bool mine = row < w.R;
+                    const int wq = mine ? row / w.gq : 0, wh = mine ? row % w.gq : 0;
+                    const __nv_bfloat16* src = a.q + ((size_t)(w.row0 + wq) * a.nh + w.head0 + wh) * (NG * HD);
+                    for (int c = lane; c < per_row; c += 32)
+                        cp_async16(base + (c / CH) * L::Q_BYTES + swz<ROWS>(row, c % CH), src + c * 8, mine ? 16 : 0);
+                }
+                asm volatile("cp.async.commit_group;" ::: "memory");
+                return;
+            }
             const bool mine = there && r < w.R;
             const int wq = mine ? r / w.gq : 0, wh = mine ? r % w.gq : 0;
             const __nv_bfloat16* src = a.q + (mine ? ((size_t)(w.row0 + wq) * a.nh + w.head0 + wh) * HD : 0);
 #pragma unroll
-            for (int c = 0; c < CH; ++c) qv[c] = mine ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
+            for (int c = 0; c < (WIDE ? 1 : CH); ++c) qv[c] = mine ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0, 0, 0, 0);
         };
         Unit u;
         int unit = (int)blockIdx.x, seq = 0;
-        bool has = read_unit(a, unit, u);
+        bool has = read_unit<OPT>(a, unit, u);
         ask_query(u, has);
         while (unit >= 0 && ok) {
             if (!has) {
@@ -595,7 +651,7 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
             const bool row_ok = r < u.R;
             const int iq = r / u.gq, ih = r % u.gq;
             const int pos_r = u.pos0 + iq;
-            const int lo_r = W > 0 ? max(0, pos_r - W + 1) : 0;
+            const int lo_r = first_key<OPT>(a, pos_r), lo_last = first_key<OPT>(a, u.pos_last);
             const int KF = OPT && W > 0 ? a.keep_first : 0;
             // the distance penalty of the row's head, in the base-2 domain the weights are computed in: a log2(1 + b d)
             const bool penal = OPT && a.dist_a != nullptr;
@@ -611,8 +667,12 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
             // The row's query -> shared memory (rows beyond R are zero).  The products of the unit before have all
             // been waited for (its last P . V, and with it everything issued earlier), so nothing reads the old rows.
             {
+                if constexpr (WIDE) {
+                    asm volatile("cp.async.wait_all;" ::: "memory");
+                } else {
 #pragma unroll
-                for (int c = 0; c < CH; ++c) *reinterpret_cast<uint4*>(gen + swz<ROWS>(r, c)) = qv[c];
+                    for (int c = 0; c < CH; ++c) *reinterpret_cast<uint4*>(gen + swz<ROWS>(r, c)) = qv[c];
+                }
                 fence_async_smem();
                 tc_fence_before();   // this row's reads of O for the unit before come before the products to follow
                 mbar_arrive(q_ready);
@@ -627,7 +687,7 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                 ok = mbar_wait(s_full(b), (gj >> 1) & 1, abort_flag, a.status);
                 if (!ok) break;
                 tl.mark(TL_ROW_SCORES, gj);
-                if (tid == 64) mbar_arrive(k_empty(gj % KS));   // the scores are there: the keys of this stage have been read
+                if (!WIDE && tid == 64) mbar_arrive(k_empty(gj % KS));   // the scores are there: the keys of this stage have been read
                 tc_fence_after();
                 uint32_t sv[4][16];
 #pragma unroll
@@ -638,7 +698,7 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
                 // Scores stay unscaled in sv; only tiles that touch a row's own position or the window's edge mask.
                 // (a tile of kept first keys: every row sees all of it that counts)
                 const bool plain_tile = OPT && j < u.n_ft ? k0 + BNK <= kend
-                                                   : (k0 >= u.lo && k0 + BNK - 1 <= u.pos0 && (W == 0 || k0 >= u.pos_last - W + 1 || k0 + BNK <= KF));   // uniform over the block
+                                                   : (k0 >= u.lo && k0 + BNK - 1 <= u.pos0 && (W == 0 || k0 >= lo_last || k0 + BNK <= KF));   // uniform over the block
                 float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
                 if (penal) {
                     // scaled scores less the penalty, times log2(e): one multiply-add, one logarithm, one multiply-add each
@@ -757,7 +817,8 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
 
             if (ok) {
                 tc_fence_after();
-                const float inv = l_end > 0.f ? 1.f / l_end : 0.f;
+                float inv = l_end > 0.f ? 1.f / l_end : 0.f;
+                if (OPT && a.out_gate != nullptr && row_ok) inv *= a.out_gate[(size_t)out_row * a.nh + out_head];
                 __nv_bfloat16* dst = a.out + ((size_t)out_row * a.nh + out_head) * HD;
 #pragma unroll
                 for (int c0 = 0; c0 < HD; c0 += 16) {   // 16 columns at a time: the query of the unit to come is in registers too
@@ -787,11 +848,11 @@ __global__ __launch_bounds__(NTHREADS, 2) void attn_tc_kernel(const __grid_const
     }
 }
 
-template <int HD, bool OPT>
+template <int HD, bool OPT, bool WIDE = false>
 int launch(const CUtensorMap& map, const TcArgs& a, int n_items, cudaStream_t stream) {
-    constexpr int KS = 3, VS = 2;
-    using L = Layout<HD, KS, VS>;
-    auto kern = attn_tc_kernel<HD, KS, VS, OPT>;
+    constexpr int KS = WIDE ? (HD == 64 ? 8 : 4) : 3, VS = 2;
+    using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1>;
+    auto kern = attn_tc_kernel<HD, KS, VS, OPT, WIDE>;
     static bool opted = false;
     if (!opted) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
@@ -801,14 +862,14 @@ int launch(const CUtensorMap& map, const TcArgs& a, int n_items, cudaStream_t st
         }
         opted = true;
     }
-    static int resident = 0;   // blocks that run at once: two an SM
+    static int resident = 0;   // blocks that run at once: two an SM, with wide rows one
     if (resident == 0) {
         int dev = 0, sms = 0;
         if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) {
             vcb_set_error("attn_tc: the device does not say how many SMs it has");
             return -2;
         }
-        resident = 2 * sms;
+        resident = (WIDE ? 1 : 2) * sms;
     }
     launch_pdl(kern, dim3((unsigned)(a.n_units < resident ? a.n_units : resident)), dim3(NTHREADS), (size_t)L::TOTAL, stream, map, a);
     VCB_CHECK_LAUNCH("attn_tc");
@@ -825,10 +886,16 @@ VCB_API int vcb_attn_tc_supported(int dtype, int hd, int page_size) {
            (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64);
 }
 
+// ... and for query rows of one block per KV head.
+VCB_API int vcb_attn_tc_wide_supported(int dtype, int hd, int page_size, int nkv) {
+    return vcb_attn_tc_supported(dtype, hd, page_size) && nkv <= wide_blocks(hd);
+}
+
 VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                            const int* table_row, int max_blocks, const int* q_start, const int* q_len, const int* ctx_len,
                            const int* items, int n_items, int nh, int nkv, int hd, int page_size, int num_pages, int window,
-                           float scale, int keep_first, const float* dist_a, const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int* status, int* work,
+                           float scale, int keep_first, const float* dist_a, const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
+                           const float* out_gate, int* status, int* work,
                            cudaStream_t stream);
 
 // Prompt portions only: every item has slice 0 of 1 and at most 128 rows (tokens x query heads per KV head).
@@ -839,13 +906,14 @@ VCB_API int vcb_attn_tc(const void* q, void* out, const void* pages, long long p
                         const int* items, int n_items, int nh, int nkv, int hd, int page_size, int num_pages, int window,
                         float scale, int* status, int* work, cudaStream_t stream) {
     return vcb_attn_tc_ex(q, out, pages, page_stride, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items, n_items,
-                          nh, nkv, hd, page_size, num_pages, window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, status, work, stream);
+                          nh, nkv, hd, page_size, num_pages, window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, 0, 0, nullptr, status, work, stream);
 }
 
 VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                            const int* table_row, int max_blocks, const int* q_start, const int* q_len, const int* ctx_len,
                            const int* items, int n_items, int nh, int nkv, int hd, int page_size, int num_pages, int window,
-                           float scale, int keep_first, const float* dist_a, const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int* status, int* work,
+                           float scale, int keep_first, const float* dist_a, const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
+                           const float* out_gate, int* status, int* work,
                            cudaStream_t stream) {
     if (n_items == 0) return 0;
     VCB_CHECK_ARG(keep_first >= 0 && (dist_a == nullptr) == (dist_b == nullptr), "attn_tc: bad keep_first %d or half a distance penalty", keep_first);
@@ -862,8 +930,10 @@ VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long lon
     const int g = nh / nkv;
     const int hchunks = (g + ROWS - 1) / ROWS;
     TcArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, block_table, table_row, max_blocks, q_start, q_len, ctx_len,
-             items, nh, nkv, page_size, num_pages, window, scale, status, n_items * nkv * hchunks, work, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value};
+             items, nh, nkv, page_size, num_pages, window, scale, status, n_items * nkv * hchunks, work, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate};
     VCB_CHECK_ARG(softcap >= 0.f && (dist_a == nullptr || slope == nullptr), "attn_tc: a negative cap, or a logarithmic penalty and a slope at once");
-    if (keep_first > 0 || dist_a != nullptr || softcap > 0.f || slope != nullptr || sink) return hd == 64 ? launch<64, true>(map, a, n_items, stream) : launch<128, true>(map, a, n_items, stream);
+    VCB_CHECK_ARG(!wide || nkv <= wide_blocks(hd), "attn_tc: wide query rows of %d x %d lanes (up to 512)", nkv, hd);
+    if (wide) return hd == 64 ? launch<64, true, true>(map, a, n_items, stream) : launch<128, true, true>(map, a, n_items, stream);
+    if (chunked || out_gate != nullptr || keep_first > 0 || dist_a != nullptr || softcap > 0.f || slope != nullptr || sink) return hd == 64 ? launch<64, true>(map, a, n_items, stream) : launch<128, true>(map, a, n_items, stream);
     return hd == 64 ? launch<64, false>(map, a, n_items, stream) : launch<128, false>(map, a, n_items, stream);
 }

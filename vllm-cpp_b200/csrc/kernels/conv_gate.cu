@@ -10,7 +10,7 @@
 //                        and key head divided by its root mean square, queries to a buffer, keys and values to
 //                        the tokens' cache slots
 //  * gated_norm_add      x_t += w * n(y_t * sigmoid(g_t + b)),  n(v) = v / sqrt(mean(v^2) + eps)
-//  * bias_act            act(u + b) for the feed-forward's hidden layer (erf or tanh GELU)
+//  * bias_act            act(u + b) for the feed-forward's hidden layer (erf or tanh GELU, SiLU, squared ReLU, tanh, xIELU)
 //
 // All arithmetic is 32-bit; inputs that are matrix products arrive as 32-bit sums, possibly as k-slice partial sums
 // [S, T, C] that are added here in slice order.  A step's rows belong to entries (q_start, q_len per entry, rows in
@@ -523,10 +523,16 @@ __global__ __launch_bounds__(1024) void gated_norm_add_vec_kernel(float* __restr
     }
 }
 
+// two branches with the slope 1/2 at zero: up z^2 + z/2 above it, down (e^z - 1 - z) + z/2 below
+__device__ __forceinline__ float xielu(float z, float up, float down) {
+    return z > 0.f ? fmaf(up * z, z, 0.5f * z) : fmaf(down, expm1f(z) - z, 0.5f * z);
+}
+
 template <typename TOUT>
-__global__ void bias_act_vec_kernel(RowsIn in, TOUT* __restrict__ out, int T, int C4, int kind) {
+__global__ void bias_act_vec_kernel(RowsIn in, TOUT* __restrict__ out, int T, int C4, int kind, const float* __restrict__ coef) {
     pdl_trigger();
     pdl_wait();
+    const float up = kind == 6 ? coef[0] : 0.f, down = kind == 6 ? coef[1] : 0.f;
     // a row a block in turn, four channels a thread: no division on the way to an address
     for (int t = blockIdx.y; t < T; t += gridDim.y)
     for (int c4 = blockIdx.x * blockDim.x + threadIdx.x; c4 < C4; c4 += gridDim.x * blockDim.x) {
@@ -540,13 +546,16 @@ __global__ void bias_act_vec_kernel(RowsIn in, TOUT* __restrict__ out, int T, in
             else if (kind == 1) f[k] = 0.5f * x * (1.f + tanhf(0.79788456080286535588f * (x + 0.044715f * x * x * x)));
             else if (kind == 2) f[k] = x / (1.f + expf(-x));
             else if (kind == 3) { const float r = fmaxf(x, 0.f); f[k] = r * r; }
+            else if (kind == 5) f[k] = tanhf(x);
+            else if (kind == 6) f[k] = xielu(x, up, down);
         }
         store4<TOUT>(out + (size_t)t * (4 * (size_t)C4) + c, z);
     }
 }
 
 template <typename TOUT>
-__global__ void bias_act_kernel(RowsIn in, TOUT* __restrict__ out, long long total, int C, int kind) {
+__global__ void bias_act_kernel(RowsIn in, TOUT* __restrict__ out, long long total, int C, int kind,
+                                const float* __restrict__ coef) {
     pdl_trigger();
     pdl_wait();
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
@@ -558,6 +567,8 @@ __global__ void bias_act_kernel(RowsIn in, TOUT* __restrict__ out, long long tot
         else if (kind == 1) r = 0.5f * z * (1.f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
         else if (kind == 2) r = z / (1.f + expf(-z));
         else if (kind == 3) { const float p = fmaxf(z, 0.f); r = p * p; }
+        else if (kind == 5) r = tanhf(z);
+        else if (kind == 6) r = xielu(z, coef[0], coef[1]);
         else r = z;
         out[i] = from_f32<TOUT>(r);
     }
@@ -714,24 +725,26 @@ VCB_API int vcb_gated_norm_add(float* resid, const float* y, int Sy, long long y
     return 0;
 }
 
-// kind 0: GELU with erf, 1: GELU with tanh, 2: SiLU, 3: the square of ReLU, 4: none (the sums, plus bias, in out_dtype)
+// kind 0: GELU with erf, 1: GELU with tanh, 2: SiLU, 3: the square of ReLU, 4: none (the sums, plus bias, in out_dtype),
+// 5: tanh, 6: xIELU with the two factors coef [2] on the device (of its parabola and of its exponential branch)
 VCB_API int vcb_bias_act(const float* in, int S, long long s_stride, long long ld, const float* bias, void* out, int out_dtype,
-                         int T, int C, int kind, cudaStream_t stream) {
+                         int T, int C, int kind, const float* coef, cudaStream_t stream) {
     if (T == 0 || C == 0) return 0;
-    VCB_CHECK_ARG(kind >= 0 && kind <= 4, "bias_act: unknown activation %d", kind);
+    VCB_CHECK_ARG(kind != 6 || coef != nullptr, "bias_act: the xIELU needs its two factors");
+    VCB_CHECK_ARG(kind >= 0 && kind <= 6, "bias_act: unknown activation %d", kind);
     RowsIn r{in, S < 1 ? 1 : S, s_stride, ld, bias};
     const long long total = (long long)T * C;
     if (C % 4 == 0 && rows_vec_ok(r) && (uintptr_t)out % 16 == 0) {
         const int bx = (C / 4 + 255) / 256 < 64 ? (C / 4 + 255) / 256 : 64;
         const dim3 grid4(bx, T < 65535 ? T : 65535);
-        if (out_dtype == VCB_F32) launch_pdl(bias_act_vec_kernel<float>, grid4, dim3(256), 0, stream, r, (float*)out, T, C / 4, kind);
-        else launch_pdl(bias_act_vec_kernel<__nv_bfloat16>, grid4, dim3(256), 0, stream, r, (__nv_bfloat16*)out, T, C / 4, kind);
+        if (out_dtype == VCB_F32) launch_pdl(bias_act_vec_kernel<float>, grid4, dim3(256), 0, stream, r, (float*)out, T, C / 4, kind, coef);
+        else launch_pdl(bias_act_vec_kernel<__nv_bfloat16>, grid4, dim3(256), 0, stream, r, (__nv_bfloat16*)out, T, C / 4, kind, coef);
         VCB_CHECK_LAUNCH("bias_act");
         return 0;
     }
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-    if (out_dtype == VCB_F32) launch_pdl(bias_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, r, (float*)out, total, C, kind);
-    else launch_pdl(bias_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, r, (__nv_bfloat16*)out, total, C, kind);
+    if (out_dtype == VCB_F32) launch_pdl(bias_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, r, (float*)out, total, C, kind, coef);
+    else launch_pdl(bias_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, r, (__nv_bfloat16*)out, total, C, kind, coef);
     VCB_CHECK_LAUNCH("bias_act");
     return 0;
 }

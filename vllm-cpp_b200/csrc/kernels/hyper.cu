@@ -187,10 +187,29 @@ __global__ void hyper_mix_norm_kernel(HyperArgs a) {
     for (int c = threadIdx.x; c < W; c += blockDim.x) o[c] = from_f32<TOUT>(u_s[c] * rstd * a.gain[c]);
 }
 
-template <typename TOUT>
-__global__ void token_shift_kernel(const float* __restrict__ h, const float* __restrict__ mu, float* __restrict__ state,
+// n_mix mixes of a row with the row before it, h + (h' - h) mu_m, each into a buffer of its own, from one reading of both
+// rows; V neighbouring channels a thread.
+template <typename TOUT, int V> __device__ __forceinline__ void store_mix(TOUT* p, const float (&x)[V]);
+template <> __device__ __forceinline__ void store_mix<float, 1>(float* p, const float (&x)[1]) { *p = x[0]; }
+template <> __device__ __forceinline__ void store_mix<__nv_bfloat16, 1>(__nv_bfloat16* p, const float (&x)[1]) { *p = __float2bfloat16_rn(x[0]); }
+template <> __device__ __forceinline__ void store_mix<float, 4>(float* p, const float (&x)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+}
+template <> __device__ __forceinline__ void store_mix<__nv_bfloat16, 4>(__nv_bfloat16* p, const float (&x)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(x[0], x[1]), b = __floats2bfloat162_rn(x[2], x[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <int V> __device__ __forceinline__ void load_row(const float* p, float (&x)[V]) {
+    if constexpr (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+    } else x[0] = *p;
+}
+
+template <typename TOUT, int V>
+__global__ void token_shift_kernel(const float* __restrict__ h, const float* __restrict__ mu, int n_mix, float* __restrict__ state,
                                    long long state_stride, const int* __restrict__ q_start, const int* __restrict__ q_len,
-                                   const int* __restrict__ slots, int E, int T, int W, TOUT* __restrict__ out) {
+                                   const int* __restrict__ slots, int E, int T, int W, TOUT* __restrict__ out, long long mix_stride) {
     pdl_trigger();
     pdl_wait();
     for (int t = blockIdx.y; t < T; t += gridDim.y) {
@@ -198,16 +217,24 @@ __global__ void token_shift_kernel(const float* __restrict__ h, const float* __r
         if (e < 0) continue;
         const int first = q_start[e], n = q_len[e];
         float* st = state + (size_t)slots[e] * state_stride;
-        for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < W; c += gridDim.x * blockDim.x) {
-            const float v = h[(size_t)t * W + c];
-            float prev;
+        for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * V; c < W; c += gridDim.x * blockDim.x * V) {
+            float v[V], prev[V];
+            load_row<V>(h + (size_t)t * W + c, v);
             if (t == first) {
-                prev = st[c];
-                st[c] = h[(size_t)(first + n - 1) * W + c];
+                load_row<V>(st + c, prev);
+                float last[V];
+                load_row<V>(h + (size_t)(first + n - 1) * W + c, last);
+                store_mix<float, V>(st + c, last);
             } else {
-                prev = h[(size_t)(t - 1) * W + c];
+                load_row<V>(h + (size_t)(t - 1) * W + c, prev);
             }
-            out[(size_t)t * W + c] = from_f32<TOUT>(fmaf(prev - v, mu[c], v));
+            for (int m = 0; m < n_mix; ++m) {
+                float w[V], x[V];
+                load_row<V>(mu + (size_t)m * W + c, w);
+#pragma unroll
+                for (int k = 0; k < V; ++k) x[k] = fmaf(prev[k] - v[k], w[k], v[k]);
+                store_mix<TOUT, V>(out + m * mix_stride + (size_t)t * W + c, x);
+            }
         }
     }
 }
@@ -240,17 +267,22 @@ VCB_API int vcb_hyper_mix_norm(float* streams, const float* init, const float* y
     return 0;
 }
 
-// h [T][W] 32-bit; mu [W]; state [slots][state_stride]: the last row every request's mixer input had; out [T][W].
-VCB_API int vcb_token_shift(const float* h, const float* mu, float* state, long long state_stride, const int* q_start,
-                            const int* q_len, const int* slots, int E, int T, int W, void* out, int out_dtype,
+// h [T][W] 32-bit; mu [n_mix][W]; state [slots][state_stride]: the last row every request's mixer input had; out: n_mix
+// buffers [T][W], mix_stride elements apart.
+VCB_API int vcb_token_shift(const float* h, const float* mu, int n_mix, float* state, long long state_stride, const int* q_start,
+                            const int* q_len, const int* slots, int E, int T, int W, void* out, int out_dtype, long long mix_stride,
                             cudaStream_t stream) {
-    if (T == 0 || E == 0) return 0;
-    const dim3 grid((W + 255) / 256, T < 65535 ? T : 65535);
-    if (out_dtype == VCB_F32)
-        launch_pdl(token_shift_kernel<float>, grid, dim3(256), 0, stream, h, mu, state, state_stride, q_start, q_len, slots, E, T, W, (float*)out);
-    else
-        launch_pdl(token_shift_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, h, mu, state, state_stride, q_start, q_len, slots, E, T,
-                   W, (__nv_bfloat16*)out);
+    if (T == 0 || E == 0 || n_mix == 0) return 0;
+    const uintptr_t bases = (uintptr_t)h | (uintptr_t)mu | (uintptr_t)state | (uintptr_t)out;
+    const bool vec = W % 4 == 0 && state_stride % 4 == 0 && mix_stride % 4 == 0 && bases % 16 == 0;
+    const int lanes = vec ? W / 4 : W;
+    const int threads = lanes >= 256 ? 256 : (lanes + 31) / 32 * 32;
+    const dim3 grid((lanes + threads - 1) / threads, T < 65535 ? T : 65535);
+#define VCB_SHIFT(TOUT, V) launch_pdl(token_shift_kernel<TOUT, V>, grid, dim3(threads), 0, stream, h, mu, n_mix, state, state_stride, q_start, \
+                                      q_len, slots, E, T, W, (TOUT*)out, mix_stride)
+    if (out_dtype == VCB_F32) { if (vec) VCB_SHIFT(float, 4); else VCB_SHIFT(float, 1); }
+    else { if (vec) VCB_SHIFT(__nv_bfloat16, 4); else VCB_SHIFT(__nv_bfloat16, 1); }
+#undef VCB_SHIFT
     VCB_CHECK_LAUNCH("token_shift");
     return 0;
 }

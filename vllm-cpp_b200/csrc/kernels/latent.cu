@@ -14,7 +14,8 @@
 //                             space, latent sums out to the heads' values)
 //  * rope_rows                the rotation alone, on a slice of every head of a 32-bit buffer (the queries' rotated part)
 //
-// Rotation pairs lane i with lane i + dims / 2; the angle is position * freq[i] in 32-bit, cos and sin times `gain`.
+// Without a query latent (q_rank 0: queries straight from the input) the first of them has only the latter two to do.
+// Rotation pairs lane i with lane i + dims / 2, or neighbouring lanes (`interleaved`); the angle is position * freq[i] in 32-bit, cos and sin times `gain`.
 // Norms, angles and all sums are 32-bit.
 #include "common.cuh"
 
@@ -48,6 +49,7 @@ struct LatentArgs {
     long long page_stride;
     int page_size, num_pages;
     int q_rank, kv_rank, rot, T;
+    int interleaved;        // lanes pair as neighbours
     int v_width;            // lanes of a value row: kv_rank, or more (the lanes behind the latent are zeros)
     int* status;
 };
@@ -67,9 +69,9 @@ __global__ void latent_norm_rope_store_kernel(LatentArgs a) {
         if (c < nq) sq = fmaf(v, v, sq);
         else if (c < nq + nk) sk = fmaf(v, v, sk);
     }
-    sq = block_sum(sq, red);
+    if (nq > 0) sq = block_sum(sq, red);
     sk = block_sum(sk, red);
-    const float rq = rsqrtf(sq / (float)nq + a.eps), rk = rsqrtf(sk / (float)nk + a.eps);
+    const float rq = nq > 0 ? rsqrtf(sq / (float)nq + a.eps) : 0.f, rk = rsqrtf(sk / (float)nk + a.eps);
     TC* cq = (TC*)a.cq_out + (size_t)t * nq;
     for (int c = threadIdx.x; c < nq; c += blockDim.x) cq[c] = from_f32<TC>(row[c] * rq * a.gq[c]);
     const int slot = a.slot_map[t];
@@ -97,9 +99,10 @@ __global__ void latent_norm_rope_store_kernel(LatentArgs a) {
         sincosf(pos * a.freq[i], &sn, &cs);
         sn *= a.gain;
         cs *= a.gain;
-        const float x = r[i], y = r[i + half];
-        krow[nk + i] = from_f32<TC>(x * cs - y * sn);
-        krow[nk + half + i] = from_f32<TC>(y * cs + x * sn);
+        const int la = a.interleaved ? 2 * i : i, lb = a.interleaved ? 2 * i + 1 : i + half;
+        const float x = r[la], y = r[lb];
+        krow[nk + la] = from_f32<TC>(x * cs - y * sn);
+        krow[nk + lb] = from_f32<TC>(y * cs + x * sn);
     }
     for (int i = 2 * half + threadIdx.x; i < nr; i += blockDim.x) krow[nk + i] = from_f32<TC>(r[i]);
 }
@@ -176,6 +179,7 @@ struct RopeArgs {
     int out_dtype;
     long long ld_out;
     int out_head_stride, out_off;
+    int interleaved;
     int T, H, dims, width;  // `width` lanes of the slice are copied, the first `dims` of them rotated
 };
 
@@ -195,9 +199,10 @@ __global__ void rope_rows_kernel(RopeArgs a) {
                 sincosf(pos * a.freq[k], &sn, &cs);
                 sn *= a.gain;
                 cs *= a.gain;
-                const float x = rows_at(a.in, t, ib + k), y = rows_at(a.in, t, ib + k + half);
-                store_from_f32(a.out, a.out_dtype, ob + k, x * cs - y * sn);
-                store_from_f32(a.out, a.out_dtype, ob + k + half, y * cs + x * sn);
+                const int la = a.interleaved ? 2 * k : k, lb = a.interleaved ? 2 * k + 1 : k + half;
+                const float x = rows_at(a.in, t, ib + la), y = rows_at(a.in, t, ib + lb);
+                store_from_f32(a.out, a.out_dtype, ob + la, x * cs - y * sn);
+                store_from_f32(a.out, a.out_dtype, ob + lb, y * cs + x * sn);
             } else {
                 const int c = 2 * half + (k - half);
                 store_from_f32(a.out, a.out_dtype, ob + c, rows_at(a.in, t, ib + c));
@@ -214,12 +219,12 @@ __global__ void rope_rows_kernel(RopeArgs a) {
 VCB_API int vcb_latent_norm_rope_store(const float* u, int S, long long s_stride, long long ld, const float* gq, const float* gkv,
                                        float eps, const int* positions, const float* freq, float gain, const int* slot_map,
                                        void* cq_out, void* pages, long long page_stride, int page_size, int num_pages, int q_rank,
-                                       int kv_rank, int rot, int v_width, int T, int dtype, int* status, cudaStream_t stream) {
+                                       int kv_rank, int rot, int interleaved, int v_width, int T, int dtype, int* status, cudaStream_t stream) {
     if (T == 0) return 0;
-    VCB_CHECK_ARG(q_rank > 0 && kv_rank > 0 && rot >= 0, "latent_norm_rope_store: bad sizes %d %d %d", q_rank, kv_rank, rot);
+    VCB_CHECK_ARG(q_rank >= 0 && kv_rank > 0 && rot >= 0, "latent_norm_rope_store: bad sizes %d %d %d", q_rank, kv_rank, rot);
     VCB_CHECK_ARG(v_width >= kv_rank && v_width <= kv_rank + rot, "latent_norm_rope_store: value rows of %d lanes", v_width);
     LatentArgs a{Rows{u, S < 1 ? 1 : S, s_stride, ld}, gq, gkv, eps, positions, freq, gain, slot_map, cq_out, pages, page_stride,
-                 page_size, num_pages, q_rank, kv_rank, rot, T, v_width, status};
+                 page_size, num_pages, q_rank, kv_rank, rot, T, interleaved, v_width, status};
     const size_t smem = (size_t)(q_rank + kv_rank + rot) * sizeof(float);
     VCB_CHECK_ARG(smem <= 48 * 1024, "latent_norm_rope_store: %d lanes are more than the kernel's shared memory holds", q_rank + kv_rank + rot);
     if (dtype == VCB_F32) launch_pdl(latent_norm_rope_store_kernel<float>, dim3(T), dim3(256), smem, stream, a);
@@ -304,11 +309,11 @@ VCB_API int vcb_head_linear(const void* in, int in_dtype, int S, long long s_str
 
 VCB_API int vcb_rope_rows(const float* in, int S, long long s_stride, long long ld, int in_head_stride, int in_off,
                           const int* positions, const float* freq, float gain, void* out, int out_dtype, long long ld_out,
-                          int out_head_stride, int out_off, int T, int H, int dims, int width, cudaStream_t stream) {
+                          int out_head_stride, int out_off, int T, int H, int dims, int width, int interleaved, cudaStream_t stream) {
     if (T == 0 || H == 0 || width == 0) return 0;
     VCB_CHECK_ARG(dims >= 0 && dims <= width, "rope_rows: %d rotated lanes of %d", dims, width);
     RopeArgs a{Rows{in, S < 1 ? 1 : S, s_stride, ld}, in_head_stride, in_off, positions, freq, gain, out, out_dtype, ld_out,
-               out_head_stride, out_off, T, H, dims, width};
+               out_head_stride, out_off, interleaved, T, H, dims, width};
     const int per_head = dims / 2 + (width - 2 * (dims / 2));
     const dim3 grid((H * per_head + 127) / 128, T < 65535 ? T : 65535);
     launch_pdl(rope_rows_kernel, grid, dim3(128), 0, stream, a);

@@ -11,7 +11,11 @@
 //  * retention               S <- decay_h S + k v^T;  o = S^T q
 //                            one fixed decay per head; the first `rot` lanes of q and k turned by position * freq[i]
 //                            (pairs in halves or interleaved), k then times d^(-1/2)
-//  * head_norm_gate          every head of o divided by its root mean square, times a gain shared by the heads, times
+//  * the wkv form            o = (S + diag(u) k v^T)^T q;  S <- diag(f) S + k v^T
+//                            q, k, v from one row of 32-bit sums each; f = exp(-exp(z + bias)) per state row, z the sums of a
+//                            second (low-rank) projection, in 32-bit; the token's own write is read out with the bonus u
+//                            alone: o = S^T q + (sum_i q_i u_i k_i) v, the bracket one number per token and head
+//  * head_norm_gate          every head of o divided by its root mean square, times a gain (shared by the heads, or of its own), times
 //                            silu(gate) where there is a gate
 //
 // One token after the other is the only order the recurrences allow.  A block owns (entry, head, a tile of value columns).
@@ -88,7 +92,9 @@ __device__ __forceinline__ uint64_t mul_pair(uint64_t x, uint64_t y) {
 }
 __device__ __forceinline__ void group_barrier(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
-enum { MODE_DELTA = 0, MODE_GATED = 1, MODE_DECAYED = 2, MODE_RETAIN = 3 };
+enum { MODE_DELTA = 0, MODE_GATED = 1, MODE_DECAYED = 2, MODE_RETAIN = 3, MODE_WKV = 4 };
+// the forms whose decay is a number per state row, staged beside q and k
+constexpr bool row_decay(int mode) { return mode == MODE_DECAYED || mode == MODE_WKV; }
 
 struct RnnArgs {
     Rows u;                 // the projection's sums
@@ -109,18 +115,19 @@ struct RnnArgs {
     float* out;             // [T][H * dv]
     int H, G, d, dv, L;     // G heads of q and k (MODE_DELTA; head h reads h / (H / G))
     int TB, dp_shift, ct_shift;     // tokens staged at a time; log2(L * R); log2(value columns a block owns)
-    Rows z;                 // MODE_DECAYED: the decay's sums [T][H * d]; f_bias is their bias
+    Rows z;                 // MODE_DECAYED, MODE_WKV: the decay's sums [T][H * d]; f_bias is their bias
     float inv_tau;          // MODE_DECAYED: 1 / tau
     const float* decay;     // MODE_RETAIN: [H]
     const int* ctx_len;     // MODE_RETAIN: an entry's tokens end at this position
     const float* freq;      // MODE_RETAIN: [rot / 2]
     int rot, interleaved;   // MODE_RETAIN: lanes of q and k that turn, and how they pair
+    const float* bonus;     // MODE_WKV: [H * d]
 };
 
 struct Stage {              // one half of the double buffer
     float* q;               // [TB][L * R]
     float* k;               // [TB][L * R]   (MODE_GATED: the forget gate)
-    float* f;               // [TB][L * R]   (MODE_DECAYED only: the decay of every state row)
+    float* f;               // [TB][L * R]   (MODE_DECAYED, MODE_WKV: the decay of every state row)
     float* v;               // [TB][CT]
     float* g;               // [TB]
     float* b;               // [TB]
@@ -163,22 +170,22 @@ __device__ __forceinline__ void stage_tokens(const RnnArgs& a, const Stage& s, i
         } else {
             qp = a.u.p + t_first * a.u.ld + a.q_col + h * d + i;
             kp = a.u.p + t_first * a.u.ld + a.k_col + h * d + i;
-            if (in) {
+            if (MODE == MODE_GATED && in) {
                 low = a.lower[h * d + i];
                 fb = a.f_bias[h * d + i];
             }
         }
-        if (MODE == MODE_DECAYED && in) fb = a.f_bias[h * d + i];
+        if (row_decay(MODE) && in) fb = a.f_bias[h * d + i];
         const float dscale = rsqrtf((float)d);
         const int ldq = MODE == MODE_DELTA ? ldx : ldu;
         for (int tb = tt0; tb < TB; tb += U * tpr) {
-            float qv[U], kv[U], fv[MODE == MODE_DECAYED ? U : 1];
+            float qv[U], kv[U], fv[row_decay(MODE) ? U : 1];
 #pragma unroll
             for (int w = 0; w < U; ++w) {
                 const int tt = tb + w * tpr;
                 qv[w] = 0.f;
                 kv[w] = 0.f;
-                if constexpr (MODE == MODE_DECAYED) fv[w] = 0.f;
+                if constexpr (row_decay(MODE)) fv[w] = 0.f;
                 if (in && tt < nb) {
                     if (MODE == MODE_DELTA || ONE) {
                         qv[w] = qp[tt * ldq];
@@ -187,7 +194,7 @@ __device__ __forceinline__ void stage_tokens(const RnnArgs& a, const Stage& s, i
                         qv[w] = rows_at(a.u, t_first + tt, a.q_col + h * d + i);
                         kv[w] = rows_at(a.u, t_first + tt, a.k_col + h * d + i);
                     }
-                    if constexpr (MODE == MODE_DECAYED) fv[w] = rows_at(a.z, t_first + tt, h * d + i);
+                    if constexpr (row_decay(MODE)) fv[w] = sums_at<ONE>(a.z, t_first + tt, h * d + i);
                 }
             }
 #pragma unroll
@@ -203,6 +210,7 @@ __device__ __forceinline__ void stage_tokens(const RnnArgs& a, const Stage& s, i
                         // sigmoid(x)^(1/tau) = exp(-softplus(-x) / tau); rows beyond d keep a zero state whatever they hold
                         s.f[tt * DPP + pi] = in && tt < nb ? expf(-softplus_f(-(fv[w] + fb)) * a.inv_tau) : 0.f;
                     }
+                    if constexpr (MODE == MODE_WKV) s.f[tt * DPP + pi] = in && tt < nb ? expf(-expf(fv[w] + fb)) : 0.f;
                     if (MODE == MODE_RETAIN && i >= a.rot) kv[w] *= dscale;     // (the turning lanes after their turn)
                     s.q[tt * DPP + pi] = qv[w];
                     s.k[tt * DPP + pi] = kv[w];
@@ -242,6 +250,20 @@ __device__ __forceinline__ void stage_tokens(const RnnArgs& a, const Stage& s, i
             }
         }
     }
+    if (MODE == MODE_WKV) {
+        group_barrier(1, STAGERS);
+        // the weight of a token's own write in its read-out (a warp a token)
+        const int lane = ltid & 31, warp = ltid >> 5;
+        const float* u = a.bonus + h * d;
+        for (int tt = warp; tt < nb; tt += STAGERS / 32) {
+            const float* q = s.q + tt * DPP;
+            const float* k = s.k + tt * DPP;
+            float sum = 0.f;
+            for (int i = lane; i < d; i += 32) sum = fmaf(q[i] * u[i], k[i], sum);
+            sum = warp_sum(sum);
+            if (lane == 0) s.b[tt] = sum;
+        }
+    }
     if (MODE == MODE_RETAIN && a.rot > 0) {
         group_barrier(1, STAGERS);
         // q and k turned by the token's position, a thread a pair of lanes; k then times d^(-1/2)
@@ -277,7 +299,7 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
     if (n <= 0) return;
     const int L = a.L, CT = 1 << a.ct_shift, DPP = L * R, TB = a.TB;
     const int d = a.d, dv = a.dv;
-    constexpr int NQK = MODE == MODE_DECAYED ? 3 : 2;
+    constexpr int NQK = row_decay(MODE) ? 3 : 2;
     const int half = NQK * TB * DPP + TB * CT + 2 * TB;       // (a multiple of four lanes)
     auto stage_at = [&](int which) {
         Stage s;
@@ -298,7 +320,7 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
     const int c0 = blockIdx.x * CT;
     const long long t0 = a.q_start[e];
     const int hk = MODE == MODE_DELTA ? h / (a.H / a.G) : h;
-    const bool one = a.u.S == 1 && (MODE != MODE_DECAYED || a.z.S == 1);
+    const bool one = a.u.S == 1 && (!row_decay(MODE) || a.z.S == 1);
     const int pos0 = MODE == MODE_RETAIN ? a.ctx_len[e] - n : 0;       // position of the entry's first token
     float* st = a.state + (size_t)a.slots[e] * a.state_stride + (size_t)h * d * dv;     // [dv][d]: a column's rows in a run
     // this thread's rows: the pieces of four 4 (kl + L m) .. + 3, m < R / 4, so that the L threads of a column read
@@ -374,7 +396,7 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
             };
             // a token's k (then q) is fetched as soon as the token before has used its own for the last time, so the
             // shared-memory reads run beside the arithmetic
-            uint64_t kr[R / 2], qr[R / 2], fr[MODE == MODE_DECAYED ? R / 2 : 1];
+            uint64_t kr[R / 2], qr[R / 2], fr[row_decay(MODE) ? R / 2 : 1];
             auto fetch = [&](uint64_t* dst, const ulonglong2* src, int tt_of) {
 #pragma unroll
                 for (int r = 0; r < R / 4; ++r) {
@@ -385,7 +407,7 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
             };
             fetch(kr, k4, 0);
             fetch(qr, q4, 0);
-            if constexpr (MODE == MODE_DECAYED) fetch(fr, f4, 0);
+            if constexpr (row_decay(MODE)) fetch(fr, f4, 0);
             const float head_decay = MODE == MODE_RETAIN ? a.decay[h] : 0.f;
             for (int tt = 0; tt < nb; ++tt) {
                 const int next = min(tt + 1, nb - 1);
@@ -395,7 +417,27 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
                 uint64_t o2[C];      // (sum over even rows, sum over odd rows)
 #pragma unroll
                 for (int c = 0; c < C; ++c) o2[c] = 0ull;
-                if constexpr (MODE == MODE_DELTA) {
+                float own[C];        // (MODE_WKV: the token's own write in its read-out, on the first of the L lanes)
+                if constexpr (MODE == MODE_WKV) {
+                    // the state as it was is read out, then it takes the token
+                    const float bonus = kl == 0 ? s.b[tt] : 0.f;
+                    uint64_t vv[C];
+#pragma unroll
+                    for (int c = 0; c < C; ++c) {
+                        own[c] = bonus * v[c];
+                        vv[c] = pair_f32(v[c], v[c]);
+                    }
+#pragma unroll
+                    for (int m = 0; m < R / 2; ++m) {
+#pragma unroll
+                        for (int c = 0; c < C; ++c) {
+                            o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
+                            S[c][m] = fma_pair(kr[m], vv[c], mul_pair(fr[row_decay(MODE) ? m : 0], S[c][m]));
+                        }
+                    }
+                    if (tt > 0) reduce(tt - 1, false, nullptr);
+                    fetch(fr, f4, next);
+                } else if constexpr (MODE == MODE_DELTA) {
                     const float g = s.g[tt], beta = s.b[tt];
                     const uint64_t gg = pair_f32(g, g);
                     uint64_t p2[C];
@@ -452,10 +494,12 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
                     if (tt > 0) reduce(tt - 1, false, nullptr);
                 }
                 fetch(kr, k4, next);
+                if constexpr (MODE != MODE_WKV) {
 #pragma unroll
-                for (int m = 0; m < R / 2; ++m) {
+                    for (int m = 0; m < R / 2; ++m) {
 #pragma unroll
-                    for (int c = 0; c < C; ++c) o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
+                        for (int c = 0; c < C; ++c) o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
+                    }
                 }
                 fetch(qr, q4, next);
 #pragma unroll
@@ -463,6 +507,7 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
                     float even, oddp;
                     unpair_f32(o2[c], even, oddp);
                     o_prev[c] = even + oddp;
+                    if constexpr (MODE == MODE_WKV) o_prev[c] += own[c];
                 }
             }
             reduce(nb - 1, false, nullptr);
@@ -507,7 +552,7 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
 
 // a warp a (token, head)
 template <typename TOUT>
-__global__ void head_norm_gate_kernel(const float* __restrict__ o, Rows gate, int gate_col, const float* __restrict__ w, float eps,
+__global__ void head_norm_gate_kernel(const float* __restrict__ o, Rows gate, int gate_col, const float* __restrict__ w, int w_stride, float eps,
                                       const int* __restrict__ q_start, const int* __restrict__ q_len, int E, int T, int H, int dv,
                                       TOUT* __restrict__ out) {
     pdl_trigger();
@@ -526,7 +571,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, Rows gate, in
     ss = warp_sum(ss);
     const float rstd = rsqrtf(ss / (float)dv + eps);
     for (int c = lane; c < dv; c += 32) {
-        float v = o[base + c] * rstd * (w != nullptr ? w[c] : 1.f);
+        float v = o[base + c] * rstd * (w != nullptr ? w[h * w_stride + c] : 1.f);
         if (gate.p != nullptr) v *= silu_f(rows_at(gate, t, gate_col + h * dv + c));
         out[base + c] = from_f32<TOUT>(v);
     }
@@ -555,8 +600,9 @@ int rnn_launch(RnnArgs a, bool split, dim3 grid, size_t smem, cudaStream_t strea
 
 }  // namespace
 
-// mode 0: the gated delta rule; 1: the gated linear form; 2: the decayed form; 3: retention (see the head of this file).
-// u [S][T][ld] the projection's sums; x [T][ldx] the convolved rows (mode 0); z [zS][T][zld] the decay's sums (mode 2).
+// mode 0: the gated delta rule; 1: the gated linear form; 2: the decayed form; 3: retention; 4: the wkv form (see the head of this file).
+// u [S][T][ld] the projection's sums; x [T][ldx] the convolved rows (mode 0); z [zS][T][zld] the decay's sums (modes 2 and 4).
+// The columns may lie in other row blocks of u's buffer (q, k and v as results of products of their own): they are offsets.
 // state [slots][H][dv][d] (a value column's d rows in a run).  out [rows][H * dv] 32-bit, rows >= the entries' tokens.
 // Entries of no tokens are left out.
 VCB_API int vcb_matrix_rnn(int mode, const float* u, int S, long long s_stride, long long ld, const float* x, long long ldx,
@@ -564,10 +610,11 @@ VCB_API int vcb_matrix_rnn(int mode, const float* u, int S, long long s_stride, 
                            const float* f_bias, const float* lower, float* state, long long state_stride, const int* q_start,
                            const int* q_len, const int* slots, int E, int rows, int H, int G, int d, int dv, float* out,
                            const float* z, int zS, long long z_stride, long long zld, float inv_tau, const float* decay,
-                           const int* ctx_len, const float* freq, int rot, int interleaved, cudaStream_t stream) {
+                           const int* ctx_len, const float* freq, int rot, int interleaved, const float* bonus, cudaStream_t stream) {
     if (E == 0) return 0;
-    VCB_CHECK_ARG(mode >= 0 && mode <= 3, "matrix_rnn: unknown mode %d", mode);
+    VCB_CHECK_ARG(mode >= 0 && mode <= 4, "matrix_rnn: unknown mode %d", mode);
     VCB_CHECK_ARG(mode != 2 || (z != nullptr && f_bias != nullptr), "matrix_rnn: the decayed form needs the decay's sums and bias");
+    VCB_CHECK_ARG(mode != 4 || (z != nullptr && f_bias != nullptr && bonus != nullptr), "matrix_rnn: the wkv form needs the decay's sums and bias and the bonus");
     VCB_CHECK_ARG(mode != 3 || (decay != nullptr && ctx_len != nullptr && rot >= 0 && rot <= d && rot % 2 == 0 && (rot == 0 || freq != nullptr)),
                   "matrix_rnn: retention needs a decay per head, the entries' positions and %d <= %d turning lanes with their frequencies", rot, d);
     VCB_CHECK_ARG(d >= 1 && d <= 512, "matrix_rnn: %d state rows a head (1 to 512)", d);
@@ -587,24 +634,25 @@ VCB_API int vcb_matrix_rnn(int mode, const float* u, int S, long long s_stride, 
     while ((1 << ct_shift) < CT) ++ct_shift;
     RnnArgs a{Rows{u, S < 1 ? 1 : S, s_stride, ld}, x, ldx, q_col, k_col, v_col, b_col, a_col, dt_bias, rate, f_bias, lower, state,
               state_stride, q_start, q_len, slots, out, H, G, d, dv, L, TB, dp_shift, ct_shift,
-              Rows{z, zS < 1 ? 1 : zS, z_stride, zld}, inv_tau, decay, ctx_len, freq, rot, interleaved};
-    const size_t smem = (size_t)(2 * ((mode == 2 ? 3 : 2) * TB * DP + TB * CT + 2 * TB) + TB * CT) * sizeof(float);
+              Rows{z, zS < 1 ? 1 : zS, z_stride, zld}, inv_tau, decay, ctx_len, freq, rot, interleaved, bonus};
+    const size_t smem = (size_t)(2 * ((row_decay(mode) ? 3 : 2) * TB * DP + TB * CT + 2 * TB) + TB * CT) * sizeof(float);
     const dim3 grid((dv + CT - 1) / CT, H, E);
     const bool split = rows > 4 * E;    // some entry has more than four tokens
     int rc;
 #define VCB_RNN_GO(MODE_, R_) (C == 1 ? rnn_launch<MODE_, R_, 1>(a, split, grid, smem, stream) : rnn_launch<MODE_, R_, 2>(a, split, grid, smem, stream))
-    if (R == 8) rc = mode == 0 ? VCB_RNN_GO(MODE_DELTA, 8) : mode == 1 ? VCB_RNN_GO(MODE_GATED, 8) : mode == 2 ? VCB_RNN_GO(MODE_DECAYED, 8) : VCB_RNN_GO(MODE_RETAIN, 8);
-    else rc = mode == 0 ? VCB_RNN_GO(MODE_DELTA, 16) : mode == 1 ? VCB_RNN_GO(MODE_GATED, 16) : mode == 2 ? VCB_RNN_GO(MODE_DECAYED, 16) : VCB_RNN_GO(MODE_RETAIN, 16);
+    if (R == 8) rc = mode == 0 ? VCB_RNN_GO(MODE_DELTA, 8) : mode == 1 ? VCB_RNN_GO(MODE_GATED, 8) : mode == 2 ? VCB_RNN_GO(MODE_DECAYED, 8) : mode == 3 ? VCB_RNN_GO(MODE_RETAIN, 8) : VCB_RNN_GO(MODE_WKV, 8);
+    else rc = mode == 0 ? VCB_RNN_GO(MODE_DELTA, 16) : mode == 1 ? VCB_RNN_GO(MODE_GATED, 16) : mode == 2 ? VCB_RNN_GO(MODE_DECAYED, 16) : mode == 3 ? VCB_RNN_GO(MODE_RETAIN, 16) : VCB_RNN_GO(MODE_WKV, 16);
 #undef VCB_RNN_GO
     if (rc != 0) return rc;
     VCB_CHECK_LAUNCH("matrix_rnn");
     return 0;
 }
 
-// o [T][H * dv] 32-bit; gate (or null) [S][T][ld] sums whose columns gate_col .. gate_col + H dv gate o through a SiLU; w [dv];
+// o [T][H * dv] 32-bit; gate (or null) [S][T][ld] sums whose columns gate_col .. gate_col + H dv gate o through a SiLU; w: a gain of
+// dv lanes per head, w_stride apart (0: one for all heads), or null;
 // out [T][H * dv] of out_dtype (zeros in rows outside every entry).
 VCB_API int vcb_head_norm_gate(const float* o, const float* gate, int S, long long s_stride, long long ld, int gate_col,
-                               const float* w, float eps, const int* q_start, const int* q_len, int E, int T, int H, int dv,
+                               const float* w, int w_stride, float eps, const int* q_start, const int* q_len, int E, int T, int H, int dv,
                                void* out, int out_dtype, cudaStream_t stream) {
     if (T == 0 || H == 0) return 0;
     const long long items = (long long)T * H;
@@ -612,9 +660,9 @@ VCB_API int vcb_head_norm_gate(const float* o, const float* gate, int S, long lo
     const dim3 grid((unsigned)((items + warps - 1) / warps));
     Rows g{gate, S < 1 ? 1 : S, s_stride, ld};
     if (out_dtype == VCB_F32)
-        launch_pdl(head_norm_gate_kernel<float>, grid, dim3(32 * warps), 0, stream, o, g, gate_col, w, eps, q_start, q_len, E, T, H, dv, (float*)out);
+        launch_pdl(head_norm_gate_kernel<float>, grid, dim3(32 * warps), 0, stream, o, g, gate_col, w, w_stride, eps, q_start, q_len, E, T, H, dv, (float*)out);
     else
-        launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, grid, dim3(32 * warps), 0, stream, o, g, gate_col, w, eps, q_start, q_len, E, T, H,
+        launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, grid, dim3(32 * warps), 0, stream, o, g, gate_col, w, w_stride, eps, q_start, q_len, E, T, H,
                    dv, (__nv_bfloat16*)out);
     VCB_CHECK_LAUNCH("head_norm_gate");
     return 0;

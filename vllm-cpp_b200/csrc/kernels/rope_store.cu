@@ -6,7 +6,15 @@
 //                     key lanes likewise; the first `rot` lanes of every q and k head turned by position * freq[i], lanes
 //                     paired in halves (i, i + rot/2) or interleaved (2i, 2i+1); optionally every value head turned the
 //                     same way over `vrot` of its lanes with frequencies of its own; queries to a buffer, keys and values
-//                     to the token's place in the paged cache.
+//                     to the token's place in the paged cache.  Further options: a bias on every lane before all else;
+//                     every value head divided by its root mean square; columns behind the projection that are one
+//                     gate per query head (their sigmoids go to a buffer for the attention kernels' epilogues); and
+//                     queries mixed across heads on their way out, see below.
+//
+// Mixed queries: where the scores of the heads are mixed before the softmax, score_h <- sum_g T[h][g] (q_g . k_kv(g)), the sum
+// over g can be drawn into the queries: with q'_h[G] = sum over the heads g that read KV head G of T[h][g] q_g,
+// score_h = sum_G q'_h[G] . k_G.  So a query row of head h becomes nkv * hd lanes, one block per KV head, and the attention
+// kernels (whose option for such wide rows adds up the blocks' products) need no other head's scores.
 //  * rotate_heads     every head of a buffer turned in place by sign * position * freq[i] (the heads' weighted sums of
 //                     rotated values turned back by the query's position).
 //
@@ -47,6 +55,10 @@ struct StoreArgs {
     int interleaved;        // pairing of the rotated lanes
     int v_from_k;           // values are the key lanes as projected (before norm and rotation); vd == hd
     int* status;
+    const float* bias;      // [nh hd + nkv hd (+ nkv vd)] or null
+    int unit_v;             // every value head divided by its root mean square (eps inside the root)
+    const float* talk;      // [nh][nh] or null: queries mixed across heads, q_out is [T][nh][nkv * hd]
+    float* gate_out;        // [T][nh] or null: sigmoid of the nh columns behind the projection's
 };
 
 // lanes (a, b) of pair k of a head whose first `dims` lanes turn; b < 0: lane a passes unchanged
@@ -61,6 +73,12 @@ __device__ __forceinline__ void pair_lanes(int k, int dims, int interleaved, int
     }
 }
 
+template <typename TC> __device__ __forceinline__ void store_pair(TC* p, float x, float y);
+template <> __device__ __forceinline__ void store_pair<float>(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
+template <> __device__ __forceinline__ void store_pair<__nv_bfloat16>(__nv_bfloat16* p, float x, float y) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x, y);
+}
+
 template <typename TC>
 __global__ void qkv_rope_store_kernel(StoreArgs a) {
     extern __shared__ __align__(16) float sm[];
@@ -73,6 +91,8 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
     float* row = sm;                    // [n]
     float* cs = sm + n;                 // [rot]: cosines, then sines
     float* vcs = cs + a.rot;            // [vrot]
+    float* vscale = vcs + a.vrot;       // [nkv] with unit values
+    float* talk = vscale + (a.unit_v ? a.nkv : 0);      // [nh][nh] with mixed queries
     const float pos = (float)a.positions[t];
     const int half = a.rot >> 1, vhalf = a.vrot >> 1;
     for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
@@ -80,11 +100,17 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         for (int i = threadIdx.x; i < vhalf; i += blockDim.x) sincosf(pos * a.vfreq[i], &vcs[vhalf + i], &vcs[i]);
     float sq = 0.f, sk = 0.f;
     for (int c = threadIdx.x; c < n; c += blockDim.x) {
-        const float v = rows_at(a.qkv, t, c);
+        float v = rows_at(a.qkv, t, c);
+        if (a.bias != nullptr) v += a.bias[c];
         row[c] = v;
         if (c < nq) sq = fmaf(v, v, sq);
         else if (c < nq + nk) sk = fmaf(v, v, sk);
     }
+    if (a.gate_out != nullptr)
+        for (int h = threadIdx.x; h < a.nh; h += blockDim.x)
+            a.gate_out[(size_t)t * a.nh + h] = 1.f / (1.f + expf(-rows_at(a.qkv, t, n + h)));
+    if (a.talk != nullptr)
+        for (int i = threadIdx.x; i < a.nh * a.nh; i += blockDim.x) talk[i] = a.talk[i];
     float rq = 1.f, rk = 1.f;
     if (a.q_gain != nullptr) {
         sq = block_sum(sq, red);
@@ -92,10 +118,66 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         rq = 1.0f / sqrtf(sq / (float)nq + a.eps);
         rk = 1.0f / sqrtf(sk / (float)nk + a.eps);
     } else __syncthreads();
+    if (a.unit_v) {
+        // a warp a value head; the factors are read behind the next barrier
+        const int lane = threadIdx.x & 31;
+        for (int g = threadIdx.x >> 5; g < a.nkv; g += blockDim.x >> 5) {
+            const float* v = row + (a.v_from_k ? nq + g * a.hd : nq + nk + g * a.vd);
+            float ss = 0.f;
+            for (int c = lane; c < a.vd; c += 32) ss = fmaf(v[c], v[c], ss);
+            ss = warp_sum(ss);
+            if (lane == 0) vscale[g] = 1.0f / sqrtf(ss / (float)a.vd + a.eps);
+        }
+    }
+    const int per_q = half + (a.hd - 2 * half);
+    if (a.talk != nullptr) {
+        // the queries turned in place, then mixed: 4 heads and two neighbouring lanes of one KV head's block a thread
+        for (int i = threadIdx.x; i < a.nh * half; i += blockDim.x) {
+            const int k = i % half;
+            float* p = row + (i / half) * a.hd;
+            int la, lb;
+            pair_lanes(k, a.rot, a.interleaved, la, lb);
+            const float x = p[la], y = p[lb], c = cs[k], s = cs[half + k];
+            p[la] = x * c - y * s;
+            p[lb] = y * c + x * s;
+        }
+        __syncthreads();
+        const int gs = a.nh / a.nkv, wide = a.nkv * a.hd, pairs = (a.hd + 1) / 2;
+        const bool even = (a.hd & 1) == 0;
+        TC* wq = (TC*)a.q_out + (size_t)t * a.nh * wide;
+        const int hb = (a.nh + 3) / 4;
+        for (int i = threadIdx.x; i < hb * a.nkv * pairs; i += blockDim.x) {
+            const int d = 2 * (i % pairs), G = (i / pairs) % a.nkv, h0 = 4 * (i / (pairs * a.nkv));
+            const bool two = even || d + 1 < a.hd;
+            const float* src = row + (size_t)G * gs * a.hd + d;
+            float acc[4][2];
+#pragma unroll
+            for (int m = 0; m < 4; ++m) acc[m][0] = acc[m][1] = 0.f;
+            for (int g = 0; g < gs; ++g) {
+                const float x = src[g * a.hd], y = two ? src[g * a.hd + 1] : 0.f;
+#pragma unroll
+                for (int m = 0; m < 4; ++m) {
+                    const float w = h0 + m < a.nh ? talk[(h0 + m) * a.nh + G * gs + g] : 0.f;
+                    acc[m][0] = fmaf(w, x, acc[m][0]);
+                    acc[m][1] = fmaf(w, y, acc[m][1]);
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < 4; ++m) {
+                if (h0 + m < a.nh) {
+                    TC* dst = wq + (size_t)(h0 + m) * wide + G * a.hd + d;
+                    if (even) store_pair<TC>(dst, acc[m][0], acc[m][1]);
+                    else {
+                        dst[0] = from_f32<TC>(acc[m][0]);
+                        if (two) dst[1] = from_f32<TC>(acc[m][1]);
+                    }
+                }
+            }
+        }
+    } else if (a.unit_v) __syncthreads();
     // queries
     TC* q_out = (TC*)a.q_out + (size_t)t * nq;
-    const int per_q = half + (a.hd - 2 * half);
-    for (int i = threadIdx.x; i < a.nh * per_q; i += blockDim.x) {
+    for (int i = threadIdx.x; a.talk == nullptr && i < a.nh * per_q; i += blockDim.x) {
         const int h = i / per_q, base = h * a.hd;
         int la, lb;
         pair_lanes(i % per_q, a.rot, a.interleaved, la, lb);
@@ -140,10 +222,11 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         TC* dst = vp + ((size_t)g * a.page_size + off) * a.vd;
         int la, lb;
         pair_lanes(i % per_v, vr, a.interleaved, la, lb);
-        const float x = row[base + la];
+        const float vs = a.unit_v ? vscale[g] : 1.f;
+        const float x = row[base + la] * vs;
         if (lb < 0) dst[la] = from_f32<TC>(x);
         else {
-            const float y = row[base + lb];
+            const float y = row[base + lb] * vs;
             const float c = vcs[i % per_v], s = vcs[vhalf + i % per_v];
             dst[la] = from_f32<TC>(x * c - y * s);
             dst[lb] = from_f32<TC>(y * c + x * s);
@@ -176,11 +259,12 @@ __global__ void rotate_heads_kernel(TC* x, const int* __restrict__ positions, co
 }  // namespace
 
 // qkv [S][T][ld] 32-bit sums; q_out [T][nh hd] and the pages of `dtype`; vfreq null: values stored unturned.
+// bias, talk (q_out then [T][nh][nkv hd]), gate_out (or null each) and unit_v: the options of StoreArgs.
 VCB_API int vcb_qkv_rope_store(const float* qkv, int S, long long s_stride, long long ld, const float* q_gain, const float* k_gain,
                                float eps, const int* positions, const float* freq, const float* vfreq, const int* slot_map,
                                void* q_out, void* pages, long long page_stride, int page_size, int num_pages, int nh, int nkv,
                                int hd, int vd, int rot, int vrot, int interleaved, int v_from_k, int T, int dtype, int* status,
-                               cudaStream_t stream) {
+                               const float* bias, int unit_v, const float* talk, float* gate_out, cudaStream_t stream) {
     if (T == 0) return 0;
     VCB_CHECK_ARG(nh > 0 && nkv > 0 && hd > 0 && vd > 0, "qkv_rope_store: bad sizes %d %d %d %d", nh, nkv, hd, vd);
     VCB_CHECK_ARG(rot >= 0 && rot <= hd && rot % 2 == 0, "qkv_rope_store: %d turning lanes of %d", rot, hd);
@@ -189,8 +273,11 @@ VCB_API int vcb_qkv_rope_store(const float* qkv, int S, long long s_stride, long
     VCB_CHECK_ARG((q_gain == nullptr) == (k_gain == nullptr), "qkv_rope_store: one gain without the other");
     VCB_CHECK_ARG(rot == 0 || freq != nullptr, "qkv_rope_store: no frequencies");
     StoreArgs a{Rows{qkv, S < 1 ? 1 : S, s_stride, ld}, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q_out, pages, page_stride,
-                page_size, num_pages, nh, nkv, hd, vd, rot, vfreq ? vrot : 0, interleaved, v_from_k, status};
-    const size_t smem = (size_t)(nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0)) * sizeof(float);
+                page_size, num_pages, nh, nkv, hd, vd, rot, vfreq ? vrot : 0, interleaved, v_from_k, status, bias, unit_v, talk, gate_out};
+    const size_t smem = (size_t)(nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0)
+                                 + (unit_v ? nkv : 0) + (talk ? nh * nh : 0)) * sizeof(float);
+    VCB_CHECK_ARG(talk == nullptr || nh % nkv == 0, "qkv_rope_store: %d heads mixed over %d KV heads", nh, nkv);
+    VCB_CHECK_ARG(talk == nullptr || q_gain == nullptr, "qkv_rope_store: mixed queries come without a norm over the whole projection");
     VCB_CHECK_ARG(smem <= 200 * 1024, "qkv_rope_store: a token's %zu bytes are more than the kernel's shared memory holds", smem);
     auto kern = dtype == VCB_F32 ? qkv_rope_store_kernel<float> : qkv_rope_store_kernel<__nv_bfloat16>;
     if (smem + 1024 > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {

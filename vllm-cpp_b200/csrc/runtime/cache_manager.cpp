@@ -104,8 +104,8 @@ void CacheManager::commit(int64_t request, int32_t new_len) {
     for (size_t g = 0; g < groups_.size(); ++g) {
         const GroupSpec& spec = groups_[g];
         if (spec.window == 0) continue;
-        // the next query sits at position new_len and reads keys >= new_len - W + 1
-        const int32_t first_needed = std::max(0, new_len - spec.window + 1);
+        // the next query sits at position new_len
+        const int32_t first_needed = spec.first_read(new_len);
         const int32_t dead_blocks = std::min<int32_t>(first_needed / spec.page_size, (int32_t)q.tables[g].size());
         // the pages of the kept first positions stay
         for (int32_t b = ceil_div(spec.keep_first, spec.page_size); b < dead_blocks; ++b) {

@@ -47,6 +47,16 @@ struct GroupSpec {
     int32_t num_pages = 0;   // pages in this group's pool
     int32_t window = 0;      // 0: every key stays; W > 0: position p reads keys (p - W, p]
     int32_t keep_first = 0;  // with a window: positions [0, keep_first) stay readable for good, so their pages are kept
+    // with a window: it stands still -- position p reads the keys of its own chunk, [p - p % W, p], chunks of W positions
+    // counted from position 0 -- so when a chunk is through, all its pages go at once
+    bool chunked = false;
+
+    // the first position that a query at position p can read (kept first positions aside)
+    int32_t first_read(int32_t p) const {
+        if (window == 0) return 0;
+        const int32_t lo = chunked ? p - p % window : p - window + 1;
+        return lo > 0 ? lo : 0;
+    }
 };
 
 class CacheManager {

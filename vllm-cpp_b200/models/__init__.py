@@ -11,6 +11,7 @@ from . import rimopel  # registers Rimopel
 from . import nagavik  # registers Nagavik
 from . import fifudra  # registers Fifudra
 from . import mefupel  # registers Mefupel
+from . import nufetar  # registers Nufetar
 from .decoder import DecoderModel
 
 

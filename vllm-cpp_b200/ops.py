@@ -69,7 +69,7 @@ def _declare(L):
         "vcb_sgemm_tn": [P, P, P, I, I, I, LL, LL, LL, P],
         "vcb_gemm_bf16_plain": [P, P, P, I, I, I, I, LL, LL, LL, P],
         "vcb_attn_paged": [P, P, I, P, LL, P, P, I, P, P, P, P, I, I, P, P, I, I, I, I, I, I, F, P, P],
-        "vcb_attn_paged_ex": [P, P, I, P, LL, P, P, I, P, P, P, P, I, I, P, P, I, I, I, I, I, I, F, I, P, P, I, F, P, I, P, P, P],
+        "vcb_attn_paged_ex": [P, P, I, P, LL, P, P, I, P, P, P, P, I, I, P, P, I, I, I, I, I, I, F, I, P, P, I, F, P, I, P, I, I, P, P, P],
         "vcb_embed_sinusoid": [P, I, P, P, P, P, I, I, I, P, P],
         "vcb_causal_conv": [P, I, LL, LL, P, P, P, LL, P, P, P, I, I, I, I, I, P, P, I, P, I, P],
         "vcb_embed_scaled_pos": [P, I, P, P, P, I, F, P, I, I, I, I, P, P],
@@ -81,18 +81,18 @@ def _declare(L):
         "vcb_gated_group_norm": [P, P, I, LL, LL, P, F, P, P, I, I, I, I, P, I, P],
         "vcb_moe_route": [P, I, LL, LL, P, P, I, I, I, I, I, P, P, P],
         "vcb_hyper_mix_norm": [P, P, P, I, LL, LL, P, P, P, P, F, P, I, P, I, I, I, I, P],
-        "vcb_token_shift": [P, P, P, LL, P, P, P, I, I, I, P, I, P],
-        "vcb_latent_norm_rope_store": [P, I, LL, LL, P, P, F, P, P, F, P, P, P, LL, I, I, I, I, I, I, I, I, P, P],
+        "vcb_token_shift": [P, P, I, P, LL, P, P, P, I, I, I, P, I, LL, P],
+        "vcb_latent_norm_rope_store": [P, I, LL, LL, P, P, F, P, P, F, P, P, P, LL, I, I, I, I, I, I, I, I, I, P, P],
         "vcb_head_linear": [P, I, I, LL, LL, I, I, P, I, P, I, LL, I, I, I, I, I, I, P],
-        "vcb_rope_rows": [P, I, LL, LL, I, I, P, P, F, P, I, LL, I, I, I, I, I, I, P],
+        "vcb_rope_rows": [P, I, LL, LL, I, I, P, P, F, P, I, LL, I, I, I, I, I, I, I, P],
         "vcb_matrix_rnn": [I, P, I, LL, LL, P, LL, I, I, I, I, I, P, P, P, P, P, LL, P, P, P, I, I, I, I, I, I, P,
-                           P, I, LL, LL, F, P, P, P, I, I, P],
+                           P, I, LL, LL, F, P, P, P, I, I, P, P],
         "vcb_sum_add_rmsnorm": [P, I, P, P, P, P, P, P, P, F, P, I, P, I, I, P],
         "vcb_branch_norm_mean": [I, P, P, P, P, P, F, P, I, I, P],
         "vcb_polynorm": [P, I, LL, LL, P, F, P, I, I, I, P],
-        "vcb_qkv_rope_store": [P, I, LL, LL, P, P, F, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, I, I, P, P],
+        "vcb_qkv_rope_store": [P, I, LL, LL, P, P, F, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, P],
         "vcb_rotate_heads": [P, I, P, P, F, I, I, I, I, I, P],
-        "vcb_head_norm_gate": [P, P, I, LL, LL, I, P, F, P, P, I, I, I, I, P, I, P],
+        "vcb_head_norm_gate": [P, P, I, LL, LL, I, P, I, F, P, P, I, I, I, I, P, I, P],
         "vcb_moe_route_grouped": [P, I, LL, LL, P, I, I, F, P, P, I, I, I, I, P, P, P],
         "vcb_moe_group": [P, I, I, I, I, P, P, P, P],
         "vcb_moe_gather": [P, LL, I, P, P, I, I, I, P, P],
@@ -102,23 +102,25 @@ def _declare(L):
         "vcb_conv_state_update": [P, I, LL, LL, P, P, LL, P, P, P, I, I, I, P],
         "vcb_qkv_conv_norm_store": [P, I, LL, LL, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P, LL, I, I, I, I, P, P],
         "vcb_gated_norm_add": [P, P, I, LL, LL, P, I, LL, LL, P, P, F, P, P, I, I, I, P, I, P],
-        "vcb_bias_act": [P, I, LL, LL, P, P, I, I, I, I, P],
+        "vcb_bias_act": [P, I, LL, LL, P, P, I, I, I, I, P, P],
         "vcb_scatter_i32": [P, P, P, P, I, LL, P],
         "vcb_selftest_wait_timeout": [LL, P, P, P],
         "vcb_state_reset": [P, I, LL, LL, LL, I, I, P, P, P, I, ctypes.c_uint, P, P],
         "vcb_attn_mma": [P, P, P, LL, P, P, I, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, I, F, P, I, I, P],
-        "vcb_attn_mma_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, I, F, I, P, P, F, P, I, P, P, I, I, P],
+        "vcb_attn_mma_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, P, I, I, P],
+        "vcb_attn_mma_wide_rows": [I, I, I],
         "vcb_attn_mma_supported": [I, I],
         "vcb_attn_mma_max_clusters": [I, I, I],
         "vcb_attn_mma_fused_supported": [I, I, I],
         "vcb_attn_mma_decode_fused": [P, I, LL, P, P, I, I, F, P, I, P, P, P, LL, P, P, I, P, P, P, P, I, P, P, P, P, I, I,
                                       I, I, I, I, F, P, I, P],
         "vcb_attn_tc": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, P, P, P],
-        "vcb_attn_tc_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, F, P, I, P, P, P, P],
+        "vcb_attn_tc_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, P, P, P],
+        "vcb_attn_tc_wide_supported": [I, I, I, I],
         "vcb_attn_tc_supported": [I, I, I],
         "vcb_attn_stream": [P, P, P, LL, P, P, I, P, P, P, I, P, I, I, I, I, I, I, F, P, I, P],
         "vcb_attn_stream_supported": [I, I, I, I, I],
-        "vcb_attn_merge": [P, P, P, P, I, I, I, I, I, P],
+        "vcb_attn_merge": [P, P, P, P, I, I, I, I, I, P, P],
         "vcb_sample": [P, LL, I, I, P, P, P, P],
         "vcb_sample_split": [P, LL, I, I, P, P, P, P, I, P, P],
         "vcb_count_tokens": [P, P, P, I, I, I, P],
@@ -409,6 +411,19 @@ def attn_paged(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_ite
           page_size, num_pages, int(window or 0), 1.0 / math.sqrt(hd), _p(status), _stream())
 
 
+def _q_width(q, nh, nkv, hd, wide):
+    """The queries' width: nh heads of hd lanes or, wide, of one block of hd lanes per KV head."""
+    width = nh * hd * (nkv if wide else 1)
+    if q.shape[-1] != width:
+        raise KernelError(f"queries of {q.shape[-1]} lanes, expected {width}")
+
+
+def _gate_ok(out_gate, out, nh):
+    if out_gate is not None:
+        _need(out_gate, "out_gate", torch.float32)
+        assert out_gate.shape[0] >= out.shape[0] and out_gate.shape[1] == nh, (out_gate.shape, out.shape, nh)
+
+
 def _sink_scores(sink, nh):
     """``sink`` as the attention wrappers take it (False, True, or a float32 tensor [nh] of scores) -> the tensor or None."""
     if not torch.is_tensor(sink):
@@ -431,13 +446,17 @@ def kv_page_views(pages, nkv, hd, hd_v):
 
 def attn_window_bias(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, rows_max, part_o, part_ml,
                      nh, nkv, hd, window, status, table_row=None, *, scale, keep_first=0, dist_a=None, dist_b=None, hd_v=None,
-                     softcap=0.0, slope=None, sink=False):
+                     softcap=0.0, slope=None, sink=False, chunked=False, wide=False, out_gate=None):
     """:func:`attn_paged` with its options: scores scaled by ``scale``; with a window, the first ``keep_first`` keys of
     a request stay visible; ``dist_a``/``dist_b`` (float32 [nh]): a_h ln(1 + b_h (pos - j)) is taken off key j's
     score; values of head size ``hd_v`` (``pages`` then [num_pages, nkv * page_size * (hd + hd_v)]); ``softcap`` c > 0:
     the scaled score becomes c tanh(s / c); ``slope`` (float32 [nh]): slope_h (pos - j) is taken off after the cap;
     ``sink``: a silent key of score 0 and no value takes part in every softmax; given as a float32 tensor [nh], the
-    silent key's score per head (not scaled)."""
+    silent key's score per head (not scaled); ``chunked``: the window stands still, a query sees the keys of its own chunk
+    of ``window`` positions counted from position 0; ``wide``: ``q`` is [T, nh * nkv * hd], a query row has a block of
+    lanes per KV head and its score is the sum of the blocks' products with those heads' keys; ``out_gate`` (float32
+    [T, nh]): what the result of a token and head is multiplied by."""
+    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, wide)
     hd_v = hd if hd_v is None else int(hd_v)
     sink_value = sink if torch.is_tensor(sink) else None
     if sink_value is not None:
@@ -456,7 +475,8 @@ def attn_window_bias(q, out, pages, block_table, q_start, q_len, ctx_len, items,
     _call("vcb_attn_paged_ex", _p(q), _p(out), _dt(q), _p(pages), pages.stride(0), _p(block_table), _p(table_row),
           block_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, rows_max, _p(part_o), _p(part_ml),
           nh, nkv, hd, page_size, num_pages, int(window or 0), float(scale), int(keep_first or 0), _p(dist_a), _p(dist_b),
-          hd_v, float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), _p(status), _stream())
+          hd_v, float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), int(bool(chunked)),
+          int(bool(wide)), _p(out_gate), _p(status), _stream())
 
 
 def embed_sinusoid(table, ids, positions, inv_freq, out, status):
@@ -568,18 +588,22 @@ def gated_norm_add(resid, y, gate, gate_bias, weight, eps, q_start, q_len, n_ent
 
 
 ACTIVATIONS = {"gelu": 0, "gelu_erf": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3}
-ELEMENTWISE = dict(ACTIVATIONS, identity=4)    # what bias_act takes: the activations, and the sums as they are
+# what bias_act takes: the activations, the sums as they are, and two more
+ELEMENTWISE = dict(ACTIVATIONS, identity=4, tanh=5, xielu=6)
 
 
-def bias_act(x, out, kind: str, bias=None):
-    """out = act(x + bias): x 32-bit [T, C] or [S, T, C] partial sums; ``kind`` one of ACTIVATIONS, or "identity" (the
-    sums themselves, added up and in ``out``'s type)."""
+def bias_act(x, out, kind: str, bias=None, coef=None):
+    """out = act(x + bias): x 32-bit [T, C] or [S, T, C] partial sums; ``kind`` one of ACTIVATIONS, "identity" (the
+    sums themselves, added up and in ``out``'s type), "tanh", or "xielu": c0 z^2 + z/2 above zero, c1 (e^z - 1 - z) + z/2
+    below, (c0, c1) = ``coef`` (float32 [2] on the device)."""
     S, ss, ld = _rows_in(x, "x")
     T, C = x.shape[-2:]
     _need(out, "out"); assert out.shape == (T, C)
     if kind not in ELEMENTWISE:
         raise KernelError(f"activation '{kind}' is not one of {sorted(ELEMENTWISE)}")
-    _call("vcb_bias_act", _p(x), S, ss, ld, _p(bias), _p(out), _dt(out), T, C, ELEMENTWISE[kind], _stream())
+    if kind == "xielu":
+        _need(coef, "coef", torch.float32); assert coef.numel() == 2
+    _call("vcb_bias_act", _p(x), S, ss, ld, _p(bias), _p(out), _dt(out), T, C, ELEMENTWISE[kind], _p(coef), _stream())
 
 
 def embed_scaled_pos(table, ids, positions, pos_table, scale, out, status):
@@ -798,10 +822,11 @@ def moe_combine(y, pos_of, top, q_start, q_len, n_entries, out, shared=None, sel
           T, W, _p(out), _stream())
 
 
-def attn_merge(part_o, part_ml, dec_rows, out, n_dec, nh, hd, nslices):
+def attn_merge(part_o, part_ml, dec_rows, out, n_dec, nh, hd, nslices, out_gate=None):
+    _gate_ok(out_gate, out, nh)
     _need(part_o, "part_o", torch.float32); _need(part_ml, "part_ml", torch.float32)
     _need(dec_rows, "dec_rows", torch.int32); _need(out, "out")
-    _call("vcb_attn_merge", _p(part_o), _p(part_ml), _p(dec_rows), _p(out), _dt(out), n_dec, nh, hd, nslices, _stream())
+    _call("vcb_attn_merge", _p(part_o), _p(part_ml), _p(dec_rows), _p(out), _dt(out), n_dec, nh, hd, nslices, _p(out_gate), _stream())
 
 
 def sample(logits, params, counts, out, no_nucleus=False):
@@ -918,17 +943,30 @@ def attn_tc_supported(dtype: torch.dtype, hd: int, page_size: int) -> bool:
     return bool(lib().vcb_attn_tc_supported(BF16 if dtype == torch.bfloat16 else F32, hd, page_size))
 
 
+def attn_tc_wide_supported(dtype: torch.dtype, hd: int, page_size: int, nkv: int) -> bool:
+    """Whether :func:`attn_tc` takes query rows of one block of ``hd`` lanes per KV head."""
+    return bool(lib().vcb_attn_tc_wide_supported(BF16 if dtype == torch.bfloat16 else F32, hd, page_size, nkv))
+
+
+def attn_mma_wide_rows(dtype: torch.dtype, hd: int, nkv: int) -> int:
+    """The rows of a prompt block (128 or 64) with which :func:`attn_mma` takes query rows of one block of ``hd`` lanes
+    per KV head; 0: it does not take them, single tokens neither."""
+    return int(lib().vcb_attn_mma_wide_rows(BF16 if dtype == torch.bfloat16 else F32, hd, nkv))
+
+
 def attn_tc(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, nh, nkv, hd, window, status,
-            table_row=None, work=None, scale=None, keep_first=0, dist_a=None, dist_b=None, softcap=0.0, slope=None, sink=False):
+            table_row=None, work=None, scale=None, keep_first=0, dist_a=None, dist_b=None, softcap=0.0, slope=None, sink=False,
+            chunked=False, wide=False, out_gate=None):
     """Attention of prompt portions on tcgen05 tensor cores (bfloat16, head_dim 64 or 128, pages of 8 to 64
     tokens), with the options of :func:`attn_window_bias` (``scale``, ``keep_first``, ``dist_a``/``dist_b``, ``softcap``,
-    ``slope``, ``sink``).
+    ``slope``, ``sink``, ``chunked``, ``out_gate``, and ``wide`` where :func:`attn_tc_wide_supported` says so).
     Items as for :func:`attn_paged` with one key slice and at most 128 rows each.  ``work``: two int32
     zeros, zero again when the kernel is through (the queue its blocks take their units from); launches that share
     them must follow one another on a stream.  Made on the spot when not given."""
     if work is None:
         work = torch.zeros(2, dtype=torch.int32, device=q.device)
     _need(work, "work", torch.int32)
+    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, wide)
     sink_value = _sink_scores(sink, nh)
     _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pages, "pages", torch.bfloat16)
     for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len),
@@ -945,19 +983,22 @@ def attn_tc(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items,
           block_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, nh, nkv, hd, page_size,
           num_pages, int(window or 0), 1.0 / math.sqrt(hd) if scale is None else float(scale), int(keep_first or 0),
           _p(dist_a), _p(dist_b), float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value),
-          _p(status), _p(work), _stream())
+          int(bool(chunked)), int(bool(wide)), _p(out_gate), _p(status), _p(work), _stream())
 
 
 def attn_mma(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, rows_max, part_o, part_ml,
              nh, nkv, hd, window, status, table_row=None, allow_tma=True, slice_counters=None, dec_rows=None,
-             cluster=0, scale=None, keep_first=0, dist_a=None, dist_b=None, softcap=0.0, slope=None, sink=False):
+             cluster=0, scale=None, keep_first=0, dist_a=None, dist_b=None, softcap=0.0, slope=None, sink=False, chunked=False,
+             wide=False, out_gate=None):
     """Tensor-core variant of :func:`attn_paged` (bfloat16, head_dim 64 or 128; rows_max 16 or 128), with the
     options of :func:`attn_window_bias` (``scale``, default 1/sqrt(hd); ``keep_first``; ``dist_a``/``dist_b``;
-    ``softcap``, ``slope``, ``sink``).
+    ``softcap``, ``slope``, ``sink``, ``chunked``, ``out_gate``, and ``wide``, with rows_max 16 or what
+    :func:`attn_mma_wide_rows` says).
     With ``slice_counters`` (int32 zeros, one per decoded token and KV head group, left at zero again) and
     ``dec_rows``, the block that finishes a token's last key slice merges the slices itself; with ``cluster`` = the
     number of slices per token (2 to 8) as well, the slices' blocks run as a cluster and merge through shared memory."""
     sink_value = _sink_scores(sink, nh)
+    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, wide)
     _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pages, "pages", torch.bfloat16)
     for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len),
                     ("items", items)):
@@ -973,8 +1014,8 @@ def attn_mma(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items
           block_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, rows_max, _p(part_o),
           _p(part_ml), _p(slice_counters), _p(dec_rows), nh, nkv, hd, page_size, num_pages, int(window or 0),
           1.0 / math.sqrt(hd) if scale is None else float(scale), int(keep_first or 0), _p(dist_a), _p(dist_b),
-          float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), _p(status), int(allow_tma),
-          int(cluster), _stream())
+          float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), int(bool(chunked)),
+          int(bool(wide)), _p(out_gate), _p(status), int(allow_tma), int(cluster), _stream())
 
 
 def attn_stream_supported(dtype: torch.dtype, hd: int, page_size: int, nh: int, nkv: int) -> bool:
@@ -1085,38 +1126,46 @@ def hyper_mix_norm(streams, *, init=None, y=None, mix=None, outw=None, inw=None,
 
 def token_shift(h, mu, state, q_start, q_len, slots, n_entries, out):
     """out[t] = h[t] + (h[t-1] - h[t]) * mu per channel over each entry's rows (32-bit ``h`` [T, W]); the row before an
-    entry's first is the request's ``state`` [slots, W] (32-bit), which then takes the entry's last row of ``h``."""
+    entry's first is the request's ``state`` [slots, W] (32-bit), which then takes the entry's last row of ``h``.
+    ``mu`` [W], ``out`` [T, W], or several mixes of the same rows at once: ``mu`` [N, W], ``out`` [N, >= T, W] (whose rows
+    beyond T are left alone)."""
     _need(h, "h", torch.float32); _need(mu, "mu", torch.float32); _need(state, "state", torch.float32, contiguous=False)
-    _need(out, "out")
+    _need(out, "out", contiguous=False)
     T, W = h.shape
-    assert mu.numel() == W and out.shape == (T, W) and state.shape[-1] == W and state.stride(-1) == 1
-    _call("vcb_token_shift", _p(h), _p(mu), _p(state), state.stride(0), _p(q_start), _p(q_len), _p(slots), n_entries, T, W,
-          _p(out), _dt(out), _stream())
+    n_mix = 1 if out.dim() == 2 else out.shape[0]
+    assert mu.numel() == n_mix * W and out.shape[-1] == W and out.shape[-2] >= T and out.stride(-1) == 1 and out.stride(-2) == W
+    assert state.shape[-1] == W and state.stride(-1) == 1
+    _call("vcb_token_shift", _p(h), _p(mu), n_mix, _p(state), state.stride(0), _p(q_start), _p(q_len), _p(slots), n_entries, T, W,
+          _p(out), _dt(out), out.stride(0) if out.dim() == 3 else 0, _stream())
 
 
 # -------------------------------------------------------------------------- attention through a latent
 
 
 def latent_norm_rope_store(u, q_gain, kv_gain, eps, positions, freq, gain, slot_map, cq_out, pages, page_size, q_rank,
-                           kv_rank, rot, status, v_width=None):
+                           kv_rank, rot, status, v_width=None, interleaved=False):
     """From the stacked down projections ``u`` (32-bit [T, q_rank + kv_rank + rot] or partial sums): the normed query
     latent to ``cq_out`` [T, q_rank]; the normed key/value latent c and the rotated shared key part into the token's
     cache row.  A page is one flat row: [page_size, kv_rank + rot] key rows [c | k_rot], then [page_size, v_width]
     value rows [c | zeros] (``v_width`` None: kv_rank lanes, c alone).  ``freq`` [rot / 2] 32-bit; cos and sin are
-    multiplied by ``gain``."""
+    multiplied by ``gain``; ``interleaved``: neighbouring lanes turn together (else lane i with lane i + rot/2).
+    ``q_rank`` 0 (``q_gain`` and ``cq_out`` None): there is no query latent."""
     v_width = int(kv_rank if v_width is None else v_width)
     S, ss, ld = _rows_in(u, "u")
     T = u.shape[-2]
     assert u.shape[-1] == q_rank + kv_rank + rot and rot % 2 == 0
-    _need(cq_out, "cq_out"); _need(pages, "pages", cq_out.dtype); _need(positions, "positions", torch.int32)
-    _need(slot_map, "slot_map", torch.int32); _need(q_gain, "q_gain", torch.float32); _need(kv_gain, "kv_gain", torch.float32)
+    if q_rank:
+        _need(cq_out, "cq_out", pages.dtype); _need(q_gain, "q_gain", torch.float32)
+        assert cq_out.shape == (T, q_rank) and q_gain.numel() == q_rank
+    _need(pages, "pages"); _need(positions, "positions", torch.int32)
+    _need(slot_map, "slot_map", torch.int32); _need(kv_gain, "kv_gain", torch.float32)
     if rot:
         _need(freq, "freq", torch.float32); assert freq.numel() == rot // 2
-    assert cq_out.shape == (T, q_rank) and q_gain.numel() == q_rank and kv_gain.numel() == kv_rank
+    assert kv_gain.numel() == kv_rank
     assert pages[0].numel() == page_size * (kv_rank + rot + v_width), (pages.shape, page_size, kv_rank, rot, v_width)
     _call("vcb_latent_norm_rope_store", _p(u), S, ss, ld, _p(q_gain), _p(kv_gain), float(eps), _p(positions), _p(freq),
           float(gain), _p(slot_map), _p(cq_out), _p(pages), pages.stride(0), int(page_size), pages.shape[0], int(q_rank),
-          int(kv_rank), int(rot), v_width, T, _dt(cq_out), _p(status), _stream())
+          int(kv_rank), int(rot), int(bool(interleaved)), v_width, T, _dt(pages), _p(status), _stream())
 
 
 def head_linear(x, m, out, *, heads, n_in, n_out, in_head_stride, in_off=0, out_head_stride, out_off=0):
@@ -1137,9 +1186,10 @@ def head_linear(x, m, out, *, heads, n_in, n_out, in_head_stride, in_off=0, out_
           out.stride(0), int(out_head_stride), int(out_off), T, int(heads), int(n_in), int(n_out), _stream())
 
 
-def rope_rows(x, positions, freq, gain, out, *, heads, dims, width, in_head_stride, in_off=0, out_head_stride, out_off=0):
+def rope_rows(x, positions, freq, gain, out, *, heads, dims, width, in_head_stride, in_off=0, out_head_stride, out_off=0,
+              interleaved=False):
     """Copies ``width`` lanes of every head's slice of the 32-bit sums ``x`` into ``out``, the first ``dims`` of them
-    rotated: lane i pairs with lane i + dims/2, the angle is position * freq[i], cos and sin times ``gain``."""
+    rotated: lane i pairs with lane i + dims/2 (``interleaved``: lane 2i with lane 2i + 1), the angle is position * freq[i], cos and sin times ``gain``."""
     S, ss, ld = _rows_in(x, "x")
     T = x.shape[-2]
     _need(out, "out", contiguous=False); _need(positions, "positions", torch.int32)
@@ -1149,7 +1199,7 @@ def rope_rows(x, positions, freq, gain, out, *, heads, dims, width, in_head_stri
     assert (heads - 1) * in_head_stride + in_off + width <= x.shape[-1]
     assert (heads - 1) * out_head_stride + out_off + width <= out.shape[-1]
     _call("vcb_rope_rows", _p(x), S, ss, ld, int(in_head_stride), int(in_off), _p(positions), _p(freq), float(gain), _p(out),
-          _dt(out), out.stride(0), int(out_head_stride), int(out_off), T, int(heads), int(dims), int(width), _stream())
+          _dt(out), out.stride(0), int(out_head_stride), int(out_off), T, int(heads), int(dims), int(width), int(bool(interleaved)), _stream())
 
 
 # -------------------------------------------------------------------------- recurrences with a matrix state per head
@@ -1157,7 +1207,7 @@ def rope_rows(x, positions, freq, gain, out, *, heads, dims, width, in_head_stri
 
 def matrix_rnn(mode, u, state, q_start, q_len, slots, n_entries, out, *, heads, d, dv, q_col, k_col, v_col, x=None,
                kv_heads=None, b_col=0, a_col=0, dt_bias=None, rate=None, f_bias=None, lower=None, z=None, tau=1.0, decay=None,
-               ctx_len=None, freq=None, rot=0, interleaved=False):
+               ctx_len=None, freq=None, rot=0, interleaved=False, bonus=None):
     """A recurrence over each entry's tokens whose state S [d, dv] per head lies in ``state`` [slots, heads, dv, d] (32-bit, a value column's rows in a run), ``out`` [T, heads dv].
 
     ``mode`` "delta": S <- g S; w = beta (v - S^T k); S <- S + k w^T; o = S^T q.  q, k, v are columns ``q_col``,
@@ -1170,11 +1220,14 @@ def matrix_rnn(mode, u, state, q_start, q_len, slots, n_entries, out, *, heads, 
     ``mode`` "retention": S <- decay_h S + k v^T; o = S^T q with q, k, v columns of u, the first ``rot`` lanes of every q
     and k head turned by position * freq[i] (lanes paired in halves, or ``interleaved``), k then times d^(-1/2);
     positions from ``ctx_len``.
-    ``u``: the projection's 32-bit sums ([S, T, C] partials)."""
+    ``mode`` "wkv": o = (S + diag(bonus) k v^T)^T q; S <- diag(f) S + k v^T with q, k, v columns of u, f = exp(-exp(z +
+    f_bias)) per state row and ``bonus`` [heads d].
+    ``u``: the projection's 32-bit sums ([S, T, C] partials).  The columns are offsets from a row's start: where q, k and v
+    are the results of products of their own, row blocks of one buffer, they reach into the other blocks."""
     S, ss, ld = _rows_in(u, "u")
     _need(state, "state", torch.float32, contiguous=False); _need(out, "out", torch.float32)
     assert state.shape[1:] == (heads, dv, d) and state[0].is_contiguous() and out.shape[1] == heads * dv
-    m = {"delta": 0, "gated": 1, "decayed": 2, "retention": 3}[mode]
+    m = {"delta": 0, "gated": 1, "decayed": 2, "retention": 3, "wkv": 4}[mode]
     ldx = 0
     zS = zss = zld = 0
     if m == 0:
@@ -1185,10 +1238,12 @@ def matrix_rnn(mode, u, state, q_start, q_len, slots, n_entries, out, *, heads, 
     elif m == 1:
         for name, t in (("f_bias", f_bias), ("lower", lower)):
             _need(t, name, torch.float32); assert t.numel() == heads * d
-    elif m == 2:
+    elif m in (2, 4):
         zS, zss, zld = _rows_in(z, "z")
         _need(f_bias, "f_bias", torch.float32); assert f_bias.numel() == heads * d and z.shape[-1] == heads * d
         assert z.shape[-2] >= out.shape[0] and tau > 0
+        if m == 4:
+            _need(bonus, "bonus", torch.float32); assert bonus.numel() == heads * d
     else:
         _need(decay, "decay", torch.float32); assert decay.numel() == heads
         _need(ctx_len, "ctx_len", torch.int32)
@@ -1197,22 +1252,24 @@ def matrix_rnn(mode, u, state, q_start, q_len, slots, n_entries, out, *, heads, 
     _call("vcb_matrix_rnn", m, _p(u), S, ss, ld, _p(x), ldx, int(q_col), int(k_col), int(v_col), int(b_col), int(a_col),
           _p(dt_bias), _p(rate), _p(f_bias), _p(lower), _p(state), state.stride(0), _p(q_start), _p(q_len), _p(slots),
           n_entries, int(out.shape[0]), int(heads), int(kv_heads or heads), int(d), int(dv), _p(out),
-          _p(z), zS, zss, zld, 1.0 / float(tau), _p(decay), _p(ctx_len), _p(freq), int(rot), int(bool(interleaved)), _stream())
+          _p(z), zS, zss, zld, 1.0 / float(tau), _p(decay), _p(ctx_len), _p(freq), int(rot), int(bool(interleaved)), _p(bonus), _stream())
 
 
 def head_norm_gate(o, weight, eps, q_start, q_len, n_entries, heads, dv, out, gate=None, gate_col=0):
     """out[t, h] = weight * o[t, h] / sqrt(mean(o[t, h]^2) + eps) (* silu(gate[t, gate_col + h dv ...]) with a gate):
-    every head of the 32-bit ``o`` [T, heads dv] by its own root mean square, one gain [dv] for all heads (None: no gain)."""
+    every head of the 32-bit ``o`` [T, heads dv] by its own root mean square, a gain [dv] for all
+    heads or [heads dv] (None: no gain)."""
     _need(o, "o", torch.float32); _need(out, "out")
     T = o.shape[0]
     assert o.shape == (T, heads * dv) and out.shape == o.shape
     if weight is not None:
-        _need(weight, "weight", torch.float32); assert weight.numel() == dv
+        _need(weight, "weight", torch.float32); assert weight.numel() in (dv, heads * dv)
     S = ss = ld = 0
     if gate is not None:
         S, ss, ld = _rows_in(gate, "gate")
         assert gate_col + heads * dv <= gate.shape[-1]
-    _call("vcb_head_norm_gate", _p(o), _p(gate), S, ss, ld, int(gate_col), _p(weight), float(eps), _p(q_start), _p(q_len),
+    _call("vcb_head_norm_gate", _p(o), _p(gate), S, ss, ld, int(gate_col), _p(weight),
+          int(dv) if weight is not None and weight.numel() == heads * dv else 0, float(eps), _p(q_start), _p(q_len),
           n_entries, T, int(heads), int(dv), _p(out), _dt(out), _stream())
 
 
@@ -1297,16 +1354,23 @@ def polynorm(u, coef, eps, out):
 
 
 def qkv_rope_store(qkv, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q_out, pages, nh, nkv, hd, vd, status, *,
-                   rot, interleaved=False, values_from_keys=False):
+                   rot, interleaved=False, values_from_keys=False, bias=None, unit_values=False, talk=None, gate_out=None):
     """From the stacked projection's 32-bit sums ``qkv`` ([T, C] or [S, T, C]; C = nh hd + nkv hd + nkv vd, or without the
     value columns where ``values_from_keys``: the keys as projected are the values): with ``q_gain`` [nh hd] / ``k_gain``
     [nkv hd] all of a token's query (key) lanes divided by their root mean square times the gain; the first ``rot`` lanes
     of every q and k head turned by position * freq[i], pairs (i, i + rot/2) or ``interleaved`` (2i, 2i+1); with
     ``vfreq`` [vd/2] every value head turned likewise over all its lanes; queries to ``q_out``, keys and values to the
-    tokens' slots of ``pages`` (see :func:`kv_page_views`)."""
+    tokens' slots of ``pages`` (see :func:`kv_page_views`).  Options: ``bias`` [C] added first; ``unit_values``: every value
+    head divided by its root mean square; ``talk`` [nh, nh]: queries mixed across heads, q'_h[G] = sum over the heads g
+    of KV head G of talk[h, g] q_g, ``q_out`` [T, nh * nkv * hd] (what the attention kernels take as ``wide``);
+    ``gate_out`` [T, nh]: the sigmoids of nh further columns behind the projection's."""
     S, ss, ld = _rows_in(qkv, "qkv")
     T, C = qkv.shape[-2:]
+    C -= nh if gate_out is not None else 0
     assert C == nh * hd + nkv * hd + (0 if values_from_keys else nkv * vd), (C, nh, nkv, hd, vd)
+    for name, t, n in (("bias", bias, C), ("talk", talk, nh * nh), ("gate_out", gate_out, T * nh)):
+        if t is not None:
+            _need(t, name, torch.float32); assert t.numel() == n, (name, t.shape, n)
     if q_gain is not None:
         _need(q_gain, "q_gain", torch.float32); _need(k_gain, "k_gain", torch.float32)
         assert q_gain.numel() == nh * hd and k_gain.numel() == nkv * hd
@@ -1315,12 +1379,13 @@ def qkv_rope_store(qkv, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q
         _need(freq, "freq", torch.float32); assert freq.numel() == rot // 2
     if vfreq is not None:
         _need(vfreq, "vfreq", torch.float32); assert vfreq.numel() == vd // 2 and vd % 2 == 0
-    _need(q_out, "q_out"); assert q_out.shape == (T, nh * hd)
+    _need(q_out, "q_out"); assert q_out.shape == (T, nh * hd * (nkv if talk is not None else 1))
     _need(pages, "pages", q_out.dtype)
     page_size, num_pages = kv_page_views(pages, nkv, hd, vd)
     _call("vcb_qkv_rope_store", _p(qkv), S, ss, ld, _p(q_gain), _p(k_gain), float(eps), _p(positions), _p(freq), _p(vfreq),
           _p(slot_map), _p(q_out), _p(pages), pages.stride(0), page_size, num_pages, nh, nkv, hd, vd, int(rot), vd,
-          int(bool(interleaved)), int(bool(values_from_keys)), T, _dt(q_out), _p(status), _stream())
+          int(bool(interleaved)), int(bool(values_from_keys)), T, _dt(q_out), _p(status), _p(bias), int(bool(unit_values)), _p(talk),
+          _p(gate_out), _stream())
 
 
 def rotate_heads(x, positions, freq, *, heads, width, dims, interleaved=False, sign=1.0):

@@ -9,7 +9,7 @@ from .gated_block import GatedPostNormBlock
 from .hyper_block import HyperStreamsBlock
 from .latent_attention import LatentAttention
 from .mamba2 import Mamba2Mixer
-from .matrix_rnn import DecayedLinearMixer, DeltaRuleMixer, GatedLinearMixer, RetentionMixer
+from .matrix_rnn import DecayedLinearMixer, DeltaRuleMixer, GatedLinearMixer, RetentionMixer, WkvMixer
 from .mlp import DenseMLP, GatedMLP, SwiGLUMLP
 from .moe import RoutedExperts
 from .sandwich_block import SandwichNormBlock
@@ -41,6 +41,7 @@ register_part("block", "hyper_streams", HyperStreamsBlock)
 register_part("mixer", "rotary_window_attention", RotaryWindowAttention)
 register_part("mixer", "decayed_linear", DecayedLinearMixer)
 register_part("mixer", "retention", RetentionMixer)
+register_part("mixer", "wkv", WkvMixer)
 register_part("mixer", "normed_branches", NormedBranchesMixer)
 register_part("block", "parallel", ParallelBlock)
 register_part("reentry", "loop_reentry", LoopReentry)
@@ -48,5 +49,5 @@ register_part("reentry", "loop_reentry", LoopReentry)
 __all__ = ["Block", "BuildContext", "CacheSpec", "FeedForward", "Mixer", "Norm", "Part", "PositionEncoding",
            "PreNormBlock", "Embedding", "Head", "LMHead", "TokenEmbedding", "SwiGLUMLP", "DenseMLP", "GatedPostNormBlock",
            "ConvWindowAttention", "SinusoidalTokenEmbedding", "PositionalTokenEmbedding",
-           "RotaryWindowAttention", "DecayedLinearMixer", "RetentionMixer", "NormedBranchesMixer", "ParallelBlock", "PendingSum", "LoopReentry",
+           "RotaryWindowAttention", "DecayedLinearMixer", "RetentionMixer", "WkvMixer", "NormedBranchesMixer", "ParallelBlock", "PendingSum", "LoopReentry",
            "Mamba2Mixer", "LatentAttention", "DeltaRuleMixer", "GatedLinearMixer", "HyperStreamsBlock", "GatedMLP", "RoutedExperts", "SandwichNormBlock", "RMSNorm", "RotaryEmbedding", "GQAAttention"]

@@ -53,6 +53,9 @@ class CacheSpec:
                   the engine's (caches that differ in it get pools of their own);
                   with a window, ``keep_first`` > 0 keeps the request's first keys
                   readable for good, so the pages that hold them are never given back;
+                  ``chunked``: the window stands still -- a position reads the keys of its
+                  own chunk of ``window`` positions, counted from position 0 --, and a
+                  chunk's pages are given back when it is through;
                   ``v_head_dim`` > 0: values of another size than keys (a page then
                   holds ``[num_kv_heads, page_size, head_dim]`` keys followed by
                   ``[num_kv_heads, page_size, v_head_dim]`` values, as one flat row).
@@ -68,6 +71,7 @@ class CacheSpec:
     initial_value: float = 0.0    # kind "state": what a request's state holds before its first token
     keep_first: int = 0
     v_head_dim: int = 0
+    chunked: bool = False
 
 
 class Part:

@@ -10,13 +10,20 @@ from .base import Block
 
 
 class PreNormBlock(Block):
-    """parts: ``norm1``, ``mixer``, ``norm2``, ``feed_forward``."""
+    """parts: ``norm1``, ``mixer`` and, unless the layer has none, ``norm2`` and ``feed_forward``."""
+
+    def __init__(self, params, prefix, build, parts):
+        super().__init__(params, prefix, build, parts)
+        if ("feed_forward" in parts) != ("norm2" in parts):
+            raise ValueError("a feed-forward and its norm come together")
 
     def forward(self, resid, pending, ctx, cache, writes=True):
         mark = getattr(ctx, "mark", lambda label: None)     # kernel groups for the profile, where the step keeps one
         y = self.parts["norm1"].forward(resid, pending)
         d = self.parts["mixer"].forward(y, ctx, cache, writes)
         mark("mixer")
+        if "feed_forward" not in self.parts:
+            return d
         y = self.parts["norm2"].forward(resid, d)
         out = self.parts["feed_forward"].forward(y, ctx)
         mark("feed_forward")

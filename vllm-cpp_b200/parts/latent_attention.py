@@ -10,8 +10,10 @@ q_plain . (W_uk[h] c) = (W_uk[h]^T q_plain) . c and sum_j w_j W_uv[h] c_j = W_uv
 into the latent space and attention runs over the cached rows themselves: one shared KV head whose keys are
 [c | rot(k_r)] (kv_rank + r lanes) and whose values are c; the heads' values are expanded from the weighted latent sums
 afterwards.  The step's cost per key no longer depends on the heads' own sizes, and nothing is expanded per cached token.
+The queries may also come straight from the input, q = W_q x (no query latent), and the keys may be those of a sliding
+window, 0 <= i - j < window, whose rows are given back as it passes.
 
-Rotation pairs lane i with lane i + r/2; the angle is position * f_i in 32-bit.  The frequencies f_i may be stretched
+Rotation pairs lane i with lane i + r/2, or neighbouring lanes (``pairing`` "interleaved"); the angle is position * f_i in 32-bit.  The frequencies f_i may be stretched
 (``rope_frequencies``): f_i / factor for pairs that turn slowly, f_i for those that turn fast, a linear ramp between,
 and cos and sin times 0.1 ln(factor) + 1.  ``scale`` is used as given.  Norms, angles, scores and softmax are 32-bit;
 the latent rows, the queries and the expanded values are stored in the compute dtype.
@@ -57,8 +59,10 @@ def rope_frequencies(dims: int, base: float, scaling: dict | None = None):
 
 class LatentAttention(Mixer):
     """params: ``hidden_size``, ``num_heads``, ``head_dim`` (plain lanes d), ``rot_dim`` (r, even), ``v_head_dim``,
-    ``q_rank``, ``kv_rank``, ``scale``, ``eps``, ``rope_base``, ``rope_scaling`` (None or factor/original/fast/slow).
-    Tensors under the prefix: ``dq`` [q_rank, H], ``dq.norm`` [q_rank], ``uq`` [heads (d + r), q_rank], ``dkv``
+    ``q_rank`` (0: no query latent), ``kv_rank``, ``scale``, ``eps``, ``rope_base``, ``rope_scaling`` (None or
+    factor/original/fast/slow), ``pairing`` ("half", the default, or "interleaved"), ``window`` (0: all keys).
+    Tensors under the prefix: ``dq`` [q_rank, H], ``dq.norm`` [q_rank], ``uq`` [heads (d + r), q_rank] -- or, without a
+    query latent, ``q`` [heads (d + r), H] --, ``dkv``
     [kv_rank + r, H], ``dkv.norm`` [kv_rank], ``uk`` [heads d, kv_rank], ``uv`` [heads vd, kv_rank], ``o`` [H, heads vd]."""
 
     def __init__(self, params, prefix, build):
@@ -66,14 +70,16 @@ class LatentAttention(Mixer):
         p = params
         self.hidden, self.nh = int(p["hidden_size"]), int(p["num_heads"])
         self.d, self.r, self.vd = int(p["head_dim"]), int(p["rot_dim"]), int(p["v_head_dim"])
-        self.q_rank, self.kv_rank = int(p["q_rank"]), int(p["kv_rank"])
+        self.q_rank, self.kv_rank = int(p.get("q_rank") or 0), int(p["kv_rank"])
+        self.window = int(p.get("window") or 0)
+        pairing = str(p.get("pairing") or "half")
+        if pairing not in ("half", "interleaved"):
+            raise ValueError(f"rotary pairing '{pairing}' is not one of 'half', 'interleaved'")
+        self.interleaved = pairing == "interleaved"
         self.scale, self.eps = float(p["scale"]), float(p.get("eps", 1e-6))
         if self.r % 2:
             raise ValueError(f"{self.r} rotated lanes: lanes turn in pairs")
         self.khd = self.kv_rank + self.r          # lanes of a cached key row
-        if not 1 <= self.khd <= 256:
-            raise ValueError(f"a latent of {self.kv_rank} lanes with {self.r} rotated ones: the attention kernels take "
-                             f"key rows of up to 256 lanes")
         freqs, self.rope_gain = rope_frequencies(self.r, float(p.get("rope_base", 10000.0)), p.get("rope_scaling")) \
             if self.r else ([], 1.0)
         self.freq = torch.tensor(freqs or [0.0], dtype=torch.float64).to(torch.float32).to(build.device)
@@ -84,24 +90,30 @@ class LatentAttention(Mixer):
         self.w_down = self.w_uq = self.w_o = self.m_uk = self.m_uv = self.q_gain = self.kv_gain = None
 
     def cache_spec(self):
-        return CacheSpec("kv", num_kv_heads=1, head_dim=self.khd, v_head_dim=0 if self.vw == self.khd else self.vw)
+        return CacheSpec("kv", num_kv_heads=1, head_dim=self.khd, window=self.window, v_head_dim=0 if self.vw == self.khd else self.vw)
 
     def tensor_specs(self):
         p, H, nh = self.prefix, self.hidden, self.nh
-        return [TensorSpec(p + "dq", (self.q_rank, H)), TensorSpec(p + "dq.norm", (self.q_rank,), "vector"),
-                TensorSpec(p + "uq", (nh * (self.d + self.r), self.q_rank)),
-                TensorSpec(p + "dkv", (self.khd, H)), TensorSpec(p + "dkv.norm", (self.kv_rank,), "vector"),
-                TensorSpec(p + "uk", (nh * self.d, self.kv_rank)), TensorSpec(p + "uv", (nh * self.vd, self.kv_rank)),
-                TensorSpec(p + "o", (H, nh * self.vd))]
+        q_rows = nh * (self.d + self.r)
+        queries = [TensorSpec(p + "q", (q_rows, H))]
+        if self.q_rank:
+            queries = [TensorSpec(p + "dq", (self.q_rank, H)), TensorSpec(p + "dq.norm", (self.q_rank,), "vector"),
+                       TensorSpec(p + "uq", (q_rows, self.q_rank))]
+        return queries + [
+            TensorSpec(p + "dkv", (self.khd, H)), TensorSpec(p + "dkv.norm", (self.kv_rank,), "vector"),
+            TensorSpec(p + "uk", (nh * self.d, self.kv_rank)), TensorSpec(p + "uv", (nh * self.vd, self.kv_rank)),
+            TensorSpec(p + "o", (H, nh * self.vd))]
 
     def bind(self, store):
         p = self.prefix
-        self.w_down = store.matrices([p + "dq", p + "dkv"])       # both down projections read the same rows: one product
-        self.w_uq, self.w_o = store.matrix(p + "uq"), store.matrix(p + "o")
+        # what reads the input is one product: the query latent (or the queries themselves) and the key/value latent
+        self.w_down = store.matrices([p + ("dq" if self.q_rank else "q"), p + "dkv"])
+        self.w_uq = store.matrix(p + "uq") if self.q_rank else None
+        self.w_o = store.matrix(p + "o")
         # head h's small matrices, [h][out][in]: W_uk[h]^T carries a query into the latent space, W_uv[h] a latent sum out
         self.m_uk = store.matrix(p + "uk").view(self.nh, self.d, self.kv_rank).transpose(1, 2).contiguous()
         self.m_uv = store.matrix(p + "uv").view(self.nh, self.vd, self.kv_rank).contiguous()
-        self.q_gain = store.vector(p + "dq.norm").float().contiguous()
+        self.q_gain = store.vector(p + "dq.norm").float().contiguous() if self.q_rank else None
         self.kv_gain = store.vector(p + "dkv.norm").float().contiguous()
 
     def forward(self, x, ctx, cache, writes=True):
@@ -112,17 +124,22 @@ class LatentAttention(Mixer):
         nh, d, r, vd, kr, khd = self.nh, self.d, self.r, self.vd, self.kv_rank, self.khd
         group = ctx.groups[kv.group]
         u = matmul_tn(x, self.w_down, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
-        cq = workspace.empty((T, self.q_rank), dt, dev)
-        ops.latent_norm_rope_store(u, self.q_gain, self.kv_gain, self.eps, ctx.positions, self.freq, self.rope_gain,
-                                   group.slot_map, cq, kv.pages, group.page_size, self.q_rank, kr, r, ctx.status, v_width=self.vw)
-        q = matmul_tn(cq, self.w_uq, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
+        q_cols = 0 if self.q_rank else nh * (d + r)      # columns of u ahead of the latents
+        cq = workspace.empty((T, self.q_rank), dt, dev) if self.q_rank else None
+        ops.latent_norm_rope_store(u[..., q_cols:], self.q_gain, self.kv_gain, self.eps, ctx.positions, self.freq, self.rope_gain,
+                                   group.slot_map, cq, kv.pages, group.page_size, self.q_rank, kr, r, ctx.status, v_width=self.vw,
+                                   interleaved=self.interleaved)
+        if self.q_rank:
+            q = matmul_tn(cq, self.w_uq, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
+        else:
+            q = u[..., :q_cols]
         ql = workspace.empty((T, nh * khd), dt, dev)
         ops.head_linear(q, self.m_uk, ql, heads=nh, n_in=d, n_out=kr, in_head_stride=d + r, out_head_stride=khd)
         if r:
             ops.rope_rows(q, ctx.positions, self.freq, self.rope_gain, ql, heads=nh, dims=r, width=r, in_head_stride=d + r,
-                          in_off=d, out_head_stride=khd, out_off=kr)
+                          in_off=d, out_head_stride=khd, out_off=kr, interleaved=self.interleaved)
         lat = workspace.empty((T, nh * self.vw), dt, dev)
-        paged_attention(ctx, kv, ql, lat, nh=nh, nkv=1, hd=khd, vd=self.vw, scale=self.scale)
+        paged_attention(ctx, kv, ql, lat, nh=nh, nkv=1, hd=khd, vd=self.vw, scale=self.scale, window=self.window)
         heads = workspace.empty((T, nh * vd), dt, dev)
         ops.head_linear(lat, self.m_uv, heads, heads=nh, n_in=kr, n_out=vd, in_head_stride=self.vw, out_head_stride=vd)
         return matmul_tn(heads, self.w_o, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)

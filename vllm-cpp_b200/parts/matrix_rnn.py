@@ -1,4 +1,4 @@
-"""Two recurrent mixers whose state is a matrix per head, S [d, dv] in 32-bit, carried in the request's slot:
+"""Recurrent mixers whose state is a matrix per head, S [d, dv] in 32-bit, carried in the request's slot:
 
 the gated delta rule (``DeltaRuleMixer``)
 
@@ -20,6 +20,7 @@ last taps - 1 inputs per request.  The recurrences run token after token (ops.ma
 """
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from .. import ops, workspace
@@ -260,3 +261,87 @@ class RetentionMixer(_MatrixStateMixer):
                        dv=self.dv, q_col=0, k_col=self.qk, v_col=2 * self.qk, decay=self.decay, ctx_len=ctx.ctx_len,
                        freq=self.freq, rot=self.rot, interleaved=self.interleaved)
         return self._read_out(o, u, 2 * self.qk + self.inner, ctx, x.dtype)
+
+
+class WkvMixer(_MatrixStateMixer):
+    """RWKV-style time mixing: a decay per state row from a low-rank projection and a bonus for the current token:
+
+        m_s = x_t + (x_(t-1) - x_t) mu_s   for s in r, k, v, g, w; x_(t-1) zeros before the request's first token
+        r, k, v = W_r m_r, W_k m_k, W_v m_v,   f = exp(-exp(W_w2 tanh(W_w1 m_w) + w0))       per head and key channel
+        o = (S + diag(u) k v^T)^T r;   S <- diag(f) S + k v^T
+        out = W_o [ gain * o_h / sqrt(mean(o_h^2) + eps) * silu(W_g m_g) ]                   a gain per lane of every head
+
+    params: ``hidden_size``, ``num_heads``, ``head_dim`` (d, of r, k and v alike), ``eps``; ``rank`` (0 or left out: the inner
+    size of the low-rank pair is whatever the checkpoint's tensors have).  Tensors under the prefix: ``mu.r``, ``mu.k``,
+    ``mu.v``, ``mu.g``, ``mu.w`` [H]; ``r``, ``k``, ``v``, ``g`` [heads d, H], ``w1`` [rank, H], ``w2`` [heads d, rank],
+    ``w0`` [heads d], ``u`` [heads, d], ``norm`` [heads d], ``o`` [H, heads d].
+
+    The input is wanted in 32-bit (its norm's ``keep_32bit``): one kernel makes all five mixes from a token's and the
+    previous token's row, in 32-bit, and rounds each once for its product; the last row stays in the request's slot
+    beside the matrices.  In bfloat16 the products of r, k, v and g, which have an input each, are one launch of the
+    grouped product (a group of token tiles per matrix).  The decay, the bonus and the state are 32-bit."""
+
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, params, prefix, build):
+        super().__init__(params, prefix, build)
+        self._sizes(dict(params, v_head_dim=params["head_dim"]))
+        self.rank = int(params.get("rank") or 0)
+        self.inner = self.heads * self.d
+        self.w_in = self.w_1 = self.w_2 = self.w_o = self.mu = self.w0 = self.bonus = self.norm_w = None
+
+    def cache_spec(self):
+        return (CacheSpec("state", shape=(self.heads, self.dv, self.d), dtype="float32"),
+                CacheSpec("state", shape=(self.hidden,), dtype="float32"))
+
+    def tensor_specs(self):
+        p, H, r = self.prefix, self.hidden, self.rank or -1     # -1: any size, as long as both tensors agree
+        return ([TensorSpec(p + "mu." + n, (H,), "unit") for n in self.MIXES]
+                + [TensorSpec(p + n, (self.inner, H)) for n in self.MIXES[:4]]
+                + [TensorSpec(p + "w1", (r, H)), TensorSpec(p + "w2", (self.inner, r)),
+                   TensorSpec(p + "w0", (self.inner,), "bias"), TensorSpec(p + "u", (self.heads, self.d), "bias"),
+                   TensorSpec(p + "norm", (self.inner,), "vector"), TensorSpec(p + "o", (H, self.inner))])
+
+    def bind(self, store):
+        p = self.prefix
+        f32 = lambda name: store.vector(p + name).float().contiguous()
+        self.mu = torch.stack([f32("mu." + n) for n in self.MIXES]).contiguous()
+        # one matrix per mix: the groups of one product
+        self.w_in = store.matrices([p + n for n in self.MIXES[:4]]).view(4, self.inner, self.hidden)
+        self.w_1, self.w_2, self.w_o = store.matrix(p + "w1"), store.matrix(p + "w2"), store.matrix(p + "o")
+        self.rank = int(self.w_1.shape[0])
+        if self.w_2.shape[1] != self.rank:
+            raise ValueError(f"{p}w1 and {p}w2 disagree about the rank of the decay's projection")
+        self.w0, self.bonus, self.norm_w = f32("w0"), f32("u"), f32("norm")
+
+    def forward(self, x, ctx, cache, writes=True):
+        if not writes:
+            raise ValueError("a recurrent mixer keeps a state of its own: it cannot read one another run left")
+        if x.dtype != torch.float32:
+            raise ValueError("this mixer reads its input in 32-bit (its norm's keep_32bit)")
+        state, last = cache[0].state, cache[1].state
+        T, W = x.shape
+        dt, dev = self.build.compute_dtype, x.device
+        n = self.inner
+        tile = next((b for b in ops.GROUPED_TILE_ROWS if T <= b), ops.GROUPED_TILE_ROWS[-1])
+        rows = -(-T // tile) * tile         # token rows of a mix: whole tiles of the grouped product
+        mixes = workspace.empty((len(self.MIXES), rows, W), dt, dev)
+        ops.token_shift(x, self.mu, last, ctx.q_start, ctx.q_len, ctx.slots, ctx.E, mixes)
+        u = workspace.empty((4, rows, n), torch.float32, dev)
+        stacked = mixes[:4].view(4 * rows, W)
+        if ops.gemm_grouped_ok(stacked, self.w_in):
+            groups = ctx.plan(("matrix_of_tile", 4, rows // tile), lambda: ctx.upload(np.repeat(np.arange(4), rows // tile)))
+            ops.gemm_bf16_grouped(self.w_in, stacked, groups, tile, u.view(4 * rows, n), ctx.status)
+        else:
+            product = ops.sgemm_tn if dt == torch.float32 else ops.gemm_bf16_plain
+            for i in range(4):
+                product(mixes[i, :T], self.w_in[i], u[i, :T])
+        low = matmul_tn(mixes[4, :T], self.w_1, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
+        low_act = workspace.empty((T, self.rank), dt, dev)
+        ops.bias_act(low, low_act, "tanh")
+        z = matmul_tn(low_act, self.w_2, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
+        o = workspace.empty((T, n), torch.float32, dev)
+        # r, k and v are row blocks of one buffer: their columns are offsets from a token's row of the first block
+        ops.matrix_rnn("wkv", u[0, :T], state, ctx.q_start, ctx.q_len, ctx.slots, ctx.E, o, heads=self.heads, d=self.d, dv=self.d,
+                       q_col=0, k_col=rows * n, v_col=2 * rows * n, z=z, f_bias=self.w0, bonus=self.bonus)
+        return self._read_out(o, u[3, :T], 0, ctx, dt)

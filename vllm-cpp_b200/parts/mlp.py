@@ -62,20 +62,23 @@ class DenseMLP(FeedForward):
     """down(act(up(y))): one hidden layer, act the exact (erf) GELU unless ``activation`` names another
     ("gelu_erf", "gelu_tanh": 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), "silu", or "polynorm": a n(z) + b n(z^2)
     + c n(z^3) + e with powers lane by lane, n(v) = v / sqrt(mean(v^2) + eps) over a token's hidden lanes and the four
-    learned numbers a, b, c, e).  The hidden layer's sums and the activation are 32-bit; what the down projection reads
+    learned numbers a, b, c, e, or "xielu": a z^2 + z/2 above zero, b (e^z - 1 - z) + z/2 below, a = softplus(p) and b =
+    1/2 + softplus(q) of two learned numbers p, q).  The hidden layer's sums and the activation are 32-bit; what the down projection reads
     is in the compute dtype.
 
     params: ``hidden_size``, ``intermediate_size``; optional ``activation``, ``up_tensor`` and ``down_tensor``
-    (names under the prefix, default "up_proj.weight" and "down_proj.weight"); with "polynorm" also ``act_tensor``
-    (default "act", a tensor [4]) and ``eps``."""
+    (names under the prefix, default "up_proj.weight" and "down_proj.weight"); with "polynorm" and "xielu" also
+    ``act_tensor`` (default "act", a tensor [4] or [2]), with "polynorm" ``eps``."""
+
+    LEARNED = {"polynorm": 4, "xielu": 2}      # activations with numbers of their own, and how many
 
     def __init__(self, params, prefix, build):
         super().__init__(params, prefix, build)
         self.hidden = int(params["hidden_size"])
         self.inter = int(params["intermediate_size"])
         self.activation = str(params.get("activation", "gelu_erf"))
-        if self.activation not in ops.ACTIVATIONS and self.activation != "polynorm":
-            raise ValueError(f"activation '{self.activation}' is not one of {sorted(ops.ACTIVATIONS) + ['polynorm']}")
+        if self.activation not in ops.ACTIVATIONS and self.activation not in self.LEARNED:
+            raise ValueError(f"activation '{self.activation}' is not one of {sorted(ops.ACTIVATIONS) + sorted(self.LEARNED)}")
         self.act_name = prefix + str(params.get("act_tensor", "act"))
         self.eps = float(params.get("eps", 1e-6))
         self.coef = None
@@ -87,15 +90,18 @@ class DenseMLP(FeedForward):
 
     def tensor_specs(self):
         specs = [TensorSpec(self.up_name, (self.inter, self.hidden)), TensorSpec(self.down_name, (self.hidden, self.inter))]
-        if self.activation == "polynorm":
-            specs.append(TensorSpec(self.act_name, (4,), "vector"))
+        if self.activation in self.LEARNED:
+            specs.append(TensorSpec(self.act_name, (self.LEARNED[self.activation],), "vector"))
         return specs
 
     def bind(self, store):
         self.w_up = store.matrix(self.up_name)
         self.w_down = store.matrix(self.down_name)
-        if self.activation == "polynorm":
+        if self.activation in self.LEARNED:
             self.coef = store.vector(self.act_name).float().contiguous()
+        if self.activation == "xielu":
+            p, q = torch.nn.functional.softplus(self.coef.double())
+            self.coef = torch.stack([p, 0.5 + q]).float().contiguous()
 
     def attach_side_rows(self, weight) -> None:
         """Stacks ``weight`` [rows, hidden] under the up projection (after ``bind``): whoever else multiplies the part's
@@ -113,7 +119,7 @@ class DenseMLP(FeedForward):
         if self.activation == "polynorm":
             ops.polynorm(u, self.coef, self.eps, act)
         else:
-            ops.bias_act(u, act, self.activation)
+            ops.bias_act(u, act, self.activation, coef=self.coef)
         return matmul_tn(act, self.w_down, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
 
 

@@ -12,7 +12,8 @@ from .base import Norm
 
 class RMSNorm(Norm):
     """params: ``size``, ``eps``; optional ``name`` (default "weight"); ``one_plus`` (default False): the tensor holds the
-    gain less one (values around zero), y = (1 + w) * x / sqrt(mean(x^2) + eps), the sum made in 32-bit.
+    gain less one (values around zero), y = (1 + w) * x / sqrt(mean(x^2) + eps), the sum made in 32-bit; ``keep_32bit``
+    (default False): the rows are handed on in 32-bit, for a mixer that computes on them before its products read them.
     Tensor: ``<prefix><name>`` [size]."""
 
     def __init__(self, params, prefix, build):
@@ -21,6 +22,7 @@ class RMSNorm(Norm):
         self.eps = float(params["eps"])
         self.name = self.prefix + str(params.get("name", "weight"))
         self.one_plus = bool(params.get("one_plus", False))
+        self.out_dtype = torch.float32 if params.get("keep_32bit", False) else self.build.compute_dtype
         self.weight = None
         self._gain32 = None
 
@@ -40,7 +42,7 @@ class RMSNorm(Norm):
 
     def forward(self, resid, delta, rows=None):
         n = resid.shape[0] if rows is None else rows.numel()
-        out = workspace.empty((n, self.size), self.build.compute_dtype, resid.device)
+        out = workspace.empty((n, self.size), self.out_dtype, resid.device)
         if delta is not None and not torch.is_tensor(delta):
             # what the arrangement before left is more than a sum to add (a result still to be normed and scaled, say):
             # it knows the kernel that does its addition and this norm in one pass

@@ -35,6 +35,7 @@ from .. import ops, workspace
 from ..weights.loader import TensorSpec
 from .attention import (CLUSTER_MERGE, DECODE_ROWS, MMA_DECODE_ROWS, MMA_SPAN_ROWS, SPAN_ROWS, TCGEN05_SPANS,
                         AttentionPlan)
+from .parallel_block import PendingSum
 from .base import CacheSpec, Mixer
 from .linear import matmul_tn
 
@@ -43,19 +44,25 @@ from .linear import matmul_tn
 MMA_ATTENTION = os.environ.get("VLLM_CPP_B200_WINDOW_ATTN_MMA", "1") != "0"
 # whether the tensor-core kernels take the cap, the slope and the sink (else steps with them run on the plain kernel)
 EXTRAS_ON_TENSOR_CORES = True
+# query lanes up to which the plain kernel keeps 32 rows of a prompt portion in a block's shared memory
+PLAIN_SPAN_LANES = 1280
 # whether they take a sink with a learned score per head (else such steps run on the plain kernel)
 SINK_SCORES_ON_TENSOR_CORES = True
 
 
 def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_first=0, dist_a=None, dist_b=None,
-                    softcap=0.0, slope=None, sink=False):
+                    softcap=0.0, slope=None, sink=False, chunked=False, wide=False, out_gate=None):
     """(``sink``: False, True -- a silent key of score 0 --, or a float32 tensor [nh] of the silent key's score per head.)
     Scores, softmax and weighted sums of one step over the paged keys and values ``kv``: ``q`` [T, nh * hd] against
     keys of ``hd`` lanes, values of ``vd`` lanes into ``out`` [T, nh * vd].  Single tokens are cut into key slices and
     merged, prompt portions into row tiles; bfloat16 with keys and values of 64 or 128 lanes runs on the tensor cores
     (tcgen05 for prompt portions where the page size allows, mma.sync for decoded tokens), everything else on the
     plain kernel.  Whoever keeps its keys in pages of this layout calls this (the window attention below; attention
-    over latent rows, whose one KV head's values are the first lanes of its keys)."""
+    over latent rows, whose one KV head's values are the first lanes of its keys).
+    ``chunked``: the window is the chunk of ``window`` positions, counted from position 0, that a query lies in.
+    ``wide``: ``q`` is [T, nh * nkv * hd], a block of lanes per KV head, and a row's score with a key position is the sum
+    of the blocks' products with all heads' keys there (queries mixed across heads).  ``out_gate`` (float32 [T, nh])
+    multiplies each head's result."""
     x = q
     # no query reads more keys than the window and the kept first ones: no more key slices than those fill
     reach = window + keep_first if window else 0
@@ -65,13 +72,23 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     has_extras = bool(softcap or slope is not None or learned_sink or sink)
     mma = (MMA_ATTENTION and vd == hd and kv.pages.dim() == 5 and ops.attn_mma_supported(x.dtype, hd)
            and (EXTRAS_ON_TENSOR_CORES or not has_extras) and (SINK_SCORES_ON_TENSOR_CORES or not learned_sink))
-    dec_rows, span_rows = (MMA_DECODE_ROWS, MMA_SPAN_ROWS) if mma else (DECODE_ROWS, SPAN_ROWS)
+    mma_rows = MMA_SPAN_ROWS
+    if mma and wide:
+        mma_rows = ops.attn_mma_wide_rows(x.dtype, hd, nkv)
+        mma = mma_rows > 0
+    dec_rows, span_rows = (MMA_DECODE_ROWS, mma_rows) if mma else (DECODE_ROWS, SPAN_ROWS)
+    if not mma and (nkv * hd if wide else hd) > PLAIN_SPAN_LANES:
+        span_rows = DECODE_ROWS      # fewer rows a block: its query rows lie in shared memory
     clustered = hd if mma and CLUSTER_MERGE and torch.cuda.is_available() else None
     group = ctx.groups[kv.group]
-    plan = ctx.plan(("attention", nh, nkv, mma, clustered, reach),
+    tcgen05 = mma and TCGEN05_SPANS and (ops.attn_tc_wide_supported(x.dtype, hd, kv.pages.shape[3], nkv) if wide
+                                         else ops.attn_tc_supported(x.dtype, hd, kv.pages.shape[3]))
+    if tcgen05:
+        span_rows = MMA_SPAN_ROWS
+    plan = ctx.plan(("attention", nh, nkv, mma, clustered, reach, span_rows),
                     lambda: AttentionPlan(ctx, nh, nkv, dec_rows, span_rows, clustered, max_keys=reach))
     common = dict(nh=nh, nkv=nkv, hd=hd, window=window, status=ctx.status, table_row=ctx.slots, scale=scale,
-                  keep_first=keep_first, dist_a=dist_a, dist_b=dist_b, **extras)
+                  keep_first=keep_first, dist_a=dist_a, dist_b=dist_b, chunked=chunked, wide=wide, out_gate=out_gate, **extras)
     args = (q, out, kv.pages, group.block_table, ctx.q_start, ctx.q_len, ctx.ctx_len)
     if plan.n_dec:
         S = plan.nslices
@@ -87,9 +104,9 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
         else:
             ops.attn_window_bias(*args, plan.dec_items, plan.n_dec * S, dec_rows, part_o, part_ml, hd_v=vd, **common)
             if S > 1:
-                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S)
+                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S, out_gate)
     if plan.n_span_items:
-        if mma and TCGEN05_SPANS and ops.attn_tc_supported(x.dtype, hd, kv.pages.shape[3]):
+        if tcgen05:
             ops.attn_tc(*args, plan.span_items, plan.n_span_items, work=plan.span_work, **common)
         elif mma:
             ops.attn_mma(*args, plan.span_items, plan.n_span_items, span_rows, None, None, **common)
@@ -215,7 +232,8 @@ def rotary_frequencies(build, base: float, dims: int) -> torch.Tensor:
 class RotaryWindowAttention(Mixer):
     """Grouped-query softmax attention with rotary positions, every variation a parameter:
 
-        q, k, v = W_q x, W_k x, W_v x                 (one stacked product; no biases)
+        q, k, v = W_q x, W_k x, W_v x                 (one stacked product)
+        ``bias``:             a bias on each of the three and on the output projection
         ``values_from_keys``: there is no W_v; v = k as projected, before any norm or rotation (v_head_dim = head_dim)
         ``whole_norm``:       q <- g_q * q / rms(q) over all of a token's query lanes at once, k likewise with g_k
         the first ``rotary_dim`` lanes of every q and k head turn by position * base^(-2i / rotary_dim), lanes paired
@@ -224,13 +242,23 @@ class RotaryWindowAttention(Mixer):
                               base^(-2m / v_head_dim)) and is cached so; a head's weighted sum at position i is turned
                               back by i, which leaves every value turned by j - i
         s_ij = scale * (q_i . k_j);  i sees j iff 0 <= i - j < window (window 0: every j <= i)
+        ``chunked``:          the window stands still: i sees j <= i in its own chunk of ``window`` positions, counted from
+                              position 0 of the request
+        ``unit_values``:      every value head divided by its root mean square (no gain) and cached so
+        ``talk``:             the heads' scores mixed before the softmax, s_h <- sum_g talk[h, g] s_g
+        ``head_gate``:        head h's weighted sum is multiplied by sigmoid(W_g x)_h
         ``sink``:             exp(sink_h), a learned score per head that is not scaled, joins the softmax's denominator
         softmax, weighted sum of the values, output projection.
 
     params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``v_head_dim`` (default head_dim), ``scale``,
     ``window``, ``rope_base``, ``rotary_dim``, ``pairing``, ``eps`` and the flags above (all default False).
     Tensors under ``<prefix>``: q [nh hd, H], k [nkv hd, H], v [nkv vd, H] (unless values_from_keys), o [H, nh vd];
-    q.norm [nh hd], k.norm [nkv hd] (whole_norm); sink [nh] (sink).
+    q.norm [nh hd], k.norm [nkv hd] (whole_norm); sink [nh] (sink); q.b, k.b, v.b, o.b (bias); talk [nh, nh] (talk);
+    g [nh, H] (head_gate).
+
+    Mixed scores cost the attention kernels no look at one another's heads: the sum over g is drawn into the queries (see
+    csrc/kernels/rope_store.cu), whose rows then have a block of lanes per KV head.  The mixing itself is 32-bit.  The
+    output projection's bias is not added here but handed on with the result.
 
     Norms, angles, scores and softmax are 32-bit; queries, keys and values are stored in the compute dtype.  Keys and
     values lie in pages that are given back as the window passes."""
@@ -252,6 +280,14 @@ class RotaryWindowAttention(Mixer):
         self.whole_norm = bool(p.get("whole_norm", False))
         self.rotate_values = bool(p.get("rotate_values", False))
         self.has_sink = bool(p.get("sink", False))
+        self.chunked = bool(p.get("chunked", False)) and self.window > 0
+        self.has_bias = bool(p.get("bias", False))
+        self.unit_values = bool(p.get("unit_values", False))
+        self.has_talk, self.has_gate = bool(p.get("talk", False)), bool(p.get("head_gate", False))
+        if self.has_talk and self.whole_norm:
+            raise ValueError("mixed scores come without a norm over the whole projection")
+        if self.has_bias and self.values_from_keys:
+            raise ValueError("keys that double as values come without biases")
         if self.nh % self.nkv:
             raise ValueError(f"{self.nh} query heads are not a multiple of {self.nkv} KV heads")
         if self.values_from_keys and self.vd != self.hd:
@@ -261,15 +297,15 @@ class RotaryWindowAttention(Mixer):
         if self.rotate_values and self.vd % 2:
             raise ValueError(f"values of {self.vd} lanes cannot turn in pairs")
         for n in (self.hd, self.vd):
-            if not 1 <= n <= 256:
-                raise ValueError(f"head size {n} is not supported: the kernels take 1 to 256")
+            if n < 1:
+                raise ValueError(f"head size {n} is not supported")
         base = float(p.get("rope_base", 10000.0))
         self.freq = rotary_frequencies(build, base, self.rot) if self.rot else None
         self.vfreq = rotary_frequencies(build, base, self.vd) if self.rotate_values else None
-        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.sink = None
+        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.sink = self.bias = self.o_bias = self.talk = None
 
     def cache_spec(self):
-        return CacheSpec("kv", num_kv_heads=self.nkv, head_dim=self.hd, window=self.window,
+        return CacheSpec("kv", num_kv_heads=self.nkv, head_dim=self.hd, window=self.window, chunked=self.chunked,
                          v_head_dim=0 if self.vd == self.hd else self.vd)
 
     def _rows(self):
@@ -283,17 +319,29 @@ class RotaryWindowAttention(Mixer):
             specs += [TensorSpec(p + "q.norm", (self.nh * self.hd,), "vector"), TensorSpec(p + "k.norm", (self.nkv * self.hd,), "vector")]
         if self.has_sink:
             specs.append(TensorSpec(p + "sink", (self.nh,), "bias"))
+        if self.has_bias:
+            specs += [TensorSpec(p + n + ".b", (r,), "bias") for n, r in self._rows() + [("o", H)]]
+        if self.has_talk:
+            specs.append(TensorSpec(p + "talk", (self.nh, self.nh), "mixing"))
+        if self.has_gate:
+            specs.append(TensorSpec(p + "g", (self.nh, H)))
         return specs
 
     def bind(self, store):
         p = self.prefix
         f32 = lambda name: store.vector(p + name).float().contiguous()
-        self.w_qkv = store.matrices([p + n for n, _ in self._rows()])
+        # the gates' rows under the projections': one product
+        self.w_qkv = store.matrices([p + n for n, _ in self._rows()] + ([p + "g"] if self.has_gate else []))
         self.w_o = store.matrix(p + "o")
         if self.whole_norm:
             self.q_gain, self.k_gain = f32("q.norm"), f32("k.norm")
         if self.has_sink:
             self.sink = f32("sink")
+        if self.has_bias:
+            self.bias = torch.cat([f32(n + ".b") for n, _ in self._rows()]).contiguous()
+            self.o_bias = f32("o.b")
+        if self.has_talk:
+            self.talk = f32("talk")
 
     def forward(self, x, ctx, cache, writes=True):
         if not writes:
@@ -303,13 +351,16 @@ class RotaryWindowAttention(Mixer):
         nh, nkv, hd, vd = self.nh, self.nkv, self.hd, self.vd
         group = ctx.groups[kv.group]
         qkv = matmul_tn(x, self.w_qkv, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
-        q = workspace.empty((T, nh * hd), x.dtype, x.device)
+        q = workspace.empty((T, nh * hd * (nkv if self.has_talk else 1)), x.dtype, x.device)
+        gate = workspace.empty((T, nh), torch.float32, x.device) if self.has_gate else None
         ops.qkv_rope_store(qkv, self.q_gain, self.k_gain, self.eps, ctx.positions, self.freq, self.vfreq, group.slot_map, q,
                            kv.pages, nh, nkv, hd, vd, ctx.status, rot=self.rot, interleaved=self.interleaved,
-                           values_from_keys=self.values_from_keys)
+                           values_from_keys=self.values_from_keys, bias=self.bias, unit_values=self.unit_values, talk=self.talk,
+                           gate_out=gate)
         out = workspace.empty((T, nh * vd), x.dtype, x.device)
         paged_attention(ctx, kv, q, out, nh=nh, nkv=nkv, hd=hd, vd=vd, scale=self.scale, window=self.window,
-                        sink=self.sink if self.has_sink else False)
+                        sink=self.sink if self.has_sink else False, chunked=self.chunked, wide=self.has_talk, out_gate=gate)
         if self.rotate_values:
             ops.rotate_heads(out, ctx.positions, self.vfreq, heads=nh, width=vd, dims=vd, interleaved=self.interleaved, sign=-1.0)
-        return matmul_tn(out, self.w_o, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
+        y = matmul_tn(out, self.w_o, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
+        return y if self.o_bias is None else PendingSum([y], vec_extra=self.o_bias)
