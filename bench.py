@@ -1,7 +1,7 @@
 #!/usr/bin/env python3
 """Benchmark of the engine on one B200.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--workloads all|headline|14b|4b|rimopel|nagavik|fifudra|mefupel] [--impl reference]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--workloads all|headline|14b|4b|rimopel|nagavik|fifudra|mefupel|nufetar] [--impl reference]
 
 Headline: decode tokens/s of the Qwen3-8B layer sizes (the baseline's third configuration) at batch 8 and context
 4,096, the median of K device-timed steps after W warm-up steps; beside it batch 1 and 64, batch 8 at context 2,176
@@ -799,6 +799,82 @@ def run_mefupel(args, pk, clocks, windows):
     return run_beside(args, pk, clocks, windows, "mefupel_beside_fifudra", MEFUPEL_SIZES, configs, numbers)
 
 
+# Nufetar at real layer sizes beside Mefupel, the closest design the engine has (recurrences on a matrix state per head with
+# a decay per state row from a low-rank projection, window attention with rotary positions), at equal width, layer count,
+# heads, recurrent state per request and feed-forward parameters: a wkv layer, a latent attention layer, a layer of
+# attention in chunks with mixed scores, and so on, each with a dense feed-forward of two matrices; Mefupel with a gated
+# linear attention layer and two window attention layers in turn.  The chunk is chosen so that a decoded token behind
+# 4,096 others sees 1,280 keys and more of its own chunk, about as many as a window holds.
+NUFETAR_SIZES = {
+    "w2048": dict(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, chunk=1408, window=1344, rot=64,
+                  l_dim=96, l_rot=32, kv_rank=96, r_heads=32, r_dim=64, rank=64, ff=6144),
+    "w4096": dict(width=4096, layers=8, vocab=32768, heads=32, kv_heads=8, dim=128, chunk=1408, window=1344, rot=64,
+                  l_dim=96, l_rot=32, kv_rank=96, r_heads=64, r_dim=64, rank=128, ff=12288),
+    # half as many KV heads: query rows that stay in shared memory once mixed
+    "w4096_kv4": dict(width=4096, layers=8, vocab=32768, heads=32, kv_heads=4, dim=128, chunk=1408, window=1344, rot=64,
+                      l_dim=96, l_rot=32, kv_rank=96, r_heads=64, r_dim=64, rank=128, ff=12288),
+}
+
+
+def run_nufetar(args, pk, clocks, windows):
+    """Nufetar at real layer sizes beside Mefupel at equal size (see NUFETAR_SIZES and run_beside)."""
+    from vllm_cpp_b200.config.mefupel import AttentionSpec, GlaSpec, MefupelConfig, MefupelLayer, MefupelMlp
+    from vllm_cpp_b200.config.mefupel import Rotation as MefupelRotation
+    from vllm_cpp_b200.config.nufetar import (ChunkAttentionSpec, LatentSpec, NufetarConfig, NufetarLayer, NufetarMlp, Rotation,
+                                              WkvSpec)
+    context, T = args.context, PREFILL_TOKENS
+
+    def kinds(z):
+        return [("wkv", "latent_attention", "attention")[i % 3] for i in range(z["layers"])]
+
+    def mefupel_kinds(z):
+        return [("gla", "attention", "attention")[i % 3] for i in range(z["layers"])]
+
+    def configs(z):
+        H, G, d, RH, rd = z["heads"], z["kv_heads"], z["dim"], z["r_heads"], z["r_dim"]
+        mixers = {"wkv": WkvSpec(heads=RH, dim=rd, rank=z["rank"]),
+                  "latent_attention": LatentSpec(heads=H, dim=z["l_dim"], rot_dim=z["l_rot"], vdim=d, kv_rank=z["kv_rank"],
+                                                 scale=(z["l_dim"] + z["l_rot"]) ** -0.5, window=z["window"], rot=Rotation(1e6, z["l_rot"])),
+                  "attention": ChunkAttentionSpec(heads=H, kv_heads=G, dim=d, vdim=d, scale=d ** -0.5, chunk=z["chunk"],
+                                                  rot=Rotation(1e6, z["rot"]))}
+        nuf = NufetarConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, max_positions=context + 4096,
+                            layers=tuple(NufetarLayer(k, mixers[k], NufetarMlp("dense", z["ff"])) for k in kinds(z)))
+        mmix = {"gla": GlaSpec(heads=RH, dim=rd, vdim=rd, tau=16.0, rank=z["rank"]),
+                "attention": AttentionSpec(heads=H, kv_heads=G, dim=d, vdim=d, scale=d ** -0.5, window=z["window"],
+                                           rot=MefupelRotation(1e6, z["rot"]))}
+        mef = MefupelConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, max_positions=context + 4096,
+                            layers=tuple(MefupelLayer(k, mmix[k], MefupelMlp("dense", z["ff"])) for k in mefupel_kinds(z)))
+        return {"nufetar": nuf, "mefupel": mef}
+
+    def numbers(z, name):
+        W, V, L = z["width"], z["vocab"], z["layers"]
+        H, G, d, RH, rd = z["heads"], z["kv_heads"], z["dim"], z["r_heads"], z["r_dim"]
+        kr, ld, lr = z["kv_rank"], z["l_dim"], z["l_rot"]
+        inner = RH * rd
+        state_bytes = 2 * 4 * RH * rd * rd              # read and written, 32-bit
+        attn_w = (H + 2 * G) * d * W + W * H * d
+        w = {"attention": attn_w, "gla": 4 * inner * W + z["rank"] * (W + inner) + W * inner,
+             "wkv": 4 * inner * W + z["rank"] * (W + inner) + W * inner,
+             "latent": (H * (ld + lr) + kr + lr) * W + H * ld * kr + H * d * kr + W * H * d}
+        names = kinds(z) if name == "nufetar" else mefupel_kinds(z)
+        n = {k: names.count(k) for k in ("attention", "gla", "wkv", "latent_attention")}
+        weights = (n["attention"] * (w["attention"] + (H * W if name == "nufetar" else 0)) + n["gla"] * w["gla"] + n["wkv"] * w["wkv"]
+                   + n["latent_attention"] * w["latent"] + L * 2 * z["ff"] * W)
+        in_window = sum(min(i + 1, z["window"]) for i in range(T))
+        in_chunk = sum(i % z["chunk"] + 1 for i in range(T))
+        seen, keys = (in_chunk, context % z["chunk"]) if name == "nufetar" else (in_window, min(context, z["window"]))
+        # scores (mixed: H more multiply-adds each) and weighted sums
+        attn_flops = 2.0 * H * (2 * d + (H if name == "nufetar" else 0)) * seen
+        rec = n["gla"] + n["wkv"]
+        return dict(weight_bytes=2 * (weights + V * W),
+                    cache_bytes=n["attention"] * 2 * G * d * 2 * keys + n["latent_attention"] * (2 * kr + lr) * 2 * min(context, z["window"])
+                                + rec * state_bytes,
+                    prefill_flops=2.0 * T * weights + 2.0 * V * W + n["attention"] * attn_flops
+                                  + n["latent_attention"] * 2.0 * H * (2 * kr + lr) * in_window + 4.0 * rec * T * RH * rd * rd)
+
+    return run_beside(args, pk, clocks, windows, "nufetar_beside_mefupel", NUFETAR_SIZES, configs, numbers)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -810,11 +886,11 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=CONTEXT)
     ap.add_argument("--impl", default="ours")
-    ap.add_argument("--workloads", default="all", choices=["all", "headline", "14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel"],
+    ap.add_argument("--workloads", default="all", choices=["all", "headline", "14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel", "nufetar"],
                     help="headline: the 8B numbers only; 14b / 4b: that workload alone (prints its own JSON line); rimopel, "
                          "nagavik: that design at real layer sizes beside Qwen3 at equal size, prefill and decode (its own JSON line); "
-                         "fifudra: that design beside Nagavik at equal size, likewise; mefupel: that design beside Fifudra at equal size, likewise")
-    ap.add_argument("--size", default="", help="rimopel, nagavik, fifudra, mefupel: one of the workload's sizes only (w2048, w4096; fifudra also w2048_k256)")
+                         "fifudra: that design beside Nagavik at equal size, likewise; mefupel: that design beside Fifudra at equal size, likewise; nufetar: that design beside Mefupel at equal size, likewise")
+    ap.add_argument("--size", default="", help="rimopel, nagavik, fifudra, mefupel, nufetar: one of the workload's sizes only (w2048, w4096; fifudra also w2048_k256)")
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (for profiling runs)")
     ap.add_argument("--no-graphs", action="store_true", help="launch decode steps kernel by kernel (for profiling runs)")
     ap.add_argument("--mode", default="all", choices=["all", "decode", "prefill"], help="what to run (profiling runs)")
@@ -836,8 +912,9 @@ def main():
     clocks.start()
     windows = []
     try:
-        if args.workloads in ("14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel"):
-            out = {"14b": run_14b, "4b": run_4b, "rimopel": run_rimopel, "nagavik": run_nagavik, "fifudra": run_fifudra, "mefupel": run_mefupel}[args.workloads](args, pk, clocks, windows)
+        if args.workloads in ("14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel", "nufetar"):
+            out = {"14b": run_14b, "4b": run_4b, "rimopel": run_rimopel, "nagavik": run_nagavik, "fifudra": run_fifudra, "mefupel": run_mefupel,
+                   "nufetar": run_nufetar}[args.workloads](args, pk, clocks, windows)
             out["clocks"] = clocks.summary(windows)
             print(json.dumps(out))
             return 0

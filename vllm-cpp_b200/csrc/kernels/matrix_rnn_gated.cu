@@ -1,0 +1,4 @@
+// The kernels of the gated linear form (matrix_rnn.cuh).
+#include "matrix_rnn.cuh"
+
+template int vcb_rnn::rnn_run<vcb_rnn::MODE_GATED>(const vcb_rnn::RnnArgs&, int, int, bool, dim3, size_t, cudaStream_t);
