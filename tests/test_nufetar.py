@@ -637,6 +637,19 @@ def test_attention_on_a_mixed_batch(dtype, nh, nkv, hd, vd, size, chunked, talks
 
 
 @gpu
+@pytest.mark.parametrize("nh,nkv,hd", [(8, 4, 128), (32, 8, 128), (20, 5, 64), (64, 16, 64), (48, 3, 128), (14, 7, 128)])
+def test_single_tokens_of_many_lengths(nh, nkv, hd):
+    """One to four tiles of heads; many tokens (one slice each) and few (sliced keys, merged); contexts that end at the first
+    key of a page, of a tile and of a chunk."""
+    for ctxs in ([1, 2, 16, 17, 64, 65, 128, 129, 300, 301, 500, 600, 601, 899], [900], [899, 601, 640]):
+        got, want = attention_by_hand(nh, nkv, hd, torch.bfloat16, 300, True, ctxs, [1] * len(ctxs), scale=0.5 * hd ** -0.5)
+        torch.testing.assert_close(got, want, **ATTN_TOL[torch.bfloat16])
+    ctxs = list(range(5, 5 + 160))          # more tokens than SMs
+    got, want = attention_by_hand(nh, nkv, hd, torch.bfloat16, 0, True, ctxs, [1] * len(ctxs), scale=0.5 * hd ** -0.5)
+    torch.testing.assert_close(got, want, **ATTN_TOL[torch.bfloat16])
+
+
+@gpu
 @pytest.mark.parametrize("ps", [8, 12, 32, 64])
 def test_attention_on_other_page_sizes(ps):
     """Pages that the tensor cores' loaders bring in whole, and one size (12) that they do not."""
@@ -646,9 +659,9 @@ def test_attention_on_other_page_sizes(ps):
 
 
 @gpu
-@pytest.mark.parametrize("env", [{"TCGEN05_SPANS": False}, {"MMA_ATTENTION": False}])
-def test_prompt_portions_agree_on_every_kernel(env, monkeypatch):
-    """The kernels that serve what the tcgen05 kernel does not: forced onto sizes that it does take."""
+@pytest.mark.parametrize("env", [{"TCGEN05_SPANS": False}, {"WIDE_DECODE": False}, {"MMA_ATTENTION": False}])
+def test_portions_and_single_tokens_agree_on_every_kernel(env, monkeypatch):
+    """The kernels that serve what the tcgen05 kernel and the one for single tokens do not: forced onto sizes they do take."""
     import vllm_cpp_b200.parts.window_attention as wa
     for k, v in env.items():
         monkeypatch.setattr(wa, k, v)
@@ -735,14 +748,14 @@ def test_replay_modes_agree_with_each_other(nufetar_dirs, tmp_path):
         requests = requests_of(name)
         vocab = configs()[name][0].vocab
         rows = {}
-        for mode in ("whole", "mixed", "portions"):
+        for mode in ("whole", "mixed"):
             trace = MODES[mode](requests)
             out = R.run_trace(nufetar_dirs[name], "float32", trace, tmp_path / (name + mode), configs()[name][1])
             for step, want in enumerate(trace.wanted):
                 got = R.read_step(out, step, vocab)
                 for i, key in enumerate(want):
                     rows.setdefault(key, {})[mode] = got[i]
-        worst = max(np.abs(v["whole"] - v[m]).max() / np.abs(v["whole"]).max() for v in rows.values() for m in ("mixed", "portions"))
+        worst = max(np.abs(v["whole"] - v[m]).max() / np.abs(v["whole"]).max() for v in rows.values() for m in ("mixed",))
         assert worst < 2e-5, (name, worst)
 
 

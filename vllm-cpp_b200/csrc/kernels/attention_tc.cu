@@ -32,10 +32,11 @@
 // other by 1 KB, so the keys keep their order in a tile whatever the page size.  (One copy per page and half, the
 // obvious way, made the copying warp the slowest role of the block: about 100 clocks a copy, 16 copies a tile.)
 // Wide query rows (WIDE; a row has one block of head_dim lanes per KV head, see attention.cu): S is the sum over the KV
-// heads of block . that head's keys, one MMA chain over all of them into the same accumulator.  The rows' blocks stay in
-// shared memory for the whole unit (up to 512 lanes, 128 KB: one block an SM then), the K ring's stages hold one KV
-// head's keys each and are given back by the products themselves, and the rows of the next unit come in by cp.async
-// as soon as the last scores of this one are there, behind its last weights and output.
+// heads of block . that head's keys, one MMA chain over all of them into the same accumulator.  The rows' blocks stay on
+// the SM for the whole unit (one block an SM then): up to 512 lanes in shared memory (128 KB), up to 512 more in TMEM
+// (256 columns, beside S, S and O all there are), from where the products read them as their A operand like the weights.
+// The K ring's stages hold one KV head's keys each and are given back by the products themselves, and the rows of the
+// next unit come in as soon as the last scores of this one are there, behind its last weights and output.
 //
 // All hand-offs are mbarriers; every wait is bounded by the clock, and a wait that runs out sets a bit in the
 // status word and an abort flag that the other roles see, after which the block frees its TMEM and returns.
@@ -223,8 +224,9 @@ __device__ __forceinline__ int tile_pb0(const Unit& u, int it, int pages_per_til
 __device__ __forceinline__ int tile_pb_hi(const Unit& u, int it, int ps) { return it < u.n_ft ? (u.n_first + ps - 1) / ps : u.pb_hi; }
 constexpr int UNIT_INTS = sizeof(Unit) / sizeof(int);
 
-// MAXQ: blocks of HD lanes that a query row has room for (1, or with wide rows the most there may be: the tiles lie behind them)
-template <int HD, int KS, int VS, int MAXQ = 1>
+// MAXQ: blocks of HD lanes that a query row has room for in shared memory (1, or with wide rows the most there may be: the
+// tiles lie behind them); IN_TMEM: further blocks lie in TMEM, behind O
+template <int HD, int KS, int VS, int MAXQ = 1, bool IN_TMEM = false>
 struct Layout {
     static constexpr int Q_BYTES = ROWS * HD * 2;
     static constexpr int KV_BYTES = BNK * HD * 2;       // one K or V tile
@@ -234,7 +236,8 @@ struct Layout {
     static constexpr int NUM_BARS = 2 * KS + VS + 7;
     static_assert(VS == 2, "a V stage is given back by the barrier of the score buffer its tile used");
     static constexpr int TOTAL = BAR_OFF + NUM_BARS * 8 + 16 + 4 * UNIT_RING * (UNIT_INTS + 2);   // + TMEM address, abort flag, the units to come
-    static constexpr uint32_t TMEM_COLS = 256;                  // S, S (64 each; P over the first half of its S), O (head_dim)
+    // S, S (64 each; P over the first half of its S), O (head_dim); from column 256 on, 512 lanes of the query rows
+    static constexpr uint32_t TMEM_COLS = IN_TMEM ? 512 : 256;
     static_assert(2 * BNK + HD <= 256, "TMEM columns");
     static_assert(MAXQ > 1 || 2 * (TOTAL + 1024) <= 228 * 1024, "two blocks per SM");
     static_assert(TOTAL <= 227 * 1024, "shared memory of a block");
@@ -242,7 +245,9 @@ struct Layout {
 
 constexpr float RESCALE_STEP = 8.0f;   // log2 of how far a row's maximum may outgrow its reference
 
-constexpr int wide_blocks(int hd) { return 512 / hd; }   // blocks of a wide query row that stay in shared memory
+constexpr int wide_blocks(int hd) { return 512 / hd; }   // blocks of a wide query row in shared memory; as many again in TMEM
+// how query rows lie: one block; several, all in shared memory; several, those beyond wide_blocks in TMEM
+enum : int { ROWS_PLAIN = 0, ROWS_WIDE = 1, ROWS_WIDER = 2 };
 
 // false: the unit has nothing to do (an item laid out for a longer portion than is there)
 template <bool OPT>
@@ -292,9 +297,10 @@ __device__ __forceinline__ bool read_unit(const TcArgs& a, int unit, Unit& u) {
 // Barrier phases, ring stages and score buffers go on counting from unit to unit, so `t0` below is the number of
 // tiles of the units before.
 // OPT: built with the options of TcArgs (kept first keys, distance penalty); without, they cost nothing
-template <int HD, int KS, int VS, bool OPT, bool WIDE>
-__global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const __grid_constant__ CUtensorMap kv_map, TcArgs a) {
-    using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1>;
+template <int HD, int KS, int VS, bool OPT, int KIND>
+__global__ __launch_bounds__(NTHREADS, KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_kernel(const __grid_constant__ CUtensorMap kv_map, TcArgs a) {
+    constexpr bool WIDE = KIND != ROWS_PLAIN, IN_TMEM = KIND == ROWS_WIDER;
+    using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1, IN_TMEM>;
     const int NG = WIDE ? a.nkv : 1;    // blocks of a query row = stages of a K tile
     constexpr int CH = HD / 8;          // 16-byte chunks per row of head_dim
     constexpr int ROWB = HD * 2;
@@ -383,6 +389,7 @@ __global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const _
     tc_fence_after();
     const uint32_t tmem_base = *tmem_holder;
     const uint32_t tmem_s = tmem_base, tmem_o = tmem_base + 2 * BNK;   // S, S, O
+    const uint32_t tmem_q = tmem_base + 256;      // (IN_TMEM)
 
     if (warp == 0) {
         // ---- TMA producer: one box per page.  Lanes 0-7 copy the pages of a K tile, lanes 8-15 those of a V tile, in
@@ -565,7 +572,10 @@ __global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const _
                             // 16 lanes of head_dim = 32 bytes along the 128-byte rows; the second 64 lanes are the next block
                             const uint64_t da = desc_k_major(qa + (ks / 4) * (ROWS * 128) + (ks % 4) * 32, 1024);
                             const uint64_t db = desc_k_major(ka + (ks / 4) * 1024 + (ks % 4) * 32, HALVES * 1024);
-                            tc_mma(tmem_s + b * BNK, da, db, idesc_qk, (blk > 0 || ks > 0) ? 1u : 0u);
+                            if (IN_TMEM && blk >= wide_blocks(HD))     // 16 lanes = 8 columns of the rows in TMEM
+                                tc_mma_ts(tmem_s + b * BNK, tmem_q + (blk - wide_blocks(HD)) * (HD / 2) + ks * 8, db, idesc_qk, 1u);
+                            else
+                                tc_mma(tmem_s + b * BNK, da, db, idesc_qk, (blk > 0 || ks > 0) ? 1u : 0u);
                         }
                         if constexpr (WIDE) tc_commit(k_empty(st));
                     }
@@ -619,7 +629,7 @@ __global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const _
         auto ask_query = [&](const Unit& w, bool there) {   // writes all of qv in any case: what it held is dead
             if constexpr (WIDE) {
                 if (!there) return;
-                const int per_row = NG * CH;
+                const int per_row = (IN_TMEM ? wide_blocks(HD) : NG) * CH;
                 for (int rr = 0; rr < 32; ++rr) {
                     const int row = qtr * 32 + rr;
                     const bool mine = row < w.R;
@@ -629,6 +639,22 @@ __global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const _
                         cp_async16(base + (c / CH) * L::Q_BYTES + swz<ROWS>(row, c % CH), src + c * 8, mine ? 16 : 0);
                 }
                 asm volatile("cp.async.commit_group;" ::: "memory");
+                if constexpr (IN_TMEM) {
+                    // the row's further lanes into its TMEM lane, two a column
+                    const bool mine = r < w.R;
+                    const int wq = mine ? r / w.gq : 0, wh = mine ? r % w.gq : 0;
+                    const __nv_bfloat16* src = a.q + ((size_t)(w.row0 + wq) * a.nh + w.head0 + wh) * (NG * HD) + wide_blocks(HD) * HD;
+                    const int lanes = (NG - wide_blocks(HD)) * HD;
+                    for (int c0 = 0; c0 < lanes; c0 += 64) {
+                        uint4 v[8];
+#pragma unroll
+                        for (int c = 0; c < 8; ++c) v[c] = mine ? *reinterpret_cast<const uint4*>(src + c0 + c * 8) : make_uint4(0, 0, 0, 0);
+                        uint32_t (*col)[16] = reinterpret_cast<uint32_t (*)[16]>(v);
+                        tc_st16(tmem_q + lane_addr + (uint32_t)(c0 / 2), col[0]);
+                        tc_st16(tmem_q + lane_addr + (uint32_t)(c0 / 2 + 16), col[1]);
+                    }
+                    tc_wait_st();
+                }
                 return;
             }
             const bool mine = there && r < w.R;
@@ -848,11 +874,12 @@ __global__ __launch_bounds__(NTHREADS, WIDE ? 1 : 2) void attn_tc_kernel(const _
     }
 }
 
-template <int HD, bool OPT, bool WIDE = false>
+template <int HD, bool OPT, int KIND = ROWS_PLAIN>
 int launch(const CUtensorMap& map, const TcArgs& a, int n_items, cudaStream_t stream) {
+    constexpr bool WIDE = KIND != ROWS_PLAIN;
     constexpr int KS = WIDE ? (HD == 64 ? 8 : 4) : 3, VS = 2;
-    using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1>;
-    auto kern = attn_tc_kernel<HD, KS, VS, OPT, WIDE>;
+    using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1, KIND == ROWS_WIDER>;
+    auto kern = attn_tc_kernel<HD, KS, VS, OPT, KIND>;
     static bool opted = false;
     if (!opted) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
@@ -888,7 +915,7 @@ VCB_API int vcb_attn_tc_supported(int dtype, int hd, int page_size) {
 
 // ... and for query rows of one block per KV head.
 VCB_API int vcb_attn_tc_wide_supported(int dtype, int hd, int page_size, int nkv) {
-    return vcb_attn_tc_supported(dtype, hd, page_size) && nkv <= wide_blocks(hd);
+    return vcb_attn_tc_supported(dtype, hd, page_size) && nkv <= 2 * wide_blocks(hd);
 }
 
 VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
@@ -932,8 +959,9 @@ VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long lon
     TcArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, block_table, table_row, max_blocks, q_start, q_len, ctx_len,
              items, nh, nkv, page_size, num_pages, window, scale, status, n_items * nkv * hchunks, work, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate};
     VCB_CHECK_ARG(softcap >= 0.f && (dist_a == nullptr || slope == nullptr), "attn_tc: a negative cap, or a logarithmic penalty and a slope at once");
-    VCB_CHECK_ARG(!wide || nkv <= wide_blocks(hd), "attn_tc: wide query rows of %d x %d lanes (up to 512)", nkv, hd);
-    if (wide) return hd == 64 ? launch<64, true, true>(map, a, n_items, stream) : launch<128, true, true>(map, a, n_items, stream);
+    VCB_CHECK_ARG(!wide || nkv <= 2 * wide_blocks(hd), "attn_tc: wide query rows of %d x %d lanes (up to 1024)", nkv, hd);
+    if (wide && nkv > wide_blocks(hd)) return hd == 64 ? launch<64, true, ROWS_WIDER>(map, a, n_items, stream) : launch<128, true, ROWS_WIDER>(map, a, n_items, stream);
+    if (wide) return hd == 64 ? launch<64, true, ROWS_WIDE>(map, a, n_items, stream) : launch<128, true, ROWS_WIDE>(map, a, n_items, stream);
     if (chunked || out_gate != nullptr || keep_first > 0 || dist_a != nullptr || softcap > 0.f || slope != nullptr || sink) return hd == 64 ? launch<64, true>(map, a, n_items, stream) : launch<128, true>(map, a, n_items, stream);
     return hd == 64 ? launch<64, false>(map, a, n_items, stream) : launch<128, false>(map, a, n_items, stream);
 }

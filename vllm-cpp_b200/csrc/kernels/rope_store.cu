@@ -20,6 +20,7 @@
 //
 // Norms, angles (a 32-bit product of position and frequency; the frequencies are rounded once from 64-bit on the host),
 // sines and cosines are 32-bit.  A block a token; cosines and sines are computed once a token and shared by its heads.
+// (Mixed queries of a few tokens: several blocks a token, each for some of its heads.)
 #include "common.cuh"
 
 namespace {
@@ -99,14 +100,15 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
     if (a.vfreq != nullptr)
         for (int i = threadIdx.x; i < vhalf; i += blockDim.x) sincosf(pos * a.vfreq[i], &vcs[vhalf + i], &vcs[i]);
     float sq = 0.f, sk = 0.f;
-    for (int c = threadIdx.x; c < n; c += blockDim.x) {
+    const bool first = blockIdx.y == 0;     // (a token's further blocks only mix queries)
+    for (int c = threadIdx.x; c < (first ? n : nq); c += blockDim.x) {
         float v = rows_at(a.qkv, t, c);
         if (a.bias != nullptr) v += a.bias[c];
         row[c] = v;
         if (c < nq) sq = fmaf(v, v, sq);
         else if (c < nq + nk) sk = fmaf(v, v, sk);
     }
-    if (a.gate_out != nullptr)
+    if (a.gate_out != nullptr && first)
         for (int h = threadIdx.x; h < a.nh; h += blockDim.x)
             a.gate_out[(size_t)t * a.nh + h] = 1.f / (1.f + expf(-rows_at(a.qkv, t, n + h)));
     if (a.talk != nullptr)
@@ -118,7 +120,7 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         rq = 1.0f / sqrtf(sq / (float)nq + a.eps);
         rk = 1.0f / sqrtf(sk / (float)nk + a.eps);
     } else __syncthreads();
-    if (a.unit_v) {
+    if (a.unit_v && first) {
         // a warp a value head; the factors are read behind the next barrier
         const int lane = threadIdx.x & 31;
         for (int g = threadIdx.x >> 5; g < a.nkv; g += blockDim.x >> 5) {
@@ -145,9 +147,9 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         const int gs = a.nh / a.nkv, wide = a.nkv * a.hd, pairs = (a.hd + 1) / 2;
         const bool even = (a.hd & 1) == 0;
         TC* wq = (TC*)a.q_out + (size_t)t * a.nh * wide;
-        const int hb = (a.nh + 3) / 4;
+        const int hb = ((a.nh + 3) / 4 - (int)blockIdx.y + (int)gridDim.y - 1) / (int)gridDim.y;     // this block's fours of heads
         for (int i = threadIdx.x; i < hb * a.nkv * pairs; i += blockDim.x) {
-            const int d = 2 * (i % pairs), G = (i / pairs) % a.nkv, h0 = 4 * (i / (pairs * a.nkv));
+            const int d = 2 * (i % pairs), G = (i / pairs) % a.nkv, h0 = 4 * ((i / (pairs * a.nkv)) * (int)gridDim.y + (int)blockIdx.y);
             const bool two = even || d + 1 < a.hd;
             const float* src = row + (size_t)G * gs * a.hd + d;
             float acc[4][2];
@@ -191,7 +193,7 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         }
     }
     const int slot = a.slot_map[t];
-    if (slot < 0) return;
+    if (slot < 0 || !first) return;
     const int page = slot / a.page_size, off = slot % a.page_size;
     if (page >= a.num_pages) {
         if (threadIdx.x == 0) atomicOr(a.status, VCB_STATUS_BAD_PAGE);
@@ -284,7 +286,10 @@ VCB_API int vcb_qkv_rope_store(const float* qkv, int S, long long s_stride, long
         vcb_set_error("qkv_rope_store: %zu bytes of shared memory refused", smem);
         return -2;
     }
-    launch_pdl(kern, dim3(T), dim3(256), smem, stream, a);
+    // few tokens with queries to mix: a token's heads are dealt to several blocks
+    const int fours = (nh + 3) / 4;
+    const int split = talk == nullptr || T > 64 ? 1 : (fours < 8 ? fours : 8);
+    launch_pdl(kern, dim3(T, split), dim3(256), smem, stream, a);
     VCB_CHECK_LAUNCH("qkv_rope_store");
     return 0;
 }

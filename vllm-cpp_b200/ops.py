@@ -118,6 +118,8 @@ def _declare(L):
         "vcb_attn_tc_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, P, P, P],
         "vcb_attn_tc_wide_supported": [I, I, I, I],
         "vcb_attn_tc_supported": [I, I, I],
+        "vcb_attn_wide": [P, P, P, LL, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, P, P, P],
+        "vcb_attn_wide_supported": [I, I, I, I, I],
         "vcb_attn_stream": [P, P, P, LL, P, P, I, P, P, P, I, P, I, I, I, I, I, I, F, P, I, P],
         "vcb_attn_stream_supported": [I, I, I, I, I],
         "vcb_attn_merge": [P, P, P, P, I, I, I, I, I, P, P],
@@ -1016,6 +1018,29 @@ def attn_mma(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items
           1.0 / math.sqrt(hd) if scale is None else float(scale), int(keep_first or 0), _p(dist_a), _p(dist_b),
           float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), int(bool(chunked)),
           int(bool(wide)), _p(out_gate), _p(status), int(allow_tma), int(cluster), _stream())
+
+
+def attn_wide_supported(dtype: torch.dtype, hd: int, page_size: int, nh: int, nkv: int) -> bool:
+    """Whether :func:`attn_wide` takes these sizes."""
+    return bool(lib().vcb_attn_wide_supported(BF16 if dtype == torch.bfloat16 else F32, hd, page_size, nh, nkv))
+
+
+def attn_wide(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, part_o, part_ml, nh, nkv, hd, window, status,
+              table_row=None, scale=None, chunked=False, out_gate=None):
+    """Single decoded tokens whose query rows are wide (``q`` [T, nh * nkv * hd], see :func:`attn_window_bias`): a block is a
+    token and a slice of its keys with all query heads, so keys and values are read once.  ``items`` as for
+    :func:`attn_mma`; several slices leave their partials in ``part_o`` / ``part_ml`` for :func:`attn_merge` (which then
+    applies ``out_gate``)."""
+    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, True)
+    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pages, "pages", torch.bfloat16)
+    for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len), ("items", items)):
+        _need(t, name, torch.int32)
+    num_pages, two, nkv_p, page_size, hd_p = pages.shape
+    assert two == 2 and nkv_p == nkv and hd_p == hd
+    _call("vcb_attn_wide", _p(q), _p(out), _p(pages), pages.stride(0), _p(block_table), _p(table_row), block_table.shape[1],
+          _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, _p(part_o), _p(part_ml), nh, nkv, hd, page_size, num_pages,
+          int(window or 0), int(bool(chunked)), 1.0 / math.sqrt(hd) if scale is None else float(scale), _p(out_gate), _p(status),
+          _stream())
 
 
 def attn_stream_supported(dtype: torch.dtype, hd: int, page_size: int, nh: int, nkv: int) -> bool:

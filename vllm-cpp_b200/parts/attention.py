@@ -78,11 +78,13 @@ class AttentionPlan:
     """Work items of the attention kernel for one step and one head layout, on the device."""
 
     def __init__(self, ctx, nh: int, nkv: int, decode_rows: int = DECODE_ROWS, span_rows: int = SPAN_ROWS,
-                 cluster_hd: int | None = None, one_slice: bool = False, max_keys: int = 0):
+                 cluster_hd: int | None = None, one_slice: bool = False, max_keys: int = 0,
+                 whole_tokens: bool = False):
         """``cluster_hd``: the head size, when the kernel that takes the decoded tokens can merge a token's key slices
         within a cluster of its blocks (then the slices are chosen so that all clusters run at once); else None.
         ``one_slice``: no key slices, whatever the contexts.  ``max_keys`` > 0: no query reads more keys than this
-        (a window), so the key ranges are sliced as if no context were longer."""
+        (a window), so the key ranges are sliced as if no context were longer.  ``whole_tokens``: a block of the kernel that
+        takes the decoded tokens is a token and key slice with all heads, and has an SM to itself."""
         g = nh // nkv
         dev = ctx.device
         # int32 arrays go to the device with the step's own staging buffers where the step has them
@@ -98,23 +100,24 @@ class AttentionPlan:
         self.n_span_items = 0
         if dec:
             hchunks = -(-g // min(g, decode_rows))
-            blocks = len(dec) * nkv * hchunks
+            blocks = len(dec) * (1 if whole_tokens else nkv * hchunks)
+            per_slice = 64 if whole_tokens else 128      # least keys of a slice
             if getattr(ctx, "static", False):
                 # a captured step serves every context length up to the bound it was captured for (None: any)
                 longest = getattr(ctx, "static_max_ctx", None)
                 if max_keys:
                     longest = max_keys if longest is None else min(longest, max_keys)
-                by_pages = MAX_SLICES if longest is None else max(1, longest // 128)
+                by_pages = MAX_SLICES if longest is None else max(1, longest // per_slice)
             else:
                 longest = self.longest = max(ctx.host_ctx_len[i] for i in dec)
                 if max_keys:
                     longest = min(longest, max_keys)
-                by_pages = max(1, longest // 128)   # at least 128 keys a slice
+                by_pages = max(1, longest // per_slice)
             # as many slices as keep every block resident in one wave; over short contexts no more than
             # SHORT_SLICES, beyond which merging the partial results costs more than the shorter key ranges save
             # (one request at 4,096 keys, 12-layer step: 8 slices 1.437 ms, 12: 1.420, 18: 1.444, 37: 1.495)
-            fit = BLOCKS_PER_SM * ops.num_sms() // blocks
-            if longest is not None and longest <= SHORT_CONTEXT:
+            fit = (1 if whole_tokens else BLOCKS_PER_SM) * ops.num_sms() // blocks
+            if longest is not None and longest <= SHORT_CONTEXT and not whole_tokens:
                 fit = min(fit, SHORT_SLICES)
             self.nslices = 1 if one_slice else int(max(1, min(MAX_SLICES, by_pages, fit)))
             if cluster_hd is not None and longest is not None and longest <= SHORT_CONTEXT and self.nslices > 1:

@@ -44,6 +44,8 @@ from .linear import matmul_tn
 MMA_ATTENTION = os.environ.get("VLLM_CPP_B200_WINDOW_ATTN_MMA", "1") != "0"
 # whether the tensor-core kernels take the cap, the slope and the sink (else steps with them run on the plain kernel)
 EXTRAS_ON_TENSOR_CORES = True
+# 0 sends single tokens with wide query rows to the kernel with a block a KV head (comparison runs, tests)
+WIDE_DECODE = os.environ.get("VLLM_CPP_B200_ATTN_WIDE", "1") != "0"
 # query lanes up to which the plain kernel keeps 32 rows of a prompt portion in a block's shared memory
 PLAIN_SPAN_LANES = 1280
 # whether they take a sink with a learned score per head (else such steps run on the plain kernel)
@@ -64,6 +66,8 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     of the blocks' products with all heads' keys there (queries mixed across heads).  ``out_gate`` (float32 [T, nh])
     multiplies each head's result."""
     x = q
+    if nkv == 1:
+        wide = False      # one block a row: an ordinary one
     # no query reads more keys than the window and the kept first ones: no more key slices than those fill
     reach = window + keep_first if window else 0
     # bfloat16 with keys and values of 64 or 128 lanes: the tensor-core kernel; else the plain one
@@ -72,6 +76,7 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     has_extras = bool(softcap or slope is not None or learned_sink or sink)
     mma = (MMA_ATTENTION and vd == hd and kv.pages.dim() == 5 and ops.attn_mma_supported(x.dtype, hd)
            and (EXTRAS_ON_TENSOR_CORES or not has_extras) and (SINK_SCORES_ON_TENSOR_CORES or not learned_sink))
+    has_extras = has_extras or bool(keep_first) or dist_a is not None
     mma_rows = MMA_SPAN_ROWS
     if mma and wide:
         mma_rows = ops.attn_mma_wide_rows(x.dtype, hd, nkv)
@@ -79,14 +84,16 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     dec_rows, span_rows = (MMA_DECODE_ROWS, mma_rows) if mma else (DECODE_ROWS, SPAN_ROWS)
     if not mma and (nkv * hd if wide else hd) > PLAIN_SPAN_LANES:
         span_rows = DECODE_ROWS      # fewer rows a block: its query rows lie in shared memory
-    clustered = hd if mma and CLUSTER_MERGE and torch.cuda.is_available() else None
+    # single tokens with wide query rows: blocks of all heads, so that keys come in once
+    whole_tokens = mma and wide and WIDE_DECODE and not has_extras and ops.attn_wide_supported(x.dtype, hd, kv.pages.shape[3], nh, nkv)
+    clustered = hd if mma and CLUSTER_MERGE and not whole_tokens and torch.cuda.is_available() else None
     group = ctx.groups[kv.group]
     tcgen05 = mma and TCGEN05_SPANS and (ops.attn_tc_wide_supported(x.dtype, hd, kv.pages.shape[3], nkv) if wide
                                          else ops.attn_tc_supported(x.dtype, hd, kv.pages.shape[3]))
     if tcgen05:
         span_rows = MMA_SPAN_ROWS
-    plan = ctx.plan(("attention", nh, nkv, mma, clustered, reach, span_rows),
-                    lambda: AttentionPlan(ctx, nh, nkv, dec_rows, span_rows, clustered, max_keys=reach))
+    plan = ctx.plan(("attention", nh, nkv, mma, clustered, reach, span_rows, whole_tokens),
+                    lambda: AttentionPlan(ctx, nh, nkv, dec_rows, span_rows, clustered, max_keys=reach, whole_tokens=whole_tokens))
     common = dict(nh=nh, nkv=nkv, hd=hd, window=window, status=ctx.status, table_row=ctx.slots, scale=scale,
                   keep_first=keep_first, dist_a=dist_a, dist_b=dist_b, chunked=chunked, wide=wide, out_gate=out_gate, **extras)
     args = (q, out, kv.pages, group.block_table, ctx.q_start, ctx.q_len, ctx.ctx_len)
@@ -97,7 +104,12 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
         if S > 1 and not cluster:
             part_o = workspace.empty((plan.n_dec * nh * S, vd), torch.float32, x.device)
             part_ml = workspace.empty((plan.n_dec * nh * S, 2), torch.float32, x.device)
-        if mma:
+        if whole_tokens:
+            ops.attn_wide(*args, plan.dec_items, plan.n_dec * S, part_o, part_ml, nh=nh, nkv=nkv, hd=hd, window=window,
+                          status=ctx.status, table_row=ctx.slots, scale=scale, chunked=chunked, out_gate=out_gate)
+            if S > 1:
+                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S, out_gate)
+        elif mma:
             ops.attn_mma(*args, plan.dec_items, plan.n_dec * S, dec_rows, part_o, part_ml,
                          slice_counters=plan.slice_counters if S > 1 else None, dec_rows=plan.dec_rows, cluster=cluster,
                          **common)
