@@ -352,22 +352,52 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     pdl_wait();
     const int n = blockIdx.x, h = blockIdx.y;
     const size_t prow0 = ((size_t)n * nh + h) * nslices;
-    float m = -CUDART_INF_F;
-    for (int s = 0; s < nslices; ++s) m = fmaxf(m, part_ml[(prow0 + s) * 2]);
+    // the slices' weights first (a batch of them at a time), each needed by every thread; then the outputs, several loads
+    // in flight
+    constexpr int MS = 64;
+    __shared__ float w_s[MS], l_s[MS], m_all;
+    if (threadIdx.x < 32) {
+        float m = -CUDART_INF_F;
+        for (int s = threadIdx.x; s < nslices; s += 32) m = fmaxf(m, part_ml[(prow0 + s) * 2]);
+        m = warp_max(m);
+        if (threadIdx.x == 0) m_all = m;
+    }
     const int row = dec_rows[n];
-    if (row < 0) return;
-    for (int d = threadIdx.x; d < hd; d += blockDim.x) {
-        float l = 0.f, o = 0.f;
-        for (int s = 0; s < nslices; ++s) {
-            const float ms = part_ml[(prow0 + s) * 2];
-            if (ms == -CUDART_INF_F) continue;
-            const float w = expf(ms - m);
-            l += part_ml[(prow0 + s) * 2 + 1] * w;
-            o += part_o[(prow0 + s) * hd + d] * w;
+    const float gate = out_gate != nullptr && row >= 0 ? out_gate[(size_t)row * nh + h] : 1.f;
+    constexpr int DPT = 4;      // value lanes a thread (of blocks of 64 to 256 threads)
+    for (int d0 = 0; d0 < hd; d0 += DPT * blockDim.x) {
+        float l = 0.f, o[DPT] = {0.f, 0.f, 0.f, 0.f};
+        for (int s0 = 0; s0 < nslices; s0 += MS) {
+            const int ns = min(MS, nslices - s0);
+            __syncthreads();
+            if (threadIdx.x < ns) {
+                const float ms = part_ml[(prow0 + s0 + threadIdx.x) * 2];
+                const float w = ms == -CUDART_INF_F ? 0.f : expf(ms - m_all);
+                w_s[threadIdx.x] = w;
+                l_s[threadIdx.x] = ms == -CUDART_INF_F ? 0.f : part_ml[(prow0 + s0 + threadIdx.x) * 2 + 1] * w;
+            }
+            __syncthreads();
+            for (int s = 0; s < ns; ++s) l += l_s[s];
+#pragma unroll
+            for (int k = 0; k < DPT; ++k) {
+                const int d = d0 + threadIdx.x + k * blockDim.x;
+                if (d < hd) {
+                    const float* p = part_o + (prow0 + s0) * hd + d;
+#pragma unroll 8
+                    for (int s = 0; s < ns; ++s) {
+                        const float w = w_s[s], x = p[(size_t)s * hd];
+                        if (w != 0.f) o[k] = fmaf(x, w, o[k]);      // (a slice without keys may have left nothing)
+                    }
+                }
+            }
         }
-        o = l > 0.f ? o / l : 0.f;
-        if (out_gate != nullptr) o *= out_gate[(size_t)row * nh + h];
-        out[((size_t)row * nh + h) * hd + d] = from_f32<T>(o);
+        if (row >= 0) {
+#pragma unroll
+            for (int k = 0; k < DPT; ++k) {
+                const int d = d0 + threadIdx.x + k * blockDim.x;
+                if (d < hd) out[((size_t)row * nh + h) * hd + d] = from_f32<T>((l > 0.f ? o[k] / l : 0.f) * gate);
+            }
+        }
     }
 }
 

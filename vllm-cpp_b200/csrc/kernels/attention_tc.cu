@@ -35,7 +35,8 @@
 // heads of block . that head's keys, one MMA chain over all of them into the same accumulator.  The rows' blocks stay on
 // the SM for the whole unit (one block an SM then): up to 512 lanes in shared memory (128 KB), up to 512 more in TMEM
 // (256 columns, beside S, S and O all there are), from where the products read them as their A operand like the weights.
-// The K ring's stages hold one KV head's keys each and are given back by the products themselves, and the rows of the
+// The K ring's stages hold one KV head's keys each and are given back by the products themselves; two warps of their own
+// bring them in, a stage in turn each (one warp took longer to issue a stage's copies than its products), and the rows of the
 // next unit come in as soon as the last scores of this one are there, behind its last weights and output.
 //
 // All hand-offs are mbarriers; every wait is bounded by the clock, and a wait that runs out sets a bit in the
@@ -52,7 +53,8 @@ namespace {
 constexpr int BNK = 64;       // keys per tile
 constexpr int ROWS = 128;     // rows per block = TMEM lanes
 constexpr int ITEM_INTS = 6;  // entry, q0, nq, slice, nslices, decode index (as in attention_mma.cu)
-constexpr int NTHREADS = 192;
+constexpr int NTHREADS = 192;         // the roles above
+constexpr int KEY_WARPS = 2;          // (wide rows: further warps that load keys)
 // Marks of the roles inside a block in a timeline build (TlRole; the block-wide marks are phases 0 to 2): the
 // loading warp asks for a stage, has it, has sent the copies; the thread that issues the products asks for a K tile,
 // has it, has issued Q.K^T, has the tile's weights (and values), has issued P.V; the first softmax row asks for a
@@ -298,7 +300,7 @@ __device__ __forceinline__ bool read_unit(const TcArgs& a, int unit, Unit& u) {
 // tiles of the units before.
 // OPT: built with the options of TcArgs (kept first keys, distance penalty); without, they cost nothing
 template <int HD, int KS, int VS, bool OPT, int KIND>
-__global__ __launch_bounds__(NTHREADS, KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_kernel(const __grid_constant__ CUtensorMap kv_map, TcArgs a) {
+__global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0), KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_kernel(const __grid_constant__ CUtensorMap kv_map, TcArgs a) {
     constexpr bool WIDE = KIND != ROWS_PLAIN, IN_TMEM = KIND == ROWS_WIDER;
     using L = Layout<HD, KS, VS, WIDE ? wide_blocks(HD) : 1, IN_TMEM>;
     const int NG = WIDE ? a.nkv : 1;    // blocks of a query row = stages of a K tile
@@ -465,10 +467,10 @@ __global__ __launch_bounds__(NTHREADS, KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_
                     const int pb = tile_pb0(u, it, pages_per_tile) + pl;
                     return (lane < 16 && it < u.n_tiles && pl < pages_per_tile && pb < tile_pb_hi(u, it, ps)) ? bt[pb] : -1;
                 };
-                // loads stage itk of the unit's K tiles (tile itk / NG, with wide rows KV head itk % NG) and V tile itv
-                // (either may be -1: none) once their stages are free; false: give up
+                // loads K tile itk and V tile itv of the unit (either may be -1: none) once their stages are free;
+                // false: give up
                 auto load_tiles = [&](int itk, int itv) {
-                    const int gk = t0 * NG + itk, gv = t0 + itv;
+                    const int gk = t0 + itk, gv = t0 + itv;
                     bool free = true;
                     tl.mark(TL_LOAD_ASKS, gv);
                     if (lane == 0) {
@@ -479,8 +481,7 @@ __global__ __launch_bounds__(NTHREADS, KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_
                     }
                     tl.mark(TL_LOAD_FREE, gv);
                     if (!__shfl_sync(0xffffffffu, free, 0)) return false;
-                    const int it = copies_v ? itv : (itk >= 0 ? itk / NG : -1);
-                    const int key_head = WIDE && itk >= 0 ? itk % NG : u.kvh;
+                    const int it = copies_v ? itv : itk;
                     const bool mine = lane < 16 && it >= 0;
                     const int st = mine ? (copies_v ? gv % VS : gk % KS) : 0;
                     const uint32_t fullb = copies_v ? v_full(st) : k_full(st);
@@ -493,25 +494,21 @@ __global__ __launch_bounds__(NTHREADS, KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_
                             atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                             page = 0;   // keep the byte count whole; the status word reports the fault
                         }
-                        const int group = (page * 2 * a.nkv + (copies_v ? u.kvh : key_head)) * groups_page + (copies_v ? groups_kv : 0);
+                        const int group = (page * 2 * a.nkv + u.kvh) * groups_page + (copies_v ? groups_kv : 0);
                         const uint32_t dst = base + (copies_v ? L::V_OFF : L::K_OFF) + st * L::KV_BYTES;
                         tma_load_groups(dst + pl * ps * ROWB, &kv_map, fullb, group);
                     }
                     tl.mark(TL_LOAD_SENT, gv);
-                    if (mine && (copies_v || !WIDE || key_head == NG - 1)) next_page = page_of(it + 1);
+                    if (mine) next_page = page_of(it + 1);
                     if (itk >= 0) armed[0] = gk + 1;
                     if (itv >= 0) armed[1] = gv + 1;
                     return true;
                 };
                 if constexpr (WIDE) {
-                    // keys one tile ahead of the values: the products of a tile's stages take several times as long
-                    for (int b = 0; b < NG && ok; ++b) ok = load_tiles(b, -1);
-                    for (int it = 0; it < u.n_tiles && ok; ++it) {
+                    for (int it = 0; it < u.n_tiles && ok; ++it) {      // the values; the keys have warps of their own
                         if (it == max(0, u.n_tiles - 4)) ask();
                         if (it == max(0, u.n_tiles - 2)) make_known();
-                        if (it + 1 < u.n_tiles)
-                            for (int b = 0; b < NG && ok; ++b) ok = load_tiles((it + 1) * NG + b, -1);
-                        if (ok) ok = load_tiles(-1, it);
+                        ok = load_tiles(-1, it);
                     }
                 } else {
                     ok = load_tiles(0, -1);
@@ -608,6 +605,57 @@ __global__ __launch_bounds__(NTHREADS, KIND != ROWS_PLAIN ? 1 : 2) void attn_tc_
                 }
                 t0 += u.n_tiles;
                 ++done;
+            }
+        }
+    } else if (WIDE && warp >= NTHREADS / 32) {
+        // ---- wide rows: the keys, a stage (a tile's keys of one KV head) in turn for each of these warps, a lane a page ----
+        const int me = warp - NTHREADS / 32;
+        const int pages_per_tile = BNK / ps, groups_page = ps / 8;
+        bool ok = true;
+        int g0 = 0, armed = -1;     // stages of the units before; the last stage this warp has asked for
+        Unit u;
+        int unit = (int)blockIdx.x;
+        bool has = read_unit<OPT>(a, unit, u);
+        for (int seq = 0; unit >= 0 && ok; unit = next_unit(seq, u), has = unit >= 0, ++seq) {
+            if (!has) continue;
+            const int* bt = a.block_table + (size_t)u.bt_row * a.max_blocks;
+            auto page_of = [&](int it) {
+                const int pb = tile_pb0(u, it, pages_per_tile) + lane;
+                return (it < u.n_tiles && lane < pages_per_tile && pb < tile_pb_hi(u, it, ps)) ? bt[pb] : -1;
+            };
+            int page = page_of(0), next_page = page_of(1), it = 0, head = (KEY_WARPS + me - g0 % KEY_WARPS) % KEY_WARPS;
+            const int n = u.n_tiles * NG;
+            for (int i = head; i < n && ok; i += KEY_WARPS, head += KEY_WARPS) {
+                while (head >= NG) {
+                    head -= NG;
+                    ++it;
+                    page = next_page;
+                    next_page = page_of(it + 1);
+                }
+                const int gk = g0 + i, st = gk % KS;
+                bool free = true;
+                if (lane == 0) free = mbar_wait(k_empty(st), ((gk / KS) & 1) ^ 1u, abort_flag, a.status);
+                ok = __shfl_sync(0xffffffffu, free, 0);
+                if (!ok) break;
+                const int np = min(pages_per_tile, tile_pb_hi(u, it, ps) - tile_pb0(u, it, pages_per_tile));
+                if (lane == 0) mbar_expect_tx(k_full(st), (uint32_t)(np * ps * ROWB));
+                __syncwarp();
+                if (lane < np) {
+                    int p = page;
+                    if (p < 0 || p >= a.num_pages) {
+                        atomicOr(a.status, VCB_STATUS_BAD_PAGE);
+                        p = 0;
+                    }
+                    tma_load_groups(base + L::K_OFF + st * L::KV_BYTES + lane * ps * ROWB, &kv_map, k_full(st), (p * 2 * a.nkv + head) * groups_page);
+                }
+                armed = gk;
+            }
+            g0 += n;
+        }
+        if (lane == 0 && *abort_flag) {   // let copies in flight land before the block goes away
+            for (int i = armed; i >= 0 && i > armed - KS; i -= KEY_WARPS) {
+                const long long c0 = clock64();
+                while (!mbar_try(k_full(i % KS), (i / KS) & 1) && clock64() - c0 < VCB_WAIT_CLOCKS) {}
             }
         }
     } else {
@@ -898,7 +946,7 @@ int launch(const CUtensorMap& map, const TcArgs& a, int n_items, cudaStream_t st
         }
         resident = (WIDE ? 1 : 2) * sms;
     }
-    launch_pdl(kern, dim3((unsigned)(a.n_units < resident ? a.n_units : resident)), dim3(NTHREADS), (size_t)L::TOTAL, stream, map, a);
+    launch_pdl(kern, dim3((unsigned)(a.n_units < resident ? a.n_units : resident)), dim3(NTHREADS + (WIDE ? 32 * KEY_WARPS : 0)), (size_t)L::TOTAL, stream, map, a);
     VCB_CHECK_LAUNCH("attn_tc");
     return 0;
 }

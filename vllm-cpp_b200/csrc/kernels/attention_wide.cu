@@ -205,10 +205,11 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
     const int q_ch = nkv * CH;
     for (int idx = tid; idx < ROWS * q_ch; idx += NT) {
         const int r = idx / q_ch, c = idx % q_ch;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (r < nh) v = *reinterpret_cast<const uint4*>(a.q + ((size_t)row0 * nh + r) * (nkv * HD) + c * 8);
-        *reinterpret_cast<uint4*>(q_s + (c / CH) * (ROWS * ROWB) + swz_rows(ROWS, r, c % CH)) = v;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n"
+                     ::"r"(smem_u32(q_s + (c / CH) * (ROWS * ROWB) + swz_rows(ROWS, r, c % CH))),
+                       "l"(a.q + ((size_t)row0 * nh + (r < nh ? r : 0)) * (nkv * HD) + c * 8), "r"(r < nh ? 16 : 0) : "memory");
     }
+    asm volatile("cp.async.wait_all;" ::: "memory");
     float o[NG][NTV][4];
 #pragma unroll
     for (int g = 0; g < NG; ++g)

@@ -59,6 +59,8 @@ struct StoreArgs {
     const float* bias;      // [nh hd + nkv hd (+ nkv vd)] or null
     int unit_v;             // every value head divided by its root mean square (eps inside the root)
     const float* talk;      // [nh][nh] or null: queries mixed across heads, q_out is [T][nh][nkv * hd]
+    int vec;                // rows, partial sums and bias lie on 16-byte words
+    int talk_off;           // where the mixing matrix lies in shared memory (floats)
     float* gate_out;        // [T][nh] or null: sigmoid of the nh columns behind the projection's
 };
 
@@ -93,7 +95,8 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
     float* cs = sm + n;                 // [rot]: cosines, then sines
     float* vcs = cs + a.rot;            // [vrot]
     float* vscale = vcs + a.vrot;       // [nkv] with unit values
-    float* talk = vscale + (a.unit_v ? a.nkv : 0);      // [nh][nh] with mixed queries
+    const int nh4 = (a.nh + 3) & ~3;
+    float* talk = sm + a.talk_off;      // [nh][nh4] with mixed queries, transposed: weights of head g's queries in all heads' scores
     const float pos = (float)a.positions[t];
     const int half = a.rot >> 1, vhalf = a.vrot >> 1;
     for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * a.freq[i], &cs[half + i], &cs[i]);
@@ -101,7 +104,34 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         for (int i = threadIdx.x; i < vhalf; i += blockDim.x) sincosf(pos * a.vfreq[i], &vcs[vhalf + i], &vcs[i]);
     float sq = 0.f, sk = 0.f;
     const bool first = blockIdx.y == 0;     // (a token's further blocks only mix queries)
-    for (int c = threadIdx.x; c < (first ? n : nq); c += blockDim.x) {
+    const int n_mine = first ? n : nq;
+    int from = 0;
+    if (a.vec) {        // 16-byte words, as far as whole ones go
+        from = n_mine & ~3;
+        for (int c = 4 * threadIdx.x; c < from; c += 4 * blockDim.x) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float* p = a.qkv.p + (long long)t * a.qkv.ld + c;
+#pragma unroll 4
+            for (int s = 0; s < a.qkv.S; ++s) {
+                const float4 w = *reinterpret_cast<const float4*>(p + (long long)s * a.qkv.s_stride);
+                v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+            }
+            if (a.bias != nullptr) {
+                const float4 b = *reinterpret_cast<const float4*>(a.bias + c);
+                v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+            }
+            *reinterpret_cast<float4*>(row + c) = v;
+            if (a.q_gain != nullptr) {
+                const float f[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    if (c + k < nq) sq = fmaf(f[k], f[k], sq);
+                    else if (c + k < nq + nk) sk = fmaf(f[k], f[k], sk);
+                }
+            }
+        }
+    }
+    for (int c = from + threadIdx.x; c < n_mine; c += blockDim.x) {
         float v = rows_at(a.qkv, t, c);
         if (a.bias != nullptr) v += a.bias[c];
         row[c] = v;
@@ -112,7 +142,10 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
         for (int h = threadIdx.x; h < a.nh; h += blockDim.x)
             a.gate_out[(size_t)t * a.nh + h] = 1.f / (1.f + expf(-rows_at(a.qkv, t, n + h)));
     if (a.talk != nullptr)
-        for (int i = threadIdx.x; i < a.nh * a.nh; i += blockDim.x) talk[i] = a.talk[i];
+        for (int i = threadIdx.x; i < a.nh * nh4; i += blockDim.x) {
+            const int g = i / nh4, h = i % nh4;
+            talk[i] = h < a.nh ? a.talk[h * a.nh + g] : 0.f;
+        }
     float rq = 1.f, rk = 1.f;
     if (a.q_gain != nullptr) {
         sq = block_sum(sq, red);
@@ -156,12 +189,21 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
 #pragma unroll
             for (int m = 0; m < 4; ++m) acc[m][0] = acc[m][1] = 0.f;
             for (int g = 0; g < gs; ++g) {
-                const float x = src[g * a.hd], y = two ? src[g * a.hd + 1] : 0.f;
+                float x, y;
+                if (even) {
+                    const float2 xy = *reinterpret_cast<const float2*>(src + g * a.hd);
+                    x = xy.x;
+                    y = xy.y;
+                } else {
+                    x = src[g * a.hd];
+                    y = two ? src[g * a.hd + 1] : 0.f;
+                }
+                const float4 w4 = *reinterpret_cast<const float4*>(talk + (G * gs + g) * nh4 + h0);
+                const float w[4] = {w4.x, w4.y, w4.z, w4.w};
 #pragma unroll
                 for (int m = 0; m < 4; ++m) {
-                    const float w = h0 + m < a.nh ? talk[(h0 + m) * a.nh + G * gs + g] : 0.f;
-                    acc[m][0] = fmaf(w, x, acc[m][0]);
-                    acc[m][1] = fmaf(w, y, acc[m][1]);
+                    acc[m][0] = fmaf(w[m], x, acc[m][0]);
+                    acc[m][1] = fmaf(w[m], y, acc[m][1]);
                 }
             }
 #pragma unroll
@@ -275,9 +317,12 @@ VCB_API int vcb_qkv_rope_store(const float* qkv, int S, long long s_stride, long
     VCB_CHECK_ARG((q_gain == nullptr) == (k_gain == nullptr), "qkv_rope_store: one gain without the other");
     VCB_CHECK_ARG(rot == 0 || freq != nullptr, "qkv_rope_store: no frequencies");
     StoreArgs a{Rows{qkv, S < 1 ? 1 : S, s_stride, ld}, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q_out, pages, page_stride,
-                page_size, num_pages, nh, nkv, hd, vd, rot, vfreq ? vrot : 0, interleaved, v_from_k, status, bias, unit_v, talk, gate_out};
-    const size_t smem = (size_t)(nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0)
-                                 + (unit_v ? nkv : 0) + (talk ? nh * nh : 0)) * sizeof(float);
+                page_size, num_pages, nh, nkv, hd, vd, rot, vfreq ? vrot : 0, interleaved, v_from_k, status, bias, unit_v, talk, 0, 0, gate_out};
+    a.vec = (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 && ld % 4 == 0 && (S <= 1 || s_stride % 4 == 0);
+    const int nh4 = (nh + 3) & ~3;
+    a.talk_off = ((nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0) + (unit_v ? nkv : 0)) + 3) & ~3;
+    const size_t smem = talk ? (size_t)(a.talk_off + nh * nh4) * sizeof(float) : (size_t)(nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0)
+                                 + (unit_v ? nkv : 0)) * sizeof(float);
     VCB_CHECK_ARG(talk == nullptr || nh % nkv == 0, "qkv_rope_store: %d heads mixed over %d KV heads", nh, nkv);
     VCB_CHECK_ARG(talk == nullptr || q_gain == nullptr, "qkv_rope_store: mixed queries come without a norm over the whole projection");
     VCB_CHECK_ARG(smem <= 200 * 1024, "qkv_rope_store: a token's %zu bytes are more than the kernel's shared memory holds", smem);
