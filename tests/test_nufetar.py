@@ -337,6 +337,24 @@ def test_xielu_and_tanh(F, S, dtype):
 
 
 @gpu
+@pytest.mark.parametrize("M,K,T", [(96, 64, 5), (300, 128, 70), (512, 200, 129), (1024, 72, 300)])
+def test_xielu_in_the_products_epilogue(M, K, T):
+    from vllm_cpp_b200 import ops
+    g = torch.Generator().manual_seed(M)
+    w = torch.randn(M, K, generator=g, dtype=F64).to(torch.bfloat16)
+    x = (torch.randn(T, K, generator=g, dtype=F64) * 2.0 * K ** -0.5).to(torch.bfloat16)
+    x[1] *= 1e-3        # sums near zero, where the branches meet
+    coef = torch.tensor([P.softplus(0.6), 0.5 + P.softplus(-1.1)], dtype=F64)
+    status = torch.zeros(1, dtype=torch.int32, device=dev())
+    want = P.xielu(x.double() @ w.double().T, 0.6, -1.1)
+    for shape in [-1] + ([i for i, n in enumerate(ops.GEMM_SHAPES) if n in ("n256", "m256_n192", "pair")] if M >= 256 and T > 128 else []):
+        out = torch.full((T, M), float("nan"), dtype=torch.bfloat16, device=dev())
+        ops.gemm_bf16_xielu(w.to(dev()), x.to(dev()), f32(coef), out, status, shape=shape)
+        assert int(status.item()) == 0
+        torch.testing.assert_close(out.double().cpu(), want, atol=2e-5, rtol=6e-3)
+
+
+@gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("nh,nkv,hd,vd,rot,S,talks", [(4, 2, 8, 6, 4, 1, True), (2, 1, 64, 64, 64, 2, True), (6, 3, 10, 14, 0, 3, True),
                                                       (5, 1, 7, 3, 6, 1, True), (8, 4, 128, 128, 96, 1, True), (3, 3, 5, 5, 2, 1, False),

@@ -132,9 +132,16 @@ struct GemmArgs {
     // Null: an ordinary product.
     const int* tile_group;
     int group_rows;
-    int act;                  // applied to the sums before they are stored: 0 none, 3 the square of ReLU, 2 SiLU
+    int act;                  // applied to the sums before they are stored: 0 none, 3 the square of ReLU, 2 SiLU, 6 xIELU
+    const float* act_coef;    // xIELU: the factors of its parabola and of its exponential branch
 };
 
+// up x^2 + x/2 above zero, down (e^x - 1 - x) + x/2 below; near zero the bracket from its series (it would cancel)
+__device__ __forceinline__ float gemm_xielu(float x, float up, float down) {
+    const float series = x * x * fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
+    const float below = x > -0.25f ? series : __expf(x) - 1.f - x;
+    return fmaf(0.5f, x, x > 0.f ? up * x * x : down * below);
+}
 __device__ __forceinline__ float gemm_act(float x, int act) {
     if (act == 3) { const float r = fmaxf(x, 0.f); return r * r; }
     if (act == 2) return x / (1.f + __expf(-x));
@@ -518,6 +525,11 @@ __global__ __launch_bounds__(NTHREADS, 1) void gemm_bf16_tn_kernel(const __grid_
                         continue;
                     }
                 }
+                if (g.act == 6) {
+                    const float up = g.act_coef[0], down = g.act_coef[1];
+#pragma unroll
+                    for (int jj = 0; jj < CHUNK; ++jj) v[jj / 16][jj % 16] = __float_as_uint(gemm_xielu(__uint_as_float(v[jj / 16][jj % 16]), up, down));
+                }
                 if (g.swiglu) {
                     swiglu_store<CHUNK>(v, reinterpret_cast<__nv_bfloat16*>(g.out), g.ldc, m, g.M, n0 + c0, g.N, lane);
                 } else if (m < g.M) {
@@ -761,6 +773,11 @@ __global__ __launch_bounds__(NTHREADS, 1) void gemm_bf16_tn_pair_kernel(const __
                         }
                     }
                     continue;
+                }
+                if (g.act == 6) {
+                    const float up = g.act_coef[0], down = g.act_coef[1];
+#pragma unroll
+                    for (int jj = 0; jj < CHUNK; ++jj) v[jj / 16][jj % 16] = __float_as_uint(gemm_xielu(__uint_as_float(v[jj / 16][jj % 16]), up, down));
                 }
                 if (g.swiglu) {
                     swiglu_store<CHUNK>(v, reinterpret_cast<__nv_bfloat16*>(g.out), g.ldc, m, g.M, n0 + c0, g.N, lane);
@@ -1100,6 +1117,22 @@ VCB_API int vcb_gemm_bf16_tn_shape(const void* W, const void* X, void* out, int 
     if ((flags & VCB_GEMM_AFTER_SMALL_KERNEL) && N <= 16 && vcb_pdl_enabled()) pf_settings(&g.pf_tiles, &g.pf_delay_ns);
     if (shape < 0 && use_pairs(M, N, K, splits)) return launch_pair(W, M, X, g, ldw, ldx, stream);
     return launch_shape(shape < 0 ? pick_shape(M, N, K, splits) : shape, W, X, g, ldw, ldx, splits, stream);
+}
+
+// out[t][m] = xIELU(W[m] . X[t]), bfloat16, the activation in the epilogue: what bias_act does with the sums of a product
+// that needs no k-slices.  coef [2] on the device: the factors of the parabola and of the exponential branch.
+VCB_API int vcb_gemm_bf16_xielu(const void* W, const void* X, void* out, int M, int N, int K, long long ldw, long long ldx, long long ldc,
+                                const float* coef, int shape, int flags, int* status, cudaStream_t stream) {
+    VCB_CHECK_ARG(M > 0 && N > 0 && K > 0 && coef != nullptr, "gemm_bf16_xielu: bad sizes M=%d N=%d K=%d, or no factors", M, N, K);
+    VCB_CHECK_ARG(K % 8 == 0 && ldw % 8 == 0 && ldx % 8 == 0,
+                  "gemm_bf16_xielu: inner size %d and row strides %lld, %lld must be multiples of 8 (16-byte rows for TMA)", K, ldw, ldx);
+    VCB_CHECK_ARG(((uintptr_t)W % 16 == 0) && ((uintptr_t)X % 16 == 0), "gemm_bf16_xielu: operands must be 16-byte aligned");
+    GemmArgs g{out, VCB_BF16, M, N, K, ldc, 0, (K + BK - 1) / BK, 1, 0, status};
+    g.act = 6;
+    g.act_coef = coef;
+    if ((flags & VCB_GEMM_AFTER_SMALL_KERNEL) && N <= 16 && vcb_pdl_enabled()) pf_settings(&g.pf_tiles, &g.pf_delay_ns);
+    if (shape < 0 && use_pairs(M, N, K, 1)) return launch_pair(W, M, X, g, ldw, ldx, stream);
+    return launch_shape(shape < 0 ? pick_shape(M, N, K, 1) : shape, W, X, g, ldw, ldx, 1, stream);
 }
 
 // A product over groups of tokens that each meet another matrix (the experts of a routed feed-forward).  W

@@ -96,6 +96,7 @@ def _declare(L):
         "vcb_moe_route_grouped": [P, I, LL, LL, P, I, I, F, P, P, I, I, I, I, P, P, P],
         "vcb_moe_group": [P, I, I, I, I, P, P, P, P],
         "vcb_moe_gather": [P, LL, I, P, P, I, I, I, P, P],
+        "vcb_gemm_bf16_xielu": [P, P, P, I, I, I, LL, LL, LL, P, I, I, P, P],
         "vcb_gemm_bf16_grouped": [P, P, P, I, I, I, I, I, I, LL, LL, LL, P, I, P, P],
         "vcb_moe_gemm": [P, LL, P, I, P, P, P, I, I, P, I, I, I, I, P],
         "vcb_moe_combine": [P, P, P, I, P, I, LL, LL, P, P, I, I, I, P, P],
@@ -356,6 +357,18 @@ def gemm_bf16_swiglu(w_gate_up, x, out, status, shape=-1, after_small_kernel=Fal
     assert I2 % 2 == 0 and x.shape[1] == K and x.stride(1) == 1 and out.shape == (T, I2 // 2)
     _call("vcb_gemm_bf16_swiglu", _p(w_gate_up), _p(x), _p(out), I2 // 2, T, K, w_gate_up.stride(0), x.stride(0),
           out.stride(0), int(shape), int(bool(after_small_kernel)), _p(status), _stream())
+
+
+def gemm_bf16_xielu(w, x, coef, out, status, shape=-1, after_small_kernel=False):
+    """out[t] = xIELU(w x_t) with the factors ``coef`` (float32 [2], see :func:`bias_act`): the product and the activation in
+    one kernel, without k-slices.  ``shape`` and ``after_small_kernel`` as in gemm_bf16_tn."""
+    _need(w, "w", torch.bfloat16); _need(x, "x", torch.bfloat16, contiguous=False); _need(out, "out", torch.bfloat16)
+    _need(coef, "coef", torch.float32); assert coef.numel() == 2
+    M, K = w.shape
+    T = x.shape[0]
+    assert x.shape[1] == K and x.stride(1) == 1 and out.shape == (T, M)
+    _call("vcb_gemm_bf16_xielu", _p(w), _p(x), _p(out), M, T, K, w.stride(0), x.stride(0), out.stride(0), _p(coef), int(shape),
+          int(bool(after_small_kernel)), _p(status), _stream())
 
 
 def gemm_qkv_rope(w_qkv, x, q_out, pages, slot_map, positions, cos_sin, q_weight, k_weight, eps, nh, nkv, status,

@@ -111,6 +111,13 @@ class DenseMLP(FeedForward):
         self.side_rows = int(weight.shape[0])
 
     def forward(self, x, ctx):
+        T, K = x.shape
+        if (self.activation == "xielu" and not self.side_rows and x.dtype == torch.bfloat16 and ops.gemm_tma_ok(x, self.w_up)
+                and (T > FUSE_ABOVE_TOKENS or ops.gemm_effective_splits(K, choose_splits(self.inter, T, K)) == 1)):
+            # no k-slices are needed, or they no longer pay: the activation runs in the product's epilogue
+            act = workspace.empty((T, self.inter), x.dtype, x.device)
+            ops.gemm_bf16_xielu(self.w_up, x, self.coef, act, ctx.status, after_small_kernel=True)     # (after a norm)
+            return matmul_tn(act, self.w_down, ctx.status, out_dtype=torch.float32, allow_partials=True)
         u = matmul_tn(x, self.w_up, ctx.status, out_dtype=torch.float32, allow_partials=True)
         if self.side_rows:
             self.side = u[..., self.inter:]
