@@ -3,17 +3,19 @@
 // rope_store.cu), bfloat16, head_dim 64 or 128, pages of 8, 16, 32 or 64 tokens.
 //
 // Where every head reads every KV head's keys, a block per KV head would fetch all keys once per KV head.  So one block is
-// a token and a slice of its keys with ALL query heads: keys and values come in once.  Per tile of 64 keys:
+// a token and a slice of its keys with ALL query heads: keys and values come in once.  Per tile of up to 128 keys:
 //
-//   S = sum over KV heads of Q_block . K^T   mma.sync m16n8k16, a warp 8 keys of all rows (16 rows a tile of heads), the
+//   S = sum over KV heads of Q_block . K^T   mma.sync m16n8k16, a warp 16 keys of all rows (16 rows a tile of heads), the
 //                    sums stay in registers over the KV heads;
 //   softmax          the scores meet in shared memory, a warp a row in turn: running maximum and sum in 32-bit,
 //                    P = exp(s - m) rounded to bfloat16;
 //   O += P . V       per KV head the rows of its own query heads (up to 16), a warp head_dim / 8 of its value lanes; O stays
 //                    in registers over the tiles.
 //
-// A ninth warp brings in the pages by TMA (one box per page through the grouped view of the cache, as attention_mma.cu does):
-// a stage is 64 keys (or values) of one KV head, a tile's keys first, then its values.  Slices leave (maximum, sum,
+// Two more warps bring in the pages by TMA, a stage each in turn (issuing a stage's copies takes a warp longer than the
+// products on it take the others; one box per page through the grouped view of the cache, as attention_mma.cu does):
+// a stage is a tile's keys (or values) of one KV head, keys first; it is as long as the slice's keys need, so that a short
+// slice has more of them on their way.  Slices leave (maximum, sum,
 // unnormalised output) partials for vcb_attn_merge.  Every wait is bounded and reports through the status word.
 #include "common.cuh"
 #include "mbarrier.cuh"
@@ -24,11 +26,12 @@
 
 namespace {
 
-constexpr int BN = 64;          // keys per tile
+constexpr int BN = 128;         // most keys of a tile
 constexpr int NW = 8;           // multiplying warps
 constexpr int NT = NW * 32;
+constexpr int LW = 2;           // loading warps
 constexpr int ITEM_INTS = 6;    // entry, q0, nq, slice, nslices, decode index (as in attention_mma.cu)
-constexpr int MAX_SLOTS = 24;
+constexpr int MAX_SLOTS = 32;
 
 struct WideArgs {
     const __nv_bfloat16* q;     // [tokens][nh][nkv * HD]
@@ -45,7 +48,7 @@ struct WideArgs {
     int nh, nkv, page_size, num_pages, window, chunked;
     float scale;
     const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
-    int slots;                  // stages of the ring
+    int ring_bytes;             // of shared memory for the stages
     int* status;
 };
 
@@ -79,25 +82,24 @@ __device__ __forceinline__ int first_key(int pos, int W, int chunked) {
     return max(0, chunked ? pos - pos % W : pos - W + 1);
 }
 
-constexpr int S_LD = BN + 8;      // floats of a row of scores in shared memory
+constexpr int S_LD = BN + 4;      // floats of a row of scores in shared memory (its weights then lie over their first half)
 
 // bytes behind the ring: the query rows, scores, weights, per-row numbers, barriers
 __host__ __device__ inline int tail_bytes(int hd, int mt, int nkv) {
     const int rows = 16 * mt;
-    return nkv * rows * hd * 2 + rows * S_LD * 4 + rows * BN * 2 + 3 * rows * 4 + 2 * MAX_SLOTS * 8 + 16;
+    return nkv * rows * hd * 2 + rows * S_LD * 4 + 3 * rows * 4 + 2 * MAX_SLOTS * 8 + 16;
 }
 
 // MT tiles of 16 rows hold the query heads; up to NG KV heads
 template <int HD, int MT, int NG>
-__global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_constant__ CUtensorMap kv_map, WideArgs a) {
-    constexpr int ROWS = 16 * MT, CH = HD / 8, ROWB = HD * 2, HALVES = HD / 64, SUB = BN * ROWB;
+__global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid_constant__ CUtensorMap kv_map, WideArgs a) {
+    constexpr int ROWS = 16 * MT, CH = HD / 8, ROWB = HD * 2, HALVES = HD / 64;
     constexpr int NTV = HD / 64;        // n-tiles of 8 value lanes a warp owns
     constexpr float LOG2E = 1.4426950408889634f;
     extern __shared__ __align__(1024) uint8_t smem[];
-    uint8_t* q_s = smem + a.slots * SUB;
+    uint8_t* q_s = smem + a.ring_bytes;
     float* s_s = reinterpret_cast<float*>(q_s + a.nkv * ROWS * ROWB);       // [ROWS][S_LD]
-    uint8_t* p_s = reinterpret_cast<uint8_t*>(s_s + ROWS * S_LD);           // [ROWS][128 bytes], swizzled
-    float* al_s = reinterpret_cast<float*>(p_s + ROWS * BN * 2);            // [ROWS] rescale factors of the tile
+    float* al_s = s_s + ROWS * S_LD;                                        // [ROWS] rescale factors of the tile
     float* m_s = al_s + ROWS;                                               // [ROWS] at the end: maxima, sums
     float* l_s = m_s + ROWS;
     uint8_t* bar_s = reinterpret_cast<uint8_t*>(l_s + ROWS);
@@ -133,9 +135,11 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
     const int my_lo = pb_lo + slice * pps, my_hi = min(pb_hi, my_lo + pps);
     const int k_begin = max(lo, my_lo * ps), k_end = min(hi, my_hi * ps);
     const int t_first = my_lo * ps;         // tiles start on a page boundary: whole pages come in
-    const int n_tiles = k_end > k_begin ? (k_end - t_first + BN - 1) / BN : 0;
+    const int tile_keys = min(BN, max(1, my_hi - my_lo) * ps);        // whole pages
+    const int n_tiles = k_end > k_begin ? (k_end - t_first + tile_keys - 1) / tile_keys : 0;
     const int per_tile = 2 * nkv, n_loads = n_tiles * per_tile;     // a tile: nkv stages of keys, then nkv of values
-    const int slots = a.slots;
+    const int stage_bytes = tile_keys * ROWB;
+    const int slots = min(MAX_SLOTS, a.ring_bytes / stage_bytes);
 
     if (tid == 0) {
         for (int st = 0; st < slots; ++st) {
@@ -148,10 +152,11 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
     }
     __syncthreads();
 
-    if (warp == NW) {
-        // ---- loads: a lane a page of the tile ----
+    if (warp >= NW) {
+        // ---- loads: every LW-th stage, a lane a page of the tile ----
+        const int me = warp - NW;
         const int* bt = a.block_table + (size_t)(a.table_row ? a.table_row[e] : e) * a.max_blocks;
-        const int pages_per_tile = BN / ps, groups_page = ps / 8, groups_kv = nkv * groups_page;
+        const int pages_per_tile = tile_keys / ps, groups_page = ps / 8, groups_kv = nkv * groups_page;
         auto page_of = [&](int tile) {
             const int pb = my_lo + tile * pages_per_tile + lane;
             return (tile < n_tiles && lane < pages_per_tile && pb < my_hi) ? bt[pb] : -1;
@@ -164,10 +169,10 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
                 if (lane == 0) ok = mbar_wait(empty_bar(st), ((load / slots) & 1) ^ 1u, abort_flag, a.status);
                 if (!__shfl_sync(0xffffffffu, ok, 0)) return false;
             }
-            if (tile != tile_now) {
-                tile_now = tile;
+            while (tile_now < tile) {
+                ++tile_now;
                 page = next_page;
-                next_page = page_of(tile + 1);
+                next_page = page_of(tile_now + 1);
             }
             const int np = min(pages_per_tile, my_hi - (my_lo + tile * pages_per_tile));
             if (lane == 0) mbar_expect_tx(full_bar(st), (uint32_t)(np * ps * ROWB));
@@ -180,20 +185,23 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
                 }
                 const bool is_v = sub >= nkv;
                 const int group = (p * 2 * nkv + (is_v ? sub - nkv : sub)) * groups_page + (is_v ? groups_kv : 0);
-                tma_load_groups(smem_u32(smem + st * SUB) + lane * ps * ROWB, &kv_map, full_bar(st), group);
+                tma_load_groups(smem_u32(smem + st * stage_bytes) + lane * ps * ROWB, &kv_map, full_bar(st), group);
             }
             return true;
         };
         // tiles whose pages hold only tokens of earlier steps are asked for before the wait
-        int load = 0;
+        int load = me;
         bool ok = true;
         while (ok && load < n_loads && load < slots &&
                min(my_hi, my_lo + (load / per_tile + 1) * pages_per_tile) * ps <= ctx - qlen)
-            ok = issue(load++);
+        {
+            ok = issue(load);
+            load += LW;
+        }
         pdl_wait();
-        for (; ok && load < n_loads; ++load) ok = issue(load);
+        for (; ok && load < n_loads; load += LW) ok = issue(load);
         if (lane == 0 && *abort_flag) {     // let copies in flight land before the block goes away
-            for (int i = max(0, load - slots); i < load; ++i) {
+            for (int i = load - LW; i >= 0 && i > load - LW - slots; i -= LW) {
                 const long long c0 = clock64();
                 while (!mbar_try(full_bar(i % slots), (i / slots) & 1) && clock64() - c0 < VCB_WAIT_CLOCKS) {}
             }
@@ -227,56 +235,64 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
     bool ok = true;
     const int mi = lane >> 3;
     for (int t = 0; t < n_tiles; ++t) {
-        const int t0 = t_first + t * BN, load0 = t * per_tile;
-        // ---- S: this warp's 8 keys, all rows ----
-        float s[MT][4];
+        const int t0 = t_first + t * tile_keys, load0 = t * per_tile;
+        // ---- S: this warp's 16 keys, all rows ----
+        float s[MT][2][4];
 #pragma unroll
-        for (int m = 0; m < MT; ++m) s[m][0] = s[m][1] = s[m][2] = s[m][3] = 0.f;
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int n = 0; n < 2; ++n) s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f;
+        const int t_keys = min(tile_keys, k_end - t0);        // keys of this tile that count (from its start)
         for (int g = 0; g < nkv; ++g) {
             const int load = load0 + g, st = load % slots;
             if (ok) ok = mbar_wait(full_bar(st), (load / slots) & 1, abort_flag, a.status);
             if (!ok) break;
-            const uint32_t kt = smem_u32(smem + st * SUB), qb = smem_u32(q_s + g * (ROWS * ROWB));
+            const uint32_t kt = smem_u32(smem + st * stage_bytes), qb = smem_u32(q_s + g * (ROWS * ROWB));
+            if (ok && warp * 16 < t_keys) {
+                // (keys beyond the stage's are read off it -- whatever lies there, within the block's memory -- and masked)
 #pragma unroll
-            for (int k2 = 0; k2 < HD / 32; ++k2) {
-                uint32_t b[4];
-                ldmatrix_x4(b, kt + swz_kv<HALVES>(warp * 8 + (lane & 7), k2 * 4 + mi));
+                for (int ks = 0; ks < HD / 16; ++ks) {
+                    uint32_t b[4];      // keys 0 .. 7 and 8 .. 15 of this warp's, 16 lanes each
+                    ldmatrix_x4(b, kt + swz_kv<HALVES>(warp * 16 + (mi >> 1) * 8 + (lane & 7), ks * 2 + (mi & 1)));
 #pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    uint32_t q0[4], q1[4];
-                    ldmatrix_x4(q0, qb + swz_rows(ROWS, m * 16 + (lane & 15), k2 * 4 + (lane >> 4)));
-                    ldmatrix_x4(q1, qb + swz_rows(ROWS, m * 16 + (lane & 15), k2 * 4 + 2 + (lane >> 4)));
-                    mma_16816(s[m], q0, b[0], b[1]);
-                    mma_16816(s[m], q1, b[2], b[3]);
+                    for (int m = 0; m < MT; ++m) {
+                        uint32_t qf[4];
+                        ldmatrix_x4(qf, qb + swz_rows(ROWS, m * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+                        mma_16816(s[m][0], qf, b[0], b[1]);
+                        mma_16816(s[m][1], qf, b[2], b[3]);
+                    }
                 }
             }
             __syncwarp();
             if (lane == 0) mbar_arrive(empty_bar(st));
         }
-        {
-            const int c = warp * 8 + 2 * (lane & 3), key = t0 + c;
-            const bool in0 = key >= k_begin && key < k_end, in1 = key + 1 >= k_begin && key + 1 < k_end;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            const int c = warp * 16 + n * 8 + 2 * (lane & 3), key = t0 + c;
+            const bool in0 = key >= k_begin && c < t_keys, in1 = key + 1 >= k_begin && c + 1 < t_keys;
 #pragma unroll
             for (int m = 0; m < MT; ++m) {
                 float* dst = s_s + (m * 16 + (lane >> 2)) * S_LD + c;
-                *reinterpret_cast<float2*>(dst) = make_float2(in0 ? s[m][0] * a.scale : -CUDART_INF_F, in1 ? s[m][1] * a.scale : -CUDART_INF_F);
-                *reinterpret_cast<float2*>(dst + 8 * S_LD) = make_float2(in0 ? s[m][2] * a.scale : -CUDART_INF_F, in1 ? s[m][3] * a.scale : -CUDART_INF_F);
+                *reinterpret_cast<float2*>(dst) = make_float2(in0 ? s[m][n][0] * a.scale : -CUDART_INF_F, in1 ? s[m][n][1] * a.scale : -CUDART_INF_F);
+                *reinterpret_cast<float2*>(dst + 8 * S_LD) = make_float2(in0 ? s[m][n][2] * a.scale : -CUDART_INF_F, in1 ? s[m][n][3] * a.scale : -CUDART_INF_F);
             }
         }
         warps_barrier();
-        // ---- softmax: a warp a row in turn, two keys a lane ----
+        // ---- softmax: a warp a row in turn, four keys a lane ----
 #pragma unroll
         for (int i = 0; i < 2 * MT; ++i) {
             const int r = warp + 8 * i;
-            const float2 v = *reinterpret_cast<const float2*>(s_s + r * S_LD + 2 * lane);
-            const float m_new = fmaxf(m_run[i], warp_max(fmaxf(v.x, v.y)));
+            const float4 v = *reinterpret_cast<const float4*>(s_s + r * S_LD + 4 * lane);
+            const float m_new = fmaxf(m_run[i], warp_max(fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w))));
             const float use = m_new == -CUDART_INF_F ? 0.f : m_new;
             const float alpha = exp2f((m_run[i] - use) * LOG2E);
-            const float p0 = exp2f((v.x - use) * LOG2E), p1 = exp2f((v.y - use) * LOG2E);
-            l_run[i] = l_run[i] * alpha + warp_sum(p0 + p1);
+            const float p0 = exp2f((v.x - use) * LOG2E), p1 = exp2f((v.y - use) * LOG2E), p2 = exp2f((v.z - use) * LOG2E), p3 = exp2f((v.w - use) * LOG2E);
+            l_run[i] = l_run[i] * alpha + warp_sum((p0 + p1) + (p2 + p3));
             m_run[i] = m_new;
-            const __nv_bfloat162 p = __floats2bfloat162_rn(p0, p1);
-            *reinterpret_cast<__nv_bfloat162*>(p_s + r * 128 + (((lane >> 2) ^ (r & 7)) << 4) + (lane & 3) * 4) = p;
+            const __nv_bfloat162 pa = __floats2bfloat162_rn(p0, p1), pc = __floats2bfloat162_rn(p2, p3);
+            __syncwarp();       // (the row's scores have been read: its weights go over them)
+            *reinterpret_cast<uint2*>(s_s + r * S_LD + 2 * lane) =
+                make_uint2(*reinterpret_cast<const uint32_t*>(&pa), *reinterpret_cast<const uint32_t*>(&pc));
             if (lane == 0) al_s[r] = alpha;
         }
         warps_barrier();
@@ -287,14 +303,14 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
                 const int load = load0 + nkv + g, st = load % slots;
                 ok = mbar_wait(full_bar(st), (load / slots) & 1, abort_flag, a.status);
                 if (ok) {
-                    uint8_t* vt = smem + st * SUB;
-                    const bool tail = t0 + BN > k_end;
+                    uint8_t* vt = smem + st * stage_bytes;
+                    const int k_rows = (t_keys + 31) & ~31;     // keys multiplied: those behind the last weigh nothing
+                    const bool tail = t_keys < k_rows;
                     if (tail) {
                         // slots beyond the sequence and rows of pages that were not loaded: a zero weight times NaN is NaN
-                        for (int idx = lane; idx < BN * NTV; idx += 32) {
-                            const int key = idx / NTV, c = warp * NTV + idx % NTV;
-                            if (t0 + key >= k_end) *reinterpret_cast<uint4*>(vt + swz_kv<HALVES>(key, c)) = make_uint4(0, 0, 0, 0);
-                        }
+                        // (rows beyond the stage belong to the next one and are not touched: see below)
+                        for (int idx = lane; idx < (min(k_rows, tile_keys) - t_keys) * NTV; idx += 32)
+                            *reinterpret_cast<uint4*>(vt + swz_kv<HALVES>(t_keys + idx / NTV, warp * NTV + idx % NTV)) = make_uint4(0, 0, 0, 0);
                         __syncwarp();
                     }
                     const int ra = lane >> 2;
@@ -304,21 +320,22 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
                         o[g][n][0] *= al_a; o[g][n][1] *= al_a; o[g][n][2] *= al_b; o[g][n][3] *= al_b;
                     }
                     const int pr = g * gs + min(lane & 15, gs - 1);     // (rows beyond the group's repeat its last: never read)
-                    const uint32_t vb = smem_u32(vt), pb = smem_u32(p_s);
-#pragma unroll
-                    for (int k2 = 0; k2 < BN / 32; ++k2) {
+                    const uint32_t vb = smem_u32(vt), pb = smem_u32(s_s + pr * S_LD);
+                    const int last_key = tile_keys - 8;     // (of the last group of eight in the stage)
+                    for (int k0 = 0; k0 < k_rows; k0 += 32) {
                         uint32_t a0[4], a1[4], b[4];
-                        ldmatrix_x4(a0, pb + pr * 128 + (((k2 * 4 + (lane >> 4)) ^ (pr & 7)) << 4));
-                        ldmatrix_x4(a1, pb + pr * 128 + (((k2 * 4 + 2 + (lane >> 4)) ^ (pr & 7)) << 4));
+                        ldmatrix_x4(a0, pb + k0 * 2 + (lane >> 4) * 16);
+                        ldmatrix_x4(a1, pb + k0 * 2 + 32 + (lane >> 4) * 16);
+                        // groups of eight keys beyond the stage: the last group once more (finite, and weighed by zero)
                         if constexpr (NTV == 2) {
-                            ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(k2 * 32 + (mi & 1) * 8 + (lane & 7), warp * 2 + (mi >> 1)));
+                            ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(min(k0 + (mi & 1) * 8, last_key) + (lane & 7), warp * 2 + (mi >> 1)));
                             mma_16816(o[g][0], a0, b[0], b[1]);
                             mma_16816(o[g][1], a0, b[2], b[3]);
-                            ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(k2 * 32 + 16 + (mi & 1) * 8 + (lane & 7), warp * 2 + (mi >> 1)));
+                            ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(min(k0 + 16 + (mi & 1) * 8, last_key) + (lane & 7), warp * 2 + (mi >> 1)));
                             mma_16816(o[g][0], a1, b[0], b[1]);
                             mma_16816(o[g][1], a1, b[2], b[3]);
                         } else {
-                            ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(k2 * 32 + mi * 8 + (lane & 7), warp));
+                            ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(min(k0 + mi * 8, last_key) + (lane & 7), warp));
                             mma_16816(o[g][0], a0, b[0], b[1]);
                             mma_16816(o[g][0], a1, b[2], b[3]);
                         }
@@ -329,7 +346,7 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
                 }
             }
         }
-        // (the next tile's scores are written behind a barrier that every warp reaches after its products here)
+        if (t + 1 < n_tiles) warps_barrier();       // (the next tile's scores go over these weights)
     }
 #pragma unroll
     for (int i = 0; i < 2 * MT; ++i)
@@ -372,16 +389,17 @@ __global__ __launch_bounds__(NT + 32, 1) void attn_wide_kernel(const __grid_cons
 
 constexpr int MAX_SMEM = 227 * 1024;
 
-// stages the ring has room for (0: the query rows leave too little)
-int ring_slots(int hd, int nh, int nkv) {
+// shared memory that is left for the stages, in whole pieces of 1 KB (0: the query rows leave too little -- less than four
+// stages of 64 keys)
+int ring_bytes(int hd, int nh, int nkv) {
     const int mt = nh <= 16 ? 1 : (nh <= 32 ? 2 : 4);
-    const int n = (MAX_SMEM - tail_bytes(hd, mt, nkv)) / (BN * hd * 2);
-    return n < 4 ? 0 : (n < MAX_SLOTS ? n : MAX_SLOTS);
+    const int n = (MAX_SMEM - tail_bytes(hd, mt, nkv)) & ~1023;
+    return n < 4 * 64 * hd * 2 ? 0 : n;
 }
 
 template <int HD, int MT, int NG>
 int launch(const CUtensorMap& map, const WideArgs& a, int n_items, cudaStream_t stream) {
-    const size_t smem = (size_t)a.slots * BN * HD * 2 + tail_bytes(HD, MT, a.nkv);
+    const size_t smem = (size_t)a.ring_bytes + tail_bytes(HD, MT, a.nkv);
     auto kern = attn_wide_kernel<HD, MT, NG>;
     static size_t opted = 0;
     if (opted < smem) {
@@ -392,7 +410,7 @@ int launch(const CUtensorMap& map, const WideArgs& a, int n_items, cudaStream_t 
         }
         opted = smem;
     }
-    launch_pdl(kern, dim3(n_items), dim3(NT + 32), smem, stream, map, a);
+    launch_pdl(kern, dim3(n_items), dim3(NT + 32 * LW), smem, stream, map, a);
     VCB_CHECK_LAUNCH("attn_wide");
     return 0;
 }
@@ -410,7 +428,7 @@ int launch_heads(const CUtensorMap& map, const WideArgs& a, int n_items, cudaStr
 // What the kernel takes: up to 64 query heads, up to 16 of them (and 8 KV heads of 128 lanes, 16 of 64) a KV head.
 VCB_API int vcb_attn_wide_supported(int dtype, int hd, int page_size, int nh, int nkv) {
     return dtype == VCB_BF16 && (hd == 64 || hd == 128) && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64) &&
-           nkv >= 1 && nh % nkv == 0 && nh <= 64 && nh / nkv <= 16 && nkv <= (hd == 64 ? 16 : 8) && ring_slots(hd, nh, nkv) > 0;
+           nkv >= 1 && nh % nkv == 0 && nh <= 64 && nh / nkv <= 16 && nkv <= (hd == 64 ? 16 : 8) && ring_bytes(hd, nh, nkv) > 0;
 }
 
 // items: single tokens, [n_items][6] as vcb_attn_mma's; part_o [tokens][nh][slices][hd], part_ml [tokens][nh][slices][2] where
@@ -429,7 +447,7 @@ VCB_API int vcb_attn_wide(const void* q, void* out, const void* pages, long long
     CUtensorMap map;
     if (!vcb_kv_tensor_map(pages, (long long)num_pages * 2 * nkv * page_size, hd, page_size, &map, true)) return -3;
     WideArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items, part_o,
-               part_ml, nh, nkv, page_size, num_pages, window, chunked, scale, out_gate, ring_slots(hd, nh, nkv), status};
+               part_ml, nh, nkv, page_size, num_pages, window, chunked, scale, out_gate, ring_bytes(hd, nh, nkv), status};
     if (hd == 64) return nh <= 16 ? launch_heads<64, 1>(map, a, n_items, stream) : nh <= 32 ? launch_heads<64, 2>(map, a, n_items, stream) : launch_heads<64, 4>(map, a, n_items, stream);
     return nh <= 16 ? launch_heads<128, 1>(map, a, n_items, stream) : nh <= 32 ? launch_heads<128, 2>(map, a, n_items, stream) : launch_heads<128, 4>(map, a, n_items, stream);
 }

@@ -136,10 +136,10 @@ struct GemmArgs {
     const float* act_coef;    // xIELU: the factors of its parabola and of its exponential branch
 };
 
-// up x^2 + x/2 above zero, down (e^x - 1 - x) + x/2 below; near zero the bracket from its series (it would cancel)
+// up x^2 + x/2 above zero, down (e^x - 1 - x) + x/2 below.  (The bracket cancels near zero, to an error of 1e-7 beside the
+// x/2 that is added to it.)
 __device__ __forceinline__ float gemm_xielu(float x, float up, float down) {
-    const float series = x * x * fmaf(x, fmaf(x, fmaf(x, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
-    const float below = x > -0.25f ? series : __expf(x) - 1.f - x;
+    const float below = __expf(fminf(x, 0.f)) - 1.f - x;
     return fmaf(0.5f, x, x > 0.f ? up * x * x : down * below);
 }
 __device__ __forceinline__ float gemm_act(float x, int act) {
@@ -190,6 +190,42 @@ __device__ __forceinline__ void swiglu_store(uint32_t (*v)[16], __nv_bfloat16* o
 #pragma unroll
         for (int jj = 0; jj < CHUNK; ++jj)
             if (n_first + jj < N) o[(size_t)jj * ldc] = __float2bfloat16_rn(r[jj]);
+    }
+}
+
+// xIELU of a chunk's sums, bfloat16, two neighbouring features (lanes) a store: of every two tokens the even lane stores
+// the first and the odd lane the second, each with its neighbour's value.
+template <int CHUNK>
+__device__ __forceinline__ void xielu_store(const uint32_t (&v)[CHUNK / 16][16], __nv_bfloat16* out, long long ldc, int m, int M, int t0,
+                                            int N, int lane, float up, float down) {
+    // all values first, without a branch, so that their latencies overlap (as in swiglu_store)
+    float r[CHUNK];
+#pragma unroll
+    for (int jj = 0; jj < CHUNK; ++jj) r[jj] = gemm_xielu(__uint_as_float(v[jj / 16][jj % 16]), up, down);
+    const bool odd = lane & 1;
+    if (((M | (int)ldc) & 1) == 0) {        // uniform
+        __nv_bfloat162 p[CHUNK / 2];
+#pragma unroll
+        for (int jj = 0; jj < CHUNK; jj += 2) {
+            const float other = __shfl_xor_sync(0xffffffffu, odd ? r[jj] : r[jj + 1], 1);
+            p[jj / 2] = odd ? __floats2bfloat162_rn(other, r[jj + 1]) : __floats2bfloat162_rn(r[jj], other);
+        }
+        __nv_bfloat16* o = out + (size_t)(t0 + (odd ? 1 : 0)) * ldc + (m & ~1);
+        if (m < M) {
+            if (t0 + CHUNK <= N) {
+#pragma unroll
+                for (int jj = 0; jj < CHUNK; jj += 2) *reinterpret_cast<__nv_bfloat162*>(o + (size_t)jj * ldc) = p[jj / 2];
+            } else {
+#pragma unroll
+                for (int jj = 0; jj < CHUNK; jj += 2)
+                    if (t0 + jj + (odd ? 1 : 0) < N) *reinterpret_cast<__nv_bfloat162*>(o + (size_t)jj * ldc) = p[jj / 2];
+            }
+        }
+    } else if (m < M) {
+        __nv_bfloat16* o = out + (size_t)t0 * ldc + m;
+#pragma unroll
+        for (int jj = 0; jj < CHUNK; ++jj)
+            if (t0 + jj < N) o[(size_t)jj * ldc] = __float2bfloat16_rn(r[jj]);
     }
 }
 
@@ -490,6 +526,7 @@ __global__ __launch_bounds__(NTHREADS, 1) void gemm_bf16_tn_kernel(const __grid_
         // ---- epilogue: warps 2..5 own TMEM lane quarters 2, 3, 0, 1 ----
         const int q = warp & 3;
         int j = 0;
+        const float act_up = g.act == 6 ? g.act_coef[0] : 0.f, act_down = g.act == 6 ? g.act_coef[1] : 0.f;
         if (g.tile_group != nullptr) pdl_wait();
         for (int u = blockIdx.x; u < units; u += gridDim.x) {
             int m0, n0, kb0, nkb, z, mo;
@@ -525,13 +562,23 @@ __global__ __launch_bounds__(NTHREADS, 1) void gemm_bf16_tn_kernel(const __grid_
                         continue;
                     }
                 }
-                if (g.act == 6) {
-                    const float up = g.act_coef[0], down = g.act_coef[1];
-#pragma unroll
-                    for (int jj = 0; jj < CHUNK; ++jj) v[jj / 16][jj % 16] = __float_as_uint(gemm_xielu(__uint_as_float(v[jj / 16][jj % 16]), up, down));
-                }
                 if (g.swiglu) {
                     swiglu_store<CHUNK>(v, reinterpret_cast<__nv_bfloat16*>(g.out), g.ldc, m, g.M, n0 + c0, g.N, lane);
+                } else if (g.act == 6) {
+                    xielu_store<CHUNK>(v, reinterpret_cast<__nv_bfloat16*>(g.out), g.ldc, m, g.M, n0 + c0, g.N, lane, act_up, act_down);
+                } else if (g.act == 0 && n0 + c0 + CHUNK <= g.N) {
+                    // a whole chunk of tokens, the sums as they are: no branch a column
+                    if (m < g.M) {
+                        if (g.out_dtype == VCB_F32) {
+                            float* o = reinterpret_cast<float*>(g.out) + zoff + (size_t)(n0 + c0) * g.ldc + m;
+#pragma unroll
+                            for (int jj = 0; jj < CHUNK; ++jj) o[(size_t)jj * g.ldc] = __uint_as_float(v[jj / 16][jj % 16]);
+                        } else {
+                            __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(g.out) + zoff + (size_t)(n0 + c0) * g.ldc + m;
+#pragma unroll
+                            for (int jj = 0; jj < CHUNK; ++jj) o[(size_t)jj * g.ldc] = __float2bfloat16_rn(__uint_as_float(v[jj / 16][jj % 16]));
+                        }
+                    }
                 } else if (m < g.M) {
                     if (g.out_dtype == VCB_F32) {
                         float* o = reinterpret_cast<float*>(g.out) + zoff;
@@ -744,6 +791,7 @@ __global__ __launch_bounds__(NTHREADS, 1) void gemm_bf16_tn_pair_kernel(const __
         // ---- epilogue (both blocks): each owns its 128 lanes of the accumulator ----
         const int q = warp & 3;
         int j = 0;
+        const float act_up = g.act == 6 ? g.act_coef[0] : 0.f, act_down = g.act == 6 ? g.act_coef[1] : 0.f;
         for (int u = pair; u < units; u += pairs, ++j) {
             int m0, n0, kb0, nkb, z;
             unit_at(u, m0, n0, kb0, nkb, z);
@@ -774,13 +822,23 @@ __global__ __launch_bounds__(NTHREADS, 1) void gemm_bf16_tn_pair_kernel(const __
                     }
                     continue;
                 }
-                if (g.act == 6) {
-                    const float up = g.act_coef[0], down = g.act_coef[1];
-#pragma unroll
-                    for (int jj = 0; jj < CHUNK; ++jj) v[jj / 16][jj % 16] = __float_as_uint(gemm_xielu(__uint_as_float(v[jj / 16][jj % 16]), up, down));
-                }
                 if (g.swiglu) {
                     swiglu_store<CHUNK>(v, reinterpret_cast<__nv_bfloat16*>(g.out), g.ldc, m, g.M, n0 + c0, g.N, lane);
+                } else if (g.act == 6) {
+                    xielu_store<CHUNK>(v, reinterpret_cast<__nv_bfloat16*>(g.out), g.ldc, m, g.M, n0 + c0, g.N, lane, act_up, act_down);
+                } else if (g.act == 0 && n0 + c0 + CHUNK <= g.N) {
+                    // a whole chunk of tokens, the sums as they are: no branch a column
+                    if (m < g.M) {
+                        if (g.out_dtype == VCB_F32) {
+                            float* o = reinterpret_cast<float*>(g.out) + zoff + (size_t)(n0 + c0) * g.ldc + m;
+#pragma unroll
+                            for (int jj = 0; jj < CHUNK; ++jj) o[(size_t)jj * g.ldc] = __uint_as_float(v[jj / 16][jj % 16]);
+                        } else {
+                            __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(g.out) + zoff + (size_t)(n0 + c0) * g.ldc + m;
+#pragma unroll
+                            for (int jj = 0; jj < CHUNK; ++jj) o[(size_t)jj * g.ldc] = __float2bfloat16_rn(__uint_as_float(v[jj / 16][jj % 16]));
+                        }
+                    }
                 } else if (m < g.M) {
                     if (g.out_dtype == VCB_F32) {
                         float* o = reinterpret_cast<float*>(g.out) + zoff;
