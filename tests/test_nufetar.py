@@ -437,6 +437,27 @@ def test_latent_rows_without_a_query_latent(dtype, kv_rank, rot, ps, v_width, S)
         torch.testing.assert_close(out.double().cpu().view(T, nh, -1)[..., kv_rank:], want, **tol)
 
 
+@gpu
+@pytest.mark.parametrize("T", [3, 40, 64, 200])
+@pytest.mark.parametrize("H,n_in,n_out,S", [(3, 96, 128, 1), (2, 40, 33, 2), (5, 7, 70, 1), (1, 16, 300, 3), (2, 250, 24, 1)])
+def test_a_small_matrix_per_head_on_steps_of_every_length(T, H, n_in, n_out, S):
+    from vllm_cpp_b200 import ops
+    g = torch.Generator().manual_seed(T + n_in)
+    stride_in, in_off, stride_out, out_off = n_in + 6, 2, n_out + 4, 3
+    x = torch.randn(T, H * stride_in, generator=g, dtype=F64)
+    m = (torch.randn(H, n_out, n_in, generator=g, dtype=F64) * n_in ** -0.5).to(torch.bfloat16)
+    heads = lambda t: torch.einsum("hjc,thc->thj", m.double(), t.view(T, H, stride_in)[..., in_off:in_off + n_in])
+    for sums in (True, False):
+        src = partial_sums(x, S, g) if sums else x.to(torch.bfloat16).to(dev())
+        want = heads(x if sums else x.to(torch.bfloat16).double())
+        out = torch.full((T, H * stride_out), 7.0, dtype=torch.bfloat16, device=dev())
+        ops.head_linear(src, m.to(dev()), out, heads=H, n_in=n_in, n_out=n_out, in_head_stride=stride_in, in_off=in_off,
+                        out_head_stride=stride_out, out_off=out_off)
+        got = out.double().cpu().view(T, H, stride_out)
+        torch.testing.assert_close(got[..., out_off:out_off + n_out], want, atol=1e-3, rtol=6e-3)     # rounded once, on the way out
+        assert bool((got[..., :out_off] == 7.0).all()) and bool((got[..., out_off + n_out:] == 7.0).all())
+
+
 PORTION_STEPS = [(3, 1), (1, 1), (2, 7), (1, 2), (9, 1), (1, 0), (2, 2), (1, 1), (1, 1), (1, 1), (16, 1), (1, 17)]
 DECODE_STEPS = [(4, 2)] + [(1, 1)] * 45
 # portions of several staged batches each (the kernels stage 8 or 16 tokens at a time), ending on, before and behind a batch's edge

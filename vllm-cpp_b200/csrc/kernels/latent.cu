@@ -12,6 +12,7 @@
 //                             token's cache row (key row [c | k_rot], value row c)
 //  * head_linear              out[t, h, :] = M[h] in[t, h, :] for every head's own small matrix (queries into the latent
 //                             space, latent sums out to the heads' values)
+//                             (long steps with bfloat16 matrices: on the tensor cores)
 //  * rope_rows                the rotation alone, on a slice of every head of a 32-bit buffer (the queries' rotated part)
 //
 // Without a query latent (q_rank 0: queries straight from the input) the first of them has only the latter two to do.
@@ -147,7 +148,8 @@ __global__ void head_linear_kernel(HeadLinearArgs a) {
         x_s[i] = v;
     }
     __syncthreads();
-    for (int j = warp; j < a.n_out; j += nwarps) {
+    // (few tokens: a head's output lanes are dealt to several blocks)
+    for (int j = blockIdx.z * nwarps + warp; j < a.n_out; j += gridDim.z * nwarps) {
         float acc[HL_TOKENS];
 #pragma unroll
         for (int tt = 0; tt < HL_TOKENS; ++tt) acc[tt] = 0.f;
@@ -286,6 +288,115 @@ __global__ __launch_bounds__(128) void head_linear_tile_kernel(HeadLinearArgs a)
     }
 }
 
+// The same on the tensor cores (mma.sync m16n8k16), for long steps with bfloat16 matrices: one block is head h and HM_TOKENS
+// tokens, a warp 16 of them; the matrix comes in 64 rows at a time.  32-bit inputs go in as two bfloat16 parts, x = hi + lo
+// (lo what rounding to hi leaves), two products into one 32-bit sum, so that they are not rounded on the way in.
+constexpr int HM_TOKENS = 128, HM_OUT = 64, HM_THREADS = 256;
+
+__device__ __forceinline__ uint32_t hm_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void hm_ldmatrix(uint32_t (&r)[4], const void* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(hm_smem(p)));
+}
+__device__ __forceinline__ void hm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// lanes of a row in shared memory: whole steps of 16 and a pad that keeps neighbouring rows off the same banks
+__host__ __device__ constexpr int hm_ld(int n_in) { return ((n_in + 15) & ~15) + 8; }
+
+template <bool SPLIT>       // 32-bit inputs
+__global__ __launch_bounds__(HM_THREADS) void head_linear_mma_kernel(HeadLinearArgs a) {
+    extern __shared__ __align__(16) __nv_bfloat16 hm[];
+    const int ld = hm_ld(a.n_in), K = ld - 8;
+    __nv_bfloat16* x_hi = hm;                                               // [HM_TOKENS][ld]
+    __nv_bfloat16* x_lo = x_hi + (SPLIT ? HM_TOKENS * ld : 0);              // [HM_TOKENS][ld]
+    __nv_bfloat16* m_s = x_lo + HM_TOKENS * ld;                             // [HM_OUT][ld]
+    pdl_trigger();
+    pdl_wait();
+    const int h = blockIdx.y, t0 = blockIdx.x * HM_TOKENS;
+    const int nt = min(HM_TOKENS, a.T - t0);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    // a warp a row in turn
+    for (int tt = warp; tt < HM_TOKENS; tt += HM_THREADS / 32) {
+        const size_t at = (size_t)(t0 + tt) * a.ld_in + (size_t)h * a.in_head_stride + a.in_off;
+#pragma unroll 4
+        for (int c = lane; c < K; c += 32) {
+            if constexpr (SPLIT) {
+                float v = 0.f;
+                if (tt < nt && c < a.n_in)
+                    for (int s = 0; s < a.S; ++s) v += ((const float*)a.in)[at + (size_t)s * a.s_stride + c];
+                const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+                x_hi[tt * ld + c] = hi;
+                x_lo[tt * ld + c] = __float2bfloat16_rn(v - __bfloat162float(hi));
+            } else {
+                x_hi[tt * ld + c] = tt < nt && c < a.n_in ? ((const __nv_bfloat16*)a.in)[at + c] : __float2bfloat16_rn(0.f);
+            }
+        }
+    }
+    const __nv_bfloat16* m = (const __nv_bfloat16*)a.m + (size_t)h * a.n_out * a.n_in;
+    const bool vec = (a.n_in & 7) == 0 && (reinterpret_cast<uintptr_t>(m) & 15) == 0;
+    __nv_bfloat16* out = (__nv_bfloat16*)a.out + (size_t)h * a.out_head_stride + a.out_off;
+    const bool pairs = ((a.out_head_stride | a.out_off | (int)a.ld_out) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.out) & 3) == 0;
+    for (int j0 = 0; j0 < a.n_out; j0 += HM_OUT) {
+        if (vec) {
+            const int ch = K / 8;
+            for (int i = threadIdx.x; i < HM_OUT * ch; i += HM_THREADS) {
+                const int j = i / ch, c = 8 * (i % ch);
+                uint4 v = make_uint4(0, 0, 0, 0);
+                if (j0 + j < a.n_out && c < a.n_in) v = *reinterpret_cast<const uint4*>(m + (size_t)(j0 + j) * a.n_in + c);
+                *reinterpret_cast<uint4*>(m_s + j * ld + c) = v;
+            }
+        } else {
+            for (int i = threadIdx.x; i < HM_OUT * K; i += HM_THREADS) {
+                const int j = i / K, c = i % K;
+                m_s[j * ld + c] = j0 + j < a.n_out && c < a.n_in ? m[(size_t)(j0 + j) * a.n_in + c] : __float2bfloat16_rn(0.f);
+            }
+        }
+        __syncthreads();
+        float acc[HM_OUT / 8][4];
+#pragma unroll
+        for (int n = 0; n < HM_OUT / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+        const int xr = (warp * 16 + (lane & 15)) * ld + (lane >> 4) * 8;
+        const int mr = ((lane >> 4) * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8;
+        for (int k = 0; k < K; k += 16) {
+            uint32_t xh[4], xl[4];
+            hm_ldmatrix(xh, x_hi + xr + k);
+            if constexpr (SPLIT) hm_ldmatrix(xl, x_lo + xr + k);
+#pragma unroll
+            for (int n = 0; n < HM_OUT / 16; ++n) {
+                uint32_t b[4];
+                hm_ldmatrix(b, m_s + n * 16 * ld + mr + k);
+                hm_mma(acc[2 * n], xh, b[0], b[1]);
+                hm_mma(acc[2 * n + 1], xh, b[2], b[3]);
+                if constexpr (SPLIT) {
+                    hm_mma(acc[2 * n], xl, b[0], b[1]);
+                    hm_mma(acc[2 * n + 1], xl, b[2], b[3]);
+                }
+            }
+        }
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int tt = warp * 16 + (lane >> 2) + 8 * half;
+            if (tt < nt) {
+                __nv_bfloat16* o = out + (size_t)(t0 + tt) * a.ld_out;
+#pragma unroll
+                for (int n = 0; n < HM_OUT / 8; ++n) {
+                    const int j = j0 + n * 8 + 2 * (lane & 3);
+                    const float u = acc[n][2 * half], v = acc[n][2 * half + 1];
+                    if (pairs && j + 1 < a.n_out) *reinterpret_cast<__nv_bfloat162*>(o + j) = __floats2bfloat162_rn(u, v);
+                    else {
+                        if (j < a.n_out) o[j] = __float2bfloat16_rn(u);
+                        if (j + 1 < a.n_out) o[j + 1] = __float2bfloat16_rn(v);
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+}
+
 VCB_API int vcb_head_linear(const void* in, int in_dtype, int S, long long s_stride, long long ld_in, int in_head_stride, int in_off,
                             const void* m, int m_dtype, void* out, int out_dtype, long long ld_out, int out_head_stride,
                             int out_off, int T, int H, int n_in, int n_out, cudaStream_t stream) {
@@ -296,13 +407,27 @@ VCB_API int vcb_head_linear(const void* in, int in_dtype, int S, long long s_str
     VCB_CHECK_ARG(H <= 65535, "head_linear: %d heads", H);
     HeadLinearArgs a{in, in_dtype, S < 1 ? 1 : S, s_stride, ld_in, in_head_stride, in_off, m, m_dtype, out, out_dtype, ld_out,
                      out_head_stride, out_off, T, H, n_in, n_out};
+    const bool split = in_dtype == VCB_F32;
+    const size_t mma_smem = (size_t)(HM_TOKENS * (split ? 2 : 1) + HM_OUT) * hm_ld(n_in) * 2;
+    if (T >= HM_TOKENS / 2 && m_dtype == VCB_BF16 && out_dtype == VCB_BF16 && mma_smem <= 200 * 1024) {
+        auto kern = split ? head_linear_mma_kernel<true> : head_linear_mma_kernel<false>;
+        if (mma_smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)mma_smem) != cudaSuccess) {
+            vcb_set_error("head_linear: %zu bytes of shared memory refused", mma_smem);
+            return -2;
+        }
+        launch_pdl(kern, dim3((T + HM_TOKENS - 1) / HM_TOKENS, H), dim3(HM_THREADS), mma_smem, stream, a);
+        VCB_CHECK_LAUNCH("head_linear");
+        return 0;
+    }
     const size_t tile_smem = (size_t)HT_TOKENS * n_in * sizeof(float);
     if (T >= 2 * HT_TOKENS && (n_in & 3) == 0 && tile_smem <= 48 * 1024 && (reinterpret_cast<uintptr_t>(m) & 15) == 0) {
         launch_pdl(head_linear_tile_kernel, dim3((T + HT_TOKENS - 1) / HT_TOKENS, H), dim3(128), tile_smem, stream, a);
         VCB_CHECK_LAUNCH("head_linear");
         return 0;
     }
-    launch_pdl(head_linear_kernel, dim3((T + HL_TOKENS - 1) / HL_TOKENS, H), dim3(256), smem, stream, a);
+    const int token_blocks = (T + HL_TOKENS - 1) / HL_TOKENS;
+    const int deal = token_blocks <= 4 ? (n_out + 31) / 32 : 1;
+    launch_pdl(head_linear_kernel, dim3(token_blocks, H, deal < 64 ? deal : 64), dim3(256), smem, stream, a);
     VCB_CHECK_LAUNCH("head_linear");
     return 0;
 }
