@@ -83,7 +83,7 @@ VCB_API int vcb_matrix_rnn(int mode, const float* u, int S, long long s_stride, 
     RnnArgs a{Rows{u, S < 1 ? 1 : S, s_stride, ld}, x, ldx, q_col, k_col, v_col, b_col, a_col, dt_bias, rate, f_bias, lower, state,
               state_stride, q_start, q_len, slots, out, H, G, d, dv, L, TB, dp_shift, ct_shift,
               Rows{z, zS < 1 ? 1 : zS, z_stride, zld}, inv_tau, decay, ctx_len, freq, rot, interleaved, bonus};
-    const size_t smem = (size_t)(2 * ((row_decay(mode) ? 3 : 2) * TB * DP + TB * CT + 2 * TB) + TB * CT) * sizeof(float);
+    const size_t smem = (size_t)(2 * ((row_decay(mode) ? 3 : 2) * TB * DP + TB * CT + 2 * TB) + TB * (CT + 1)) * sizeof(float);
     const dim3 grid((dv + CT - 1) / CT, H, E);
     const bool split = rows > 4 * E;    // some entry has more than four tokens
     const int rc = mode == MODE_DELTA     ? rnn_run<MODE_DELTA>(a, R, C, split, grid, smem, stream)

@@ -309,7 +309,8 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
         s.b = s.g + TB;
         return s;
     };
-    float* o_s = sm + 2 * half;         // [TB][CT]
+    const int OL = CT + 1;
+    float* o_s = sm + 2 * half;         // [TB][OL] (a pad: a token's lanes and a column's tokens both lie on different banks)
     const int tid = threadIdx.x;
     const bool walker = !SPLIT || tid < WALKERS;
     const bool stager = !SPLIT || tid >= WALKERS;
@@ -386,10 +387,10 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
                             for (int c = 0; c < C; ++c) p[c] += __shfl_xor_sync(0xffffffffu, p[c], off);
                         }
                     }
-                    if (tt_of >= 0 && kl < C) o_s[tt_of * CT + cg * C + kl] = keep;
+                    if (tt_of >= 0 && kl < C) o_s[tt_of * OL + cg * C + kl] = keep;
                 } else if (tt_of >= 0) {
 #pragma unroll
-                    for (int c = 0; c < C; ++c) o_s[tt_of * CT + cg * C + c] = o_prev[c];
+                    for (int c = 0; c < C; ++c) o_s[tt_of * OL + cg * C + c] = o_prev[c];
                 }
             };
             // a token's k (then q) is fetched as soon as the token before has used its own for the last time, so the
@@ -403,117 +404,166 @@ __global__ __launch_bounds__(SPLIT ? THREADS : WALKERS, SPLIT ? 1 : 2) void matr
                     dst[2 * r + 1] = t.y;
                 }
             };
-            fetch(kr, k4, 0);
-            fetch(qr, q4, 0);
-            if constexpr (row_decay(MODE)) fetch(fr, f4, 0);
-            const float head_decay = MODE == MODE_RETAIN ? a.decay[h] : 0.f;
-            for (int tt = 0; tt < nb; ++tt) {
-                const int next = min(tt + 1, nb - 1);
-                float v[C];
+            int tt0 = 0;
+            if constexpr (C == 1 && MODE != MODE_DELTA) {
+                // Eight tokens at a time where a column is shared by eight lanes or more: their read-outs are reduced
+                // together, the lanes swapping tokens as they add (7 shuffles where eight alone take 24), each lane ending
+                // with the sum of one token.  The pairs that are added are the same, so the sums are too.
+                if (L >= 8) {
+                    const float hd8 = MODE == MODE_RETAIN ? a.decay[h] : 0.f;
+                    const uint64_t gg = pair_f32(hd8, hd8);
+                    for (; tt0 + 8 <= nb; tt0 += 8) {
+                        float op[8];
 #pragma unroll
-                for (int c = 0; c < C; ++c) v[c] = vcol[tt * CT + c];
-                uint64_t o2[C];      // (sum over even rows, sum over odd rows)
+                        for (int x = 0; x < 8; ++x) {
+                            const int tt = tt0 + x;
+                            fetch(kr, k4, tt);
+                            fetch(qr, q4, tt);
+                            if constexpr (row_decay(MODE)) fetch(fr, f4, tt);
+                            const float v = vcol[tt * CT];
+                            const uint64_t vv = pair_f32(v, v);
+                            uint64_t o2 = 0ull;
 #pragma unroll
-                for (int c = 0; c < C; ++c) o2[c] = 0ull;
-                float own[C];        // (MODE_WKV: the token's own write in its read-out, on the first of the L lanes)
-                if constexpr (MODE == MODE_WKV) {
-                    // the state as it was is read out, then it takes the token
-                    const float bonus = kl == 0 ? s.b[tt] : 0.f;
-                    uint64_t vv[C];
+                            for (int m = 0; m < R / 2; ++m) {
+                                if constexpr (MODE == MODE_WKV) o2 = fma_pair(S[0][m], qr[m], o2);
+                                if constexpr (MODE == MODE_GATED) {
+                                    const uint64_t f = kr[m], nf = fma_pair(f, pair_f32(-1.f, -1.f), pair_f32(1.f, 1.f));
+                                    S[0][m] = fma_pair(f, S[0][m], mul_pair(nf, vv));
+                                } else {
+                                    S[0][m] = fma_pair(kr[m], vv, mul_pair(row_decay(MODE) ? fr[row_decay(MODE) ? m : 0] : gg, S[0][m]));
+                                }
+                                if constexpr (MODE != MODE_WKV) o2 = fma_pair(S[0][m], qr[m], o2);
+                            }
+                            float even, oddp;
+                            unpair_f32(o2, even, oddp);
+                            op[x] = even + oddp;
+                            if constexpr (MODE == MODE_WKV) op[x] += kl == 0 ? s.b[tt] * v : 0.f;
+                        }
+                        const bool b1 = kl & 2, b2 = kl & 4;
+                        float o1[4], o2v[2];
 #pragma unroll
-                    for (int c = 0; c < C; ++c) {
-                        own[c] = bonus * v[c];
-                        vv[c] = pair_f32(v[c], v[c]);
+                        for (int x = 0; x < 4; ++x) o1[x] = (odd ? op[2 * x + 1] : op[2 * x]) + __shfl_xor_sync(0xffffffffu, odd ? op[2 * x] : op[2 * x + 1], 1);
+#pragma unroll
+                        for (int x = 0; x < 2; ++x) o2v[x] = (b1 ? o1[2 * x + 1] : o1[2 * x]) + __shfl_xor_sync(0xffffffffu, b1 ? o1[2 * x] : o1[2 * x + 1], 2);
+                        float keep = (b2 ? o2v[1] : o2v[0]) + __shfl_xor_sync(0xffffffffu, b2 ? o2v[0] : o2v[1], 4);
+                        for (int off = 8; off < L; off <<= 1) keep += __shfl_xor_sync(0xffffffffu, keep, off);
+                        if (kl < 8) o_s[(tt0 + kl) * OL + cg] = keep;
                     }
+                }
+            }
+            if (tt0 < nb) {
+                fetch(kr, k4, tt0);
+                fetch(qr, q4, tt0);
+                if constexpr (row_decay(MODE)) fetch(fr, f4, tt0);
+                const float head_decay = MODE == MODE_RETAIN ? a.decay[h] : 0.f;
+                for (int tt = tt0; tt < nb; ++tt) {
+                    const int next = min(tt + 1, nb - 1);
+                    float v[C];
 #pragma unroll
-                    for (int m = 0; m < R / 2; ++m) {
+                    for (int c = 0; c < C; ++c) v[c] = vcol[tt * CT + c];
+                    uint64_t o2[C];      // (sum over even rows, sum over odd rows)
+#pragma unroll
+                    for (int c = 0; c < C; ++c) o2[c] = 0ull;
+                    float own[C];        // (MODE_WKV: the token's own write in its read-out, on the first of the L lanes)
+                    if constexpr (MODE == MODE_WKV) {
+                        // the state as it was is read out, then it takes the token
+                        const float bonus = kl == 0 ? s.b[tt] : 0.f;
+                        uint64_t vv[C];
 #pragma unroll
                         for (int c = 0; c < C; ++c) {
-                            o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
-                            S[c][m] = fma_pair(kr[m], vv[c], mul_pair(fr[row_decay(MODE) ? m : 0], S[c][m]));
+                            own[c] = bonus * v[c];
+                            vv[c] = pair_f32(v[c], v[c]);
+                        }
+#pragma unroll
+                        for (int m = 0; m < R / 2; ++m) {
+#pragma unroll
+                            for (int c = 0; c < C; ++c) {
+                                o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
+                                S[c][m] = fma_pair(kr[m], vv[c], mul_pair(fr[row_decay(MODE) ? m : 0], S[c][m]));
+                            }
+                        }
+                        if (tt > tt0) reduce(tt - 1, false, nullptr);
+                        fetch(fr, f4, next);
+                    } else if constexpr (MODE == MODE_DELTA) {
+                        const float g = s.g[tt], beta = s.b[tt];
+                        const uint64_t gg = pair_f32(g, g);
+                        uint64_t p2[C];
+#pragma unroll
+                        for (int c = 0; c < C; ++c) p2[c] = 0ull;
+#pragma unroll
+                        for (int m = 0; m < R / 2; ++m) {
+#pragma unroll
+                            for (int c = 0; c < C; ++c) p2[c] = fma_pair(S[c][m], kr[m], p2[c]);
+                        }
+                        float p[C];
+#pragma unroll
+                        for (int c = 0; c < C; ++c) {
+                            float even, oddp;
+                            unpair_f32(p2[c], even, oddp);
+                            p[c] = even + oddp;
+                        }
+                        reduce(tt - 1, true, p);
+                        uint64_t w[C];
+#pragma unroll
+                        for (int c = 0; c < C; ++c) {
+                            const float wc = beta * (v[c] - g * p[c]);
+                            w[c] = pair_f32(wc, wc);
+                        }
+#pragma unroll
+                        for (int m = 0; m < R / 2; ++m) {
+#pragma unroll
+                            for (int c = 0; c < C; ++c) S[c][m] = fma_pair(kr[m], w[c], mul_pair(gg, S[c][m]));
+                        }
+                    } else if constexpr (MODE == MODE_DECAYED || MODE == MODE_RETAIN) {
+                        const uint64_t gg = pair_f32(head_decay, head_decay);
+                        uint64_t vv[C];
+#pragma unroll
+                        for (int c = 0; c < C; ++c) vv[c] = pair_f32(v[c], v[c]);
+#pragma unroll
+                        for (int m = 0; m < R / 2; ++m) {
+                            const uint64_t f = MODE == MODE_DECAYED ? fr[MODE == MODE_DECAYED ? m : 0] : gg;
+#pragma unroll
+                            for (int c = 0; c < C; ++c) S[c][m] = fma_pair(kr[m], vv[c], mul_pair(f, S[c][m]));
+                        }
+                        if (tt > tt0) reduce(tt - 1, false, nullptr);
+                        if constexpr (MODE == MODE_DECAYED) fetch(fr, f4, next);
+                    } else {
+                        const uint64_t ones = pair_f32(1.f, 1.f), neg = pair_f32(-1.f, -1.f);
+                        uint64_t vv[C];
+#pragma unroll
+                        for (int c = 0; c < C; ++c) vv[c] = pair_f32(v[c], v[c]);
+#pragma unroll
+                        for (int m = 0; m < R / 2; ++m) {
+                            const uint64_t f = kr[m], nf = fma_pair(f, neg, ones);      // 1 - f
+#pragma unroll
+                            for (int c = 0; c < C; ++c) S[c][m] = fma_pair(f, S[c][m], mul_pair(nf, vv[c]));
+                        }
+                        if (tt > tt0) reduce(tt - 1, false, nullptr);
+                    }
+                    fetch(kr, k4, next);
+                    if constexpr (MODE != MODE_WKV) {
+#pragma unroll
+                        for (int m = 0; m < R / 2; ++m) {
+#pragma unroll
+                            for (int c = 0; c < C; ++c) o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
                         }
                     }
-                    if (tt > 0) reduce(tt - 1, false, nullptr);
-                    fetch(fr, f4, next);
-                } else if constexpr (MODE == MODE_DELTA) {
-                    const float g = s.g[tt], beta = s.b[tt];
-                    const uint64_t gg = pair_f32(g, g);
-                    uint64_t p2[C];
-#pragma unroll
-                    for (int c = 0; c < C; ++c) p2[c] = 0ull;
-#pragma unroll
-                    for (int m = 0; m < R / 2; ++m) {
-#pragma unroll
-                        for (int c = 0; c < C; ++c) p2[c] = fma_pair(S[c][m], kr[m], p2[c]);
-                    }
-                    float p[C];
+                    fetch(qr, q4, next);
 #pragma unroll
                     for (int c = 0; c < C; ++c) {
                         float even, oddp;
-                        unpair_f32(p2[c], even, oddp);
-                        p[c] = even + oddp;
-                    }
-                    reduce(tt - 1, true, p);
-                    uint64_t w[C];
-#pragma unroll
-                    for (int c = 0; c < C; ++c) {
-                        const float wc = beta * (v[c] - g * p[c]);
-                        w[c] = pair_f32(wc, wc);
-                    }
-#pragma unroll
-                    for (int m = 0; m < R / 2; ++m) {
-#pragma unroll
-                        for (int c = 0; c < C; ++c) S[c][m] = fma_pair(kr[m], w[c], mul_pair(gg, S[c][m]));
-                    }
-                } else if constexpr (MODE == MODE_DECAYED || MODE == MODE_RETAIN) {
-                    const uint64_t gg = pair_f32(head_decay, head_decay);
-                    uint64_t vv[C];
-#pragma unroll
-                    for (int c = 0; c < C; ++c) vv[c] = pair_f32(v[c], v[c]);
-#pragma unroll
-                    for (int m = 0; m < R / 2; ++m) {
-                        const uint64_t f = MODE == MODE_DECAYED ? fr[MODE == MODE_DECAYED ? m : 0] : gg;
-#pragma unroll
-                        for (int c = 0; c < C; ++c) S[c][m] = fma_pair(kr[m], vv[c], mul_pair(f, S[c][m]));
-                    }
-                    if (tt > 0) reduce(tt - 1, false, nullptr);
-                    if constexpr (MODE == MODE_DECAYED) fetch(fr, f4, next);
-                } else {
-                    const uint64_t ones = pair_f32(1.f, 1.f), neg = pair_f32(-1.f, -1.f);
-                    uint64_t vv[C];
-#pragma unroll
-                    for (int c = 0; c < C; ++c) vv[c] = pair_f32(v[c], v[c]);
-#pragma unroll
-                    for (int m = 0; m < R / 2; ++m) {
-                        const uint64_t f = kr[m], nf = fma_pair(f, neg, ones);      // 1 - f
-#pragma unroll
-                        for (int c = 0; c < C; ++c) S[c][m] = fma_pair(f, S[c][m], mul_pair(nf, vv[c]));
-                    }
-                    if (tt > 0) reduce(tt - 1, false, nullptr);
-                }
-                fetch(kr, k4, next);
-                if constexpr (MODE != MODE_WKV) {
-#pragma unroll
-                    for (int m = 0; m < R / 2; ++m) {
-#pragma unroll
-                        for (int c = 0; c < C; ++c) o2[c] = fma_pair(S[c][m], qr[m], o2[c]);
+                        unpair_f32(o2[c], even, oddp);
+                        o_prev[c] = even + oddp;
+                        if constexpr (MODE == MODE_WKV) o_prev[c] += own[c];
                     }
                 }
-                fetch(qr, q4, next);
-#pragma unroll
-                for (int c = 0; c < C; ++c) {
-                    float even, oddp;
-                    unpair_f32(o2[c], even, oddp);
-                    o_prev[c] = even + oddp;
-                    if constexpr (MODE == MODE_WKV) o_prev[c] += own[c];
-                }
+                reduce(nb - 1, false, nullptr);
             }
-            reduce(nb - 1, false, nullptr);
             group_barrier(2, WALKERS);
             float* orow = a.out + (size_t)(t0 + b0) * (a.H * dv) + h * dv + c0;
             for (int idx = tid; idx < nb * CT; idx += WALKERS) {
                 const int tt = idx >> a.ct_shift, c = idx & (CT - 1);
-                if (c0 + c < dv) orow[(size_t)tt * (a.H * dv) + c] = o_s[idx];
+                if (c0 + c < dv) orow[(size_t)tt * (a.H * dv) + c] = o_s[tt * OL + c];
             }
         }
         if (stager && b + 1 < batches) {
