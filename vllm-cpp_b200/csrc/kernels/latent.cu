@@ -318,20 +318,62 @@ __global__ __launch_bounds__(HM_THREADS) void head_linear_mma_kernel(HeadLinearA
     const int h = blockIdx.y, t0 = blockIdx.x * HM_TOKENS;
     const int nt = min(HM_TOKENS, a.T - t0);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    // a warp a row in turn
-    for (int tt = warp; tt < HM_TOKENS; tt += HM_THREADS / 32) {
-        const size_t at = (size_t)(t0 + tt) * a.ld_in + (size_t)h * a.in_head_stride + a.in_off;
-#pragma unroll 4
-        for (int c = lane; c < K; c += 32) {
-            if constexpr (SPLIT) {
-                float v = 0.f;
-                if (tt < nt && c < a.n_in)
-                    for (int s = 0; s < a.S; ++s) v += ((const float*)a.in)[at + (size_t)s * a.s_stride + c];
-                const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-                x_hi[tt * ld + c] = hi;
-                x_lo[tt * ld + c] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    // four lanes a thread, several loads in flight (16- or 8-byte words where rows and slices lie on them)
+    const int quads = K / 4;
+    const size_t elem = SPLIT ? 4 : 2;
+    const bool words = ((a.n_in | a.in_head_stride | a.in_off | (int)(a.ld_in & 3) | (int)(a.s_stride & 3)) & 3) == 0 &&
+                       (reinterpret_cast<uintptr_t>(a.in) & (4 * elem - 1)) == 0;
+    auto fetch4 = [&](int idx) {
+        const int tt = idx / quads, c = 4 * (idx % quads);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (idx >= HM_TOKENS * quads || tt >= nt || c >= a.n_in) return v;
+        const size_t at = (size_t)(t0 + tt) * a.ld_in + (size_t)h * a.in_head_stride + a.in_off + c;
+        float* f = reinterpret_cast<float*>(&v);
+        if constexpr (SPLIT) {
+            const float* p = (const float*)a.in + at;
+            for (int s = 0; s < a.S; ++s, p += a.s_stride) {
+                if (words) {
+                    const float4 w = *reinterpret_cast<const float4*>(p);
+                    v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+                } else {
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+                        if (c + k < a.n_in) f[k] += p[k];
+                }
+            }
+        } else {
+            const __nv_bfloat16* p = (const __nv_bfloat16*)a.in + at;
+            if (words) {
+                const uint2 raw = *reinterpret_cast<const uint2*>(p);
+                const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+                const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+                v = make_float4(lo.x, lo.y, hi.x, hi.y);
             } else {
-                x_hi[tt * ld + c] = tt < nt && c < a.n_in ? ((const __nv_bfloat16*)a.in)[at + c] : __float2bfloat16_rn(0.f);
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (c + k < a.n_in) f[k] = __bfloat162float(p[k]);
+            }
+        }
+        return v;
+    };
+    for (int i0 = threadIdx.x; i0 < HM_TOKENS * quads; i0 += 4 * HM_THREADS) {
+        float4 v[4];
+#pragma unroll
+        for (int w = 0; w < 4; ++w) v[w] = fetch4(i0 + w * HM_THREADS);
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+            const int idx = i0 + w * HM_THREADS;
+            if (idx < HM_TOKENS * quads) {
+                const int at = (idx / quads) * ld + 4 * (idx % quads);
+                const float f[4] = {v[w].x, v[w].y, v[w].z, v[w].w};
+                __align__(8) __nv_bfloat16 hi[4], lo[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    hi[k] = __float2bfloat16_rn(f[k]);
+                    lo[k] = __float2bfloat16_rn(f[k] - __bfloat162float(hi[k]));
+                }
+                *reinterpret_cast<uint2*>(x_hi + at) = *reinterpret_cast<const uint2*>(hi);
+                if constexpr (SPLIT) *reinterpret_cast<uint2*>(x_lo + at) = *reinterpret_cast<const uint2*>(lo);
             }
         }
     }
