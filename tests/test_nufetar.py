@@ -84,7 +84,10 @@ def hand_made(cfg, tensors, seed):
             out[p + "u"] = tensors[p + "u"] * 8.0
             for m in "rkvgw":
                 out[p + "mu." + m] = torch.rand(cfg.width, generator=g)
+        # sublayers whose results outweigh the embedding they are added to: what is generated depends on all that came before
+        out[p + "o"] = tensors[p + "o"] * 3.0
         if layer.mlp is not None:
+            out[f"l{i}.mlp.down"] = tensors[f"l{i}.mlp.down"] * 3.0
             out[f"l{i}.mlp.act"] = torch.tensor([0.7, -0.9]) + 0.3 * i
             out[f"l{i}.mlp.up"] = tensors[f"l{i}.mlp.up"] * 8.0
     return {k: v.to(torch.bfloat16) for k, v in out.items()}

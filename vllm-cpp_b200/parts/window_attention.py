@@ -63,7 +63,8 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     over latent rows, whose one KV head's values are the first lanes of its keys).
     ``chunked``: the window is the chunk of ``window`` positions, counted from position 0, that a query lies in.
     ``wide``: ``q`` is [T, nh * nkv * hd], a block of lanes per KV head, and a row's score with a key position is the sum
-    of the blocks' products with all heads' keys there (queries mixed across heads).  ``out_gate`` (float32 [T, nh])
+    of the blocks' products with all heads' keys there (queries mixed across heads); single tokens with such rows run on a
+    kernel whose block is a token and key slice with all heads (ops.attn_wide), where it takes the sizes.  ``out_gate`` (float32 [T, nh])
     multiplies each head's result."""
     x = q
     if nkv == 1:
