@@ -257,21 +257,23 @@ def test_what_a_layer_run_keeps_per_request():
     for run in range(6):
         assert (specs[(run, 0)].kind, specs[(run, 0)].shape, specs[(run, 0)].dtype) == ("state", (48,), "float32")
     kv = specs[(0, 1)]
-    assert (kv.kind, kv.num_kv_heads, kv.head_dim, kv.v_head_dim) == ("kv", 1, 12 + 4, 12)       # the latent and the rotated key part
+    assert (kv.kind, kv.num_kv_heads, kv.head_dim, kv.one_row) == ("kv", 1, 12 + 4, True)       # the latent and the rotated key part
     for run in (1, 3):
         assert (specs[(run, 1)].shape, specs[(run, 1)].dtype) == ((4, 12, 8), "float32")          # heads, value columns, rows
         assert specs[(run, 2)].shape == (2, 2 * 16 + 48)                                       # the convolution's last inputs
     for run in (2, 4):
         assert specs[(run, 1)].shape == (2, 10, 6)
-    assert (specs[(5, 1)].head_dim, specs[(5, 1)].v_head_dim) == (5 + 8, 5)
+    assert (specs[(5, 1)].head_dim, specs[(5, 1)].one_row) == (5 + 8, True)
     c, _ = configs()["C"]
     specs = models.build_model(c, torch.float32, "cpu").cache_specs()
     assert specs[(2, 1)].shape == (5, 10, 20) and (2, 2) not in specs       # one tap: the convolution keeps nothing
-    # cached rows of 64 lanes in bfloat16: value rows as wide as key rows, for the attention kernels on the tensor cores
+    # in bfloat16 rows are as wide as the attention kernels on the tensor cores take; values are read from the key rows
     b, _ = configs()["B"]
     kv32 = models.build_model(b, torch.float32, "cpu").cache_specs()[(1, 1)]
     kv16 = models.build_model(b, torch.bfloat16, "cpu").cache_specs()[(1, 1)]
-    assert (kv32.head_dim, kv32.v_head_dim) == (64, 48) and (kv16.head_dim, kv16.v_head_dim) == (64, 0)
+    assert (kv32.head_dim, kv16.head_dim) == (64, 64) and kv32.one_row and kv16.one_row
+    kv16 = models.build_model(cfg, torch.bfloat16, "cpu").cache_specs()[(0, 1)]
+    assert (kv16.num_kv_heads, kv16.head_dim, kv16.v_head_dim) == (1, 64, 0)
 
 
 def test_stretched_frequencies_agree_with_the_plain_ones():

@@ -206,7 +206,7 @@ def test_what_a_layer_keeps_per_request():
     kv = specs[1]
     assert (kv.kind, kv.num_kv_heads, kv.head_dim, kv.v_head_dim, kv.window, kv.chunked) == ("kv", 2, 8, 6, 10, True)
     kv = specs[2]
-    assert (kv.kind, kv.num_kv_heads, kv.head_dim, kv.v_head_dim, kv.window, kv.chunked) == ("kv", 1, 13, 9, 9, False)
+    assert (kv.kind, kv.num_kv_heads, kv.head_dim, kv.one_row, kv.window, kv.chunked) == ("kv", 1, 13, True, 9, False)
     from vllm_cpp_b200.cache.device_cache import CacheLayout
     lay = CacheLayout(specs)
     assert len(lay.paged) == 2       # a standing and a sliding window are different pools

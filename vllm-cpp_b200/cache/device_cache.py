@@ -8,7 +8,8 @@ mixers keep, and owns the tensors:
   and the same window -- is one tensor
   ``[caches in group, num_pages, 2 (K,V), kv_heads, page_size, head_dim]`` (where values
   have another head size than keys: ``[caches, num_pages, kv_heads * page_size *
-  (head_dim + v_head_dim)]``, keys first): a page id
+  (head_dim + v_head_dim)]``, keys first; where the key rows double as values:
+  ``[caches, num_pages, 1, kv_heads, page_size, head_dim]``): a page id
   means the same page in every cache of the group (as a page of the reference
   covers every layer, src/kv_cache_manager.cpp:15-29), head-major inside a page so
   the keys of one KV head are contiguous runs of page_size * head_dim;
@@ -83,8 +84,8 @@ class CacheLayout:
                 for g in self.paged]
 
     def bytes_per_token(self, elem_size: int) -> int:
-        return sum(len(g.cache_ids) * g.spec.num_kv_heads * (g.spec.head_dim + (g.spec.v_head_dim or g.spec.head_dim)) * elem_size
-                   for g in self.paged)
+        lanes = lambda s: s.head_dim if s.one_row else s.head_dim + (s.v_head_dim or s.head_dim)
+        return sum(len(g.cache_ids) * g.spec.num_kv_heads * lanes(g.spec) * elem_size for g in self.paged)
 
 
 class DeviceCache:
@@ -100,7 +101,7 @@ class DeviceCache:
                     # values of another size than keys: a page is one flat row, keys first
                     shape = (n, pages, g.spec.num_kv_heads * ps * (g.spec.head_dim + g.spec.v_head_dim))
                 else:
-                    shape = (n, pages, 2, g.spec.num_kv_heads, ps, g.spec.head_dim)
+                    shape = (n, pages, 1 if g.spec.one_row else 2, g.spec.num_kv_heads, ps, g.spec.head_dim)
                 self.tensors.append(torch.zeros(shape, dtype=dtype, device=device))
             else:
                 sdt = _TORCH_DTYPES[g.spec.dtype]

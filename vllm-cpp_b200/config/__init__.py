@@ -6,5 +6,6 @@ from .nagavik import NagavikConfig
 from .fifudra import FifudraConfig
 from .mefupel import MefupelConfig
 from .nufetar import NufetarConfig
+from .disorax import DisoraxConfig
 
-__all__ = ["ConfigError", "ModelConfig", "EngineConfig", "Qwen3Config", "RimopelConfig", "NagavikConfig", "FifudraConfig", "MefupelConfig", "NufetarConfig", "load_config_dict"]
+__all__ = ["ConfigError", "ModelConfig", "EngineConfig", "Qwen3Config", "RimopelConfig", "NagavikConfig", "FifudraConfig", "MefupelConfig", "NufetarConfig", "DisoraxConfig", "load_config_dict"]

@@ -25,6 +25,11 @@
 // sum over the KV heads of block . that head's key (queries mixed across heads, see rope_store.cu), while its values are
 // still those of the row's own KV head.  A gate per (token, head) may multiply the result (`out_gate`).  Key rows may be as
 // wide as shared memory has room for; values wider than a block's threads hold are dealt to further blocks (grid z).
+// The gate may be per output lane (`gate_lanes`).  A page may hold key rows alone (`one_row`): the values are the first hd_v
+// lanes of the key rows.  And where rows are wide because one shared row is kept in blocks (`blocks`: attention over latent
+// rows wider than a tile), the KV heads are those blocks, every query head meets all of them, and nh counts (block, query
+// head) pairs, block after block: pair (G, h) has the wide row of query head h and sums the values of block G.  Results
+// lie query head by query head, its blocks side by side.
 // Items whose key range is sliced write (max, sum, unnormalised output) partials,
 // merged by attn_merge_kernel in slice order.
 #include "common.cuh"
@@ -69,7 +74,10 @@ struct AttnArgs {
     const float* sink_value;    // with a sink: its score per head (null: 0); it is not scaled
     int chunked;                // the window is the chunk of `window` positions that pos lies in
     int wide;                   // q rows are [nkv][hd] lanes, one block per KV head
-    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
+    const float* out_gate;      // [tokens][query heads] or null: what the result of a (token, head) is multiplied by
+    int gate_lanes;             // out_gate is laid out as the result, a factor per lane
+    int one_row;                // pages hold keys only: values are the first hd_v lanes of the key rows
+    int blocks;                 // the KV heads are blocks of one shared row (see above)
 };
 
 template <typename T> struct Vec8;
@@ -136,13 +144,17 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
         // an empty entry: its slices still say "nothing here" (max = -inf, sum = 0), so that the merge writes zeros
         // rather than whatever the partial buffers held before
         if (nslices > 1 && a.part_ml != nullptr && tid < gq) {
-            const size_t prow = ((size_t)dec_index * a.nh + head0 + tid) * nslices + slice;
+            const int oh = a.blocks ? (head0 - kvh * g + tid) * a.nkv + kvh : head0 + tid;
+            const size_t prow = ((size_t)dec_index * a.nh + oh) * nslices + slice;
             a.part_ml[prow * 2] = -CUDART_INF_F;
             a.part_ml[prow * 2 + 1] = 0.f;
         }
         return;
     }
     const int R = nq * gq;  // rows in use: r = iq * gq + ih
+    // query heads, the first one here, and where head ih's result lies among a token's
+    const int nqh = a.blocks ? g : a.nh, qh0 = a.blocks ? head0 - kvh * g : head0;
+    auto out_head = [&](int ih) { return a.blocks ? (qh0 + ih) * a.nkv + kvh : head0 + ih; };
 
     const int row0 = a.q_start[e] + q0;       // flat token index of the first query
     const int pos0 = ctx - qlen + q0;         // its position
@@ -169,11 +181,11 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
     for (int idx = tid; idx < R * qw; idx += TK) {
         const int r = idx / qw, d = idx % qw;
         const int iq = r / gq, ih = r % gq;
-        q_s[r * qw + d] = to_f32(qg[((size_t)(row0 + iq) * a.nh + head0 + ih) * qw + d]) * a.scale;
+        q_s[r * qw + d] = to_f32(qg[((size_t)(row0 + iq) * nqh + qh0 + ih) * qw + d]) * a.scale;
     }
     if (tid < RMAX) {
         const bool with_sink = a.sink && slice == 0;
-        const int h = head0 + tid % gq;
+        const int h = qh0 + tid % gq;
         m_s[tid] = with_sink ? (a.sink_value != nullptr && tid < R ? a.sink_value[h] : 0.f) : -CUDART_INF_F;
         l_s[tid] = with_sink ? 1.f : 0.f;
         da_s[tid] = a.dist_a != nullptr && tid < R ? a.dist_a[h] : (a.slope != nullptr && tid < R ? a.slope[h] : 0.f);
@@ -209,7 +221,8 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
                     valid = false;
                     voff_s[tid] = -1;
                 } else {
-                    voff_s[tid] = (long long)page * a.page_stride + (long long)a.nkv * ps * hd + ((long long)kvh * ps + kidx % ps) * hdv;
+                    voff_s[tid] = (long long)page * a.page_stride + (a.one_row ? ((long long)kvh * ps + kidx % ps) * hd
+                                  : (long long)a.nkv * ps * hd + ((long long)kvh * ps + kidx % ps) * hdv);
                     for (int b = 0; b < (a.wide ? a.nkv : 1); ++b) {
                         const T* kp = pages + (long long)page * a.page_stride + ((long long)(a.wide ? b : kvh) * ps + kidx % ps) * hd;
                         const float* q_b = q_s + b * hd;
@@ -315,9 +328,9 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
                     if (r < R) {
                         const float l = l_s[r];
                         const int iq = r / gq, ih = r % gq;
-                        const size_t row = (size_t)(row0 + iq) * a.nh + head0 + ih;
+                        const size_t row = (size_t)(row0 + iq) * a.nh + out_head(ih);
                         float o = l > 0.f ? acc_o[r][i] / l : 0.f;
-                        if (a.out_gate != nullptr) o *= a.out_gate[row];
+                        if (a.out_gate != nullptr) o *= a.out_gate[a.gate_lanes ? row * hdv + d : (size_t)(row0 + iq) * nqh + qh0 + ih];
                         og[row * hdv + d] = from_f32<T>(o);
                     }
                 }
@@ -328,7 +341,7 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
 #pragma unroll
         for (int r = 0; r < RMAX; ++r) {
             if (r < R) {
-                const size_t prow = ((size_t)dec_index * a.nh + head0 + r) * nslices + slice;
+                const size_t prow = ((size_t)dec_index * a.nh + out_head(r)) * nslices + slice;
 #pragma unroll
                 for (int i = 0; i < DPT; ++i) {
                     const int d = d0 + tid + i * TK;
@@ -347,7 +360,7 @@ __global__ __launch_bounds__(TK) void attn_paged_kernel(AttnArgs a) {
 template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   const int* __restrict__ dec_rows, T* __restrict__ out, int nh, int hd, int nslices,
-                                  const float* __restrict__ out_gate) {
+                                  const float* __restrict__ out_gate, int gate_lanes, int gate_blocks) {
     pdl_trigger();
     pdl_wait();
     const int n = blockIdx.x, h = blockIdx.y;
@@ -363,7 +376,8 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
         if (threadIdx.x == 0) m_all = m;
     }
     const int row = dec_rows[n];
-    const float gate = out_gate != nullptr && row >= 0 ? out_gate[(size_t)row * nh + h] : 1.f;
+    // (gate_blocks results side by side belong to one head)
+    const float gate = out_gate != nullptr && !gate_lanes && row >= 0 ? out_gate[((size_t)row * nh + h) / gate_blocks] : 1.f;
     constexpr int DPT = 4;      // value lanes a thread (of blocks of 64 to 256 threads)
     for (int d0 = 0; d0 < hd; d0 += DPT * blockDim.x) {
         float l = 0.f, o[DPT] = {0.f, 0.f, 0.f, 0.f};
@@ -395,7 +409,10 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
 #pragma unroll
             for (int k = 0; k < DPT; ++k) {
                 const int d = d0 + threadIdx.x + k * blockDim.x;
-                if (d < hd) out[((size_t)row * nh + h) * hd + d] = from_f32<T>((l > 0.f ? o[k] / l : 0.f) * gate);
+                if (d < hd) {
+                    const size_t at = ((size_t)row * nh + h) * hd + d;
+                    out[at] = from_f32<T>((l > 0.f ? o[k] / l : 0.f) * (gate_lanes && out_gate != nullptr ? out_gate[at] : gate));
+                }
             }
         }
     }
@@ -434,9 +451,11 @@ VCB_API int vcb_attn_paged_ex(const void* q, void* out, int dtype, const void* p
                               float* part_ml, int nh, int nkv, int hd, int page_size, int num_pages, int window,
                               float scale, int keep_first, const float* dist_a, const float* dist_b, int hd_v,
                               float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
-                              const float* out_gate, int* status, cudaStream_t stream) {
+                              const float* out_gate, int gate_lanes, int one_row, int blocks, int* status, cudaStream_t stream) {
     if (n_items == 0) return 0;
     if (hd_v <= 0) hd_v = hd;
+    VCB_CHECK_ARG(!one_row || hd_v <= hd, "attn_paged: values of %d lanes in key rows of %d", hd_v, hd);
+    VCB_CHECK_ARG(!blocks || (wide && dist_a == nullptr && slope == nullptr), "attn_paged: blocks of one shared row want wide query rows and no distance terms");
     VCB_CHECK_ARG(nh > 0 && nkv > 0 && nh % nkv == 0, "attn_paged: %d query heads are not a multiple of %d KV heads", nh, nkv);
     VCB_CHECK_ARG(hd >= 1 && hd_v >= 1, "attn_paged: head sizes %d (keys) and %d (values)", hd, hd_v);
     VCB_CHECK_ARG(hd % 8 != 0 || (page_stride % 8 == 0 && ((long long)nkv * page_size * hd) % 8 == 0),
@@ -448,7 +467,7 @@ VCB_API int vcb_attn_paged_ex(const void* q, void* out, int dtype, const void* p
     VCB_CHECK_ARG(softcap >= 0.f, "attn_paged: a negative cap");
     AttnArgs a{q, out, pages, page_stride, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items, part_o, part_ml,
                nh, nkv, hd, page_size, num_pages, window, scale, status, 0, 0, keep_first, dist_a, dist_b, hd_v,
-               softcap, slope, sink, sink_value, chunked, wide, out_gate};
+               softcap, slope, sink, sink_value, chunked, wide, out_gate, gate_lanes, one_row, blocks};
     if (dtype == VCB_F32) return rows_max == 8 ? launch_attn<float, 8>(a, n_items, stream) : launch_attn<float, 32>(a, n_items, stream);
     return rows_max == 8 ? launch_attn<__nv_bfloat16, 8>(a, n_items, stream) : launch_attn<__nv_bfloat16, 32>(a, n_items, stream);
 }
@@ -470,13 +489,13 @@ VCB_API int vcb_attn_paged(const void* q, void* out, int dtype, const void* page
 }
 
 VCB_API int vcb_attn_merge(const float* part_o, const float* part_ml, const int* dec_rows, void* out, int dtype,
-                           int n_dec, int nh, int hd, int nslices, const float* out_gate, cudaStream_t stream) {
+                           int n_dec, int nh, int hd, int nslices, const float* out_gate, int gate_lanes, int gate_blocks, cudaStream_t stream) {
     if (n_dec == 0) return 0;
     const int threads = hd <= 64 ? 64 : (hd <= 128 ? 128 : 256);
     if (dtype == VCB_F32)
-        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices, out_gate);
+        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices, out_gate, gate_lanes, gate_blocks);
     else
-        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices, out_gate);
+        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices, out_gate, gate_lanes, gate_blocks);
     VCB_CHECK_LAUNCH("attn_merge");
     return 0;
 }
@@ -560,9 +579,9 @@ VCB_API int vcb_attn_decode_no_alloc(const void* q, void* out, int dtype, const 
     if (rc) return rc;
     const int threads = hd <= 64 ? 64 : (hd <= 128 ? 128 : 256);
     if (dtype == VCB_F32)
-        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices, (const float*)nullptr);
+        launch_pdl(attn_merge_kernel<float>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (float*)out, nh, hd, nslices, (const float*)nullptr, 0, 1);
     else
-        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices, (const float*)nullptr);
+        launch_pdl(attn_merge_kernel<__nv_bfloat16>, dim3(n_dec, nh), dim3(threads), 0, stream, part_o, part_ml, dec_rows, (__nv_bfloat16*)out, nh, hd, nslices, (const float*)nullptr, 0, 1);
     VCB_CHECK_LAUNCH("attn_decode_no_alloc merge");
     return 0;
 }

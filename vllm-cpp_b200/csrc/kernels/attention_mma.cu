@@ -97,7 +97,10 @@ struct AttnArgs {
     int sink;
     const float* sink_value;    // with a sink: the silent key's score per head, not scaled (null: 0)
     int chunked;                // the window stands still: the chunk of `window` positions that a query's position lies in
-    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
+    const float* out_gate;      // [tokens][query heads] or null: what the result of a (token, head) is multiplied by
+    int gate_lanes;             // out_gate is laid out as the result, a factor per lane
+    int one_row;                // pages hold keys only: the values are the key rows
+    int blocks;                 // (with wide rows) the KV heads are blocks of one shared row, see attention.cu
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, int src_bytes) {
@@ -229,6 +232,15 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     const int head0 = kvh * g + hc * gq_max;
     const int gq = min(gq_max, g - hc * gq_max);
     const int R = nq * gq;
+    // query heads, the first one here, and where head ih's result lies among a token's
+    const bool in_blocks = WIDE && a.blocks;
+    const int nqh = in_blocks ? g : a.nh, qh0 = in_blocks ? head0 - kvh * g : head0;
+    auto out_head = [&](int ih) { return in_blocks ? (qh0 + ih) * a.nkv + kvh : head0 + ih; };
+    auto gate_at = [&](int row, int ih, int d) {      // the gate's factors for lanes d, d + 1
+        if (a.gate_lanes) return *reinterpret_cast<const float2*>(a.out_gate + ((size_t)row * a.nh + out_head(ih)) * HD + d);
+        const float f = a.out_gate[(size_t)row * nqh + qh0 + ih];
+        return make_float2(f, f);
+    };
 
     const int row0 = a.q_start[e] + q0;
     const int pos0 = ctx - qlen + q0;
@@ -271,7 +283,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
     // block-table read, took about as long as the tile's share of HBM time. ----
     const int pages_per_tile = BN / ps;
     const int groups_page = ps / 8;
-    const int groups_kv = a.nkv * groups_page;   // groups of 8 rows from a page's K to its V
+    const int parts = a.one_row ? 1 : 2;
+    const int groups_kv = a.one_row ? 0 : a.nkv * groups_page;   // groups of 8 rows from a page's K to its V
     const int my_pg = lane >> 1, my_v = lane & 1;
     const int first_pb_hi = (n_first + ps - 1) / ps;   // pages that hold the kept first keys read here
     auto tile_pb0 = [&](int it) { return it < n_ft ? it * pages_per_tile : my_pb_lo + (it - n_ft) * pages_per_tile; };
@@ -309,7 +322,7 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                 atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                 page = 0;   // keep the byte count whole; the status word reports the fault
             }
-            const int group = (page * 2 * a.nkv + (my_v ? kvh : key_head)) * groups_page + (my_v ? groups_kv : 0);
+            const int group = (page * parts * a.nkv + (my_v ? kvh : key_head)) * groups_page + (my_v ? groups_kv : 0);
             const uint32_t dst = smem_u32((my_v ? v_s : k_s) + st * TILE_BYTES) + my_pg * ps * ROWB;
             tma_load_groups(dst, &kv_map, full_bar(st), group);
         }
@@ -476,7 +489,7 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
             uint4 v = make_uint4(0, 0, 0, 0);
             if (r < R) {
                 const int iq = r / gq, ih = r % gq;
-                v = *reinterpret_cast<const uint4*>(a.q + ((size_t)(row0 + iq) * a.nh + head0 + ih) * (NG * HD) + c * 8);
+                v = *reinterpret_cast<const uint4*>(a.q + ((size_t)(row0 + iq) * nqh + qh0 + ih) * (NG * HD) + c * 8);
             }
             *reinterpret_cast<uint4*>(q_s + (c / CH) * (RMAX * ROWB) + swz<RMAX>(r, c % CH)) = v;
         }
@@ -507,7 +520,7 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
             }
             const int off = swz_kv<HD / 64>(j, c);
             cp_async16(smem_u32(kd + off), src, bytes);
-            if (with_v) cp_async16(smem_u32(vd + off), bytes ? src + ((size_t)a.nkv + kvh - key_head) * ps * HD : src, bytes);
+            if (with_v) cp_async16(smem_u32(vd + off), bytes ? src + ((a.one_row ? 0 : a.nkv) + kvh - key_head) * ps * HD : src, bytes);
         }
     };
 
@@ -550,8 +563,8 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
         ok_a[mr] = r_a[mr] < R;
         ok_b[mr] = r_a[mr] + 8 < R;
         const bool scored = with_sink && a.sink_value != nullptr;
-        m_run[mr][0] = with_sink ? (scored && ok_a[mr] ? a.sink_value[head0 + r_a[mr] % gq] : 0.f) : -CUDART_INF_F;
-        m_run[mr][1] = with_sink ? (scored && ok_b[mr] ? a.sink_value[head0 + (r_a[mr] + 8) % gq] : 0.f) : -CUDART_INF_F;
+        m_run[mr][0] = with_sink ? (scored && ok_a[mr] ? a.sink_value[qh0 + r_a[mr] % gq] : 0.f) : -CUDART_INF_F;
+        m_run[mr][1] = with_sink ? (scored && ok_b[mr] ? a.sink_value[qh0 + (r_a[mr] + 8) % gq] : 0.f) : -CUDART_INF_F;
         l_run[mr][0] = l_run[mr][1] = with_sink && (lane & 3) == 0 ? 1.f : 0.f;   // per-thread partial sums (reduced over the quad at the end)
     }
     float da_a[MR], db_a[MR], da_b[MR], db_b[MR];   // the distance penalty's a_h ln 2 and b_h of rows a and b
@@ -846,15 +859,15 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
         }
         const int iq = r / gq, ih = r % gq;
         if (nslices == 1) {
-            float inv = l > 0.f ? 1.f / l : 0.f;
-            if (a.out_gate != nullptr) inv *= a.out_gate[(size_t)(row0 + iq) * a.nh + head0 + ih];
-            *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)(row0 + iq) * a.nh + head0 + ih) * HD + d) =
-                __floats2bfloat162_rn(o0 * inv, o1 * inv);
+            const float inv = l > 0.f ? 1.f / l : 0.f;
+            const float2 gt = a.out_gate != nullptr ? gate_at(row0 + iq, ih, d) : make_float2(1.f, 1.f);
+            *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)(row0 + iq) * a.nh + out_head(ih)) * HD + d) =
+                __floats2bfloat162_rn(o0 * inv * gt.x, o1 * inv * gt.y);
         } else if (in_cluster) {
             *reinterpret_cast<float2*>(cl_o + (size_t)r * HD + d) = make_float2(o0, o1);
             if (d == 0) *reinterpret_cast<float2*>(cl_ml + r * 2) = make_float2(m, l);
         } else {
-            const size_t prow = ((size_t)dec_index * a.nh + head0 + r) * nslices + slice;
+            const size_t prow = ((size_t)dec_index * a.nh + out_head(r)) * nslices + slice;
             *reinterpret_cast<float2*>(a.part_o + prow * HD + d) = make_float2(o0, o1);
             if (d == 0) {
                 a.part_ml[prow * 2] = m;
@@ -895,10 +908,10 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                         o1 += ov[j].y * w;
                     }
                 }
-                float inv = l > 0.f ? 1.f / l : 0.f;
-                if (a.out_gate != nullptr) inv *= a.out_gate[(size_t)out_row * a.nh + head0 + ih];
-                *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)out_row * a.nh + head0 + ih) * HD + d) =
-                    __floats2bfloat162_rn(o0 * inv, o1 * inv);
+                const float inv = l > 0.f ? 1.f / l : 0.f;
+                const float2 gt = a.out_gate != nullptr ? gate_at(out_row, ih, d) : make_float2(1.f, 1.f);
+                *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)out_row * a.nh + out_head(ih)) * HD + d) =
+                    __floats2bfloat162_rn(o0 * inv * gt.x, o1 * inv * gt.y);
             }
         }
         cluster_barrier();          // nobody leaves while its result may still be read
@@ -929,7 +942,7 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                 constexpr int MS = VCB_MS;     // slices merged per batch (more run through the loop again)
                 for (int idx = tid; idx < gq * (HD / 2); idx += blockDim.x) {
                     const int ih = idx / (HD / 2), d = (idx % (HD / 2)) * 2;
-                    const size_t prow0 = ((size_t)dec_index * a.nh + head0 + ih) * nslices;
+                    const size_t prow0 = ((size_t)dec_index * a.nh + out_head(ih)) * nslices;
                     float m = -CUDART_INF_F, l = 0.f, o0 = 0.f, o1 = 0.f;
                     if (nslices <= MS) {
                         float2 mlv[MS], ov[MS];
@@ -974,10 +987,10 @@ __global__ __launch_bounds__(WR * WK * 32 + (TMA ? 32 : 0)) void attn_mma_kernel
                             }
                         }
                     }
-                    float inv = l > 0.f ? 1.f / l : 0.f;
-                    if (a.out_gate != nullptr) inv *= a.out_gate[(size_t)out_row * a.nh + head0 + ih];
-                    *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)out_row * a.nh + head0 + ih) * HD + d) =
-                        __floats2bfloat162_rn(o0 * inv, o1 * inv);
+                    const float inv = l > 0.f ? 1.f / l : 0.f;
+                    const float2 gt = a.out_gate != nullptr ? gate_at(out_row, ih, d) : make_float2(1.f, 1.f);
+                    *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)out_row * a.nh + out_head(ih)) * HD + d) =
+                        __floats2bfloat162_rn(o0 * inv * gt.x, o1 * inv * gt.y);
                 }
             }
         }
@@ -1092,8 +1105,8 @@ int launch(const AttnArgs& a, int n_items, cudaStream_t stream) {
     CUtensorMap map;
     memset(&map, 0, sizeof(map));
     if (TMA) {
-        const long long rows = (long long)a.num_pages * 2 * a.nkv * a.page_size;
-        if (a.page_stride != (long long)2 * a.nkv * a.page_size * HD) {
+        const long long rows = (long long)a.num_pages * (a.one_row ? 1 : 2) * a.nkv * a.page_size;
+        if (a.page_stride != (long long)(a.one_row ? 1 : 2) * a.nkv * a.page_size * HD) {
             vcb_set_error("attn_mma: the pages of a layer must be contiguous for TMA loads");
             return -1;
         }
@@ -1163,7 +1176,7 @@ VCB_API int vcb_attn_mma_ex(const void* q, void* out, const void* pages, long lo
                             float* part_ml, int* slice_counters, const int* dec_rows, int nh, int nkv, int hd,
                             int page_size, int num_pages, int window, float scale, int keep_first, const float* dist_a,
                             const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
-                            const float* out_gate, int* status, int allow_tma, int cluster, cudaStream_t stream);
+                            const float* out_gate, int gate_lanes, int one_row, int blocks, int* status, int allow_tma, int cluster, cudaStream_t stream);
 
 VCB_API int vcb_attn_mma(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                          const int* table_row, int max_blocks, const int* q_start, const int* q_len,
@@ -1173,17 +1186,17 @@ VCB_API int vcb_attn_mma(const void* q, void* out, const void* pages, long long 
                          int cluster, cudaStream_t stream) {
     return vcb_attn_mma_ex(q, out, pages, page_stride, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items,
                            n_items, rows_max, part_o, part_ml, slice_counters, dec_rows, nh, nkv, hd, page_size, num_pages,
-                           window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, 0, 0, nullptr, status, allow_tma, cluster, stream);
+                           window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, 0, 0, nullptr, 0, 0, 0, status, allow_tma, cluster, stream);
 }
 
-// keep_first, dist_a, dist_b, softcap, slope, sink, chunked, wide, out_gate: the options described with AttnArgs.
+// keep_first, dist_a, dist_b, softcap, slope, sink, chunked, wide, out_gate, gate_lanes, one_row, blocks: the options described with AttnArgs.
 VCB_API int vcb_attn_mma_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                             const int* table_row, int max_blocks, const int* q_start, const int* q_len,
                             const int* ctx_len, const int* items, int n_items, int rows_max, float* part_o,
                             float* part_ml, int* slice_counters, const int* dec_rows, int nh, int nkv, int hd,
                             int page_size, int num_pages, int window, float scale, int keep_first, const float* dist_a,
                             const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
-                            const float* out_gate, int* status, int allow_tma, int cluster, cudaStream_t stream) {
+                            const float* out_gate, int gate_lanes, int one_row, int blocks, int* status, int allow_tma, int cluster, cudaStream_t stream) {
     if (n_items == 0) return 0;
     VCB_CHECK_ARG(keep_first >= 0 && (dist_a == nullptr) == (dist_b == nullptr), "attn_mma: bad keep_first %d or half a distance penalty", keep_first);
     VCB_CHECK_ARG(nh > 0 && nkv > 0 && nh % nkv == 0, "attn_mma: %d query heads are not a multiple of %d KV heads", nh, nkv);
@@ -1193,10 +1206,11 @@ VCB_API int vcb_attn_mma_ex(const void* q, void* out, const void* pages, long lo
     VCB_CHECK_ARG(page_size > 0 && window >= 0, "attn_mma: bad page_size %d or window %d", page_size, window);
     AttnArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)pages, page_stride, block_table,
                table_row, max_blocks, q_start, q_len, ctx_len, items, part_o, part_ml, slice_counters, dec_rows, nh, nkv,
-               page_size, num_pages, window, scale, status, FusedQkv{}, cluster, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate};
+               page_size, num_pages, window, scale, status, FusedQkv{}, cluster, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate, gate_lanes, one_row, blocks};
     VCB_CHECK_ARG(softcap >= 0.f && (dist_a == nullptr || slope == nullptr), "attn_mma: a negative cap, or a logarithmic penalty and a slope at once");
     const bool tma = allow_tma && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64) &&
-                     ((uintptr_t)pages % 16 == 0) && page_stride == (long long)2 * nkv * page_size * hd;
+                     ((uintptr_t)pages % 16 == 0) && page_stride == (long long)(one_row ? 1 : 2) * nkv * page_size * hd;
+    VCB_CHECK_ARG(!blocks || (wide && dist_a == nullptr && slope == nullptr), "attn_mma: blocks of one shared row want wide query rows and no distance terms");
     if (wide && hd == 64) return tma ? launch_wide<64, true>(a, n_items, rows_max, stream) : launch_wide<64, false>(a, n_items, rows_max, stream);
     if (wide) return tma ? launch_wide<128, true>(a, n_items, rows_max, stream) : launch_wide<128, false>(a, n_items, rows_max, stream);
     if (hd == 64) return tma ? launch_rows<64, true>(a, n_items, rows_max, stream) : launch_rows<64, false>(a, n_items, rows_max, stream);

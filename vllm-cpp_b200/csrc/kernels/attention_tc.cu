@@ -91,8 +91,16 @@ struct TcArgs {
     int sink;
     const float* sink_value;    // with a sink: the silent key's score per head, not scaled (null: 0)
     int chunked;                // the window stands still: the chunk of `window` positions that a query's position lies in
-    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
+    const float* out_gate;      // [tokens][query heads] or null: what the result of a (token, head) is multiplied by
+    int gate_lanes;             // out_gate is laid out as the result, a factor per lane
+    int one_row;                // pages hold keys only: the values are the key rows
+    int blocks;                 // (with wide rows) the KV heads are blocks of one shared row, see attention.cu
 };
+
+// query heads of a token, the row a query head has in `q`, and where its result (of KV head or block kvh) lies in `out`
+__device__ __forceinline__ int query_heads(const TcArgs& a) { return a.blocks ? a.nh / a.nkv : a.nh; }
+__device__ __forceinline__ int query_head(const TcArgs& a, int kvh, int head) { return a.blocks ? head - kvh * (a.nh / a.nkv) : head; }
+__device__ __forceinline__ int out_head(const TcArgs& a, int kvh, int head) { return a.blocks ? query_head(a, kvh, head) * a.nkv + kvh : head; }
 
 // the first key a query at `pos` sees (kept first keys aside)
 template <bool OPT> __device__ __forceinline__ int first_key(const TcArgs& a, int pos) {
@@ -400,7 +408,8 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
         // themselves were a third, and made it the slowest role of the block). ----
         const int pages_per_tile = BNK / ps;
         const int groups_page = ps / 8;
-        const int groups_kv = a.nkv * groups_page;   // groups of 8 rows from a page's K to its V
+        const int parts = a.one_row ? 1 : 2;
+        const int groups_kv = a.one_row ? 0 : a.nkv * groups_page;   // groups of 8 rows from a page's K to its V
         const bool copies_v = lane >= 8;
         const int pl = lane & 7;
         int armed[2] = {0, 0};
@@ -494,7 +503,7 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
                             atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                             page = 0;   // keep the byte count whole; the status word reports the fault
                         }
-                        const int group = (page * 2 * a.nkv + u.kvh) * groups_page + (copies_v ? groups_kv : 0);
+                        const int group = (page * parts * a.nkv + u.kvh) * groups_page + (copies_v ? groups_kv : 0);
                         const uint32_t dst = base + (copies_v ? L::V_OFF : L::K_OFF) + st * L::KV_BYTES;
                         tma_load_groups(dst + pl * ps * ROWB, &kv_map, fullb, group);
                     }
@@ -646,7 +655,7 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
                         atomicOr(a.status, VCB_STATUS_BAD_PAGE);
                         p = 0;
                     }
-                    tma_load_groups(base + L::K_OFF + st * L::KV_BYTES + lane * ps * ROWB, &kv_map, k_full(st), (p * 2 * a.nkv + head) * groups_page);
+                    tma_load_groups(base + L::K_OFF + st * L::KV_BYTES + lane * ps * ROWB, &kv_map, k_full(st), (p * (a.one_row ? 1 : 2) * a.nkv + head) * groups_page);
                 }
                 armed = gk;
             }
@@ -682,7 +691,7 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
                     const int row = qtr * 32 + rr;
                     const bool mine = row < w.R;
                     const int wq = mine ? row / w.gq : 0, wh = mine ? row % w.gq : 0;
-                    const __nv_bfloat16* src = a.q + ((size_t)(w.row0 + wq) * a.nh + w.head0 + wh) * (NG * HD);
+                    const __nv_bfloat16* src = a.q + ((size_t)(w.row0 + wq) * query_heads(a) + query_head(a, w.kvh, w.head0 + wh)) * (NG * HD);
                     for (int c = lane; c < per_row; c += 32)
                         cp_async16(base + (c / CH) * L::Q_BYTES + swz<ROWS>(row, c % CH), src + c * 8, mine ? 16 : 0);
                 }
@@ -691,7 +700,7 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
                     // the row's further lanes into its TMEM lane, two a column
                     const bool mine = r < w.R;
                     const int wq = mine ? r / w.gq : 0, wh = mine ? r % w.gq : 0;
-                    const __nv_bfloat16* src = a.q + ((size_t)(w.row0 + wq) * a.nh + w.head0 + wh) * (NG * HD) + wide_blocks(HD) * HD;
+                    const __nv_bfloat16* src = a.q + ((size_t)(w.row0 + wq) * query_heads(a) + query_head(a, w.kvh, w.head0 + wh)) * (NG * HD) + wide_blocks(HD) * HD;
                     const int lanes = (NG - wide_blocks(HD)) * HD;
                     for (int c0 = 0; c0 < lanes; c0 += 64) {
                         uint4 v[8];
@@ -733,7 +742,7 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
             // a cap on the scaled score and a slope times the distance, likewise brought to the base-2 domain here
             const bool lin = OPT && (a.slope != nullptr || a.softcap > 0.f);
             const bool sink = OPT && a.sink != 0;
-            const float sink_l2 = sink && a.sink_value != nullptr && row_ok ? a.sink_value[u.head0 + ih] * LOG2E : 0.f;
+            const float sink_l2 = sink && a.sink_value != nullptr && row_ok ? a.sink_value[query_head(a, u.kvh, u.head0 + ih)] * LOG2E : 0.f;
             const float slope_l2 = lin && a.slope != nullptr && row_ok ? a.slope[u.head0 + ih] * LOG2E : 0.f;
             const float cap_l2 = a.softcap * LOG2E, cap_in = a.softcap > 0.f ? 2.f * scale_log2 / a.softcap : 0.f;
             const float sl2 = penal || lin ? 1.f : scale_log2;   // what is left to multiply the scores by on their way to weights
@@ -882,7 +891,8 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
             const int g_last = t0 + u.n_tiles - 1;
             t0 += u.n_tiles;
             const float l_end = l_run;
-            const int out_row = u.row0 + iq, out_head = u.head0 + ih;
+            const int out_row = u.row0 + iq, q_head = WIDE ? query_head(a, u.kvh, u.head0 + ih) : u.head0 + ih;
+            const size_t out_at = ((size_t)out_row * a.nh + (WIDE ? out_head(a, u.kvh, u.head0 + ih) : u.head0 + ih)) * HD;
             // the unit to come, and this row's query of it on its way
             unit = ok ? next_unit(seq++, u) : -1;
             has = unit >= 0;
@@ -892,8 +902,9 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
             if (ok) {
                 tc_fence_after();
                 float inv = l_end > 0.f ? 1.f / l_end : 0.f;
-                if (OPT && a.out_gate != nullptr && row_ok) inv *= a.out_gate[(size_t)out_row * a.nh + out_head];
-                __nv_bfloat16* dst = a.out + ((size_t)out_row * a.nh + out_head) * HD;
+                const bool gated = OPT && a.out_gate != nullptr && row_ok;
+                if (gated && !a.gate_lanes) inv *= a.out_gate[(size_t)out_row * (WIDE ? query_heads(a) : a.nh) + q_head];
+                __nv_bfloat16* dst = a.out + out_at;
 #pragma unroll
                 for (int c0 = 0; c0 < HD; c0 += 16) {   // 16 columns at a time: the query of the unit to come is in registers too
                     uint32_t v[16];
@@ -905,6 +916,12 @@ __global__ __launch_bounds__(NTHREADS + (KIND != ROWS_PLAIN ? 32 * KEY_WARPS : 0
                             float f[8];
 #pragma unroll
                             for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[8 * c + i]) * inv;
+                            if (gated && a.gate_lanes) {
+                                const float4* gl = reinterpret_cast<const float4*>(a.out_gate + out_at + c0 + 8 * c);
+                                const float4 g0 = gl[0], g1 = gl[1];
+                                f[0] *= g0.x; f[1] *= g0.y; f[2] *= g0.z; f[3] *= g0.w;
+                                f[4] *= g1.x; f[5] *= g1.y; f[6] *= g1.z; f[7] *= g1.w;
+                            }
                             *reinterpret_cast<uint4*>(dst + c0 + 8 * c) =
                                 make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
                         }
@@ -970,7 +987,7 @@ VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long lon
                            const int* table_row, int max_blocks, const int* q_start, const int* q_len, const int* ctx_len,
                            const int* items, int n_items, int nh, int nkv, int hd, int page_size, int num_pages, int window,
                            float scale, int keep_first, const float* dist_a, const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
-                           const float* out_gate, int* status, int* work,
+                           const float* out_gate, int gate_lanes, int one_row, int blocks, int* status, int* work,
                            cudaStream_t stream);
 
 // Prompt portions only: every item has slice 0 of 1 and at most 128 rows (tokens x query heads per KV head).
@@ -981,14 +998,14 @@ VCB_API int vcb_attn_tc(const void* q, void* out, const void* pages, long long p
                         const int* items, int n_items, int nh, int nkv, int hd, int page_size, int num_pages, int window,
                         float scale, int* status, int* work, cudaStream_t stream) {
     return vcb_attn_tc_ex(q, out, pages, page_stride, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items, n_items,
-                          nh, nkv, hd, page_size, num_pages, window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, 0, 0, nullptr, status, work, stream);
+                          nh, nkv, hd, page_size, num_pages, window, scale, 0, nullptr, nullptr, 0.f, nullptr, 0, nullptr, 0, 0, nullptr, 0, 0, 0, status, work, stream);
 }
 
 VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                            const int* table_row, int max_blocks, const int* q_start, const int* q_len, const int* ctx_len,
                            const int* items, int n_items, int nh, int nkv, int hd, int page_size, int num_pages, int window,
                            float scale, int keep_first, const float* dist_a, const float* dist_b, float softcap, const float* slope, int sink, const float* sink_value, int chunked, int wide,
-                           const float* out_gate, int* status, int* work,
+                           const float* out_gate, int gate_lanes, int one_row, int blocks, int* status, int* work,
                            cudaStream_t stream) {
     if (n_items == 0) return 0;
     VCB_CHECK_ARG(keep_first >= 0 && (dist_a == nullptr) == (dist_b == nullptr), "attn_tc: bad keep_first %d or half a distance penalty", keep_first);
@@ -996,20 +1013,22 @@ VCB_API int vcb_attn_tc_ex(const void* q, void* out, const void* pages, long lon
     VCB_CHECK_ARG(vcb_attn_tc_supported(VCB_BF16, hd, page_size), "attn_tc: head_dim %d with pages of %d tokens is not supported", hd, page_size);
     VCB_CHECK_ARG(window >= 0, "attn_tc: bad window %d", window);
     VCB_CHECK_ARG((long long)n_items * nh < (1ll << 31), "attn_tc: %d items of %d heads are more blocks than a grid holds", n_items, nh);
-    VCB_CHECK_ARG(((uintptr_t)pages % 16 == 0) && page_stride == (long long)2 * nkv * page_size * hd,
+    VCB_CHECK_ARG(((uintptr_t)pages % 16 == 0) && page_stride == (long long)(one_row ? 1 : 2) * nkv * page_size * hd,
                   "attn_tc: the pages of a layer must be contiguous and 16-byte aligned for TMA loads");
     VCB_CHECK_ARG(((uintptr_t)q % 16 == 0) && ((uintptr_t)out % 16 == 0), "attn_tc: q and out must be 16-byte aligned");
     VCB_CHECK_ARG(work != nullptr, "attn_tc: no work counters");
     CUtensorMap map;
-    if (!vcb_kv_tensor_map(pages, (long long)num_pages * 2 * nkv * page_size, hd, page_size, &map, true)) return -3;
+    if (!vcb_kv_tensor_map(pages, (long long)num_pages * (one_row ? 1 : 2) * nkv * page_size, hd, page_size, &map, true)) return -3;
     const int g = nh / nkv;
     const int hchunks = (g + ROWS - 1) / ROWS;
     TcArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, block_table, table_row, max_blocks, q_start, q_len, ctx_len,
-             items, nh, nkv, page_size, num_pages, window, scale, status, n_items * nkv * hchunks, work, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate};
+             items, nh, nkv, page_size, num_pages, window, scale, status, n_items * nkv * hchunks, work, keep_first, dist_a, dist_b, softcap, slope, sink, sink_value, chunked, out_gate, gate_lanes, one_row, blocks};
+    VCB_CHECK_ARG(!blocks || (wide && dist_a == nullptr && slope == nullptr), "attn_tc: blocks of one shared row want wide query rows and no distance terms");
+    VCB_CHECK_ARG(!gate_lanes || (uintptr_t)out_gate % 16 == 0, "attn_tc: the gates must be 16-byte aligned");
     VCB_CHECK_ARG(softcap >= 0.f && (dist_a == nullptr || slope == nullptr), "attn_tc: a negative cap, or a logarithmic penalty and a slope at once");
     VCB_CHECK_ARG(!wide || nkv <= 2 * wide_blocks(hd), "attn_tc: wide query rows of %d x %d lanes (up to 1024)", nkv, hd);
     if (wide && nkv > wide_blocks(hd)) return hd == 64 ? launch<64, true, ROWS_WIDER>(map, a, n_items, stream) : launch<128, true, ROWS_WIDER>(map, a, n_items, stream);
     if (wide) return hd == 64 ? launch<64, true, ROWS_WIDE>(map, a, n_items, stream) : launch<128, true, ROWS_WIDE>(map, a, n_items, stream);
-    if (chunked || out_gate != nullptr || keep_first > 0 || dist_a != nullptr || softcap > 0.f || slope != nullptr || sink) return hd == 64 ? launch<64, true>(map, a, n_items, stream) : launch<128, true>(map, a, n_items, stream);
+    if (chunked || out_gate != nullptr || one_row || keep_first > 0 || dist_a != nullptr || softcap > 0.f || slope != nullptr || sink) return hd == 64 ? launch<64, true>(map, a, n_items, stream) : launch<128, true>(map, a, n_items, stream);
     return hd == 64 ? launch<64, false>(map, a, n_items, stream) : launch<128, false>(map, a, n_items, stream);
 }

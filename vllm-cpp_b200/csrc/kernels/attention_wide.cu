@@ -16,7 +16,10 @@
 // products on it take the others; one box per page through the grouped view of the cache, as attention_mma.cu does):
 // a stage is a tile's keys (or values) of one KV head, keys first; it is as long as the slice's keys need, so that a short
 // slice has more of them on their way.  Slices leave (maximum, sum,
-// unnormalised output) partials for vcb_attn_merge.  Every wait is bounded and reports through the status word.
+// unnormalised output) partials for vcb_attn_merge.
+//
+// BLOCKS: the KV heads are blocks of one shared row (attention over latent rows wider than a tile, see attention.cu): all
+// rows meet the values of every block, and a head's result is its blocks side by side.  Every wait is bounded and reports through the status word.
 #include "common.cuh"
 #include "mbarrier.cuh"
 #include "kv_tensor_map.h"
@@ -47,7 +50,10 @@ struct WideArgs {
     float* part_ml;
     int nh, nkv, page_size, num_pages, window, chunked;
     float scale;
-    const float* out_gate;      // [tokens][nh] or null: what the result of a (token, head) is multiplied by
+    const float* out_gate;      // [tokens][query heads] or null: what the result of a (token, head) is multiplied by
+    int gate_lanes;             // out_gate is laid out as the result, a factor per lane
+    int one_row;                // pages hold keys only: the values are the key rows
+    const float* sink;          // [query heads] or null: the score of a silent key without a value in every softmax
     int ring_bytes;             // of shared memory for the stages
     int* status;
 };
@@ -91,10 +97,11 @@ __host__ __device__ inline int tail_bytes(int hd, int mt, int nkv) {
 }
 
 // MT tiles of 16 rows hold the query heads; up to NG KV heads
-template <int HD, int MT, int NG>
+template <int HD, int MT, int NG, bool BLOCKS = false>
 __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid_constant__ CUtensorMap kv_map, WideArgs a) {
     constexpr int ROWS = 16 * MT, CH = HD / 8, ROWB = HD * 2, HALVES = HD / 64;
     constexpr int NTV = HD / 64;        // n-tiles of 8 value lanes a warp owns
+    constexpr int MTV = BLOCKS ? MT : 1;        // tiles of 16 rows that meet a KV head's values
     constexpr float LOG2E = 1.4426950408889634f;
     extern __shared__ __align__(1024) uint8_t smem[];
     uint8_t* q_s = smem + a.ring_bytes;
@@ -112,15 +119,16 @@ __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid
     const int* item = a.items + (size_t)blockIdx.x * ITEM_INTS;
     const int e = item[0], slice = item[3], nslices = item[4], dec_index = item[5];
     const int qlen = a.q_len[e], ctx = a.ctx_len[e];
-    const int nh = a.nh, nkv = a.nkv, gs = nh / nkv;
+    // query rows; those that a KV head's values belong to; results of a token
+    const int nh = BLOCKS ? a.nh / a.nkv : a.nh, nkv = a.nkv, gs = BLOCKS ? nh : nh / nkv, n_out = a.nh;
     if (qlen <= 0 || ctx <= 0 || (smem_u32(smem) & 1023u)) {
         pdl_wait();
         if (qlen > 0 && ctx > 0) {
             if (tid == 0) atomicOr(a.status, VCB_STATUS_BAD_LAYOUT);
         } else if (nslices > 1) {
             // an empty entry: its slices still say "nothing here", so that the merge writes zeros
-            for (int h = tid; h < nh; h += blockDim.x) {
-                const size_t prow = ((size_t)dec_index * nh + h) * nslices + slice;
+            for (int h = tid; h < n_out; h += blockDim.x) {
+                const size_t prow = ((size_t)dec_index * n_out + h) * nslices + slice;
                 a.part_ml[prow * 2] = -CUDART_INF_F;
                 a.part_ml[prow * 2 + 1] = 0.f;
             }
@@ -156,7 +164,7 @@ __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid
         // ---- loads: every LW-th stage, a lane a page of the tile ----
         const int me = warp - NW;
         const int* bt = a.block_table + (size_t)(a.table_row ? a.table_row[e] : e) * a.max_blocks;
-        const int pages_per_tile = tile_keys / ps, groups_page = ps / 8, groups_kv = nkv * groups_page;
+        const int pages_per_tile = tile_keys / ps, groups_page = ps / 8, groups_kv = a.one_row ? 0 : nkv * groups_page;
         auto page_of = [&](int tile) {
             const int pb = my_lo + tile * pages_per_tile + lane;
             return (tile < n_tiles && lane < pages_per_tile && pb < my_hi) ? bt[pb] : -1;
@@ -184,7 +192,7 @@ __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid
                     p = 0;      // keep the byte count whole; the status word reports the fault
                 }
                 const bool is_v = sub >= nkv;
-                const int group = (p * 2 * nkv + (is_v ? sub - nkv : sub)) * groups_page + (is_v ? groups_kv : 0);
+                const int group = (p * (a.one_row ? 1 : 2) * nkv + (is_v ? sub - nkv : sub)) * groups_page + (is_v ? groups_kv : 0);
                 tma_load_groups(smem_u32(smem + st * stage_bytes) + lane * ps * ROWB, &kv_map, full_bar(st), group);
             }
             return true;
@@ -218,16 +226,20 @@ __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid
                        "l"(a.q + ((size_t)row0 * nh + (r < nh ? r : 0)) * (nkv * HD) + c * 8), "r"(r < nh ? 16 : 0) : "memory");
     }
     asm volatile("cp.async.wait_all;" ::: "memory");
-    float o[NG][NTV][4];
+    float o[NG][MTV][NTV][4];
 #pragma unroll
     for (int g = 0; g < NG; ++g)
 #pragma unroll
-        for (int n = 0; n < NTV; ++n) o[g][n][0] = o[g][n][1] = o[g][n][2] = o[g][n][3] = 0.f;
+        for (int m = 0; m < MTV; ++m)
+#pragma unroll
+            for (int n = 0; n < NTV; ++n) o[g][m][n][0] = o[g][m][n][1] = o[g][m][n][2] = o[g][m][n][3] = 0.f;
     float m_run[2 * MT], l_run[2 * MT];         // of rows warp, warp + 8, ... (every lane holds them)
 #pragma unroll
     for (int i = 0; i < 2 * MT; ++i) {
-        m_run[i] = -CUDART_INF_F;
-        l_run[i] = 0.f;
+        // (the silent key is the first slice's starting state)
+        const bool sink = a.sink != nullptr && slice == 0 && warp + 8 * i < nh;
+        m_run[i] = sink ? a.sink[warp + 8 * i] : -CUDART_INF_F;
+        l_run[i] = sink ? 1.f : 0.f;
     }
     warps_barrier();
 
@@ -313,31 +325,49 @@ __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid
                             *reinterpret_cast<uint4*>(vt + swz_kv<HALVES>(t_keys + idx / NTV, warp * NTV + idx % NTV)) = make_uint4(0, 0, 0, 0);
                         __syncwarp();
                     }
-                    const int ra = lane >> 2;
-                    const float al_a = al_s[g * gs + min(ra, gs - 1)], al_b = al_s[g * gs + min(ra + 8, gs - 1)];
+                    const int r_first = BLOCKS ? 0 : g * gs;        // the first row that meets these values
+                    const uint32_t vb = smem_u32(vt);
+                    uint32_t pb[MTV];
 #pragma unroll
-                    for (int n = 0; n < NTV; ++n) {
-                        o[g][n][0] *= al_a; o[g][n][1] *= al_a; o[g][n][2] *= al_b; o[g][n][3] *= al_b;
+                    for (int m = 0; m < MTV; ++m) {
+                        const int ra = m * 16 + (lane >> 2);
+                        const float al_a = al_s[r_first + min(ra, gs - 1)], al_b = al_s[r_first + min(ra + 8, gs - 1)];
+#pragma unroll
+                        for (int n = 0; n < NTV; ++n) {
+                            o[g][m][n][0] *= al_a; o[g][m][n][1] *= al_a; o[g][m][n][2] *= al_b; o[g][m][n][3] *= al_b;
+                        }
+                        // (rows beyond the group's repeat its last: never read)
+                        pb[m] = smem_u32(s_s + (r_first + min(m * 16 + (lane & 15), gs - 1)) * S_LD);
                     }
-                    const int pr = g * gs + min(lane & 15, gs - 1);     // (rows beyond the group's repeat its last: never read)
-                    const uint32_t vb = smem_u32(vt), pb = smem_u32(s_s + pr * S_LD);
                     const int last_key = tile_keys - 8;     // (of the last group of eight in the stage)
                     for (int k0 = 0; k0 < k_rows; k0 += 32) {
-                        uint32_t a0[4], a1[4], b[4];
-                        ldmatrix_x4(a0, pb + k0 * 2 + (lane >> 4) * 16);
-                        ldmatrix_x4(a1, pb + k0 * 2 + 32 + (lane >> 4) * 16);
+                        uint32_t a0[MTV][4], a1[MTV][4], b[4];
+#pragma unroll
+                        for (int m = 0; m < MTV; ++m) {
+                            ldmatrix_x4(a0[m], pb[m] + k0 * 2 + (lane >> 4) * 16);
+                            ldmatrix_x4(a1[m], pb[m] + k0 * 2 + 32 + (lane >> 4) * 16);
+                        }
                         // groups of eight keys beyond the stage: the last group once more (finite, and weighed by zero)
                         if constexpr (NTV == 2) {
                             ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(min(k0 + (mi & 1) * 8, last_key) + (lane & 7), warp * 2 + (mi >> 1)));
-                            mma_16816(o[g][0], a0, b[0], b[1]);
-                            mma_16816(o[g][1], a0, b[2], b[3]);
+#pragma unroll
+                            for (int m = 0; m < MTV; ++m) {
+                                mma_16816(o[g][m][0], a0[m], b[0], b[1]);
+                                mma_16816(o[g][m][1], a0[m], b[2], b[3]);
+                            }
                             ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(min(k0 + 16 + (mi & 1) * 8, last_key) + (lane & 7), warp * 2 + (mi >> 1)));
-                            mma_16816(o[g][0], a1, b[0], b[1]);
-                            mma_16816(o[g][1], a1, b[2], b[3]);
+#pragma unroll
+                            for (int m = 0; m < MTV; ++m) {
+                                mma_16816(o[g][m][0], a1[m], b[0], b[1]);
+                                mma_16816(o[g][m][1], a1[m], b[2], b[3]);
+                            }
                         } else {
                             ldmatrix_x4_trans(b, vb + swz_kv<HALVES>(min(k0 + mi * 8, last_key) + (lane & 7), warp));
-                            mma_16816(o[g][0], a0, b[0], b[1]);
-                            mma_16816(o[g][0], a1, b[2], b[3]);
+#pragma unroll
+                            for (int m = 0; m < MTV; ++m) {
+                                mma_16816(o[g][m][0], a0[m], b[0], b[1]);
+                                mma_16816(o[g][m][0], a1[m], b[2], b[3]);
+                            }
                         }
                     }
                     if (tail) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // the clearing stores above
@@ -359,23 +389,26 @@ __global__ __launch_bounds__(NT + 32 * LW, 1) void attn_wide_kernel(const __grid
     for (int g = 0; g < NG; ++g) {
         if (g < nkv) {
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int rg = (lane >> 2) + 8 * half, h = g * gs + rg;
+            for (int i = 0; i < 2 * MTV; ++i) {
+                const int m = i >> 1, half = i & 1;
+                const int rg = m * 16 + (lane >> 2) + 8 * half, h = BLOCKS ? rg : g * gs + rg, oh = BLOCKS ? rg * nkv + g : h;
                 if (rg < gs) {
                     float f = 1.f;
                     if (nslices == 1) {
                         f = l_s[h] > 0.f ? 1.f / l_s[h] : 0.f;
-                        if (a.out_gate != nullptr) f *= a.out_gate[(size_t)row0 * nh + h];
+                        if (a.out_gate != nullptr && !a.gate_lanes) f *= a.out_gate[(size_t)row0 * nh + h];
                     }
-                    const size_t prow = ((size_t)dec_index * nh + h) * nslices + slice;
+                    const size_t prow = ((size_t)dec_index * n_out + oh) * nslices + slice;
 #pragma unroll
                     for (int n = 0; n < NTV; ++n) {
                         const int d = (warp * NTV + n) * 8 + 2 * (lane & 3);
-                        if (nslices == 1)
-                            *reinterpret_cast<__nv_bfloat162*>(a.out + ((size_t)row0 * nh + h) * HD + d) =
-                                __floats2bfloat162_rn(o[g][n][2 * half] * f, o[g][n][2 * half + 1] * f);
-                        else
-                            *reinterpret_cast<float2*>(a.part_o + prow * HD + d) = make_float2(o[g][n][2 * half], o[g][n][2 * half + 1]);
+                        if (nslices == 1) {
+                            const size_t at = ((size_t)row0 * n_out + oh) * HD + d;
+                            const float2 gl = a.out_gate != nullptr && a.gate_lanes ? *reinterpret_cast<const float2*>(a.out_gate + at) : make_float2(1.f, 1.f);
+                            *reinterpret_cast<__nv_bfloat162*>(a.out + at) =
+                                __floats2bfloat162_rn(o[g][m][n][2 * half] * f * gl.x, o[g][m][n][2 * half + 1] * f * gl.y);
+                        } else
+                            *reinterpret_cast<float2*>(a.part_o + prow * HD + d) = make_float2(o[g][m][n][2 * half], o[g][m][n][2 * half + 1]);
                     }
                     if (nslices > 1 && warp == 0 && (lane & 3) == 0) {
                         a.part_ml[prow * 2] = m_s[h];
@@ -397,10 +430,10 @@ int ring_bytes(int hd, int nh, int nkv) {
     return n < 4 * 64 * hd * 2 ? 0 : n;
 }
 
-template <int HD, int MT, int NG>
+template <int HD, int MT, int NG, bool BLOCKS = false>
 int launch(const CUtensorMap& map, const WideArgs& a, int n_items, cudaStream_t stream) {
     const size_t smem = (size_t)a.ring_bytes + tail_bytes(HD, MT, a.nkv);
-    auto kern = attn_wide_kernel<HD, MT, NG>;
+    auto kern = attn_wide_kernel<HD, MT, NG, BLOCKS>;
     static size_t opted = 0;
     if (opted < smem) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -425,6 +458,12 @@ int launch_heads(const CUtensorMap& map, const WideArgs& a, int n_items, cudaStr
 
 }  // namespace
 
+// What the kernel takes for blocks of one shared row: up to 32 query heads, up to 8 blocks of 128 lanes.
+VCB_API int vcb_attn_wide_blocks_supported(int dtype, int hd, int page_size, int query_heads, int blocks) {
+    return dtype == VCB_BF16 && hd == 128 && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64) &&
+           query_heads >= 1 && query_heads <= (blocks <= 4 ? 32 : 16) && blocks >= 1 && blocks <= 8 && ring_bytes(hd, query_heads, blocks) > 0;
+}
+
 // What the kernel takes: up to 64 query heads, up to 16 of them (and 8 KV heads of 128 lanes, 16 of 64) a KV head.
 VCB_API int vcb_attn_wide_supported(int dtype, int hd, int page_size, int nh, int nkv) {
     return dtype == VCB_BF16 && (hd == 64 || hd == 128) && (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64) &&
@@ -436,18 +475,22 @@ VCB_API int vcb_attn_wide_supported(int dtype, int hd, int page_size, int nh, in
 VCB_API int vcb_attn_wide(const void* q, void* out, const void* pages, long long page_stride, const int* block_table,
                           const int* table_row, int max_blocks, const int* q_start, const int* q_len, const int* ctx_len,
                           const int* items, int n_items, float* part_o, float* part_ml, int nh, int nkv, int hd, int page_size,
-                          int num_pages, int window, int chunked, float scale, const float* out_gate, int* status,
-                          cudaStream_t stream) {
+                          int num_pages, int window, int chunked, float scale, const float* out_gate, int gate_lanes, int one_row,
+                          int blocks, const float* sink, int* status, cudaStream_t stream) {
     if (n_items == 0) return 0;
-    VCB_CHECK_ARG(vcb_attn_wide_supported(VCB_BF16, hd, page_size, nh, nkv), "attn_wide: %d heads on %d of %d lanes with pages of %d tokens are not supported", nh, nkv, hd, page_size);
+    VCB_CHECK_ARG(nh > 0 && nkv > 0 && nh % nkv == 0, "attn_wide: %d heads on %d KV heads", nh, nkv);
+    const int rows = blocks ? nh / nkv : nh;
+    VCB_CHECK_ARG(blocks ? vcb_attn_wide_blocks_supported(VCB_BF16, hd, page_size, rows, nkv) : vcb_attn_wide_supported(VCB_BF16, hd, page_size, nh, nkv), "attn_wide: %d heads on %d of %d lanes with pages of %d tokens are not supported", nh, nkv, hd, page_size);
     VCB_CHECK_ARG(window >= 0, "attn_wide: bad window %d", window);
-    VCB_CHECK_ARG(((uintptr_t)pages % 16 == 0) && page_stride == (long long)2 * nkv * page_size * hd,
+    VCB_CHECK_ARG(((uintptr_t)pages % 16 == 0) && page_stride == (long long)(one_row ? 1 : 2) * nkv * page_size * hd,
                   "attn_wide: the pages of a layer must be contiguous and 16-byte aligned for TMA loads");
     VCB_CHECK_ARG((uintptr_t)q % 16 == 0, "attn_wide: q must be 16-byte aligned");
     CUtensorMap map;
-    if (!vcb_kv_tensor_map(pages, (long long)num_pages * 2 * nkv * page_size, hd, page_size, &map, true)) return -3;
+    if (!vcb_kv_tensor_map(pages, (long long)num_pages * (one_row ? 1 : 2) * nkv * page_size, hd, page_size, &map, true)) return -3;
     WideArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, block_table, table_row, max_blocks, q_start, q_len, ctx_len, items, part_o,
-               part_ml, nh, nkv, page_size, num_pages, window, chunked, scale, out_gate, ring_bytes(hd, nh, nkv), status};
+               part_ml, nh, nkv, page_size, num_pages, window, chunked, scale, out_gate, gate_lanes, one_row, sink, ring_bytes(hd, rows, nkv), status};
+    if (blocks && nkv > 4) return launch<128, 1, 8, true>(map, a, n_items, stream);
+    if (blocks) return rows <= 16 ? launch<128, 1, 4, true>(map, a, n_items, stream) : launch<128, 2, 4, true>(map, a, n_items, stream);
     if (hd == 64) return nh <= 16 ? launch_heads<64, 1>(map, a, n_items, stream) : nh <= 32 ? launch_heads<64, 2>(map, a, n_items, stream) : launch_heads<64, 4>(map, a, n_items, stream);
     return nh <= 16 ? launch_heads<128, 1>(map, a, n_items, stream) : nh <= 32 ? launch_heads<128, 2>(map, a, n_items, stream) : launch_heads<128, 4>(map, a, n_items, stream);
 }

@@ -1,10 +1,11 @@
 // Row kernels of layers whose sublayers run side by side on one normed input, all 32-bit arithmetic on 32-bit sums or
 // k-slice partial sums:
 //
-//  * sum_add_rmsnorm    x[t] += sum over up to four results (each maybe in k-slices) + a row of a second stream (the
+//  * sum_add_rmsnorm    x[t] += scale * (sum over up to four results, each maybe in k-slices) + a row of a second stream (the
 //                       embedding's, where a repeated stretch of layers starts over) + a vector; out[t] = gain * x[t] /
 //                       sqrt(mean(x[t]^2) + eps).  One pass over the row: the additions of everything a layer left
-//                       pending and the next norm.  On a list of rows the stream itself is left alone.
+//                       pending and the next norm (or the next two norms of the same row, which differ in their gains).
+//                       On a list of rows the stream itself is left alone.
 //  * branch_norm_mean   out[t] = 1/N sum_b gain_b * y_b[t] / sqrt(mean(y_b[t]^2) + eps): the results of N mixers that
 //                       read the same input, each normed over the model width with its own gain, averaged.
 //  * polynorm           out[t] = a n(z) + b n(z^2) + c n(z^3) + e with n(v) = v / sqrt(mean(v^2) + eps) over a token's
@@ -37,6 +38,9 @@ struct SumArgs {
     int out_dtype;
     const int* rows;            // null: every row, and the stream is written back
     int H;
+    float scale;                // on the results' sum
+    const float* gain2;         // with out2: a second norm of the same row
+    void* out2;
 };
 
 template <int V> struct Pack;
@@ -54,14 +58,14 @@ template <> struct Pack<4> {
     __device__ __forceinline__ void store(float* p) const { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
 };
 
-template <int V>
-__device__ __forceinline__ void add_rows(Pack<V>& x, const Rows& in, size_t r, int c) {
+template <int V, bool SCALED = false>
+__device__ __forceinline__ void add_rows(Pack<V>& x, const Rows& in, size_t r, int c, float scale = 1.f) {
     const float* p = in.p + r * in.ld + c;
     for (int s = 0; s < in.S; ++s) {
         Pack<V> t;
         t.load(p + (size_t)s * in.s_stride);
 #pragma unroll
-        for (int i = 0; i < V; ++i) x.v[i] += t.v[i];
+        for (int i = 0; i < V; ++i) x.v[i] = SCALED ? fmaf(scale, t.v[i], x.v[i]) : x.v[i] + t.v[i];
     }
 }
 
@@ -104,8 +108,9 @@ __device__ __forceinline__ void block_sums(float (&v)[N], float* scratch /* >= N
     for (int k = 0; k < N; ++k) v[k] = scratch[k * 33 + 32];
 }
 
-template <int V>
-__global__ __launch_bounds__(512, 3) void sum_add_rmsnorm_kernel(SumArgs a) {
+// MORE: with a factor on the results' sum and a second norm
+template <int V, bool MORE>
+__global__ __launch_bounds__(512, MORE ? 2 : 3) void sum_add_rmsnorm_kernel(SumArgs a) {
     extern __shared__ __align__(16) float row_s[];      // [H]
     __shared__ float red[33];
     pdl_trigger();
@@ -117,7 +122,7 @@ __global__ __launch_bounds__(512, 3) void sum_add_rmsnorm_kernel(SumArgs a) {
     for (int c = threadIdx.x * V; c < H; c += blockDim.x * V) {
         Pack<V> x;
         x.load(a.resid + r * H + c);
-        for (int k = 0; k < a.n_terms; ++k) add_rows<V>(x, a.term[k], r, c);
+        for (int k = 0; k < a.n_terms; ++k) add_rows<V, MORE>(x, a.term[k], r, c, a.scale);
         if (a.row_extra != nullptr) {
             Pack<V> t;
             t.load(a.row_extra + r * H + c);
@@ -143,8 +148,16 @@ __global__ __launch_bounds__(512, 3) void sum_add_rmsnorm_kernel(SumArgs a) {
         x.load(row_s + c);
         g.load(a.gain + c);
 #pragma unroll
-        for (int j = 0; j < V; ++j) x.v[j] = g.v[j] * x.v[j] * inv;
-        store_out<V>(a.out, a.out_dtype, (size_t)i * H + c, x);
+        for (int j = 0; j < V; ++j) x.v[j] *= inv;
+#pragma unroll
+        for (int j = 0; j < V; ++j) g.v[j] *= x.v[j];
+        store_out<V>(a.out, a.out_dtype, (size_t)i * H + c, g);
+        if (MORE && a.out2 != nullptr) {
+            g.load(a.gain2 + c);
+#pragma unroll
+            for (int j = 0; j < V; ++j) g.v[j] *= x.v[j];
+            store_out<V>(a.out2, a.out_dtype, (size_t)i * H + c, g);
+        }
     }
 }
 
@@ -272,16 +285,18 @@ int want_smem(K kern, size_t smem, const char* name) {
 // resid [T][H]; terms: n_terms results, term k [S_k][T][ld_k] 32-bit (pointers, slice counts, slice strides, row strides in
 // four arrays); row_extra [T][H] or null; vec_extra [H] or null; gain [H] 32-bit; out [n][H] of out_dtype or null (then
 // only the additions are done); rows: null (every row i < n, the stream written back) or n row indices (stream untouched).
+// scale multiplies the results' sum (not row_extra and vec_extra); gain2 [H] and out2 [n][H] (or null): a second norm.
 VCB_API int vcb_sum_add_rmsnorm(float* resid, int n_terms, const float* const* term_p, const int* term_S, const long long* term_ss,
                                 const long long* term_ld, const float* row_extra, const float* vec_extra, const float* gain, float eps,
-                                void* out, int out_dtype, const int* rows, int n, int H, cudaStream_t stream) {
+                                void* out, int out_dtype, const int* rows, int n, int H, float scale, const float* gain2, void* out2, cudaStream_t stream) {
     if (n == 0) return 0;
     VCB_CHECK_ARG(n_terms >= 0 && n_terms <= MAX_TERMS, "sum_add_rmsnorm: %d results at once (up to %d)", n_terms, MAX_TERMS);
     VCB_CHECK_ARG(H > 0 && (out == nullptr || gain != nullptr), "sum_add_rmsnorm: bad arguments (H=%d)", H);
+    VCB_CHECK_ARG(out2 == nullptr || (out != nullptr && gain2 != nullptr), "sum_add_rmsnorm: a second norm without its gain, or without a first");
     SumArgs a{};
     a.resid = resid;
     bool vec = H % 4 == 0 && (uintptr_t)resid % 16 == 0 && (uintptr_t)row_extra % 16 == 0 && (uintptr_t)vec_extra % 16 == 0 &&
-               (uintptr_t)gain % 16 == 0 && (uintptr_t)out % 16 == 0;
+               (uintptr_t)gain % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)gain2 % 16 == 0 && (uintptr_t)out2 % 16 == 0;
     for (int k = 0; k < n_terms; ++k) {
         a.term[k] = Rows{term_p[k], term_S[k] < 1 ? 1 : term_S[k], term_ss[k], term_ld[k]};
         vec = vec && rows_vec_ok(a.term[k]);
@@ -295,14 +310,15 @@ VCB_API int vcb_sum_add_rmsnorm(float* resid, int n_terms, const float* const* t
     a.out_dtype = out_dtype;
     a.rows = rows;
     a.H = H;
+    a.scale = scale;
+    a.gain2 = gain2;
+    a.out2 = out2;
     const size_t smem = (size_t)H * sizeof(float);
-    if (vec) {
-        if (int rc = want_smem(sum_add_rmsnorm_kernel<4>, smem, "sum_add_rmsnorm")) return rc;
-        launch_pdl(sum_add_rmsnorm_kernel<4>, dim3(n), dim3(block_for(H, 4)), smem, stream, a);
-    } else {
-        if (int rc = want_smem(sum_add_rmsnorm_kernel<1>, smem, "sum_add_rmsnorm")) return rc;
-        launch_pdl(sum_add_rmsnorm_kernel<1>, dim3(n), dim3(block_for(H, 1)), smem, stream, a);
-    }
+    const bool more = scale != 1.f || out2 != nullptr;
+    auto kern = vec ? (more ? sum_add_rmsnorm_kernel<4, true> : sum_add_rmsnorm_kernel<4, false>)
+                    : (more ? sum_add_rmsnorm_kernel<1, true> : sum_add_rmsnorm_kernel<1, false>);
+    if (int rc = want_smem(kern, smem, "sum_add_rmsnorm")) return rc;
+    launch_pdl(kern, dim3(n), dim3(block_for(H, vec ? 4 : 1)), smem, stream, a);
     VCB_CHECK_LAUNCH("sum_add_rmsnorm");
     return 0;
 }

@@ -298,7 +298,7 @@ VCB_API int vcb_add_rmsnorm(float* resid, const void* delta, int delta_dtype, in
 // SiLU-gate product: out[t,i] = silu(gu[t,2i]) * gu[t,2i+1]   (gate and up alternate along a row)
 // ---------------------------------------------------------------------------
 template <typename TIN, typename T>
-__global__ void swiglu_kernel(const TIN* __restrict__ gu, int S, size_t s_stride, T* __restrict__ out, int I, size_t total) {
+__global__ void swiglu_kernel(const TIN* __restrict__ gu, int S, size_t s_stride, size_t ld, T* __restrict__ out, int I, size_t total) {
     pdl_trigger();
     tl_mark(VCB_TL_SWIGLU, 0);
     pdl_wait();
@@ -312,8 +312,8 @@ __global__ void swiglu_kernel(const TIN* __restrict__ gu, int S, size_t s_stride
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 if (s0 + j < S) {
-                    gs[j] = to_f32(gu[(s0 + j) * s_stride + t * 2 * I + 2 * i]);
-                    us[j] = to_f32(gu[(s0 + j) * s_stride + t * 2 * I + 2 * i + 1]);
+                    gs[j] = to_f32(gu[(s0 + j) * s_stride + t * ld + 2 * i]);
+                    us[j] = to_f32(gu[(s0 + j) * s_stride + t * ld + 2 * i + 1]);
                 }
             }
 #pragma unroll
@@ -328,7 +328,7 @@ __global__ void swiglu_kernel(const TIN* __restrict__ gu, int S, size_t s_stride
 
 // 32-bit k-slice partial sums in, bfloat16 out, I a multiple of 4: a thread makes four outputs from two 16-byte loads a
 // slice (g0 u0 g1 u1, g2 u2 g3 u3), all slices' loads of up to four slices in flight together, added in slice order.
-__global__ void swiglu_partials_vec_kernel(const float* __restrict__ gu, int S, size_t s_stride, __nv_bfloat16* __restrict__ out,
+__global__ void swiglu_partials_vec_kernel(const float* __restrict__ gu, int S, size_t s_stride, size_t ld, __nv_bfloat16* __restrict__ out,
                                            int I4, size_t total4) {
     pdl_trigger();
     tl_mark(VCB_TL_SWIGLU, 0);
@@ -336,7 +336,7 @@ __global__ void swiglu_partials_vec_kernel(const float* __restrict__ gu, int S, 
     tl_mark(VCB_TL_SWIGLU, 1);
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total4; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t t = idx / I4, i = idx % I4;
-        const float4* src = reinterpret_cast<const float4*>(gu + t * 8 * (size_t)I4) + 2 * i;
+        const float4* src = reinterpret_cast<const float4*>(gu + t * ld) + 2 * i;
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
         for (int s0 = 0; s0 < S; s0 += 4) {
             float4 ta[4], tb[4];
@@ -386,14 +386,14 @@ __global__ void swiglu_bf16_vec_kernel(const __nv_bfloat16* __restrict__ gu, __n
     }
 }
 
-// gate_up: [S, T, 2I] of in_dtype (S partial sums, s_stride elements apart), gate_i at 2i and up_i at 2i+1;
-// out: [T, I] of out_dtype
-VCB_API int vcb_swiglu(const void* gate_up, int in_dtype, int S, long long s_stride, void* out, int out_dtype, int T,
+// gate_up: [S, T, 2I] of in_dtype (S partial sums, s_stride elements apart; rows ld elements apart), gate_i at 2i and up_i at
+// 2i+1; out: [T, I] of out_dtype
+VCB_API int vcb_swiglu(const void* gate_up, int in_dtype, int S, long long s_stride, long long ld, void* out, int out_dtype, int T,
                        int I, cudaStream_t stream) {
     if (T == 0) return 0;
     VCB_CHECK_ARG(T > 0 && I > 0 && S >= 1, "swiglu: bad sizes T=%d I=%d S=%d", T, I, S);
     const size_t total = (size_t)T * I;
-    if (in_dtype == VCB_BF16 && out_dtype == VCB_BF16 && S == 1 && I % 8 == 0 && ((uintptr_t)gate_up % 16 == 0) &&
+    if (in_dtype == VCB_BF16 && out_dtype == VCB_BF16 && S == 1 && I % 8 == 0 && ld == 2LL * I && ((uintptr_t)gate_up % 16 == 0) &&
         ((uintptr_t)out % 16 == 0)) {
         const size_t total8 = total / 8;
         const int nb = (int)((total8 + 255) / 256 < 148 * 32 ? (total8 + 255) / 256 : 148 * 32);
@@ -401,22 +401,22 @@ VCB_API int vcb_swiglu(const void* gate_up, int in_dtype, int S, long long s_str
         VCB_CHECK_LAUNCH("swiglu");
         return 0;
     }
-    if (in_dtype == VCB_F32 && out_dtype == VCB_BF16 && I % 4 == 0 && s_stride % 4 == 0 && ((uintptr_t)gate_up % 16 == 0) &&
+    if (in_dtype == VCB_F32 && out_dtype == VCB_BF16 && I % 4 == 0 && s_stride % 4 == 0 && ld % 4 == 0 && ((uintptr_t)gate_up % 16 == 0) &&
         ((uintptr_t)out % 8 == 0)) {
         const size_t total4 = total / 4;
         const int nb = (int)((total4 + 255) / 256 < 148 * 8 ? (total4 + 255) / 256 : 148 * 8);   // all blocks resident at once
         launch_pdl(swiglu_partials_vec_kernel, dim3(nb), dim3(256), 0, stream, (const float*)gate_up, S, (size_t)s_stride,
-                   (__nv_bfloat16*)out, I / 4, total4);
+                   (size_t)ld, (__nv_bfloat16*)out, I / 4, total4);
         VCB_CHECK_LAUNCH("swiglu");
         return 0;
     }
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     if (in_dtype == VCB_F32 && out_dtype == VCB_F32)
-        launch_pdl(swiglu_kernel<float, float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, S, (size_t)s_stride, (float*)out, I, total);
+        launch_pdl(swiglu_kernel<float, float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, S, (size_t)s_stride, (size_t)ld, (float*)out, I, total);
     else if (in_dtype == VCB_F32)
-        launch_pdl(swiglu_kernel<float, __nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, S, (size_t)s_stride, (__nv_bfloat16*)out, I, total);
+        launch_pdl(swiglu_kernel<float, __nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, S, (size_t)s_stride, (size_t)ld, (__nv_bfloat16*)out, I, total);
     else if (out_dtype == VCB_BF16)
-        launch_pdl(swiglu_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gate_up, S, (size_t)s_stride, (__nv_bfloat16*)out, I, total);
+        launch_pdl(swiglu_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gate_up, S, (size_t)s_stride, (size_t)ld, (__nv_bfloat16*)out, I, total);
     else { vcb_set_error("swiglu: bfloat16 input with 32-bit output is not a combination the engine uses"); return -1; }
     VCB_CHECK_LAUNCH("swiglu");
     return 0;

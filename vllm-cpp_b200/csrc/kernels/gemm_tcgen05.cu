@@ -1197,7 +1197,8 @@ VCB_API int vcb_gemm_bf16_xielu(const void* W, const void* X, void* out, int M, 
 // [groups * group_rows, K]: the groups' matrices stacked; X [tiles * tile_rows, K]: the tokens sorted by group, every
 // group's run padded to whole tiles of tile_rows rows (16, 32, 64, 128 or 256); tile_group [tiles] (device): the group
 // of each tile, -1 for a tile beyond the last, whose rows are neither read nor written.  out [tiles * tile_rows,
-// group_rows] of out_dtype, after `act` (0: none, 2: SiLU, 3: the square of ReLU).  The grid is laid out for all
+// group_rows] of out_dtype, after `act` (0: none, 2: SiLU, 3: the square of ReLU; 7: rows 2i and 2i + 1 of a group are gate_i
+// and up_i, and out is silu(gate) * up, [tiles * tile_rows, group_rows / 2] bfloat16).  The grid is laid out for all
 // `tiles`; which of them hold tokens is read on the device, so a captured step replays the launch.
 VCB_API int vcb_gemm_bf16_grouped(const void* W, const void* X, void* out, int out_dtype, int groups, int group_rows, int tiles,
                                   int tile_rows, int K, long long ldw, long long ldx, long long ldc, const int* tile_group,
@@ -1207,12 +1208,14 @@ VCB_API int vcb_gemm_bf16_grouped(const void* W, const void* X, void* out, int o
     VCB_CHECK_ARG(K % 8 == 0 && ldw % 8 == 0 && ldx % 8 == 0,
                   "gemm_bf16_grouped: inner size %d and row strides %lld, %lld must be multiples of 8 (16-byte rows for TMA)", K, ldw, ldx);
     VCB_CHECK_ARG(((uintptr_t)W % 16 == 0) && ((uintptr_t)X % 16 == 0), "gemm_bf16_grouped: operands must be 16-byte aligned");
-    VCB_CHECK_ARG(tile_group != nullptr && (act == 0 || act == 2 || act == 3), "gemm_bf16_grouped: no tile table, or an unknown activation");
+    VCB_CHECK_ARG(tile_group != nullptr && (act == 0 || act == 2 || act == 3 || act == 7), "gemm_bf16_grouped: no tile table, or an unknown activation");
+    VCB_CHECK_ARG(act != 7 || (out_dtype == VCB_BF16 && group_rows % 2 == 0), "gemm_bf16_grouped: a SiLU gate wants pairs of rows and a bfloat16 result");
     const int total_kb = (K + BK - 1) / BK;
     GemmArgs g{out, out_dtype, group_rows, tiles * tile_rows, K, ldc, 0, total_kb, 1, 0, status};
     g.tile_group = tile_group;
     g.group_rows = group_rows;
-    g.act = act;
+    g.act = act == 7 ? 0 : act;
+    g.swiglu = act == 7;
     const long long w_rows = (long long)groups * group_rows;
     switch (tile_rows) {
         case 16: return launch_maps<16, 8, 1, 2>(W, w_rows, X, g, ldw, ldx, 1, stream);

@@ -9,7 +9,8 @@
 //
 //  * latent_norm_rope_store   from the stacked down projections [q latent | kv latent | rotated key part] (32-bit sums):
 //                             c_q = g_q n(q latent) to a buffer; c = g_kv n(kv latent) and the rotated key part to the
-//                             token's cache row (key row [c | k_rot], value row c)
+//                             token's cache row (key row [c | k_rot | zeros], and value row c unless the key rows double as
+//                             values); optionally one gate per head from further columns (its sigmoid to a buffer)
 //  * head_linear              out[t, h, :] = M[h] in[t, h, :] for every head's own small matrix (queries into the latent
 //                             space, latent sums out to the heads' values)
 //                             (long steps with bfloat16 matrices: on the tensor cores)
@@ -51,7 +52,11 @@ struct LatentArgs {
     int page_size, num_pages;
     int q_rank, kv_rank, rot, T;
     int interleaved;        // lanes pair as neighbours
-    int v_width;            // lanes of a value row: kv_rank, or more (the lanes behind the latent are zeros)
+    int v_width;            // lanes of a value row: kv_rank, or more (the lanes behind the latent are zeros); 0: there are none
+    int k_width;            // lanes of a key row: kv_rank + rot, or more (zeros)
+    int k_block;            // a key row lies in pieces of this many lanes, all tokens' first pieces first (k_width: one piece)
+    float* gate_out;        // [T][n_gates] or null: sigmoids of the columns behind the others
+    int n_gates;
     int* status;
 };
 
@@ -73,6 +78,8 @@ __global__ void latent_norm_rope_store_kernel(LatentArgs a) {
     if (nq > 0) sq = block_sum(sq, red);
     sk = block_sum(sk, red);
     const float rq = nq > 0 ? rsqrtf(sq / (float)nq + a.eps) : 0.f, rk = rsqrtf(sk / (float)nk + a.eps);
+    for (int h = threadIdx.x; h < a.n_gates; h += blockDim.x)
+        a.gate_out[(size_t)t * a.n_gates + h] = 1.f / (1.f + expf(-rows_at(a.u, t, n + h)));
     TC* cq = (TC*)a.cq_out + (size_t)t * nq;
     for (int c = threadIdx.x; c < nq; c += blockDim.x) cq[c] = from_f32<TC>(row[c] * rq * a.gq[c]);
     const int slot = a.slot_map[t];
@@ -82,15 +89,15 @@ __global__ void latent_norm_rope_store_kernel(LatentArgs a) {
         if (threadIdx.x == 0) atomicOr(a.status, VCB_STATUS_BAD_PAGE);
         return;
     }
-    const int hd = nk + nr;
     TC* base = (TC*)a.pages + (size_t)page * a.page_stride;
-    TC* krow = base + (size_t)off * hd;
-    TC* vrow = base + (size_t)a.page_size * hd + (size_t)off * a.v_width;
+    auto key = [&](int c) -> TC& { return base[((size_t)(c / a.k_block) * a.page_size + off) * a.k_block + c % a.k_block]; };
+    TC* vrow = base + (size_t)a.page_size * a.k_width + (size_t)off * a.v_width;
     for (int c = threadIdx.x; c < nk; c += blockDim.x) {
         const TC v = from_f32<TC>(row[nq + c] * rk * a.gkv[c]);
-        krow[c] = v;
-        vrow[c] = v;
+        key(c) = v;
+        if (a.v_width > 0) vrow[c] = v;
     }
+    for (int c = nk + nr + threadIdx.x; c < a.k_width; c += blockDim.x) key(c) = from_f32<TC>(0.f);
     for (int c = nk + threadIdx.x; c < a.v_width; c += blockDim.x) vrow[c] = from_f32<TC>(0.f);
     const int half = nr / 2;
     const float pos = (float)a.positions[t];
@@ -102,10 +109,10 @@ __global__ void latent_norm_rope_store_kernel(LatentArgs a) {
         cs *= a.gain;
         const int la = a.interleaved ? 2 * i : i, lb = a.interleaved ? 2 * i + 1 : i + half;
         const float x = r[la], y = r[lb];
-        krow[nk + la] = from_f32<TC>(x * cs - y * sn);
-        krow[nk + lb] = from_f32<TC>(y * cs + x * sn);
+        key(nk + la) = from_f32<TC>(x * cs - y * sn);
+        key(nk + lb) = from_f32<TC>(y * cs + x * sn);
     }
-    for (int i = 2 * half + threadIdx.x; i < nr; i += blockDim.x) krow[nk + i] = from_f32<TC>(r[i]);
+    for (int i = 2 * half + threadIdx.x; i < nr; i += blockDim.x) key(nk + i) = from_f32<TC>(r[i]);
 }
 
 // One block: head h, a tile of TT tokens.  A warp an output lane: its lanes walk the inner dimension (coalesced reads of the
@@ -183,13 +190,14 @@ struct RopeArgs {
     int out_head_stride, out_off;
     int interleaved;
     int T, H, dims, width;  // `width` lanes of the slice are copied, the first `dims` of them rotated
+    int pad;                // so many zero lanes go behind them
 };
 
 __global__ void rope_rows_kernel(RopeArgs a) {
     pdl_trigger();
     pdl_wait();
     const int half = a.dims / 2;
-    const int per_head = half + (a.width - 2 * half);     // one thread a pair, one a lane that passes unchanged
+    const int per_head = half + (a.width - 2 * half) + a.pad;     // one thread a pair, one a lane that passes unchanged
     for (int t = blockIdx.y; t < a.T; t += gridDim.y) {
         const float pos = (float)a.positions[t];
         for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < a.H * per_head; i += gridDim.x * blockDim.x) {
@@ -207,7 +215,7 @@ __global__ void rope_rows_kernel(RopeArgs a) {
                 store_from_f32(a.out, a.out_dtype, ob + lb, y * cs + x * sn);
             } else {
                 const int c = 2 * half + (k - half);
-                store_from_f32(a.out, a.out_dtype, ob + c, rows_at(a.in, t, ib + c));
+                store_from_f32(a.out, a.out_dtype, ob + c, c < a.width ? rows_at(a.in, t, ib + c) : 0.f);
             }
         }
     }
@@ -216,17 +224,21 @@ __global__ void rope_rows_kernel(RopeArgs a) {
 }  // namespace
 
 // u [S][T][ld]: q_rank + kv_rank + rot columns.  cq_out [T][q_rank] and the pages in `dtype`.  A page is one flat row:
-// [page_size][kv_rank + rot] key rows, then [page_size][v_width] value rows (v_width >= kv_rank; the latent, then zeros:
-// value rows as wide as key rows are what the tensor-core attention kernels read).
+// [page_size][k_width] key rows (in pieces of k_block lanes, see LatentArgs), then [page_size][v_width] value rows (v_width >=
+// kv_rank; the latent, then zeros: value rows as wide as key rows are what the tensor-core attention kernels read; 0: none,
+// the key rows double as values).  gate_out [T][n_gates] (or null): sigmoids of n_gates columns behind the others.
 VCB_API int vcb_latent_norm_rope_store(const float* u, int S, long long s_stride, long long ld, const float* gq, const float* gkv,
                                        float eps, const int* positions, const float* freq, float gain, const int* slot_map,
                                        void* cq_out, void* pages, long long page_stride, int page_size, int num_pages, int q_rank,
-                                       int kv_rank, int rot, int interleaved, int v_width, int T, int dtype, int* status, cudaStream_t stream) {
+                                       int kv_rank, int rot, int interleaved, int k_width, int k_block, int v_width, float* gate_out, int n_gates,
+                                       int T, int dtype, int* status, cudaStream_t stream) {
     if (T == 0) return 0;
     VCB_CHECK_ARG(q_rank >= 0 && kv_rank > 0 && rot >= 0, "latent_norm_rope_store: bad sizes %d %d %d", q_rank, kv_rank, rot);
-    VCB_CHECK_ARG(v_width >= kv_rank && v_width <= kv_rank + rot, "latent_norm_rope_store: value rows of %d lanes", v_width);
+    VCB_CHECK_ARG(k_width >= kv_rank + rot && k_block > 0 && k_width % k_block == 0, "latent_norm_rope_store: key rows of %d lanes in pieces of %d", k_width, k_block);
+    VCB_CHECK_ARG(v_width == 0 || (v_width >= kv_rank && v_width <= k_width), "latent_norm_rope_store: value rows of %d lanes", v_width);
+    VCB_CHECK_ARG(n_gates >= 0 && (n_gates == 0) == (gate_out == nullptr), "latent_norm_rope_store: %d gates without a buffer, or none with one", n_gates);
     LatentArgs a{Rows{u, S < 1 ? 1 : S, s_stride, ld}, gq, gkv, eps, positions, freq, gain, slot_map, cq_out, pages, page_stride,
-                 page_size, num_pages, q_rank, kv_rank, rot, T, interleaved, v_width, status};
+                 page_size, num_pages, q_rank, kv_rank, rot, T, interleaved, v_width, k_width, k_block, gate_out, n_gates, status};
     const size_t smem = (size_t)(q_rank + kv_rank + rot) * sizeof(float);
     VCB_CHECK_ARG(smem <= 48 * 1024, "latent_norm_rope_store: %d lanes are more than the kernel's shared memory holds", q_rank + kv_rank + rot);
     if (dtype == VCB_F32) launch_pdl(latent_norm_rope_store_kernel<float>, dim3(T), dim3(256), smem, stream, a);
@@ -476,12 +488,12 @@ VCB_API int vcb_head_linear(const void* in, int in_dtype, int S, long long s_str
 
 VCB_API int vcb_rope_rows(const float* in, int S, long long s_stride, long long ld, int in_head_stride, int in_off,
                           const int* positions, const float* freq, float gain, void* out, int out_dtype, long long ld_out,
-                          int out_head_stride, int out_off, int T, int H, int dims, int width, int interleaved, cudaStream_t stream) {
+                          int out_head_stride, int out_off, int T, int H, int dims, int width, int pad, int interleaved, cudaStream_t stream) {
     if (T == 0 || H == 0 || width == 0) return 0;
-    VCB_CHECK_ARG(dims >= 0 && dims <= width, "rope_rows: %d rotated lanes of %d", dims, width);
+    VCB_CHECK_ARG(pad >= 0 && dims >= 0 && dims <= width, "rope_rows: %d rotated lanes of %d", dims, width);
     RopeArgs a{Rows{in, S < 1 ? 1 : S, s_stride, ld}, in_head_stride, in_off, positions, freq, gain, out, out_dtype, ld_out,
-               out_head_stride, out_off, interleaved, T, H, dims, width};
-    const int per_head = dims / 2 + (width - 2 * (dims / 2));
+               out_head_stride, out_off, interleaved, T, H, dims, width, pad};
+    const int per_head = dims / 2 + (width - 2 * (dims / 2)) + pad;
     const dim3 grid((H * per_head + 127) / 128, T < 65535 ? T : 65535);
     launch_pdl(rope_rows_kernel, grid, dim3(128), 0, stream, a);
     VCB_CHECK_LAUNCH("rope_rows");

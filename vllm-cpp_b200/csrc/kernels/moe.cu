@@ -9,7 +9,7 @@
 //                  compute dtype as a stored activation would be) and applies the activation; the down projection
 //                  writes 32-bit sums per pair
 //  * moe_combine   per token: the sums of its pairs, in the order the router chose them (times the pair's weight where
-//                  it belongs on the output), plus a shared expert's result
+//                  it belongs on the output), plus a shared expert's result (times a gate per token, if it has one)
 //
 // Nothing here asks the host how many tokens an expert got: the grids are laid out for the most tiles the step can
 // need and a tile beyond the last one returns at once, so a captured step replays it.  Products accumulate in 32-bit
@@ -51,7 +51,7 @@ __device__ __forceinline__ int entry_of_row(const int* __restrict__ q_start, con
 }
 
 // a warp a token; the logits of the warp's token lie in shared memory while its lanes look for the next largest
-__global__ void moe_route_kernel(Rows logits, const int* __restrict__ q_start, const int* __restrict__ q_len, int n_entries,
+__global__ void moe_route_kernel(Rows logits, const float* __restrict__ bias, const int* __restrict__ q_start, const int* __restrict__ q_len, int n_entries,
                                  int T, int E, int top, int softmax_weights, int* __restrict__ sel_e, float* __restrict__ sel_w) {
     extern __shared__ float zs[];   // [warps][E]
     pdl_trigger();
@@ -64,7 +64,7 @@ __global__ void moe_route_kernel(Rows logits, const int* __restrict__ q_start, c
         return;
     }
     float* z = zs + (size_t)warp * E;
-    for (int e = lane; e < E; e += 32) z[e] = rows_at(logits, t, e);
+    for (int e = lane; e < E; e += 32) z[e] = rows_at(logits, t, e) + (bias != nullptr ? bias[e] : 0.f);
     __syncwarp();
     float first = 0.f, denom = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -328,7 +328,7 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, long long ldx, const 
 
 // grid (ceil(W / 256), rows): out[t] = shared[t] + sum over the token's pairs, in the router's order
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, const float* __restrict__ sel_w,
-                                   int top, Rows shared, const int* __restrict__ q_start, const int* __restrict__ q_len,
+                                   int top, Rows shared, Rows gate, const int* __restrict__ q_start, const int* __restrict__ q_len,
                                    int n_entries, int W, float* __restrict__ out) {
     pdl_trigger();
     pdl_wait();
@@ -336,6 +336,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= W || entry_of_row(q_start, q_len, n_entries, t) < 0) return;
     float v = shared.p != nullptr ? rows_at(shared, t, c) : 0.f;
+    if (gate.p != nullptr) v *= 1.f / (1.f + expf(-rows_at(gate, t, 0)));
     for (int k = 0; k < top; ++k) {
         const int pos = pos_of[(size_t)t * top + k];
         if (pos >= 0) {
@@ -348,7 +349,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 
 // four channels a thread (W a multiple of 4, every base and stride a multiple of 4 elements)
 __global__ void moe_combine_vec_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, const float* __restrict__ sel_w,
-                                       int top, Rows shared, const int* __restrict__ q_start, const int* __restrict__ q_len,
+                                       int top, Rows shared, Rows gate, const int* __restrict__ q_start, const int* __restrict__ q_len,
                                        int n_entries, int W, float* __restrict__ out) {
     pdl_trigger();
     pdl_wait();
@@ -361,6 +362,10 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ y, const int* _
         for (int s = 0; s < shared.S; ++s) {
             const float4 a = *reinterpret_cast<const float4*>(p + (long long)s * shared.s_stride);
             v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+        }
+        if (gate.p != nullptr) {
+            const float g = 1.f / (1.f + expf(-rows_at(gate, t, 0)));
+            v.x *= g; v.y *= g; v.z *= g; v.w *= g;
         }
     }
     for (int k = 0; k < top; ++k) {
@@ -380,8 +385,9 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ y, const int* _
 VCB_API int vcb_moe_tile_rows() { return BM; }
 
 // logits [S][T][ld] 32-bit sums with E columns.  sel_e, sel_w [T * top]: expert (-1 for rows outside every entry) and weight of
-// each choice.  softmax_weights 0: the sigmoid of the chosen logit; 1: the softmax over the chosen logits.
-VCB_API int vcb_moe_route(const float* logits, int S, long long s_stride, long long ld, const int* q_start, const int* q_len,
+// each choice.  bias [E] (or null) is added to the logits first.  softmax_weights 0: the sigmoid of the chosen logit; 1: the
+// softmax over the chosen logits.
+VCB_API int vcb_moe_route(const float* logits, int S, long long s_stride, long long ld, const float* bias, const int* q_start, const int* q_len,
                           int n_entries, int T, int E, int top, int softmax_weights, int* sel_e, float* sel_w,
                           cudaStream_t stream) {
     if (T == 0) return 0;
@@ -390,7 +396,7 @@ VCB_API int vcb_moe_route(const float* logits, int S, long long s_stride, long l
     const size_t smem = (size_t)warps * E * sizeof(float);
     VCB_CHECK_ARG(smem <= 48 * 1024, "moe_route: %d experts are more than the kernel's shared memory holds", E);
     launch_pdl(moe_route_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, stream,
-               Rows{logits, S < 1 ? 1 : S, s_stride, ld}, q_start, q_len, n_entries, T, E, top, softmax_weights, sel_e, sel_w);
+               Rows{logits, S < 1 ? 1 : S, s_stride, ld}, bias, q_start, q_len, n_entries, T, E, top, softmax_weights, sel_e, sel_w);
     VCB_CHECK_LAUNCH("moe_route");
     return 0;
 }
@@ -467,22 +473,23 @@ VCB_API int vcb_moe_gather(const void* x, long long ldx, int dtype, const int* s
     return 0;
 }
 
-// y [tiles_cap * BM][W] 32-bit sums per pair; shared (or null): a shared expert's sums [S][T][ld]; sel_w (or null): the
-// pairs' weights where they belong on the output; out [T][W] 32-bit.
+// y [tiles_cap * BM][W] 32-bit sums per pair; shared (or null): a shared expert's sums [S][T][ld]; gate (or null): a column of
+// sums [gS][T][gld] whose sigmoid multiplies the shared expert's result; sel_w (or null): the pairs' weights where they
+// belong on the output; out [T][W] 32-bit.
 VCB_API int vcb_moe_combine(const float* y, const int* pos_of, const float* sel_w, int top, const float* shared, int S,
-                            long long s_stride, long long ld, const int* q_start, const int* q_len, int n_entries, int T, int W,
-                            float* out, cudaStream_t stream) {
+                            long long s_stride, long long ld, const float* gate, int gS, long long g_stride, long long gld,
+                            const int* q_start, const int* q_len, int n_entries, int T, int W, float* out, cudaStream_t stream) {
     if (T == 0) return 0;
     VCB_CHECK_ARG(T <= 65535, "moe_combine: %d rows in one step (at most 65535)", T);
     if (W % 4 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)out % 16 == 0 &&
         (shared == nullptr || ((uintptr_t)shared % 16 == 0 && ld % 4 == 0 && (S <= 1 || s_stride % 4 == 0)))) {
         launch_pdl(moe_combine_vec_kernel, dim3((W / 4 + 127) / 128, T), dim3(128), 0, stream, y, pos_of, sel_w, top,
-                   Rows{shared, S < 1 ? 1 : S, s_stride, ld}, q_start, q_len, n_entries, W, out);
+                   Rows{shared, S < 1 ? 1 : S, s_stride, ld}, Rows{gate, gS < 1 ? 1 : gS, g_stride, gld}, q_start, q_len, n_entries, W, out);
         VCB_CHECK_LAUNCH("moe_combine");
         return 0;
     }
     launch_pdl(moe_combine_kernel, dim3((W + 255) / 256, T), dim3(256), 0, stream, y, pos_of, sel_w, top,
-               Rows{shared, S < 1 ? 1 : S, s_stride, ld}, q_start, q_len, n_entries, W, out);
+               Rows{shared, S < 1 ? 1 : S, s_stride, ld}, Rows{gate, gS < 1 ? 1 : gS, g_stride, gld}, q_start, q_len, n_entries, W, out);
     VCB_CHECK_LAUNCH("moe_combine");
     return 0;
 }

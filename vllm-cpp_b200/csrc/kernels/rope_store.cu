@@ -8,8 +8,10 @@
 //                     same way over `vrot` of its lanes with frequencies of its own; queries to a buffer, keys and values
 //                     to the token's place in the paged cache.  Further options: a bias on every lane before all else;
 //                     every value head divided by its root mean square; columns behind the projection that are one
-//                     gate per query head (their sigmoids go to a buffer for the attention kernels' epilogues); and
-//                     queries mixed across heads on their way out, see below.
+//                     gate per query head or per lane of the heads' results (their sigmoids go to a buffer for the
+//                     attention kernels' epilogues); queries mixed across heads on their way out, see below; and values
+//                     mixed with those that an earlier layer made of the same token, v <- (1 - l) v + l v_first, l a
+//                     learned number (that layer leaves its values, 32-bit, in a buffer of the step).
 //
 // Mixed queries: where the scores of the heads are mixed before the softmax, score_h <- sum_g T[h][g] (q_g . k_kv(g)), the sum
 // over g can be drawn into the queries: with q'_h[G] = sum over the heads g that read KV head G of T[h][g] q_g,
@@ -61,7 +63,11 @@ struct StoreArgs {
     const float* talk;      // [nh][nh] or null: queries mixed across heads, q_out is [T][nh][nkv * hd]
     int vec;                // rows, partial sums and bias lie on 16-byte words
     int talk_off;           // where the mixing matrix lies in shared memory (floats)
-    float* gate_out;        // [T][nh] or null: sigmoid of the nh columns behind the projection's
+    float* gate_out;        // [T][n_gates] or null: sigmoids of the columns behind the projection's
+    int n_gates;            // nh, or nh * vd: one per lane of the heads' results
+    float* v_keep;          // [T][nkv vd] or null: receives the values as projected
+    const float* v_first;   // [T][nkv vd] or null: an earlier layer's values of the same tokens
+    const float* v_share;   // how much of them is mixed in (one number)
 };
 
 // lanes (a, b) of pair k of a head whose first `dims` lanes turn; b < 0: lane a passes unchanged
@@ -103,6 +109,14 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
     if (a.vfreq != nullptr)
         for (int i = threadIdx.x; i < vhalf; i += blockDim.x) sincosf(pos * a.vfreq[i], &vcs[vhalf + i], &vcs[i]);
     float sq = 0.f, sk = 0.f;
+    const float share = a.v_first != nullptr ? *a.v_share : 0.f;
+    // what becomes of lane c of the values on its way into the row
+    auto value_lane = [&](int c, float v) {
+        const size_t at = (size_t)t * nv + (c - nq - nk);
+        if (a.v_keep != nullptr) a.v_keep[at] = v;
+        return a.v_first != nullptr ? fmaf(share, a.v_first[at] - v, v) : v;
+    };
+    const bool mixes = a.v_keep != nullptr || a.v_first != nullptr;
     const bool first = blockIdx.y == 0;     // (a token's further blocks only mix queries)
     const int n_mine = first ? n : nq;
     int from = 0;
@@ -120,6 +134,12 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
                 const float4 b = *reinterpret_cast<const float4*>(a.bias + c);
                 v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
             }
+            if (mixes && c + 3 >= nq + nk) {
+                float* f = reinterpret_cast<float*>(&v);
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (c + k >= nq + nk) f[k] = value_lane(c + k, f[k]);
+            }
             *reinterpret_cast<float4*>(row + c) = v;
             if (a.q_gain != nullptr) {
                 const float f[4] = {v.x, v.y, v.z, v.w};
@@ -134,13 +154,30 @@ __global__ void qkv_rope_store_kernel(StoreArgs a) {
     for (int c = from + threadIdx.x; c < n_mine; c += blockDim.x) {
         float v = rows_at(a.qkv, t, c);
         if (a.bias != nullptr) v += a.bias[c];
+        if (mixes && c >= nq + nk) v = value_lane(c, v);
         row[c] = v;
         if (c < nq) sq = fmaf(v, v, sq);
         else if (c < nq + nk) sk = fmaf(v, v, sk);
     }
-    if (a.gate_out != nullptr && first)
-        for (int h = threadIdx.x; h < a.nh; h += blockDim.x)
-            a.gate_out[(size_t)t * a.nh + h] = 1.f / (1.f + expf(-rows_at(a.qkv, t, n + h)));
+    if (a.gate_out != nullptr && first) {
+        int h0 = 0;
+        if (a.vec && (n & 3) == 0 && (a.n_gates & 3) == 0) {
+            h0 = a.n_gates;
+            for (int h = 4 * threadIdx.x; h < h0; h += 4 * blockDim.x) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float* p = a.qkv.p + (long long)t * a.qkv.ld + n + h;
+#pragma unroll 4
+                for (int s = 0; s < a.qkv.S; ++s) {
+                    const float4 w = *reinterpret_cast<const float4*>(p + (long long)s * a.qkv.s_stride);
+                    v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+                }
+                *reinterpret_cast<float4*>(a.gate_out + (size_t)t * a.n_gates + h) =
+                    make_float4(1.f / (1.f + expf(-v.x)), 1.f / (1.f + expf(-v.y)), 1.f / (1.f + expf(-v.z)), 1.f / (1.f + expf(-v.w)));
+            }
+        }
+        for (int h = h0 + threadIdx.x; h < a.n_gates; h += blockDim.x)
+            a.gate_out[(size_t)t * a.n_gates + h] = 1.f / (1.f + expf(-rows_at(a.qkv, t, n + h)));
+    }
     if (a.talk != nullptr)
         for (int i = threadIdx.x; i < a.nh * nh4; i += blockDim.x) {
             const int g = i / nh4, h = i % nh4;
@@ -303,12 +340,14 @@ __global__ void rotate_heads_kernel(TC* x, const int* __restrict__ positions, co
 }  // namespace
 
 // qkv [S][T][ld] 32-bit sums; q_out [T][nh hd] and the pages of `dtype`; vfreq null: values stored unturned.
-// bias, talk (q_out then [T][nh][nkv hd]), gate_out (or null each) and unit_v: the options of StoreArgs.
+// bias, talk (q_out then [T][nh][nkv hd]), gate_out with n_gates, v_keep, v_first with v_share (or null each) and unit_v: the
+// options of StoreArgs.
 VCB_API int vcb_qkv_rope_store(const float* qkv, int S, long long s_stride, long long ld, const float* q_gain, const float* k_gain,
                                float eps, const int* positions, const float* freq, const float* vfreq, const int* slot_map,
                                void* q_out, void* pages, long long page_stride, int page_size, int num_pages, int nh, int nkv,
                                int hd, int vd, int rot, int vrot, int interleaved, int v_from_k, int T, int dtype, int* status,
-                               const float* bias, int unit_v, const float* talk, float* gate_out, cudaStream_t stream) {
+                               const float* bias, int unit_v, const float* talk, float* gate_out, int n_gates, float* v_keep,
+                               const float* v_first, const float* v_share, cudaStream_t stream) {
     if (T == 0) return 0;
     VCB_CHECK_ARG(nh > 0 && nkv > 0 && hd > 0 && vd > 0, "qkv_rope_store: bad sizes %d %d %d %d", nh, nkv, hd, vd);
     VCB_CHECK_ARG(rot >= 0 && rot <= hd && rot % 2 == 0, "qkv_rope_store: %d turning lanes of %d", rot, hd);
@@ -317,8 +356,11 @@ VCB_API int vcb_qkv_rope_store(const float* qkv, int S, long long s_stride, long
     VCB_CHECK_ARG((q_gain == nullptr) == (k_gain == nullptr), "qkv_rope_store: one gain without the other");
     VCB_CHECK_ARG(rot == 0 || freq != nullptr, "qkv_rope_store: no frequencies");
     StoreArgs a{Rows{qkv, S < 1 ? 1 : S, s_stride, ld}, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q_out, pages, page_stride,
-                page_size, num_pages, nh, nkv, hd, vd, rot, vfreq ? vrot : 0, interleaved, v_from_k, status, bias, unit_v, talk, 0, 0, gate_out};
-    a.vec = (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 && ld % 4 == 0 && (S <= 1 || s_stride % 4 == 0);
+                page_size, num_pages, nh, nkv, hd, vd, rot, vfreq ? vrot : 0, interleaved, v_from_k, status, bias, unit_v, talk, 0, 0, gate_out, n_gates, v_keep, v_first, v_share};
+    VCB_CHECK_ARG(gate_out == nullptr || n_gates == nh || n_gates == nh * vd, "qkv_rope_store: %d gates for %d heads of %d lanes", n_gates, nh, vd);
+    VCB_CHECK_ARG((v_keep == nullptr && v_first == nullptr) || !v_from_k, "qkv_rope_store: keys that double as values are not mixed");
+    VCB_CHECK_ARG(v_first == nullptr || v_share != nullptr, "qkv_rope_store: values to mix in without a share");
+    a.vec = (uintptr_t)qkv % 16 == 0 && (uintptr_t)bias % 16 == 0 && ld % 4 == 0 && (S <= 1 || s_stride % 4 == 0) && (uintptr_t)gate_out % 16 == 0;
     const int nh4 = (nh + 3) & ~3;
     a.talk_off = ((nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0) + (unit_v ? nkv : 0)) + 3) & ~3;
     const size_t smem = talk ? (size_t)(a.talk_off + nh * nh4) * sizeof(float) : (size_t)(nh * hd + nkv * hd + (v_from_k ? 0 : nkv * vd) + rot + (vfreq ? vrot : 0)

@@ -12,6 +12,7 @@ from . import nagavik  # registers Nagavik
 from . import fifudra  # registers Fifudra
 from . import mefupel  # registers Mefupel
 from . import nufetar  # registers Nufetar
+from . import disorax  # registers Disorax
 from .decoder import DecoderModel
 
 

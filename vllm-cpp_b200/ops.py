@@ -58,7 +58,7 @@ def _declare(L):
     sigs = {
         "vcb_embed_gather": [P, I, P, P, I, I, I, P, P],
         "vcb_add_rmsnorm": [P, P, I, I, LL, P, I, F, P, I, P, I, I, P],
-        "vcb_swiglu": [P, I, I, LL, P, I, I, I, P],
+        "vcb_swiglu": [P, I, I, LL, LL, P, I, I, I, P],
         "vcb_qknorm_rope_kvwrite": [P, I, I, LL, I, P, P, I, I, F, P, I, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, P, P],
         "vcb_gemm_bf16_tn": [P, P, P, I, I, I, I, LL, LL, LL, I, LL, P, P],
         "vcb_gemm_bf16_tn_shape": [P, P, P, I, I, I, I, LL, LL, LL, I, LL, I, I, P, P],
@@ -69,7 +69,7 @@ def _declare(L):
         "vcb_sgemm_tn": [P, P, P, I, I, I, LL, LL, LL, P],
         "vcb_gemm_bf16_plain": [P, P, P, I, I, I, I, LL, LL, LL, P],
         "vcb_attn_paged": [P, P, I, P, LL, P, P, I, P, P, P, P, I, I, P, P, I, I, I, I, I, I, F, P, P],
-        "vcb_attn_paged_ex": [P, P, I, P, LL, P, P, I, P, P, P, P, I, I, P, P, I, I, I, I, I, I, F, I, P, P, I, F, P, I, P, I, I, P, P, P],
+        "vcb_attn_paged_ex": [P, P, I, P, LL, P, P, I, P, P, P, P, I, I, P, P, I, I, I, I, I, I, F, I, P, P, I, F, P, I, P, I, I, P, I, I, I, P, P],
         "vcb_embed_sinusoid": [P, I, P, P, P, P, I, I, I, P, P],
         "vcb_causal_conv": [P, I, LL, LL, P, P, P, LL, P, P, P, I, I, I, I, I, P, P, I, P, I, P],
         "vcb_embed_scaled_pos": [P, I, P, P, P, I, F, P, I, I, I, I, P, P],
@@ -79,18 +79,18 @@ def _declare(L):
         "vcb_softcap": [P, LL, F, P],
         "vcb_ssm_scan": [P, I, LL, LL, I, P, I, LL, P, P, P, P, LL, P, P, P, I, I, I, I, I, I, I, I, P, P, P, P],
         "vcb_gated_group_norm": [P, P, I, LL, LL, P, F, P, P, I, I, I, I, P, I, P],
-        "vcb_moe_route": [P, I, LL, LL, P, P, I, I, I, I, I, P, P, P],
+        "vcb_moe_route": [P, I, LL, LL, P, P, P, I, I, I, I, I, P, P, P],
         "vcb_hyper_mix_norm": [P, P, P, I, LL, LL, P, P, P, P, F, P, I, P, I, I, I, I, P],
         "vcb_token_shift": [P, P, I, P, LL, P, P, P, I, I, I, P, I, LL, P],
-        "vcb_latent_norm_rope_store": [P, I, LL, LL, P, P, F, P, P, F, P, P, P, LL, I, I, I, I, I, I, I, I, I, P, P],
+        "vcb_latent_norm_rope_store": [P, I, LL, LL, P, P, F, P, P, F, P, P, P, LL, I, I, I, I, I, I, I, I, I, P, I, I, I, P, P],
         "vcb_head_linear": [P, I, I, LL, LL, I, I, P, I, P, I, LL, I, I, I, I, I, I, P],
-        "vcb_rope_rows": [P, I, LL, LL, I, I, P, P, F, P, I, LL, I, I, I, I, I, I, I, P],
+        "vcb_rope_rows": [P, I, LL, LL, I, I, P, P, F, P, I, LL, I, I, I, I, I, I, I, I, P],
         "vcb_matrix_rnn": [I, P, I, LL, LL, P, LL, I, I, I, I, I, P, P, P, P, P, LL, P, P, P, I, I, I, I, I, I, P,
                            P, I, LL, LL, F, P, P, P, I, I, P, P],
-        "vcb_sum_add_rmsnorm": [P, I, P, P, P, P, P, P, P, F, P, I, P, I, I, P],
+        "vcb_sum_add_rmsnorm": [P, I, P, P, P, P, P, P, P, F, P, I, P, I, I, F, P, P, P],
         "vcb_branch_norm_mean": [I, P, P, P, P, P, F, P, I, I, P],
         "vcb_polynorm": [P, I, LL, LL, P, F, P, I, I, I, P],
-        "vcb_qkv_rope_store": [P, I, LL, LL, P, P, F, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, P],
+        "vcb_qkv_rope_store": [P, I, LL, LL, P, P, F, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, I, P, P, P, P],
         "vcb_rotate_heads": [P, I, P, P, F, I, I, I, I, I, P],
         "vcb_head_norm_gate": [P, P, I, LL, LL, I, P, I, F, P, P, I, I, I, I, P, I, P],
         "vcb_moe_route_grouped": [P, I, LL, LL, P, I, I, F, P, P, I, I, I, I, P, P, P],
@@ -99,7 +99,7 @@ def _declare(L):
         "vcb_gemm_bf16_xielu": [P, P, P, I, I, I, LL, LL, LL, P, I, I, P, P],
         "vcb_gemm_bf16_grouped": [P, P, P, I, I, I, I, I, I, LL, LL, LL, P, I, P, P],
         "vcb_moe_gemm": [P, LL, P, I, P, P, P, I, I, P, I, I, I, I, P],
-        "vcb_moe_combine": [P, P, P, I, P, I, LL, LL, P, P, I, I, I, P, P],
+        "vcb_moe_combine": [P, P, P, I, P, I, LL, LL, P, I, LL, LL, P, P, I, I, I, P, P],
         "vcb_conv_state_update": [P, I, LL, LL, P, P, LL, P, P, P, I, I, I, P],
         "vcb_qkv_conv_norm_store": [P, I, LL, LL, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P, LL, I, I, I, I, P, P],
         "vcb_gated_norm_add": [P, P, I, LL, LL, P, I, LL, LL, P, P, F, P, P, I, I, I, P, I, P],
@@ -108,7 +108,7 @@ def _declare(L):
         "vcb_selftest_wait_timeout": [LL, P, P, P],
         "vcb_state_reset": [P, I, LL, LL, LL, I, I, P, P, P, I, ctypes.c_uint, P, P],
         "vcb_attn_mma": [P, P, P, LL, P, P, I, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, I, F, P, I, I, P],
-        "vcb_attn_mma_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, P, I, I, P],
+        "vcb_attn_mma_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, I, I, I, P, I, I, P],
         "vcb_attn_mma_wide_rows": [I, I, I],
         "vcb_attn_mma_supported": [I, I],
         "vcb_attn_mma_max_clusters": [I, I, I],
@@ -116,14 +116,15 @@ def _declare(L):
         "vcb_attn_mma_decode_fused": [P, I, LL, P, P, I, I, F, P, I, P, P, P, LL, P, P, I, P, P, P, P, I, P, P, P, P, I, I,
                                       I, I, I, I, F, P, I, P],
         "vcb_attn_tc": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, P, P, P],
-        "vcb_attn_tc_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, P, P, P],
+        "vcb_attn_tc_ex": [P, P, P, LL, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, F, P, I, P, I, I, P, I, I, I, P, P, P],
         "vcb_attn_tc_wide_supported": [I, I, I, I],
         "vcb_attn_tc_supported": [I, I, I],
-        "vcb_attn_wide": [P, P, P, LL, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, P, P, P],
+        "vcb_attn_wide": [P, P, P, LL, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, P, I, I, I, P, P, P],
+        "vcb_attn_wide_blocks_supported": [I, I, I, I, I],
         "vcb_attn_wide_supported": [I, I, I, I, I],
         "vcb_attn_stream": [P, P, P, LL, P, P, I, P, P, P, I, P, I, I, I, I, I, I, F, P, I, P],
         "vcb_attn_stream_supported": [I, I, I, I, I],
-        "vcb_attn_merge": [P, P, P, P, I, I, I, I, I, P, P],
+        "vcb_attn_merge": [P, P, P, P, I, I, I, I, I, P, I, I, P],
         "vcb_sample": [P, LL, I, I, P, P, P, P],
         "vcb_sample_split": [P, LL, I, I, P, P, P, P, I, P, P],
         "vcb_count_tokens": [P, P, P, I, I, I, P],
@@ -252,11 +253,12 @@ def _partials(t: torch.Tensor, name: str):
 
 def swiglu(gate_up, out):
     """out[t, i] = silu(gate_up[t, 2i]) * gate_up[t, 2i+1]: gate and up alternate along a row.
-    gate_up [T, 2I] or [S, T, 2I] (32-bit partial sums); out [T, I]."""
-    S, stride = _partials(gate_up, "gate_up"); _need(out, "out")
+    gate_up [T, 2I] or [S, T, 2I] (32-bit partial sums), the first columns of a wider product or alone; out [T, I]."""
+    _need(gate_up, "gate_up", contiguous=False); _need(out, "out")
+    S, stride = (1, 0) if gate_up.dim() == 2 else (gate_up.shape[0], gate_up.stride(0))
     T, I2 = gate_up.shape[-2:]
-    assert out.shape == (T, I2 // 2)
-    _call("vcb_swiglu", _p(gate_up), _dt(gate_up), S, stride, _p(out), _dt(out), T, I2 // 2, _stream())
+    assert out.shape == (T, I2 // 2) and gate_up.stride(-1) == 1
+    _call("vcb_swiglu", _p(gate_up), _dt(gate_up), S, stride, gate_up.stride(-2), _p(out), _dt(out), T, I2 // 2, _stream())
 
 
 def qknorm_rope_kvwrite(qkv, q_weight, k_weight, eps, cos_sin, positions, slot_map, q_out, pages, nh, nkv, hd,
@@ -433,10 +435,22 @@ def _q_width(q, nh, nkv, hd, wide):
         raise KernelError(f"queries of {q.shape[-1]} lanes, expected {width}")
 
 
-def _gate_ok(out_gate, out, nh):
-    if out_gate is not None:
-        _need(out_gate, "out_gate", torch.float32)
-        assert out_gate.shape[0] >= out.shape[0] and out_gate.shape[1] == nh, (out_gate.shape, out.shape, nh)
+def _gate_lanes(out_gate, out, heads) -> int:
+    """``out_gate`` as the attention wrappers take it: None, float32 [T, query heads] or, a factor per lane, shaped as the
+    result -> whether it is the latter."""
+    if out_gate is None:
+        return 0
+    _need(out_gate, "out_gate", torch.float32)
+    assert out_gate.shape[0] >= out.shape[0] and out_gate.shape[1] in (heads, out.shape[1]), (out_gate.shape, out.shape, heads)
+    return int(out_gate.shape[1] != heads)
+
+
+def _kv_pages(pages, nkv, hd):
+    """Pages [pages, 2, nkv, page_size, hd], or [pages, 1, nkv, page_size, hd] whose key rows double as values ->
+    (page_size, num_pages, one_row)."""
+    num_pages, parts, nkv_p, page_size, hd_p = pages.shape
+    assert parts in (1, 2) and nkv_p == nkv and hd_p == hd, (pages.shape, nkv, hd)
+    return page_size, num_pages, int(parts == 1)
 
 
 def _sink_scores(sink, nh):
@@ -450,10 +464,11 @@ def _sink_scores(sink, nh):
 
 def kv_page_views(pages, nkv, hd, hd_v):
     """(page_size, num_pages) of one cache's pages, laid out either [pages, 2, nkv, page_size, hd] or, where values
-    have another head size than keys, [pages, nkv * page_size * (hd + hd_v)]: keys first, then values."""
+    have another head size than keys, [pages, nkv * page_size * (hd + hd_v)]: keys first, then values; or
+    [pages, 1, nkv, page_size, hd], key rows whose first hd_v lanes double as values."""
     if pages.dim() == 5:
-        num_pages, two, nkv_p, page_size, hd_p = pages.shape
-        assert two == 2 and nkv_p == nkv and hd_p == hd == hd_v, (pages.shape, nkv, hd, hd_v)
+        page_size, num_pages, one_row = _kv_pages(pages, nkv, hd)
+        assert hd_v <= hd if one_row else hd_v == hd, (pages.shape, nkv, hd, hd_v)
         return page_size, num_pages
     assert pages.dim() == 2 and pages.shape[1] % (nkv * (hd + hd_v)) == 0, (pages.shape, nkv, hd, hd_v)
     return pages.shape[1] // (nkv * (hd + hd_v)), pages.shape[0]
@@ -461,7 +476,7 @@ def kv_page_views(pages, nkv, hd, hd_v):
 
 def attn_window_bias(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, rows_max, part_o, part_ml,
                      nh, nkv, hd, window, status, table_row=None, *, scale, keep_first=0, dist_a=None, dist_b=None, hd_v=None,
-                     softcap=0.0, slope=None, sink=False, chunked=False, wide=False, out_gate=None):
+                     softcap=0.0, slope=None, sink=False, chunked=False, wide=False, out_gate=None, blocks=False):
     """:func:`attn_paged` with its options: scores scaled by ``scale``; with a window, the first ``keep_first`` keys of
     a request stay visible; ``dist_a``/``dist_b`` (float32 [nh]): a_h ln(1 + b_h (pos - j)) is taken off key j's
     score; values of head size ``hd_v`` (``pages`` then [num_pages, nkv * page_size * (hd + hd_v)]); ``softcap`` c > 0:
@@ -470,12 +485,14 @@ def attn_window_bias(q, out, pages, block_table, q_start, q_len, ctx_len, items,
     silent key's score per head (not scaled); ``chunked``: the window stands still, a query sees the keys of its own chunk
     of ``window`` positions counted from position 0; ``wide``: ``q`` is [T, nh * nkv * hd], a query row has a block of
     lanes per KV head and its score is the sum of the blocks' products with those heads' keys; ``out_gate`` (float32
-    [T, nh]): what the result of a token and head is multiplied by."""
-    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, wide)
+    [T, query heads], or shaped as ``out``): what the result of a token and head (and lane) is multiplied by.  ``pages``
+    [num_pages, 1, nkv, page_size, hd]: the key rows' first hd_v lanes double as values.  ``blocks`` (with ``wide``): the
+    KV heads are the blocks of one shared row that every query head meets; ``nh`` counts (block, query head) pairs, ``q``
+    is [T, nh / nkv * nkv * hd] and ``out`` [T, nh / nkv, nkv, hd_v], a head's result block by block."""
+    heads = nh // nkv if blocks else nh
+    lanes = _gate_lanes(out_gate, out, heads); _q_width(q, heads, nkv, hd, wide)
     hd_v = hd if hd_v is None else int(hd_v)
-    sink_value = sink if torch.is_tensor(sink) else None
-    if sink_value is not None:
-        _need(sink_value, "sink", torch.float32); assert sink_value.numel() == nh
+    sink_value = _sink_scores(sink, heads)
     _need(q, "q"); _need(out, "out", q.dtype); _need(pages, "pages", q.dtype)
     for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len),
                     ("items", items)):
@@ -491,7 +508,7 @@ def attn_window_bias(q, out, pages, block_table, q_start, q_len, ctx_len, items,
           block_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, rows_max, _p(part_o), _p(part_ml),
           nh, nkv, hd, page_size, num_pages, int(window or 0), float(scale), int(keep_first or 0), _p(dist_a), _p(dist_b),
           hd_v, float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), int(bool(chunked)),
-          int(bool(wide)), _p(out_gate), _p(status), _stream())
+          int(bool(wide)), _p(out_gate), lanes, int(pages.dim() == 5 and pages.shape[1] == 1), int(bool(blocks)), _p(status), _stream())
 
 
 def embed_sinusoid(table, ids, positions, inv_freq, out, status):
@@ -755,15 +772,18 @@ def moe_tiles_cap(n_pairs: int, n_experts: int, tile_rows: int | None = None) ->
     return min(n_pairs, n_experts) + n_pairs // (tile_rows or moe_tile_rows())
 
 
-def moe_route(logits, q_start, q_len, n_entries, top, sel_e, sel_w, softmax_weights=False):
-    """Per row of the step's entries: the ``top`` largest of the router's ``logits`` (32-bit [T, E] or [S, T, E]) ->
+def moe_route(logits, q_start, q_len, n_entries, top, sel_e, sel_w, softmax_weights=False, bias=None):
+    """Per row of the step's entries: the ``top`` largest of the router's ``logits`` (32-bit [T, E] or [S, T, E]; ``bias``
+    [E], if given, is added first) ->
     ``sel_e`` [T, top] int32 (-1 in rows outside every entry) and ``sel_w`` [T, top]: sigmoid(logit), or the softmax over
     the chosen logits."""
     S, ss, ld = _rows_in(logits, "logits")
     T, E = logits.shape[-2:]
     _need(sel_e, "sel_e", torch.int32); _need(sel_w, "sel_w", torch.float32)
     assert sel_e.numel() == T * top and sel_w.numel() == T * top
-    _call("vcb_moe_route", _p(logits), S, ss, ld, _p(q_start), _p(q_len), n_entries, T, E, int(top), int(bool(softmax_weights)),
+    if bias is not None:
+        _need(bias, "bias", torch.float32); assert bias.numel() == E
+    _call("vcb_moe_route", _p(logits), S, ss, ld, _p(bias), _p(q_start), _p(q_len), n_entries, T, E, int(top), int(bool(softmax_weights)),
           _p(sel_e), _p(sel_w), _stream())
 
 
@@ -798,16 +818,17 @@ def gemm_grouped_ok(x, w) -> bool:
 def gemm_bf16_grouped(w, x, tile_expert, tile_rows, out, status, act=None):
     """out[r, :] = act(w[tile_expert[r // tile_rows]] . x[r]) over the sorted rows (tcgen05 + TMA): w [E, N, K] bfloat16,
     x [tiles * tile_rows, K] bfloat16, out [tiles * tile_rows, N] bfloat16 or float32; tiles whose expert is -1 are
-    skipped.  ``act``: None, "silu" or "relu2"."""
+    skipped.  ``act``: None, "silu" or "relu2"; "swiglu": rows 2i and 2i + 1 of an expert are gate_i and up_i, out
+    [tiles * tile_rows, N / 2] bfloat16 is silu(gate) * up."""
     _need(w, "w", torch.bfloat16); _need(x, "x", torch.bfloat16, contiguous=False); _need(out, "out")
     _need(tile_expert, "tile_expert", torch.int32)
     E, N, K = w.shape
     tiles = tile_expert.numel()
-    assert tile_rows in GROUPED_TILE_ROWS and x.shape == (tiles * tile_rows, K) and out.shape == (tiles * tile_rows, N)
-    if act not in (None, "silu", "relu2"):
-        raise KernelError(f"gemm_bf16_grouped: activation '{act}' (None, 'silu' or 'relu2')")
+    assert tile_rows in GROUPED_TILE_ROWS and x.shape == (tiles * tile_rows, K) and out.shape == (tiles * tile_rows, N // 2 if act == "swiglu" else N)
+    if act not in (None, "silu", "relu2", "swiglu"):
+        raise KernelError(f"gemm_bf16_grouped: activation '{act}' (None, 'silu', 'relu2' or 'swiglu')")
     _call("vcb_gemm_bf16_grouped", _p(w), _p(x), _p(out), _dt(out), E, N, tiles, int(tile_rows), K, K, x.stride(0), out.stride(0),
-          _p(tile_expert), 0 if act is None else ACTIVATIONS[act], _p(status), _stream())
+          _p(tile_expert), 0 if act is None else (7 if act == "swiglu" else ACTIVATIONS[act]), _p(status), _stream())
 
 
 def moe_gemm(x, w, tile_expert, out, *, src_of=None, sel_w=None, top=1, act=None):
@@ -825,23 +846,29 @@ def moe_gemm(x, w, tile_expert, out, *, src_of=None, sel_w=None, top=1, act=None
           int(src_of is not None), _p(out), N, K, ACTIVATIONS[act] if act is not None else -1, tiles, _stream())
 
 
-def moe_combine(y, pos_of, top, q_start, q_len, n_entries, out, shared=None, sel_w=None):
-    """out[t] = shared[t] + sum over the token's pairs of y[pos_of[t, k]] (times sel_w[t, k] if given), k in order."""
+def moe_combine(y, pos_of, top, q_start, q_len, n_entries, out, shared=None, sel_w=None, shared_gate=None):
+    """out[t] = shared[t] + sum over the token's pairs of y[pos_of[t, k]] (times sel_w[t, k] if given), k in order.
+    ``shared_gate`` (32-bit [T, 1] or [S, T, 1]): its sigmoid multiplies shared[t]."""
     _need(y, "y", torch.float32); _need(pos_of, "pos_of", torch.int32); _need(out, "out", torch.float32)
     T, W = out.shape
     S = ss = ld = 0
     if shared is not None:
         S, ss, ld = _rows_in(shared, "shared")
         assert shared.shape[-1] == W and shared.shape[-2] >= T
-    _call("vcb_moe_combine", _p(y), _p(pos_of), _p(sel_w), int(top), _p(shared), S, ss, ld, _p(q_start), _p(q_len), n_entries,
-          T, W, _p(out), _stream())
+    gS = gss = gld = 0
+    if shared_gate is not None:
+        gS, gss, gld = _rows_in(shared_gate, "shared_gate")
+        assert shared is not None and shared_gate.shape[-1] == 1 and shared_gate.shape[-2] >= T
+    _call("vcb_moe_combine", _p(y), _p(pos_of), _p(sel_w), int(top), _p(shared), S, ss, ld, _p(shared_gate), gS, gss, gld,
+          _p(q_start), _p(q_len), n_entries, T, W, _p(out), _stream())
 
 
-def attn_merge(part_o, part_ml, dec_rows, out, n_dec, nh, hd, nslices, out_gate=None):
-    _gate_ok(out_gate, out, nh)
+def attn_merge(part_o, part_ml, dec_rows, out, n_dec, nh, hd, nslices, out_gate=None, gate_blocks=1):
+    """``gate_blocks``: that many results side by side belong to one head (a gate per head is then theirs together)."""
+    lanes = _gate_lanes(out_gate, out, nh // gate_blocks)
     _need(part_o, "part_o", torch.float32); _need(part_ml, "part_ml", torch.float32)
     _need(dec_rows, "dec_rows", torch.int32); _need(out, "out")
-    _call("vcb_attn_merge", _p(part_o), _p(part_ml), _p(dec_rows), _p(out), _dt(out), n_dec, nh, hd, nslices, _p(out_gate), _stream())
+    _call("vcb_attn_merge", _p(part_o), _p(part_ml), _p(dec_rows), _p(out), _dt(out), n_dec, nh, hd, nslices, _p(out_gate), lanes, int(gate_blocks), _stream())
 
 
 def sample(logits, params, counts, out, no_nucleus=False):
@@ -971,24 +998,24 @@ def attn_mma_wide_rows(dtype: torch.dtype, hd: int, nkv: int) -> int:
 
 def attn_tc(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, nh, nkv, hd, window, status,
             table_row=None, work=None, scale=None, keep_first=0, dist_a=None, dist_b=None, softcap=0.0, slope=None, sink=False,
-            chunked=False, wide=False, out_gate=None):
+            chunked=False, wide=False, out_gate=None, blocks=False):
     """Attention of prompt portions on tcgen05 tensor cores (bfloat16, head_dim 64 or 128, pages of 8 to 64
     tokens), with the options of :func:`attn_window_bias` (``scale``, ``keep_first``, ``dist_a``/``dist_b``, ``softcap``,
-    ``slope``, ``sink``, ``chunked``, ``out_gate``, and ``wide`` where :func:`attn_tc_wide_supported` says so).
+    ``slope``, ``sink``, ``chunked``, ``out_gate``, pages whose keys double as values, ``wide`` and ``blocks`` where :func:`attn_tc_wide_supported` says so).
     Items as for :func:`attn_paged` with one key slice and at most 128 rows each.  ``work``: two int32
     zeros, zero again when the kernel is through (the queue its blocks take their units from); launches that share
     them must follow one another on a stream.  Made on the spot when not given."""
     if work is None:
         work = torch.zeros(2, dtype=torch.int32, device=q.device)
     _need(work, "work", torch.int32)
-    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, wide)
-    sink_value = _sink_scores(sink, nh)
+    heads = nh // nkv if blocks else nh
+    lanes = _gate_lanes(out_gate, out, heads); _q_width(q, heads, nkv, hd, wide)
+    sink_value = _sink_scores(sink, heads)
     _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pages, "pages", torch.bfloat16)
     for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len),
                     ("items", items)):
         _need(t, name, torch.int32)
-    num_pages, two, nkv_p, page_size, hd_p = pages.shape
-    assert two == 2 and nkv_p == nkv and hd_p == hd
+    page_size, num_pages, one_row = _kv_pages(pages, nkv, hd)
     if dist_a is not None:
         _need(dist_a, "dist_a", torch.float32); _need(dist_b, "dist_b", torch.float32)
         assert dist_a.numel() == nh and dist_b.numel() == nh
@@ -998,28 +1025,29 @@ def attn_tc(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items,
           block_table.shape[1], _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, nh, nkv, hd, page_size,
           num_pages, int(window or 0), 1.0 / math.sqrt(hd) if scale is None else float(scale), int(keep_first or 0),
           _p(dist_a), _p(dist_b), float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value),
-          int(bool(chunked)), int(bool(wide)), _p(out_gate), _p(status), _p(work), _stream())
+          int(bool(chunked)), int(bool(wide)), _p(out_gate), lanes, one_row, int(bool(blocks)), _p(status), _p(work), _stream())
 
 
 def attn_mma(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, rows_max, part_o, part_ml,
              nh, nkv, hd, window, status, table_row=None, allow_tma=True, slice_counters=None, dec_rows=None,
              cluster=0, scale=None, keep_first=0, dist_a=None, dist_b=None, softcap=0.0, slope=None, sink=False, chunked=False,
-             wide=False, out_gate=None):
+             wide=False, out_gate=None, blocks=False):
     """Tensor-core variant of :func:`attn_paged` (bfloat16, head_dim 64 or 128; rows_max 16 or 128), with the
     options of :func:`attn_window_bias` (``scale``, default 1/sqrt(hd); ``keep_first``; ``dist_a``/``dist_b``;
-    ``softcap``, ``slope``, ``sink``, ``chunked``, ``out_gate``, and ``wide``, with rows_max 16 or what
+    ``softcap``, ``slope``, ``sink``, ``chunked``, ``out_gate``, pages whose keys double as values, and ``wide`` and
+    ``blocks``, with rows_max 16 or what
     :func:`attn_mma_wide_rows` says).
     With ``slice_counters`` (int32 zeros, one per decoded token and KV head group, left at zero again) and
     ``dec_rows``, the block that finishes a token's last key slice merges the slices itself; with ``cluster`` = the
     number of slices per token (2 to 8) as well, the slices' blocks run as a cluster and merge through shared memory."""
-    sink_value = _sink_scores(sink, nh)
-    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, wide)
+    heads = nh // nkv if blocks else nh
+    sink_value = _sink_scores(sink, heads)
+    lanes = _gate_lanes(out_gate, out, heads); _q_width(q, heads, nkv, hd, wide)
     _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pages, "pages", torch.bfloat16)
     for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len),
                     ("items", items)):
         _need(t, name, torch.int32)
-    num_pages, two, nkv_p, page_size, hd_p = pages.shape
-    assert two == 2 and nkv_p == nkv and hd_p == hd
+    page_size, num_pages, one_row = _kv_pages(pages, nkv, hd)
     if dist_a is not None:
         _need(dist_a, "dist_a", torch.float32); _need(dist_b, "dist_b", torch.float32)
         assert dist_a.numel() == nh and dist_b.numel() == nh
@@ -1030,30 +1058,35 @@ def attn_mma(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items
           _p(part_ml), _p(slice_counters), _p(dec_rows), nh, nkv, hd, page_size, num_pages, int(window or 0),
           1.0 / math.sqrt(hd) if scale is None else float(scale), int(keep_first or 0), _p(dist_a), _p(dist_b),
           float(softcap or 0.0), _p(slope), int(sink_value is not None or bool(sink)), _p(sink_value), int(bool(chunked)),
-          int(bool(wide)), _p(out_gate), _p(status), int(allow_tma), int(cluster), _stream())
+          int(bool(wide)), _p(out_gate), lanes, one_row, int(bool(blocks)), _p(status), int(allow_tma), int(cluster), _stream())
 
 
-def attn_wide_supported(dtype: torch.dtype, hd: int, page_size: int, nh: int, nkv: int) -> bool:
-    """Whether :func:`attn_wide` takes these sizes."""
+def attn_wide_supported(dtype: torch.dtype, hd: int, page_size: int, nh: int, nkv: int, blocks: bool = False) -> bool:
+    """Whether :func:`attn_wide` takes these sizes (``nh`` and ``blocks`` as there)."""
+    if blocks:
+        return bool(lib().vcb_attn_wide_blocks_supported(BF16 if dtype == torch.bfloat16 else F32, hd, page_size, nh // nkv, nkv))
     return bool(lib().vcb_attn_wide_supported(BF16 if dtype == torch.bfloat16 else F32, hd, page_size, nh, nkv))
 
 
 def attn_wide(q, out, pages, block_table, q_start, q_len, ctx_len, items, n_items, part_o, part_ml, nh, nkv, hd, window, status,
-              table_row=None, scale=None, chunked=False, out_gate=None):
+              table_row=None, scale=None, chunked=False, out_gate=None, sink=False, blocks=False):
     """Single decoded tokens whose query rows are wide (``q`` [T, nh * nkv * hd], see :func:`attn_window_bias`): a block is a
     token and a slice of its keys with all query heads, so keys and values are read once.  ``items`` as for
     :func:`attn_mma`; several slices leave their partials in ``part_o`` / ``part_ml`` for :func:`attn_merge` (which then
-    applies ``out_gate``)."""
-    _gate_ok(out_gate, out, nh); _q_width(q, nh, nkv, hd, True)
+    applies ``out_gate``).  ``sink`` (a float32 tensor of scores per query head) and ``blocks`` as there."""
+    heads = nh // nkv if blocks else nh
+    lanes = _gate_lanes(out_gate, out, heads); _q_width(q, heads, nkv, hd, True)
+    sink_value = _sink_scores(sink, heads)
+    if sink is True:
+        raise KernelError("attn_wide: the silent key has a score per head")
     _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(pages, "pages", torch.bfloat16)
     for name, t in (("block_table", block_table), ("q_start", q_start), ("q_len", q_len), ("ctx_len", ctx_len), ("items", items)):
         _need(t, name, torch.int32)
-    num_pages, two, nkv_p, page_size, hd_p = pages.shape
-    assert two == 2 and nkv_p == nkv and hd_p == hd
+    page_size, num_pages, one_row = _kv_pages(pages, nkv, hd)
     _call("vcb_attn_wide", _p(q), _p(out), _p(pages), pages.stride(0), _p(block_table), _p(table_row), block_table.shape[1],
           _p(q_start), _p(q_len), _p(ctx_len), _p(items), n_items, _p(part_o), _p(part_ml), nh, nkv, hd, page_size, num_pages,
-          int(window or 0), int(bool(chunked)), 1.0 / math.sqrt(hd) if scale is None else float(scale), _p(out_gate), _p(status),
-          _stream())
+          int(window or 0), int(bool(chunked)), 1.0 / math.sqrt(hd) if scale is None else float(scale), _p(out_gate), lanes, one_row,
+          int(bool(blocks)), _p(sink_value), _p(status), _stream())
 
 
 def attn_stream_supported(dtype: torch.dtype, hd: int, page_size: int, nh: int, nkv: int) -> bool:
@@ -1181,17 +1214,26 @@ def token_shift(h, mu, state, q_start, q_len, slots, n_entries, out):
 
 
 def latent_norm_rope_store(u, q_gain, kv_gain, eps, positions, freq, gain, slot_map, cq_out, pages, page_size, q_rank,
-                           kv_rank, rot, status, v_width=None, interleaved=False):
+                           kv_rank, rot, status, v_width=None, interleaved=False, k_width=None, k_block=None, gate_out=None):
     """From the stacked down projections ``u`` (32-bit [T, q_rank + kv_rank + rot] or partial sums): the normed query
     latent to ``cq_out`` [T, q_rank]; the normed key/value latent c and the rotated shared key part into the token's
     cache row.  A page is one flat row: [page_size, kv_rank + rot] key rows [c | k_rot], then [page_size, v_width]
     value rows [c | zeros] (``v_width`` None: kv_rank lanes, c alone).  ``freq`` [rot / 2] 32-bit; cos and sin are
     multiplied by ``gain``; ``interleaved``: neighbouring lanes turn together (else lane i with lane i + rot/2).
-    ``q_rank`` 0 (``q_gain`` and ``cq_out`` None): there is no query latent."""
+    ``q_rank`` 0 (``q_gain`` and ``cq_out`` None): there is no query latent.  ``v_width`` 0: no value rows, the key rows
+    double as values.  ``k_width``: lanes of a key row (zeros behind kv_rank + rot; default none); ``k_block``: it lies in
+    pieces of that many lanes, [k_width / k_block, page_size, k_block].  ``gate_out`` [T, n]: the sigmoids of n further
+    columns of ``u`` behind the others."""
     v_width = int(kv_rank if v_width is None else v_width)
+    k_width = int(kv_rank + rot if k_width is None else k_width)
+    k_block = int(k_width if k_block is None else k_block)
+    n_gates = 0
+    if gate_out is not None:
+        _need(gate_out, "gate_out", torch.float32)
+        n_gates = gate_out.shape[1]
     S, ss, ld = _rows_in(u, "u")
     T = u.shape[-2]
-    assert u.shape[-1] == q_rank + kv_rank + rot and rot % 2 == 0
+    assert u.shape[-1] == q_rank + kv_rank + rot + n_gates and rot % 2 == 0
     if q_rank:
         _need(cq_out, "cq_out", pages.dtype); _need(q_gain, "q_gain", torch.float32)
         assert cq_out.shape == (T, q_rank) and q_gain.numel() == q_rank
@@ -1200,10 +1242,10 @@ def latent_norm_rope_store(u, q_gain, kv_gain, eps, positions, freq, gain, slot_
     if rot:
         _need(freq, "freq", torch.float32); assert freq.numel() == rot // 2
     assert kv_gain.numel() == kv_rank
-    assert pages[0].numel() == page_size * (kv_rank + rot + v_width), (pages.shape, page_size, kv_rank, rot, v_width)
+    assert pages[0].numel() == page_size * (k_width + v_width), (pages.shape, page_size, kv_rank, rot, v_width)
     _call("vcb_latent_norm_rope_store", _p(u), S, ss, ld, _p(q_gain), _p(kv_gain), float(eps), _p(positions), _p(freq),
           float(gain), _p(slot_map), _p(cq_out), _p(pages), pages.stride(0), int(page_size), pages.shape[0], int(q_rank),
-          int(kv_rank), int(rot), int(bool(interleaved)), v_width, T, _dt(pages), _p(status), _stream())
+          int(kv_rank), int(rot), int(bool(interleaved)), k_width, k_block, v_width, _p(gate_out), n_gates, T, _dt(pages), _p(status), _stream())
 
 
 def head_linear(x, m, out, *, heads, n_in, n_out, in_head_stride, in_off=0, out_head_stride, out_off=0):
@@ -1225,9 +1267,10 @@ def head_linear(x, m, out, *, heads, n_in, n_out, in_head_stride, in_off=0, out_
 
 
 def rope_rows(x, positions, freq, gain, out, *, heads, dims, width, in_head_stride, in_off=0, out_head_stride, out_off=0,
-              interleaved=False):
+              interleaved=False, pad=0):
     """Copies ``width`` lanes of every head's slice of the 32-bit sums ``x`` into ``out``, the first ``dims`` of them
-    rotated: lane i pairs with lane i + dims/2 (``interleaved``: lane 2i with lane 2i + 1), the angle is position * freq[i], cos and sin times ``gain``."""
+    rotated: lane i pairs with lane i + dims/2 (``interleaved``: lane 2i with lane 2i + 1), the angle is position * freq[i], cos and sin times ``gain``.  ``pad``
+    zero lanes go behind them."""
     S, ss, ld = _rows_in(x, "x")
     T = x.shape[-2]
     _need(out, "out", contiguous=False); _need(positions, "positions", torch.int32)
@@ -1235,9 +1278,9 @@ def rope_rows(x, positions, freq, gain, out, *, heads, dims, width, in_head_stri
         _need(freq, "freq", torch.float32); assert freq.numel() == dims // 2
     assert out.stride(-1) == 1 and dims % 2 == 0
     assert (heads - 1) * in_head_stride + in_off + width <= x.shape[-1]
-    assert (heads - 1) * out_head_stride + out_off + width <= out.shape[-1]
+    assert (heads - 1) * out_head_stride + out_off + width + pad <= out.shape[-1]
     _call("vcb_rope_rows", _p(x), S, ss, ld, int(in_head_stride), int(in_off), _p(positions), _p(freq), float(gain), _p(out),
-          _dt(out), out.stride(0), int(out_head_stride), int(out_off), T, int(heads), int(dims), int(width), int(bool(interleaved)), _stream())
+          _dt(out), out.stride(0), int(out_head_stride), int(out_off), T, int(heads), int(dims), int(width), int(pad), int(bool(interleaved)), _stream())
 
 
 # -------------------------------------------------------------------------- recurrences with a matrix state per head
@@ -1338,10 +1381,11 @@ def _terms(tensors, name):
     return ptrs, counts, sstr, lds
 
 
-def sum_add_rmsnorm(resid, terms, gain, eps, out, rows=None, row_extra=None, vec_extra=None):
-    """resid[t] += sum of ``terms`` (up to four 32-bit results, each [T, H] or [S, T, H] partial sums) + row_extra[t] +
+def sum_add_rmsnorm(resid, terms, gain, eps, out, rows=None, row_extra=None, vec_extra=None, scale=1.0, gain2=None, out2=None):
+    """resid[t] += ``scale`` * sum of ``terms`` (up to four 32-bit results, each [T, H] or [S, T, H] partial sums) + row_extra[t] +
     vec_extra, then out = gain * resid[t] / sqrt(mean(resid[t]^2) + eps), in one pass.  ``gain`` 32-bit [H]; ``out`` None:
-    the additions alone.  With ``rows`` (int32 indices) only those rows are made and the stream is left alone."""
+    the additions alone.  With ``rows`` (int32 indices) only those rows are made and the stream is left alone.  ``gain2``
+    and ``out2``: a second norm of the same rows, which differs in its gain."""
     _need(resid, "resid", torch.float32)
     T, H = resid.shape
     terms = [t for t in terms if t is not None]
@@ -1358,9 +1402,12 @@ def sum_add_rmsnorm(resid, terms, gain, eps, out, rows=None, row_extra=None, vec
         _need(rows, "rows", torch.int32)
     if out is not None:
         _need(out, "out"); assert out.shape[0] >= n and out.shape[1] == H and gain is not None
+    if out2 is not None:
+        _need(out2, "out2", out.dtype); _need(gain2, "gain2", torch.float32)
+        assert out2.shape == out.shape and gain2.numel() == H
     ptrs, counts, sstr, lds = _terms(terms, "term")
     _call("vcb_sum_add_rmsnorm", _p(resid), len(terms), ptrs, counts, sstr, lds, _p(row_extra), _p(vec_extra), _p(gain), float(eps),
-          _p(out), _dt(out) if out is not None else F32, _p(rows), n, H, _stream())
+          _p(out), _dt(out) if out is not None else F32, _p(rows), n, H, float(scale), _p(gain2), _p(out2), _stream())
 
 
 def branch_norm_mean(results, gains, eps, out):
@@ -1392,7 +1439,8 @@ def polynorm(u, coef, eps, out):
 
 
 def qkv_rope_store(qkv, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q_out, pages, nh, nkv, hd, vd, status, *,
-                   rot, interleaved=False, values_from_keys=False, bias=None, unit_values=False, talk=None, gate_out=None):
+                   rot, interleaved=False, values_from_keys=False, bias=None, unit_values=False, talk=None, gate_out=None,
+                   v_keep=None, v_first=None, v_share=None):
     """From the stacked projection's 32-bit sums ``qkv`` ([T, C] or [S, T, C]; C = nh hd + nkv hd + nkv vd, or without the
     value columns where ``values_from_keys``: the keys as projected are the values): with ``q_gain`` [nh hd] / ``k_gain``
     [nkv hd] all of a token's query (key) lanes divided by their root mean square times the gain; the first ``rot`` lanes
@@ -1401,12 +1449,17 @@ def qkv_rope_store(qkv, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q
     tokens' slots of ``pages`` (see :func:`kv_page_views`).  Options: ``bias`` [C] added first; ``unit_values``: every value
     head divided by its root mean square; ``talk`` [nh, nh]: queries mixed across heads, q'_h[G] = sum over the heads g
     of KV head G of talk[h, g] q_g, ``q_out`` [T, nh * nkv * hd] (what the attention kernels take as ``wide``);
-    ``gate_out`` [T, nh]: the sigmoids of nh further columns behind the projection's."""
+    ``gate_out`` [T, nh] or [T, nh * vd]: the sigmoids of as many further columns behind the projection's; ``v_keep``
+    (float32 [T, nkv * vd]) receives the values as projected; ``v_first`` (likewise) and ``v_share`` (one number):
+    v <- (1 - v_share) v + v_share v_first before anything else happens to the values."""
     S, ss, ld = _rows_in(qkv, "qkv")
     T, C = qkv.shape[-2:]
-    C -= nh if gate_out is not None else 0
+    n_gates = gate_out.shape[1] if gate_out is not None else 0
+    C -= n_gates
+    assert n_gates in (0, nh, nh * vd), (n_gates, nh, vd)
     assert C == nh * hd + nkv * hd + (0 if values_from_keys else nkv * vd), (C, nh, nkv, hd, vd)
-    for name, t, n in (("bias", bias, C), ("talk", talk, nh * nh), ("gate_out", gate_out, T * nh)):
+    for name, t, n in (("bias", bias, C), ("talk", talk, nh * nh), ("gate_out", gate_out, T * n_gates),
+                       ("v_keep", v_keep, T * nkv * vd), ("v_first", v_first, T * nkv * vd), ("v_share", v_share, 1)):
         if t is not None:
             _need(t, name, torch.float32); assert t.numel() == n, (name, t.shape, n)
     if q_gain is not None:
@@ -1423,7 +1476,7 @@ def qkv_rope_store(qkv, q_gain, k_gain, eps, positions, freq, vfreq, slot_map, q
     _call("vcb_qkv_rope_store", _p(qkv), S, ss, ld, _p(q_gain), _p(k_gain), float(eps), _p(positions), _p(freq), _p(vfreq),
           _p(slot_map), _p(q_out), _p(pages), pages.stride(0), page_size, num_pages, nh, nkv, hd, vd, int(rot), vd,
           int(bool(interleaved)), int(bool(values_from_keys)), T, _dt(q_out), _p(status), _p(bias), int(bool(unit_values)), _p(talk),
-          _p(gate_out), _stream())
+          _p(gate_out), n_gates, _p(v_keep), _p(v_first), _p(v_share), _stream())
 
 
 def rotate_heads(x, positions, freq, *, heads, width, dims, interleaved=False, sign=1.0):

@@ -58,7 +58,8 @@ class CacheSpec:
                   chunk's pages are given back when it is through;
                   ``v_head_dim`` > 0: values of another size than keys (a page then
                   holds ``[num_kv_heads, page_size, head_dim]`` keys followed by
-                  ``[num_kv_heads, page_size, v_head_dim]`` values, as one flat row).
+                  ``[num_kv_heads, page_size, v_head_dim]`` values, as one flat row);
+                  ``one_row``: keys alone are kept, their rows double as values.
     kind "state": a block of fixed size per request, ``shape`` of ``dtype``,
                   addressed by the request's slot."""
     kind: str
@@ -72,6 +73,7 @@ class CacheSpec:
     keep_first: int = 0
     v_head_dim: int = 0
     chunked: bool = False
+    one_row: bool = False
 
 
 class Part:

@@ -53,7 +53,7 @@ SINK_SCORES_ON_TENSOR_CORES = True
 
 
 def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_first=0, dist_a=None, dist_b=None,
-                    softcap=0.0, slope=None, sink=False, chunked=False, wide=False, out_gate=None):
+                    softcap=0.0, slope=None, sink=False, chunked=False, wide=False, out_gate=None, blocks=False):
     """(``sink``: False, True -- a silent key of score 0 --, or a float32 tensor [nh] of the silent key's score per head.)
     Scores, softmax and weighted sums of one step over the paged keys and values ``kv``: ``q`` [T, nh * hd] against
     keys of ``hd`` lanes, values of ``vd`` lanes into ``out`` [T, nh * vd].  Single tokens are cut into key slices and
@@ -64,11 +64,15 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     ``chunked``: the window is the chunk of ``window`` positions, counted from position 0, that a query lies in.
     ``wide``: ``q`` is [T, nh * nkv * hd], a block of lanes per KV head, and a row's score with a key position is the sum
     of the blocks' products with all heads' keys there (queries mixed across heads); single tokens with such rows run on a
-    kernel whose block is a token and key slice with all heads (ops.attn_wide), where it takes the sizes.  ``out_gate`` (float32 [T, nh])
-    multiplies each head's result."""
+    kernel whose block is a token and key slice with all heads (ops.attn_wide), where it takes the sizes.  ``out_gate`` (float32 [T, nh],
+    or shaped as ``out``) multiplies each head's result.
+    Pages of one part, [pages, 1, nkv, page_size, hd]: the key rows' first ``vd`` lanes double as values.
+    ``blocks``: key rows wider than a kernel's tile, kept as ``nkv`` blocks of ``hd`` lanes, that all query heads share; ``nh``
+    counts (block, query head) pairs, ``q`` is [T, nh / nkv, nkv * hd] and ``out`` [T, nh / nkv, nkv * vd]."""
     x = q
+    wide = wide or blocks
     if nkv == 1:
-        wide = False      # one block a row: an ordinary one
+        wide = blocks = False      # one block a row: an ordinary one
     # no query reads more keys than the window and the kept first ones: no more key slices than those fill
     reach = window + keep_first if window else 0
     # bfloat16 with keys and values of 64 or 128 lanes: the tensor-core kernel; else the plain one
@@ -77,7 +81,7 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     has_extras = bool(softcap or slope is not None or learned_sink or sink)
     mma = (MMA_ATTENTION and vd == hd and kv.pages.dim() == 5 and ops.attn_mma_supported(x.dtype, hd)
            and (EXTRAS_ON_TENSOR_CORES or not has_extras) and (SINK_SCORES_ON_TENSOR_CORES or not learned_sink))
-    has_extras = has_extras or bool(keep_first) or dist_a is not None
+    more_than_a_sink = bool(softcap or slope is not None or sink is True or keep_first or dist_a is not None)
     mma_rows = MMA_SPAN_ROWS
     if mma and wide:
         mma_rows = ops.attn_mma_wide_rows(x.dtype, hd, nkv)
@@ -86,7 +90,7 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     if not mma and (nkv * hd if wide else hd) > PLAIN_SPAN_LANES:
         span_rows = DECODE_ROWS      # fewer rows a block: its query rows lie in shared memory
     # single tokens with wide query rows: blocks of all heads, so that keys come in once
-    whole_tokens = mma and wide and WIDE_DECODE and not has_extras and ops.attn_wide_supported(x.dtype, hd, kv.pages.shape[3], nh, nkv)
+    whole_tokens = mma and wide and WIDE_DECODE and not more_than_a_sink and ops.attn_wide_supported(x.dtype, hd, kv.pages.shape[3], nh, nkv, blocks)
     clustered = hd if mma and CLUSTER_MERGE and not whole_tokens and torch.cuda.is_available() else None
     group = ctx.groups[kv.group]
     tcgen05 = mma and TCGEN05_SPANS and (ops.attn_tc_wide_supported(x.dtype, hd, kv.pages.shape[3], nkv) if wide
@@ -96,7 +100,8 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
     plan = ctx.plan(("attention", nh, nkv, mma, clustered, reach, span_rows, whole_tokens),
                     lambda: AttentionPlan(ctx, nh, nkv, dec_rows, span_rows, clustered, max_keys=reach, whole_tokens=whole_tokens))
     common = dict(nh=nh, nkv=nkv, hd=hd, window=window, status=ctx.status, table_row=ctx.slots, scale=scale,
-                  keep_first=keep_first, dist_a=dist_a, dist_b=dist_b, chunked=chunked, wide=wide, out_gate=out_gate, **extras)
+                  keep_first=keep_first, dist_a=dist_a, dist_b=dist_b, chunked=chunked, wide=wide, out_gate=out_gate, blocks=blocks, **extras)
+    merge = dict(out_gate=out_gate, gate_blocks=nkv if blocks else 1)
     args = (q, out, kv.pages, group.block_table, ctx.q_start, ctx.q_len, ctx.ctx_len)
     if plan.n_dec:
         S = plan.nslices
@@ -107,9 +112,9 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
             part_ml = workspace.empty((plan.n_dec * nh * S, 2), torch.float32, x.device)
         if whole_tokens:
             ops.attn_wide(*args, plan.dec_items, plan.n_dec * S, part_o, part_ml, nh=nh, nkv=nkv, hd=hd, window=window,
-                          status=ctx.status, table_row=ctx.slots, scale=scale, chunked=chunked, out_gate=out_gate)
+                          status=ctx.status, table_row=ctx.slots, scale=scale, chunked=chunked, out_gate=out_gate, sink=sink, blocks=blocks)
             if S > 1:
-                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S, out_gate)
+                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S, **merge)
         elif mma:
             ops.attn_mma(*args, plan.dec_items, plan.n_dec * S, dec_rows, part_o, part_ml,
                          slice_counters=plan.slice_counters if S > 1 else None, dec_rows=plan.dec_rows, cluster=cluster,
@@ -117,7 +122,7 @@ def paged_attention(ctx, kv, q, out, *, nh, nkv, hd, vd, scale, window=0, keep_f
         else:
             ops.attn_window_bias(*args, plan.dec_items, plan.n_dec * S, dec_rows, part_o, part_ml, hd_v=vd, **common)
             if S > 1:
-                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S, out_gate)
+                ops.attn_merge(part_o, part_ml, plan.dec_rows, out, plan.n_dec, nh, vd, S, **merge)
     if plan.n_span_items:
         if tcgen05:
             ops.attn_tc(*args, plan.span_items, plan.n_span_items, work=plan.span_work, **common)
@@ -242,6 +247,11 @@ def rotary_frequencies(build, base: float, dims: int) -> torch.Tensor:
     return build.shared[key]
 
 
+def tensor_core_width(lanes: int) -> int:
+    """Lanes a key or value row is padded to so that the tensor-core attention kernels take it (64, 128); 0: too wide."""
+    return 64 if lanes <= 64 else (128 if lanes <= 128 else 0)
+
+
 class RotaryWindowAttention(Mixer):
     """Grouped-query softmax attention with rotary positions, every variation a parameter:
 
@@ -260,14 +270,21 @@ class RotaryWindowAttention(Mixer):
         ``unit_values``:      every value head divided by its root mean square (no gain) and cached so
         ``talk``:             the heads' scores mixed before the softmax, s_h <- sum_g talk[h, g] s_g
         ``head_gate``:        head h's weighted sum is multiplied by sigmoid(W_g x)_h
+        ``lane_gate``:        the heads' sums, side by side, are multiplied lane by lane by sigmoid(W_g x)
+        ``keep_first``:       with a window, a request's first keys stay visible: i also sees every j < keep_first
+        ``value_mix``:        "first": the layer's values (as projected) serve later layers of the step; "mixed": v <-
+                              (1 - l) v + l v_first with l a learned number and v_first those values of the same token, the
+                              mixed value is what is cached
         ``sink``:             exp(sink_h), a learned score per head that is not scaled, joins the softmax's denominator
         softmax, weighted sum of the values, output projection.
 
     params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``v_head_dim`` (default head_dim), ``scale``,
-    ``window``, ``rope_base``, ``rotary_dim``, ``pairing``, ``eps`` and the flags above (all default False).
+    ``window``, ``rope_base``, ``rotary_dim``, ``pairing``, ``eps`` and the options above (all off by default);
+    ``pad_heads`` (default False): in the bfloat16 engine q, k and v heads of up to 128 lanes are padded with zero lanes to a
+    width the tensor-core kernels take (zero rows in the bound matrices, zero columns in the output projection).
     Tensors under ``<prefix>``: q [nh hd, H], k [nkv hd, H], v [nkv vd, H] (unless values_from_keys), o [H, nh vd];
     q.norm [nh hd], k.norm [nkv hd] (whole_norm); sink [nh] (sink); q.b, k.b, v.b, o.b (bias); talk [nh, nh] (talk);
-    g [nh, H] (head_gate).
+    g [nh, H] (head_gate) or [nh vd, H] (lane_gate); vmix, one number (value_mix; "first" has it and does not use it).
 
     Mixed scores cost the attention kernels no look at one another's heads: the sum over g is drawn into the queries (see
     csrc/kernels/rope_store.cu), whose rows then have a block of lanes per KV head.  The mixing itself is 32-bit.  The
@@ -297,6 +314,17 @@ class RotaryWindowAttention(Mixer):
         self.has_bias = bool(p.get("bias", False))
         self.unit_values = bool(p.get("unit_values", False))
         self.has_talk, self.has_gate = bool(p.get("talk", False)), bool(p.get("head_gate", False))
+        self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
+        self.lane_gate = bool(p.get("lane_gate", False))
+        self.value_mix = str(p.get("value_mix") or "")
+        if self.value_mix not in ("", "first", "mixed"):
+            raise ValueError(f"value_mix '{self.value_mix}' is not one of 'first', 'mixed'")
+        if self.has_gate and self.lane_gate:
+            raise ValueError("a gate per head and one per lane at once")
+        if self.chunked and self.keep_first:
+            raise ValueError("a window that stands still keeps no first keys")
+        if self.value_mix and self.values_from_keys:
+            raise ValueError("keys that double as values are not mixed with earlier values")
         if self.has_talk and self.whole_norm:
             raise ValueError("mixed scores come without a norm over the whole projection")
         if self.has_bias and self.values_from_keys:
@@ -312,14 +340,21 @@ class RotaryWindowAttention(Mixer):
         for n in (self.hd, self.vd):
             if n < 1:
                 raise ValueError(f"head size {n} is not supported")
+        # lanes of a head as the kernels see it
+        self.khd, self.kvd = self.hd, self.vd
+        padded = tensor_core_width(max(self.hd, self.vd))
+        if bool(p.get("pad_heads", False)) and padded and MMA_ATTENTION and build.compute_dtype == torch.bfloat16:
+            if self.whole_norm or self.unit_values or self.rotate_values or self.has_bias or self.values_from_keys:
+                raise ValueError("padded heads come without norms over them, biases, turned values and shared keys")
+            self.khd = self.kvd = padded
         base = float(p.get("rope_base", 10000.0))
         self.freq = rotary_frequencies(build, base, self.rot) if self.rot else None
         self.vfreq = rotary_frequencies(build, base, self.vd) if self.rotate_values else None
-        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.sink = self.bias = self.o_bias = self.talk = None
+        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.sink = self.bias = self.o_bias = self.talk = self.v_share = None
 
     def cache_spec(self):
-        return CacheSpec("kv", num_kv_heads=self.nkv, head_dim=self.hd, window=self.window, chunked=self.chunked,
-                         v_head_dim=0 if self.vd == self.hd else self.vd)
+        return CacheSpec("kv", num_kv_heads=self.nkv, head_dim=self.khd, window=self.window, chunked=self.chunked,
+                         keep_first=self.keep_first, v_head_dim=0 if self.kvd == self.khd else self.kvd)
 
     def _rows(self):
         rows = [("q", self.nh * self.hd), ("k", self.nkv * self.hd)]
@@ -338,14 +373,36 @@ class RotaryWindowAttention(Mixer):
             specs.append(TensorSpec(p + "talk", (self.nh, self.nh), "mixing"))
         if self.has_gate:
             specs.append(TensorSpec(p + "g", (self.nh, H)))
+        if self.lane_gate:
+            specs.append(TensorSpec(p + "g", (self.nh * self.vd, H)))
+        if self.value_mix:
+            specs.append(TensorSpec(p + "vmix", (), "unit"))
         return specs
 
     def bind(self, store):
         p = self.prefix
         f32 = lambda name: store.vector(p + name).float().contiguous()
         # the gates' rows under the projections': one product
-        self.w_qkv = store.matrices([p + n for n, _ in self._rows()] + ([p + "g"] if self.has_gate else []))
-        self.w_o = store.matrix(p + "o")
+        gates = [p + "g"] if self.has_gate or self.lane_gate else []
+        if (self.khd, self.kvd) == (self.hd, self.vd):
+            self.w_qkv = store.matrices([p + n for n, _ in self._rows()] + gates)
+            self.w_o = store.matrix(p + "o")
+        else:
+            def padded(name, heads, lanes, to):
+                w = store.matrix(name)
+                out = w.new_zeros((heads, to, w.shape[1]))
+                out[:, :lanes] = w.view(heads, lanes, w.shape[1])
+                return out.view(heads * to, w.shape[1])
+            rows = [padded(p + "q", self.nh, self.hd, self.khd), padded(p + "k", self.nkv, self.hd, self.khd),
+                    padded(p + "v", self.nkv, self.vd, self.kvd)]
+            rows += [padded(p + "g", self.nh, self.vd, self.kvd)] if self.lane_gate else [store.matrix(g) for g in gates]
+            self.w_qkv = torch.cat(rows).contiguous()
+            w_o = store.matrix(p + "o")
+            self.w_o = w_o.new_zeros((w_o.shape[0], self.nh, self.kvd))
+            self.w_o[..., :self.vd] = w_o.view(-1, self.nh, self.vd)
+            self.w_o = self.w_o.view(-1, self.nh * self.kvd)
+        if self.value_mix == "mixed":
+            self.v_share = f32("vmix").view(1)
         if self.whole_norm:
             self.q_gain, self.k_gain = f32("q.norm"), f32("k.norm")
         if self.has_sink:
@@ -361,18 +418,25 @@ class RotaryWindowAttention(Mixer):
             raise ValueError("this attention part keeps its own keys: it cannot read a cache another run filled")
         kv = cache
         T = x.shape[0]
-        nh, nkv, hd, vd = self.nh, self.nkv, self.hd, self.vd
+        nh, nkv, hd, vd = self.nh, self.nkv, self.khd, self.kvd
         group = ctx.groups[kv.group]
         qkv = matmul_tn(x, self.w_qkv, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
         q = workspace.empty((T, nh * hd * (nkv if self.has_talk else 1)), x.dtype, x.device)
-        gate = workspace.empty((T, nh), torch.float32, x.device) if self.has_gate else None
+        gate = None
+        if self.has_gate or self.lane_gate:
+            gate = workspace.empty((T, nh if self.has_gate else nh * vd), torch.float32, x.device)
+        v_keep = v_first = None
+        if self.value_mix:
+            # one buffer a step: the first layer of the kind fills it before any other asks
+            values = ctx.plan(("first_values", nkv, vd), lambda: workspace.empty((T, nkv * vd), torch.float32, x.device))
+            v_keep, v_first = (values, None) if self.value_mix == "first" else (None, values)
         ops.qkv_rope_store(qkv, self.q_gain, self.k_gain, self.eps, ctx.positions, self.freq, self.vfreq, group.slot_map, q,
                            kv.pages, nh, nkv, hd, vd, ctx.status, rot=self.rot, interleaved=self.interleaved,
                            values_from_keys=self.values_from_keys, bias=self.bias, unit_values=self.unit_values, talk=self.talk,
-                           gate_out=gate)
+                           gate_out=gate, v_keep=v_keep, v_first=v_first, v_share=self.v_share)
         out = workspace.empty((T, nh * vd), x.dtype, x.device)
         paged_attention(ctx, kv, q, out, nh=nh, nkv=nkv, hd=hd, vd=vd, scale=self.scale, window=self.window,
-                        sink=self.sink if self.has_sink else False, chunked=self.chunked, wide=self.has_talk, out_gate=gate)
+                        keep_first=self.keep_first, sink=self.sink if self.has_sink else False, chunked=self.chunked, wide=self.has_talk, out_gate=gate)
         if self.rotate_values:
             ops.rotate_heads(out, ctx.positions, self.vfreq, heads=nh, width=vd, dims=vd, interleaved=self.interleaved, sign=-1.0)
         y = matmul_tn(out, self.w_o, ctx.status, out_dtype=torch.float32, allow_partials=True, after_small_kernel=True)
