@@ -1,7 +1,7 @@
 #!/usr/bin/env python3
 """Benchmark of the engine on one B200.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--workloads all|headline|14b|4b|rimopel|nagavik|fifudra|mefupel|nufetar] [--impl reference]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--workloads all|headline|14b|4b|rimopel|nagavik|fifudra|mefupel|nufetar|disorax] [--impl reference]
 
 Headline: decode tokens/s of the Qwen3-8B layer sizes (the baseline's third configuration) at batch 8 and context
 4,096, the median of K device-timed steps after W warm-up steps; beside it batch 1 and 64, batch 8 at context 2,176
@@ -875,6 +875,76 @@ def run_nufetar(args, pk, clocks, windows):
     return run_beside(args, pk, clocks, windows, "nufetar_beside_mefupel", NUFETAR_SIZES, configs, numbers)
 
 
+# Disorax at real layer sizes beside Fifudra, the closest design the engine has (latent attention, gated experts behind a
+# router), at equal width, layer count, heads, latent rows and feed-forward parameters per token: a layer of window
+# attention that keeps first tokens, a latent attention layer, a latent attention layer under a window, and so on, each
+# with 4 of 16 experts and a shared one of their size; Fifudra as latent attention layers on one plain stream, each with 5
+# of 16 experts.
+DISORAX_SIZES = {
+    "w2048": dict(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, window=1024, keep_first=64, rot=128,
+                  l_dim=128, l_rot=32, kv_rank=128, q_rank=1536, experts=16, top=4, ff=1024),
+    "w4096": dict(width=4096, layers=8, vocab=32768, heads=32, kv_heads=8, dim=128, window=2048, keep_first=64, rot=128,
+                  l_dim=128, l_rot=32, kv_rank=128, q_rank=3072, experts=16, top=4, ff=2048),
+    # latent rows of four blocks of the tensor-core kernels' 128 lanes
+    "w2048_k512": dict(width=2048, layers=12, vocab=32768, heads=16, kv_heads=4, dim=128, window=1024, keep_first=64, rot=128,
+                       l_dim=128, l_rot=32, kv_rank=512, q_rank=1536, experts=16, top=4, ff=1024),
+}
+
+
+def run_disorax(args, pk, clocks, windows):
+    """Disorax at real layer sizes beside Fifudra at equal size (see DISORAX_SIZES and run_beside)."""
+    from vllm_cpp_b200.config.disorax import AttentionSpec, DisoraxConfig, DisoraxLayer, DisoraxMlp, LatentSpec
+    from vllm_cpp_b200.config.fifudra import FifudraConfig, FifudraLayer, FifudraMlp, LatentAttentionSpec, RotarySpec
+    context, T = args.context, PREFILL_TOKENS
+
+    def kinds(z):
+        return [("attention", "latent_attention", "latent_attention_2")[i % 3] for i in range(z["layers"])]
+
+    def configs(z):
+        H, d, ld, r, kr = z["heads"], z["dim"], z["l_dim"], z["l_rot"], z["kv_rank"]
+        latent = dict(heads=H, dim=ld, vdim=d, kv_rank=kr, scale=ld ** -0.5)
+        mixers = {"attention": AttentionSpec(heads=H, kv_heads=z["kv_heads"], dim=d, vdim=d, scale=d ** -0.5, rope_base=1e6, rope_dims=z["rot"],
+                                             window=z["window"], keep_first=z["keep_first"], v_mix=True),
+                  "latent_attention": LatentSpec(**latent), "latent_attention_2": LatentSpec(**latent, window=z["window"])}
+        mlp = DisoraxMlp("moe", ff=z["ff"], experts=z["experts"], top=z["top"], shared_ff=z["ff"])
+        dis = DisoraxConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, residual_mult=0.5, max_positions=context + 4096,
+                            layers=tuple(DisoraxLayer(k, mixers[k], mlp) for k in kinds(z)))
+        fmix = LatentAttentionSpec(heads=H, dim=ld, rot_dim=r, vdim=d, q_rank=z["q_rank"], kv_rank=kr - r, scale=(ld + r) ** -0.5,
+                                   rot=RotarySpec(base=1e6, dims=r))
+        fmlp = FifudraMlp("moe", ff=z["ff"], experts=z["experts"], top=z["top"] + 1)
+        fif = FifudraConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-5, max_positions=context + 4096,
+                            layers=tuple(FifudraLayer("latent_attention", fmix, fmlp) for _ in range(z["layers"])))
+        return {"disorax": dis, "fifudra": fif}
+
+    def numbers(z, name):
+        W, V, L = z["width"], z["vocab"], z["layers"]
+        H, G, d, ld, r, kr, E, ff = z["heads"], z["kv_heads"], z["dim"], z["l_dim"], z["l_rot"], z["kv_rank"], z["experts"], z["ff"]
+        dis = name == "disorax"
+        top, shared = (z["top"], 1) if dis else (z["top"] + 1, 0)
+        expert, router = 3 * ff * W, E * W
+        distinct = E * (1 - (1 - top / E) ** args.batch)        # experts that a decoding batch chooses, in expectation
+        qr = z["q_rank"]
+        w = {"attention": (2 * H + 2 * G) * d * W + W * H * d, "latent": (H * ld + kr + H) * W + H * ld * kr + H * d * kr + W * H * d,
+             "fifudra": (qr + kr) * W + H * (ld + r) * qr + H * ld * (kr - r) + H * d * (kr - r) + W * H * d}
+        names = kinds(z) if dis else ["fifudra"] * L
+        n = {k: names.count(k) for k in ("attention", "latent_attention", "latent_attention_2", "fifudra")}
+        mixers = n["attention"] * w["attention"] + (n["latent_attention"] + n["latent_attention_2"]) * w["latent"] + n["fifudra"] * w["fifudra"]
+        window, keep = z["window"], z["keep_first"]
+        seen = {"all": sum(i + 1 for i in range(T)), "window": sum(min(i + 1, window) for i in range(T)),
+                "kept": sum(min(i + 1, window + keep) for i in range(T))}
+        keys = {"all": context, "window": min(context, window), "kept": min(context, window + keep)}
+        # scores and weighted sums over a latent row (Fifudra's weighted sums leave the turned lanes out)
+        row = {"latent_attention": 2 * kr, "latent_attention_2": 2 * kr, "fifudra": 2 * kr - r}
+        reach = {"latent_attention": "all", "latent_attention_2": "window", "fifudra": "all"}
+        return dict(weight_bytes=2 * (mixers + L * (router + (distinct + shared) * expert) + V * W),
+                    # a cached token: a key and a value row per KV head, or the latent row, 16-bit
+                    cache_bytes=n["attention"] * 2 * G * d * 2 * keys["kept"] + sum(n[k] * kr * 2 * keys[reach[k]] for k in row),
+                    prefill_flops=2.0 * T * (mixers + L * (router + (top + shared) * expert)) + 2.0 * V * W
+                                  + n["attention"] * 4.0 * H * d * seen["kept"] + sum(n[k] * 2.0 * H * row[k] * seen[reach[k]] for k in row))
+
+    return run_beside(args, pk, clocks, windows, "disorax_beside_fifudra", DISORAX_SIZES, configs, numbers)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -886,11 +956,11 @@ def main():
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=CONTEXT)
     ap.add_argument("--impl", default="ours")
-    ap.add_argument("--workloads", default="all", choices=["all", "headline", "14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel", "nufetar"],
+    ap.add_argument("--workloads", default="all", choices=["all", "headline", "14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel", "nufetar", "disorax"],
                     help="headline: the 8B numbers only; 14b / 4b: that workload alone (prints its own JSON line); rimopel, "
                          "nagavik: that design at real layer sizes beside Qwen3 at equal size, prefill and decode (its own JSON line); "
-                         "fifudra: that design beside Nagavik at equal size, likewise; mefupel: that design beside Fifudra at equal size, likewise; nufetar: that design beside Mefupel at equal size, likewise")
-    ap.add_argument("--size", default="", help="rimopel, nagavik, fifudra, mefupel, nufetar: one of the workload's sizes only (w2048, w4096; fifudra also w2048_k256)")
+                         "fifudra: that design beside Nagavik at equal size, likewise; mefupel: that design beside Fifudra at equal size, likewise; nufetar: that design beside Mefupel at equal size, likewise; disorax: that design beside Fifudra at equal size, likewise")
+    ap.add_argument("--size", default="", help="rimopel, nagavik, fifudra, mefupel, nufetar, disorax: one of the workload's sizes only (w2048, w4096; fifudra also w2048_k256, nufetar w4096_kv4, disorax w2048_k512)")
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (for profiling runs)")
     ap.add_argument("--no-graphs", action="store_true", help="launch decode steps kernel by kernel (for profiling runs)")
     ap.add_argument("--mode", default="all", choices=["all", "decode", "prefill"], help="what to run (profiling runs)")
@@ -912,9 +982,9 @@ def main():
     clocks.start()
     windows = []
     try:
-        if args.workloads in ("14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel", "nufetar"):
+        if args.workloads in ("14b", "4b", "rimopel", "nagavik", "fifudra", "mefupel", "nufetar", "disorax"):
             out = {"14b": run_14b, "4b": run_4b, "rimopel": run_rimopel, "nagavik": run_nagavik, "fifudra": run_fifudra, "mefupel": run_mefupel,
-                   "nufetar": run_nufetar}[args.workloads](args, pk, clocks, windows)
+                   "nufetar": run_nufetar, "disorax": run_disorax}[args.workloads](args, pk, clocks, windows)
             out["clocks"] = clocks.summary(windows)
             print(json.dumps(out))
             return 0

@@ -99,5 +99,5 @@ def write_safetensors(path, tensors: dict[str, torch.Tensor], metadata: dict[str
         f.write(struct.pack("<Q", len(blob)))
         f.write(blob)
         for name in order:
-            t = tensors[name].detach().cpu().contiguous()
+            t = tensors[name].detach().cpu().contiguous().reshape(-1)       # (a tensor of no dimension has bytes too)
             f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
