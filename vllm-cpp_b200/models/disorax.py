@@ -54,7 +54,9 @@ def describe_disorax(cfg: DisoraxConfig) -> ModelSpec:
             raise ConfigError(f"layer {i}: no mixer of type '{layer.type}' (known: {sorted(MIXERS)})")
         parts = {"norm1": (norm, "norm1"), "mixer": (MIXERS[layer.type](cfg, layer.mixer, i == first_mixing), "mix.")}
         mlp = layer.mlp
-        if mlp is not None:
+        if mlp is None:      # its checkpoint may hold a second norm all the same: nothing reads it
+            parts["norm2"] = (PartSpec("rmsnorm", {**norm.params, "unused": True}), "norm2")
+        else:
             parts["norm2"] = (norm, "norm2")
             parts["feed_forward"] = (PartSpec("routed_experts", {
                 "hidden_size": cfg.width, "num_experts": mlp.experts, "top": mlp.top, "expert_size": mlp.ff,

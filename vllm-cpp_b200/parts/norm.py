@@ -13,7 +13,8 @@ from .base import Norm
 class RMSNorm(Norm):
     """params: ``size``, ``eps``; optional ``name`` (default "weight"); ``one_plus`` (default False): the tensor holds the
     gain less one (values around zero), y = (1 + w) * x / sqrt(mean(x^2) + eps), the sum made in 32-bit; ``keep_32bit``
-    (default False): the rows are handed on in 32-bit, for a mixer that computes on them before its products read them.
+    (default False): the rows are handed on in 32-bit, for a mixer that computes on them before its products read them;
+    ``unused`` (default False): nothing reads the norm and a checkpoint may lack its tensor.
     Tensor: ``<prefix><name>`` [size]."""
 
     def __init__(self, params, prefix, build):
@@ -23,13 +24,16 @@ class RMSNorm(Norm):
         self.name = self.prefix + str(params.get("name", "weight"))
         self.one_plus = bool(params.get("one_plus", False))
         self.out_dtype = torch.float32 if params.get("keep_32bit", False) else self.build.compute_dtype
+        self.unused = bool(params.get("unused", False))
         self.weight = None
         self._gain32 = None
 
     def tensor_specs(self):
-        return [TensorSpec(self.name, (self.size,), "bias" if self.one_plus else "vector")]
+        return [TensorSpec(self.name, (self.size,), "bias" if self.one_plus else "vector", optional=self.unused)]
 
     def bind(self, store):
+        if self.unused:
+            return
         self.weight = store.vector(self.name)
         if self.one_plus:
             self.weight = (1.0 + self.weight.float()).contiguous()

@@ -77,12 +77,12 @@ class ParallelBlock(Block):
     def __init__(self, params, prefix, build, parts):
         super().__init__(params, prefix, build, parts)
         self.scale = float(params.get("result_scale", 1.0))
-        if "norm2" in parts and "feed_forward" not in parts:
+        if "feed_forward" not in parts and "norm2" in parts and not getattr(parts["norm2"], "unused", False):
             raise ValueError("a second norm comes with a feed-forward")
 
     def _normed(self, resid, pending):
         """-> (what the mixer reads, what the feed-forward reads)"""
-        n1, n2 = self.parts["norm1"], self.parts.get("norm2")
+        n1, n2 = self.parts["norm1"], self.parts.get("norm2") if "feed_forward" in self.parts else None
         if n2 is None:
             h = n1.forward(resid, pending)
             return h, h

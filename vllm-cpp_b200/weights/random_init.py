@@ -61,7 +61,7 @@ def write_random_model(config, seed: int, out_dir, dtype: str = "bfloat16") -> P
     cfg["torch_dtype"] = dtype
     (out_dir / "config.json").write_text(json.dumps(cfg, indent=2))
     tensors = {s.name: (_generate(s, seed) if s.role == "table" else _generate(s, seed).to(store_dtype))
-               for s in expected_tensors(config)}
+               for s in expected_tensors(config) if not s.optional}
     write_safetensors(out_dir / "model.safetensors", tensors, {"format": "pt", "seed": str(seed)})
     return out_dir
 
